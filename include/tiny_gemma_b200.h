@@ -72,6 +72,21 @@ int tg_config_by_name(const char *name, tg_config *out);
 
 /* ---- model -------------------------------------------------------------- */
 
+/* Models in a folder (config.json + model.safetensors). config.json's "architecture" selects the family from
+ * the library's registry; the layer list, every size and every constant are read from config.json, the weights
+ * (bfloat16) from model.safetensors. An architecture the library does not know, a config it cannot read or a
+ * tensor that is missing or has another shape is an error (TG_EINVAL / TG_EIO / TG_ESHAPE).
+ *   dtype TG_BF16: matrix products and activations in bfloat16 with 32-bit accumulation; residual stream,
+ *                  norms, attention scores and recurrent states in 32-bit.
+ *   dtype TG_F32:  everything in 32-bit (the weights are the same bfloat16 values).
+ * Architectures: "Nabelix" (pre-norm decoder whose mixer runs windowed attention with kept first tokens and a
+ * gated delta rule side by side). Entry points of this header that name a Gemma structure (tg_model_load_*,
+ * tg_model_set_*, tg_kv_read, tg_decode_hidden, the tg_dev_ calls on a handle) return TG_EINVAL on such a model. */
+enum { TG_BF16 = 0, TG_F32 = 1 };
+int tg_model_open(const char *dir, int device, int dtype, tg_model **out);
+int tg_model_vocab(tg_model *m, int *n_vocab);
+int tg_model_hidden_size(tg_model *m, int *hidden_size);
+
 /* gemma::Transformer(Config), transformer.hpp:33-46. Allocates the weight
  * store in the HBM of `device`; weights are zero until loaded. */
 int tg_model_create(const tg_config *cfg, int device, tg_model **out);
@@ -135,6 +150,21 @@ int tg_decode(tg_state *s, const int *ids_host, float *logits_host);
  * listed as a limitation in README.md:96). One sequence per state; logits_host may be NULL, otherwise it
  * receives the logits after the last token. */
 int tg_append(tg_state *s, const int *ids_host, int n, float *logits_host);
+
+/* The general step of models opened with tg_model_open: n entries, entry e being the next count[e] tokens of
+ * sequence seq[e] (0 <= seq < batch, each at most once per step); ids_host holds all entries' tokens one after
+ * the other. Sequences advance independently, a prompt may be cut into portions anywhere, and portions and single
+ * tokens may share a step. n_want[e] (n_want may be null: none) places of entry e, listed in `want` one entry after
+ * the other, are scored: logits_host receives [sum of n_want][n_vocab] fp32. tg_prefill, tg_append and tg_decode
+ * are special cases of it; after a step, the logits of each entry's last token are NOT kept for the samplers.
+ * Synchronises. tg_sequence_free empties one sequence, whose slot can then be used for another. */
+int tg_step(tg_state *s, int n, const int *seq, const int *count, const int *ids_host, const int *n_want, const int *want,
+            float *logits_host);
+int tg_sequence_free(tg_state *s, int b);
+/* A recorder for the residual stream, for comparing a model layer by layer: with on != 0 the following steps keep
+ * it after every layer run, and tg_trace_read copies out what the last step left: [layer runs][tokens][hidden]. */
+int tg_trace_enable(tg_state *s, int on);
+int tg_trace_read(tg_state *s, float *x_host, size_t cap_floats, int *runs, int *tokens);
 
 /* ops::argmax_logits, ops.hpp:744-760, on the logits of the last forward
  * (still in HBM): lowest index wins ties, NaN never wins, -1 if no logit is

@@ -13,6 +13,7 @@ import numpy as np
 HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(HERE, "libtinygemma_b200.so")
 
+TG_BF16, TG_F32 = 0, 1
 TG_OK, TG_EINVAL, TG_ENODEVICE, TG_ECUDA, TG_EIO, TG_ESHAPE, TG_ESTATE, TG_ENOMEM = range(8)
 
 
@@ -37,6 +38,13 @@ SIGNATURES = {
     "tg_version": (C.c_char_p, []),
     "tg_device_count": (C.c_int, [C.POINTER(C.c_int)]),
     "tg_config_by_name": (C.c_int, [C.c_char_p, C.POINTER(tg_config)]),
+    "tg_model_open": (C.c_int, [C.c_char_p, C.c_int, C.c_int, C.POINTER(_P)]),
+    "tg_model_vocab": (C.c_int, [_P, C.POINTER(C.c_int)]),
+    "tg_model_hidden_size": (C.c_int, [_P, C.POINTER(C.c_int)]),
+    "tg_step": (C.c_int, [_P, C.c_int, _P, _P, _P, _P, _P, _P]),
+    "tg_sequence_free": (C.c_int, [_P, C.c_int]),
+    "tg_trace_enable": (C.c_int, [_P, C.c_int]),
+    "tg_trace_read": (C.c_int, [_P, _P, C.c_size_t, C.POINTER(C.c_int), C.POINTER(C.c_int)]),
     "tg_model_create": (C.c_int, [C.POINTER(tg_config), C.c_int, C.POINTER(_P)]),
     "tg_model_free": (C.c_int, [_P]),
     "tg_model_load_file": (C.c_int, [_P, C.c_char_p]),
@@ -84,15 +92,19 @@ SIGNATURES = {
 _lib = None
 
 
-def load() -> C.CDLL:
-    """dlopen the library (once) and set signatures; raises if it is not built."""
+def load(path: str | None = None) -> C.CDLL:
+    """dlopen the library (once) and set signatures; raises if it is not built. `path`: a library that holds one
+    model family only (build.py --family), which lacks the other families' entry points."""
     global _lib
     if _lib is None:
-        if not os.path.exists(LIB_PATH):
+        lib_path = path or LIB_PATH
+        if not os.path.exists(lib_path):
             raise FileNotFoundError(
-                LIB_PATH + " is not built; run `python tiny-gemma_b200/build.py` (there is no CPU fallback)")
-        lib = C.CDLL(LIB_PATH)
+                lib_path + " is not built; run `python tiny-gemma_b200/build.py` (there is no CPU fallback)")
+        lib = C.CDLL(lib_path)
         for name, (res, args) in SIGNATURES.items():
+            if path and not hasattr(lib, name):
+                continue
             fn = getattr(lib, name)
             fn.restype = res
             fn.argtypes = args
@@ -184,14 +196,30 @@ def rmsnorm(x, w) -> np.ndarray:
 
 # ------------------------------------------------------------------ model / state
 class Model:
-    """gemma::Transformer + read_weights (reference transformer.hpp:22-47, 99-165)"""
+    """gemma::Transformer + read_weights (reference transformer.hpp:22-47, 99-165); Model.open for model folders"""
 
     def __init__(self, size: str, device: int = 0):
         self.lib = load()
         self.size = size
         self.cfg = config(size)
+        self.vocab, self.hidden_size = self.cfg.n_vocab, self.cfg.hidden_size
         self.h = C.c_void_p()
         _ck(self.lib.tg_model_create(C.byref(self.cfg), device, C.byref(self.h)))
+
+    @classmethod
+    def open(cls, folder: str, dtype: str = "bfloat16", device: int = 0) -> "Model":
+        """a folder with config.json and model.safetensors; config.json names the architecture"""
+        self = cls.__new__(cls)
+        self.lib = load()
+        self.size = os.path.basename(os.path.normpath(folder))
+        self.h = C.c_void_p()
+        code = {"bfloat16": TG_BF16, "float32": TG_F32}[dtype]
+        _ck(self.lib.tg_model_open(os.fsencode(folder), device, code, C.byref(self.h)))
+        v, d = C.c_int(0), C.c_int(0)
+        _ck(self.lib.tg_model_vocab(self.h, C.byref(v)))
+        _ck(self.lib.tg_model_hidden_size(self.h, C.byref(d)))
+        self.vocab, self.hidden_size = v.value, d.value
+        return self
 
     def load_file(self, path: str):
         _ck(self.lib.tg_model_load_file(self.h, path.encode()))
@@ -241,7 +269,7 @@ class State:
         self.m = model
         self.lib = model.lib
         self.B = batch
-        self.V = model.cfg.n_vocab
+        self.V = model.vocab
         self.h = C.c_void_p()
         _ck(self.lib.tg_state_create(model.h, batch, max_pos_global, C.byref(self.h)))
 
@@ -272,6 +300,33 @@ class State:
         logits = np.empty((1, self.V), np.float32) if want_logits else None
         _ck(self.lib.tg_append(self.h, _ptr(ids), ids.size, _ptr(logits)))
         return logits
+
+    def step(self, entries):
+        """one general step (models of Model.open): entries = [(sequence, tokens, places whose logits are wanted)];
+        returns the logits [wanted, vocab] in the order of the entries and places"""
+        seq = np.array([e[0] for e in entries], np.int32)
+        count = np.array([len(e[1]) for e in entries], np.int32)
+        ids = np.concatenate([np.asarray(e[1], np.int32).reshape(-1) for e in entries])
+        n_want = np.array([len(e[2]) for e in entries], np.int32)
+        want = np.array([w for e in entries for w in e[2]], np.int32)
+        out = np.empty((int(n_want.sum()), self.V), np.float32)
+        _ck(self.lib.tg_step(self.h, len(entries), _ptr(seq), _ptr(count), _ptr(ids), _ptr(n_want), _ptr(want), _ptr(out)))
+        return out
+
+    def free_sequence(self, b: int):
+        """empties one sequence; its slot can then be used for another"""
+        _ck(self.lib.tg_sequence_free(self.h, b))
+
+    def trace_enable(self, on: bool = True):
+        _ck(self.lib.tg_trace_enable(self.h, int(on)))
+
+    def trace(self) -> np.ndarray:
+        """residual stream after every layer run of the last step: [layer runs, tokens, hidden]"""
+        runs, tokens = C.c_int(0), C.c_int(0)
+        _ck(self.lib.tg_trace_read(self.h, None, 0, C.byref(runs), C.byref(tokens)))
+        out = np.empty((runs.value, tokens.value, self.m.hidden_size), np.float32)
+        _ck(self.lib.tg_trace_read(self.h, _ptr(out), out.size, C.byref(runs), C.byref(tokens)))
+        return out
 
     def sample_argmax(self) -> np.ndarray:
         t = np.empty(self.B, np.int32)
@@ -341,7 +396,7 @@ class State:
         return k, v
 
     def hidden(self) -> np.ndarray:
-        out = np.empty((self.B, self.m.cfg.hidden_size), np.float32)
+        out = np.empty((self.B, self.m.hidden_size), np.float32)
         _ck(self.lib.tg_hidden_read(self.h, _ptr(out)))
         return out
 

@@ -46,7 +46,7 @@
 #include <cuda.h>
 #include <cuda_bf16.h>
 
-#include "kernels_mega.cuh"  // mbarrier / TMA helpers
+#include "tc_common.cuh"
 #include "tg_common.cuh"
 
 namespace tg {
@@ -69,7 +69,6 @@ template <int MT, int BN> struct TcShape {
 	static constexpr int SMEM = NA * A_BYTES + NB * (W_BYTES + B_BYTES) + 1024;
 };
 constexpr int TC_THREADS = 224;
-constexpr int TC_SPIN_CAP = 1 << 24;
 
 // ------------------------------------------------------------------ split + pack
 // out: [3 terms][m_tiles][k_blocks][TC_TILE_BYTES]; rows >= M are zero.
@@ -341,45 +340,6 @@ __device__ __forceinline__ uint64_t tc_smem_desc(uint32_t smem_addr) {
 // instruction descriptor: D fp32, A and B bf16, A K-major, B N-major (bit 16), M = 128, N = bn
 __device__ __forceinline__ uint32_t tc_idesc(int bn) {
 	return (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | (uint32_t(bn >> 3) << 17) | (uint32_t(TC_BM >> 4) << 24);
-}
-__device__ __forceinline__ void tc_mma(uint32_t d_tmem, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
-	asm volatile(
-	    "{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
-	    "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}" ::"r"(d_tmem),
-	    "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
-	    : "memory");
-}
-__device__ __forceinline__ void tc_commit(uint64_t *bar) {
-	asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void bulk_load(void *dst, const void *src, uint32_t bytes, uint64_t *bar) {
-	asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst)),
-	             "l"(src), "r"(bytes), "r"(smem_u32(bar))
-	             : "memory");
-}
-// 32 lanes x 32 consecutive fp32 columns of TMEM -> 32 registers per thread (completion: tcgen05.wait::ld)
-__device__ __forceinline__ void tc_ld32(uint32_t taddr, uint32_t (&r)[32]) {
-	asm volatile(
-	    "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-	    "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
-	    : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-	      "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]),
-	      "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]),
-	      "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-	    : "r"(taddr)
-	    : "memory");
-}
-__device__ __forceinline__ bool tc_wait(uint64_t *bar, uint32_t parity, int *err) {
-	int spins = 0;
-	while (!mbar_try_wait(bar, parity)) {
-		if (++spins > TC_SPIN_CAP) {
-			atomicExch(err, 6);
-			return false;
-		}
-	}
-	return true;
 }
 
 struct GemmTcArgs {

@@ -1,0 +1,250 @@
+// Matrix-vector products with bfloat16 weights [N][K] for a few rows (decoding): HBM bound. Activations stay fp32.
+// The norm (and input convolution) that precedes a product is its prologue, what follows it is its epilogue, so a
+// layer is five launches: [norm + conv -> projections -> cache], token mixing, [output projection + residual],
+// [norm -> gate|up -> gated GELU], [down + residual].
+//
+// A CTA of 8 warps walks groups of output rows: a warp owns NR rows of the group (or, with KS > 1, the KS warps of a
+// row set share its K range), a lane 8 consecutive k of every 256. The next 16-byte weight words are requested before
+// the current ones are used, the very first ones before the wait for the preceding kernel.
+#pragma once
+#include "kernels_gemm_bf16.cuh"
+#include "kernels_rowwise.cuh"
+
+namespace tg {
+
+enum GemvPro { GV_VEC = 0, GV_LN = 1, GV_LN_CONV = 2 };
+enum GemvEpi { GV_PROJ = 0, GV_ADD = 1, GV_GEGLU = 2, GV_LOGITS = 3 };
+
+struct GemvArgs {
+	StepDesc d;
+	const __nv_bfloat16 *W;
+	int ldw, N, K;             // K: columns that are used (a multiple of 8; surplus columns and activations are zero)
+	const float *vec;          // GV_VEC: [R][ldv]
+	int ldv;
+	const float *x;            // residual stream [R][ldx]
+	int ldx, D;
+	const __nv_bfloat16 *embed;
+	int lde, V;
+	int embed_mode;            // 0: x; 1: x = embed[tok] (nothing written there yet); 2: x + embed[tok]
+	const float *w;            // norm weight [D]
+	float eps;
+	const float *cw;           // convolution [taps][D]
+	float *hist;               // [B][2][taps-1][D]
+	int taps;
+	float *out;                // GV_PROJ, GV_GEGLU, GV_LOGITS: [R][ldo]; GV_ADD: the residual stream [R][ldo]
+	int ldo;
+	float *norm_out;           // normed rows [R][D], written by one CTA, or null
+	float cap;
+	// GV_PROJ: columns p_k .. and p_v .. also go to the cache
+	int p_k, n_k, p_v, n_v;
+	void *kc, *vc, *ks, *vs;
+	int cap_rows, keep, keep_rows, cache_f32;
+	int *err;
+};
+
+constexpr int GV_THREADS = 256;
+__host__ __device__ inline int gv_k8(int K) { return (K + 7) / 8; }
+template <int R, int NR> __host__ __device__ constexpr int gv_red_floats() { return 2 * 8 * NR * R; }
+template <int R, int NR> size_t gv_smem(int K) { return (size_t(R) * 8 * gv_k8(K) + gv_red_floats<R, NR>() + 32) * 4; }
+
+__device__ __forceinline__ float gv_block_sum(float v, float *red) {
+	v = warp_sum(v);
+	__syncthreads();
+	if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+	__syncthreads();
+	float t = 0.0f;
+#pragma unroll
+	for (int w = 0; w < 8; w++) t += red[w];
+	return t;
+}
+
+template <int R, int NR, int KS, int PRO, int EPI>
+__global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
+	pdl_trigger();
+	extern __shared__ __align__(16) float gv_sm[];
+	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+	const int K8 = gv_k8(a.K);
+	float *xs = gv_sm;                                   // [R][two halves of 8 k][K8] float4
+	float *red = gv_sm + size_t(R) * 8 * K8;             // [2][row set][KS][NR][R]
+	float *bred = red + gv_red_floats<R, NR>();
+	constexpr int SETS = 8 / KS, GROUP = SETS * NR;      // weight rows per CTA and group
+	const int set = warp / KS, ks = warp % KS;
+	const int n_out = EPI == GV_GEGLU ? a.N / 2 : (EPI == GV_LOGITS ? a.ldo : a.N);
+	constexpr int OUTS = EPI == GV_GEGLU ? GROUP / 2 : GROUP;  // outputs per group
+	const int groups = (n_out + OUTS - 1) / OUTS;
+	const int nit = (K8 + 32 * KS - 1) / (32 * KS);
+
+	// weight row i (of NR) of this warp in a group
+	auto wrow = [&](int grp, int i) -> int {
+		if (EPI == GV_GEGLU) {
+			const int o = grp * OUTS + set * (NR / 2) + (i >> 1);
+			return (o >> 4) * 32 + (o & 15) + (i & 1) * 16;
+		}
+		return grp * GROUP + set * NR + i;
+	};
+	auto load = [&](int grp, int it, uint4 (&w)[NR]) {
+		const int k8 = (it * KS + ks) * 32 + lane;
+#pragma unroll
+		for (int i = 0; i < NR; i++) {
+			const int n = wrow(grp, i);
+			w[i] = make_uint4(0, 0, 0, 0);
+			if (grp < groups && n < a.N && k8 < K8) {
+				const int4 v = ld_stream_int4(a.W + size_t(n) * a.ldw + 8 * k8);
+				w[i] = make_uint4(v.x, v.y, v.z, v.w);
+			}
+		}
+	};
+	uint4 cur[NR], nxt[NR];
+	load(blockIdx.x, 0, cur);
+	pdl_wait();
+
+	// ---------------------------------------------------------------- prologue: activations into shared memory
+	auto xi = [&](int k) { return ((k >> 2) & 1) * 4 * K8 + (k >> 3) * 4 + (k & 3); };
+#pragma unroll 1
+	for (int r = 0; r < R; r++) {
+		float *xr = xs + size_t(r) * 8 * K8;
+		if (PRO == GV_VEC) {
+			for (int k = tid; k < 8 * K8; k += GV_THREADS) xr[xi(k)] = k < a.K ? a.vec[size_t(r) * a.ldv + k] : 0.0f;
+			continue;
+		}
+		const int seg = a.d.row_seg[r];
+		int tok = 0;
+		if (a.embed_mode) {
+			tok = a.d.tok[r];
+			if (tok < 0 || tok >= a.V) {
+				if (blockIdx.x == 0 && tid == 0) *a.err = 1;
+				tok = 0;
+			}
+		}
+		float s = 0.0f;
+		for (int k = tid; k < a.D; k += GV_THREADS) {
+			float v = a.embed_mode == 1 ? 0.0f : a.x[size_t(r) * a.ldx + k];
+			if (a.embed_mode) v += __bfloat162float(a.embed[size_t(tok) * a.lde + k]);
+			xr[xi(k)] = v;
+			s += v;
+		}
+		const float mean = gv_block_sum(s, bred) / float(a.D);
+		float q = 0.0f;
+		for (int k = tid; k < a.D; k += GV_THREADS) {
+			const float c = xr[xi(k)] - mean;
+			q = fmaf(c, c, q);
+		}
+		const float rstd = 1.0f / sqrtf(gv_block_sum(q, bred) / float(a.D) + a.eps);
+		const int H = a.taps - 1;
+		float *hb = nullptr;
+		const float *hr = nullptr;
+		float *hw = nullptr;
+		int pos = 0;
+		if (PRO == GV_LN_CONV) {
+			pos = a.d.seg_pos[seg];
+			hb = a.hist + size_t(a.d.seg_seq[seg]) * 2 * H * a.D;
+			hr = hb + size_t(a.d.seg_par[seg]) * H * a.D;
+			hw = hb + size_t(a.d.seg_par[seg] ^ 1) * H * a.D;
+		}
+		for (int k = tid; k < 8 * K8; k += GV_THREADS) {
+			float y = 0.0f;
+			if (k < a.D) {
+				const float n = (xr[xi(k)] - mean) * rstd * a.w[k];
+				y = n;
+				if (PRO == GV_LN_CONV) {
+					float c = 0.0f;
+					for (int j = 0; j < H; j++) {
+						const float v = pos - H + j >= 0 ? hr[size_t(j) * a.D + k] : 0.0f;
+						c = fmaf(a.cw[size_t(j) * a.D + k], v, c);
+						if (blockIdx.x == 0 && j > 0) hw[size_t(j - 1) * a.D + k] = v;
+					}
+					y += fmaf(a.cw[size_t(H) * a.D + k], n, c);
+					if (blockIdx.x == 0 && H > 0) hw[size_t(H - 1) * a.D + k] = n;
+				}
+				if (a.norm_out && blockIdx.x == 0) a.norm_out[size_t(r) * a.D + k] = y;
+			}
+			xr[xi(k)] = y;
+		}
+	}
+	__syncthreads();
+
+	// ---------------------------------------------------------------- products
+	int flip = 0;
+	for (int grp = blockIdx.x; grp < groups; grp += gridDim.x, flip ^= 1) {
+		float acc[R][NR] = {};
+		for (int it = 0; it < nit; it++) {
+			if (it + 1 < nit) load(grp, it + 1, nxt);
+			else load(grp + gridDim.x, 0, nxt);
+			const int k8 = (it * KS + ks) * 32 + lane;
+			if (k8 < K8) {
+#pragma unroll
+				for (int r = 0; r < R; r++) {
+					const float4 x0 = *reinterpret_cast<const float4 *>(xs + size_t(r) * 8 * K8 + 4 * k8);
+					const float4 x1 = *reinterpret_cast<const float4 *>(xs + size_t(r) * 8 * K8 + 4 * K8 + 4 * k8);
+#pragma unroll
+					for (int i = 0; i < NR; i++) {
+						float s = acc[r][i];
+						s = fmaf(bf16_lo(cur[i].x), x0.x, s);
+						s = fmaf(bf16_hi(cur[i].x), x0.y, s);
+						s = fmaf(bf16_lo(cur[i].y), x0.z, s);
+						s = fmaf(bf16_hi(cur[i].y), x0.w, s);
+						s = fmaf(bf16_lo(cur[i].z), x1.x, s);
+						s = fmaf(bf16_hi(cur[i].z), x1.y, s);
+						s = fmaf(bf16_lo(cur[i].w), x1.z, s);
+						acc[r][i] = fmaf(bf16_hi(cur[i].w), x1.w, s);
+					}
+				}
+			}
+#pragma unroll
+			for (int i = 0; i < NR; i++) cur[i] = nxt[i];
+		}
+		float *rb = red + flip * 8 * NR * R;
+#pragma unroll
+		for (int i = 0; i < NR; i++)
+#pragma unroll
+			for (int r = 0; r < R; r++) {
+				const float v = warp_sum(acc[r][i]);
+				if (lane == 0) rb[((set * KS + ks) * NR + i) * R + r] = v;
+			}
+		__syncthreads();
+		// one thread per (output, row); the other copy of `red` keeps the next group from overwriting it
+		if (tid < OUTS * R) {
+			const int o = tid / R, r = tid % R, n = grp * OUTS + o;
+			auto sum = [&](int st, int i) {
+				float v = 0.0f;
+#pragma unroll
+				for (int q = 0; q < KS; q++) v += rb[((st * KS + q) * NR + i) * R + r];
+				return v;
+			};
+			if (n < n_out) {
+				float *dst = a.out + size_t(r) * a.ldo + n;
+				if (EPI == GV_GEGLU) {
+					const int st = o / (NR / 2), i = (o % (NR / 2)) * 2;
+					*dst = gelu_tanh(sum(st, i)) * sum(st, i + 1);
+				} else {
+					const float v = sum(o / NR, o % NR);
+					if (EPI == GV_ADD) {
+						float b = a.embed_mode == 1 ? 0.0f : *dst;
+						if (a.embed_mode) b += __bfloat162float(a.embed[size_t(min(max(a.d.tok[r], 0), a.V - 1)) * a.lde + n]);
+						*dst = b + v;
+					} else if (EPI == GV_LOGITS) {
+						*dst = n < a.N ? soft_cap(v, a.cap) : -INFINITY;
+					} else {
+						*dst = v;
+						const bool isk = n >= a.p_k && n < a.p_k + a.n_k, isv = n >= a.p_v && n < a.p_v + a.n_v;
+						if (isk || isv) {
+							const int seg = a.d.row_seg[r], seq = a.d.seg_seq[seg], pos = a.d.seg_pos[seg];
+							const int w = isk ? a.n_k : a.n_v, c = n - (isk ? a.p_k : a.p_v);
+							const size_t ring = (size_t(seq) * a.cap_rows + pos % a.cap_rows) * w + c, first = (size_t(seq) * a.keep_rows + pos) * w + c;
+							void *rp = isk ? a.kc : a.vc, *fp = isk ? a.ks : a.vs;
+							if (a.cache_f32) {
+								reinterpret_cast<float *>(rp)[ring] = v;
+								if (pos < a.keep) reinterpret_cast<float *>(fp)[first] = v;
+							} else {
+								reinterpret_cast<__nv_bfloat16 *>(rp)[ring] = __float2bfloat16_rn(v);
+								if (pos < a.keep) reinterpret_cast<__nv_bfloat16 *>(fp)[first] = __float2bfloat16_rn(v);
+							}
+						}
+					}
+				}
+			}
+		}
+	}
+}
+
+}  // namespace tg

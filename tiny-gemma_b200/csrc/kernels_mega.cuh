@@ -36,6 +36,7 @@
 
 #include "kernels_decode.cuh"
 #include "kernels_sampler.cuh"
+#include "tc_common.cuh"
 #include "tg_common.cuh"
 
 namespace tg {
@@ -134,52 +135,6 @@ struct MgArgs {
 	                 // the cost around without lowering it.
 	int dbg_cap;
 };
-
-// ------------------------------------------------------------------ PTX helpers
-__device__ __forceinline__ uint32_t smem_u32(const void *p) { return uint32_t(__cvta_generic_to_shared(p)); }
-
-__device__ __forceinline__ void mbar_init(uint64_t *bar, int count) {
-	asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(bar)), "r"(count) : "memory");
-}
-__device__ __forceinline__ void mbar_expect_tx(uint64_t *bar, uint32_t bytes) {
-	asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_u32(bar)), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void mbar_arrive(uint64_t *bar) {
-	asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-__device__ __forceinline__ bool mbar_try_wait(uint64_t *bar, uint32_t parity) {
-	uint32_t ok;
-	asm volatile(
-	    "{\n\t.reg .pred p;\n\t"
-	    "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
-	    "selp.u32 %0, 1, 0, p;\n\t}"
-	    : "=r"(ok)
-	    : "r"(smem_u32(bar)), "r"(parity)
-	    : "memory");
-	return ok != 0;
-}
-// 2-D tiled TMA load into this CTA only (never cluster-wide): box at (x = byte column, y = row) -> dst, completes on bar.
-// Weights are read once per token, so they carry an L2 evict-first policy and
-// leave the L2 to the KV cache and the small exchange vectors.
-__device__ __forceinline__ uint64_t l2_evict_first_policy() {
-	uint64_t pol;
-	asm volatile("createpolicy.fractional.L2::evict_first.b64 %0, 1.0;" : "=l"(pol));
-	return pol;
-}
-__device__ __forceinline__ void tma_load_2d(void *dst, const CUtensorMap *map, int x, int y, uint64_t *bar, uint64_t pol) {
-	asm volatile(
-	    "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes.L2::cache_hint [%0], [%1, {%2, %3}], "
-	    "[%4], %5;" ::"r"(smem_u32(dst)),
-	    "l"(map), "r"(x), "r"(y), "r"(smem_u32(bar)), "l"(pol)
-	    : "memory");
-}
-__device__ __forceinline__ void prefetch_l2(const void *p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
-__device__ __forceinline__ void fence_proxy_async() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
-__device__ __forceinline__ unsigned ld_acquire_u32(const unsigned *p) {
-	unsigned v;
-	asm volatile("ld.acquire.gpu.global.u32 %0, [%1];" : "=r"(v) : "l"(p) : "memory");
-	return v;
-}
 
 // Self-validating hand-off ("LL" style): the consumer's buffer is filled with a sentinel that no
 // computation produces (all ones, a NaN the hardware never generates); the producer stores plain

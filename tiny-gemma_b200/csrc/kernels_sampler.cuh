@@ -33,7 +33,7 @@ __device__ __forceinline__ void emit_token(const SampleArgs &a, int b, int tok) 
 
 // ops::argmax_logits, reference ops.hpp:744-760: ascending scan with a strict
 // '>' — the lowest index wins ties, NaN never wins, -1 if nothing exceeds -inf.
-__global__ void __launch_bounds__(SM_THREADS) argmax_kernel(SampleArgs a) {
+static __global__ void __launch_bounds__(SM_THREADS) argmax_kernel(SampleArgs a) {
 	pdl_trigger();
 	pdl_wait();
 	__shared__ float sv[SM_NWARPS];
@@ -302,7 +302,7 @@ __device__ int cdf_cross_block(const float *p, int n, float *cum_io, float randf
 // chunks that the whole CTA stages into shared memory.
 constexpr int MP_CHUNK = 8192;
 
-__global__ void __launch_bounds__(SM_THREADS) minp_kernel(SampleArgs a) {
+static __global__ void __launch_bounds__(SM_THREADS) minp_kernel(SampleArgs a) {
 	__shared__ float red[SM_NWARPS];
 	__shared__ float chunk[MP_CHUNK];
 	__shared__ int scratch[2 * SM_NWARPS + 8];
@@ -430,7 +430,7 @@ __device__ __forceinline__ float sg_block_sum(float v, float *red) {
 }
 
 // part: [2 * G] floats of scratch, probs: [V] floats of scratch, bar: one zeroed word, err: error word
-__global__ void __launch_bounds__(SG_THREADS, 1) minp_grid_kernel(SampleArgs a, unsigned *bar, float *part, float *probs, int *err) {
+static __global__ void __launch_bounds__(SG_THREADS, 1) minp_grid_kernel(SampleArgs a, unsigned *bar, float *part, float *probs, int *err) {
 	__shared__ float red[SG_NWARPS];
 	__shared__ float chunk[MP_CHUNK];
 	__shared__ int scratch[2 * SG_NWARPS + 8];
@@ -537,7 +537,7 @@ __global__ void __launch_bounds__(SG_THREADS, 1) minp_grid_kernel(SampleArgs a, 
 // The inverse-CDF step in isolation over an explicit vector p[0..n) in global memory, starting
 // from the running sum cum0: *idx = first i with fl(cum0 + p[0] + ... + p[i]) >= randf, else -1.
 // One CTA; *cum_out receives the sum after the last element consumed.
-__global__ void __launch_bounds__(SM_THREADS) inverse_cdf_kernel(const float *p, int n, float cum0, float randf, int *idx,
+static __global__ void __launch_bounds__(SM_THREADS) inverse_cdf_kernel(const float *p, int n, float cum0, float randf, int *idx,
                                                                  float *cum_out) {
 	__shared__ float chunk[MP_CHUNK];
 	__shared__ int scratch[2 * SM_NWARPS + 8];

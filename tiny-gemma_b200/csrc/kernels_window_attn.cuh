@@ -1,0 +1,569 @@
+// Causal attention over a sliding window plus the first tokens of a sequence, with an optional per-head distance
+// bias taken off the scores:
+//     score(i, j) = scale * q_i . k_j - r1 ln(1 + r2 (i - j)),     j <= i and (i - j < window or j < keep_first)
+// No rotation; grouped key/value heads; an optional sigmoid output gate.
+//
+// Cache of one layer run, per sequence: a ring of `cap` rows (slot = position mod cap; cap is a multiple of 64 and at
+// least window + rows of a step) and, because the ring forgets them, a copy of the first keep_first rows. A query
+// takes keys within its window from the ring and the others from the copy, so no key is met twice.
+// Rows hold G heads one after the other, each padded to a multiple of 16 elements (dkp, dvp) with zeros.
+//
+//   kv_append_kernel        rows of a step -> cache
+//   window_attn_kernel      portions, CUDA cores: any sizes, fp32 or bf16
+//   window_attn_tc_kernel   portions, bf16 on tcgen05 (dkp, dvp <= 256): 128 queries of one head per CTA
+//   window_attn_token_cta   one token per sequence: a CTA per (sequence, key/value head, run of keys)
+#pragma once
+#include "kernels_gemm_bf16.cuh"
+#include "kernels_rowwise.cuh"
+
+namespace tg {
+
+struct WAttnArgs {
+	StepDesc d;
+	int H, G, dk, dv, dkp, dvp;
+	float scale;
+	int window, keep;      // keep: first tokens that stay visible
+	const float *r1, *r2;  // [H] or null
+	const void *p;         // projections, rows of ldp: q at p_q, k at p_k, v at p_v, gate at p_g (-1: none)
+	int ldp, p_q, p_k, p_v, p_g;
+	void *kc, *vc;         // [B][cap][G*dkp], [B][cap][G*dvp]
+	void *ks, *vs;         // [B][keep_rows][G*dkp], ...: the first tokens
+	int cap, keep_rows;    // keep_rows: keep rounded up to a multiple of 64 (0 if keep = 0)
+	void *out;             // [R] rows of ldo, head h at h*dvp
+	int ldo;
+	float out_scale;
+	// one token per sequence: partial results of the runs of keys
+	float *part;           // [B][G][nsplit][per][dvp + 2]
+	unsigned *tickets;     // [B][G], zero between launches
+	int nsplit;
+	int *err;
+};
+
+template <typename PT, typename CT>
+static __global__ void __launch_bounds__(256) kv_append_kernel(WAttnArgs a) {
+	pdl_trigger();
+	pdl_wait();
+	const int r = blockIdx.x, seg = a.d.row_seg[r], seq = a.d.seg_seq[seg];
+	const int pos = a.d.seg_pos[seg] + r - a.d.seg_row[seg], slot = pos % a.cap;
+	const PT *row = reinterpret_cast<const PT *>(a.p) + size_t(r) * a.ldp;
+	const int nk = a.G * a.dkp, nv = a.G * a.dvp;
+	for (int i = threadIdx.x; i < nk + nv; i += 256) {
+		const bool isk = i < nk;
+		const int c = isk ? i : i - nk, n = isk ? nk : nv;
+		const CT v = from_f32<CT>(to_f32(row[(isk ? a.p_k : a.p_v) + c]));
+		reinterpret_cast<CT *>(isk ? a.kc : a.vc)[(size_t(seq) * a.cap + slot) * n + c] = v;
+		if (pos < a.keep) reinterpret_cast<CT *>(isk ? a.ks : a.vs)[(size_t(seq) * a.keep_rows + pos) * n + c] = v;
+	}
+}
+
+// number of keys a query at position i sees, and key number n -> position
+__device__ __forceinline__ int wa_first(const WAttnArgs &a, int i) { return max(0, i - a.window + 1); }      // first window position
+__device__ __forceinline__ int wa_kept(const WAttnArgs &a, int i) { return min(a.keep, wa_first(a, i)); }    // kept tokens outside the window
+__device__ __forceinline__ float wa_bias(float r1, float r2, int dist) { return r1 * log1pf(r2 * float(dist)); }
+
+// ------------------------------------------------------------------ portions, CUDA cores
+// One warp per (row, head); a lane scores one key of 32, then the lanes own the value dimensions.
+template <typename PT, typename CT>
+static __global__ void __launch_bounds__(128) window_attn_kernel(WAttnArgs a, int R) {
+	pdl_trigger();
+	pdl_wait();
+	extern __shared__ float wa_sm[];
+	const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+	const int item = blockIdx.x * 4 + warp;
+	float *q = wa_sm + warp * (a.dkp + a.dvp), *o = q + a.dkp;
+	if (item >= R * a.H) return;
+	const int r = item / a.H, h = item % a.H, g = h / (a.H / a.G);
+	const int seg = a.d.row_seg[r], seq = a.d.seg_seq[seg], i = a.d.seg_pos[seg] + r - a.d.seg_row[seg];
+	const PT *row = reinterpret_cast<const PT *>(a.p) + size_t(r) * a.ldp;
+	for (int c = lane; c < a.dkp; c += 32) q[c] = to_f32(row[a.p_q + h * a.dkp + c]) * a.scale;
+	for (int c = lane; c < a.dvp; c += 32) o[c] = 0.0f;
+	__syncwarp();
+	const CT *kc = reinterpret_cast<const CT *>(a.kc) + size_t(seq) * a.cap * a.G * a.dkp, *vc = reinterpret_cast<const CT *>(a.vc) + size_t(seq) * a.cap * a.G * a.dvp;
+	const CT *ks = reinterpret_cast<const CT *>(a.ks) + size_t(seq) * a.keep_rows * a.G * a.dkp, *vs = reinterpret_cast<const CT *>(a.vs) + size_t(seq) * a.keep_rows * a.G * a.dvp;
+	const int first = wa_first(a, i), kept = wa_kept(a, i), total = kept + i - first + 1;
+	const float r1 = a.r1 ? a.r1[h] : 0.0f, r2 = a.r2 ? a.r2[h] : 0.0f;
+	float m = -INFINITY, l = 0.0f;
+	for (int n0 = 0; n0 < total; n0 += 32) {
+		const int n = n0 + lane;
+		float s = -INFINITY;
+		if (n < total) {
+			const int j = n < kept ? n : first + n - kept;
+			const CT *k = n < kept ? ks + size_t(j) * a.G * a.dkp + g * a.dkp : kc + size_t(j % a.cap) * a.G * a.dkp + g * a.dkp;
+			s = 0.0f;
+			for (int c = 0; c < a.dk; c++) s = fmaf(q[c], to_f32(k[c]), s);
+			if (a.r1) s -= wa_bias(r1, r2, i - j);
+		}
+		const float mn = fmaxf(m, warp_max(s)), corr = expf(m - mn), p = expf(s - mn);
+		l = l * corr + warp_sum(p);
+		m = mn;
+		for (int c = lane; c < a.dvp; c += 32) o[c] *= corr;
+		const int cnt = min(32, total - n0);
+		for (int e = 0; e < cnt; e++) {
+			const int n2 = n0 + e, j = n2 < kept ? n2 : first + n2 - kept;
+			const CT *v = n2 < kept ? vs + size_t(j) * a.G * a.dvp + g * a.dvp : vc + size_t(j % a.cap) * a.G * a.dvp + g * a.dvp;
+			const float pe = __shfl_sync(0xffffffffu, p, e);
+			for (int c = lane; c < a.dvp; c += 32) o[c] = fmaf(pe, to_f32(v[c]), o[c]);
+		}
+	}
+	PT *out = reinterpret_cast<PT *>(a.out) + size_t(r) * a.ldo + h * a.dvp;
+	const float f = a.out_scale / l;
+	for (int c = lane; c < a.dvp; c += 32) {
+		const float gate = a.p_g >= 0 ? sigmoid_f(to_f32(row[a.p_g + h * a.dvp + c])) : 1.0f;
+		out[c] = from_f32<PT>(c < a.dv ? o[c] * f * gate : 0.0f);
+	}
+}
+
+// ------------------------------------------------------------------ portions, tensor cores
+// Warps 0-3: softmax, a thread per query row. Warp 4: TMA (Q once, then K and V tiles of 64 keys through one ring).
+// Warp 5: issues the MMAs in the order QK(t+1), PV(t), with S double-buffered in TMEM. P goes through shared memory
+// (one buffer: P(t+1) waits for PV(t)); O stays in TMEM and is rescaled there only when a row's running maximum has
+// grown by more than 8 (powers of two), the sums staying exact for any reference maximum.
+constexpr int WT_THREADS = 192, WT_KEYS = 64;
+struct WtShape {
+	int q_bytes, k_bytes, v_bytes, stage, ns, p_off, total;
+};
+__host__ __device__ inline int wt_chunks(int d) { return (d + 63) / 64; }
+__host__ __device__ inline WtShape wt_shape(int dkp, int dvp) {
+	WtShape s;
+	s.q_bytes = wt_chunks(dkp) * 128 * 128;
+	s.k_bytes = wt_chunks(dkp) * WT_KEYS * 128;
+	s.v_bytes = wt_chunks(dvp) * WT_KEYS * 128;
+	s.stage = s.k_bytes > s.v_bytes ? s.k_bytes : s.v_bytes;
+	const int p = 128 * 128;
+	// two CTAs per SM where three stages allow it, else as deep as one CTA's shared memory goes (at most 4)
+	s.ns = 3;
+	if (s.q_bytes + p + 3 * s.stage + 1024 > 110 * 1024) {
+		s.ns = 4;
+		while (s.ns > 2 && s.q_bytes + p + s.ns * s.stage + 1024 > 220 * 1024) s.ns--;
+	}
+	s.p_off = s.q_bytes + s.ns * s.stage;
+	s.total = s.p_off + p + 1024;
+	return s;
+}
+__host__ __device__ inline int wt_tmem_cols(int dvp) { return dvp <= 128 ? 256 : 512; }  // O, then two S buffers of 64
+
+static __global__ void __launch_bounds__(WT_THREADS) window_attn_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap kmap,
+                                                                           const __grid_constant__ CUtensorMap vmap, const __grid_constant__ CUtensorMap ksmap,
+                                                                           const __grid_constant__ CUtensorMap vsmap, WAttnArgs a) {
+	pdl_trigger();
+	extern __shared__ uint8_t wt_raw[];
+	uint8_t *smem = reinterpret_cast<uint8_t *>((uintptr_t(wt_raw) + 1023) & ~uintptr_t(1023));
+	__shared__ uint64_t q_bar, full_bar[4], free_bar[4], s_bar[2], p_bar, pv_bar;
+	__shared__ uint32_t tmem_base_s;
+	__shared__ int s_fail, s_issued;
+	__shared__ float s_bias[2][192];
+	const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+	const WtShape sh = wt_shape(a.dkp, a.dvp);
+	const int ncols = wt_tmem_cols(a.dvp);
+	if (tid == 0) {
+		mbar_init(&q_bar, 1);
+		for (int i = 0; i < 4; i++) {
+			mbar_init(&full_bar[i], 1);
+			mbar_init(&free_bar[i], 1);
+		}
+		mbar_init(&s_bar[0], 1);
+		mbar_init(&s_bar[1], 1);
+		mbar_init(&p_bar, 4);
+		mbar_init(&pv_bar, 1);
+		s_fail = 0;
+		s_issued = 0;
+		asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+	}
+	if (warp == 5) {
+		asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_base_s)), "r"(ncols) : "memory");
+		asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+	}
+	tc_fence_before();
+	__syncthreads();
+	tc_fence_after();
+	const uint32_t tmem = tmem_base_s;
+	const uint32_t s_off = uint32_t(ncols - 128);
+	pdl_wait();
+
+	const int seg = blockIdx.z, h = blockIdx.y, g = h / (a.H / a.G);
+	const int len = a.d.seg_len[seg], row0 = a.d.seg_row[seg], pos = a.d.seg_pos[seg], seq = a.d.seg_seq[seg];
+	// the last query tiles have the most keys: they start first
+	const int qt = (len + 127) / 128 - 1 - int(blockIdx.x);
+	if (qt >= 0) {
+		const int nq = min(128, len - qt * 128), i_lo = pos + qt * 128, i_hi = i_lo + nq - 1;
+		// key tiles: of the kept first tokens (those outside the first query's .. last query's window), then of the ring
+		const int kept = wa_kept(a, i_hi), nkept = (kept + WT_KEYS - 1) / WT_KEYS;
+		const int j_first = wa_first(a, i_lo) / WT_KEYS, nring = i_hi / WT_KEYS - j_first + 1;
+		const int ntile = nkept + nring;
+		const int kch = wt_chunks(a.dkp), vch = wt_chunks(a.dvp);
+		auto stage = [&](int n) { return smem + sh.q_bytes + (n % sh.ns) * sh.stage; };
+
+		if (warp == 4) {
+			if (lane == 0) {
+				mbar_expect_tx(&q_bar, uint32_t(sh.q_bytes));
+				for (int c = 0; c < kch; c++) tma_load_2d(smem + c * 128 * 128, &qmap, a.p_q + h * a.dkp + 64 * c, row0 + qt * 128, &q_bar);
+				// load n: K of tile n/2 (even n) or V (odd n)
+				for (int n = 0; n < 2 * ntile; n++) {
+					const int s = n % sh.ns, use = n / sh.ns, t = n >> 1;
+					if (use > 0 && !tc_wait(&free_bar[s], (use - 1) & 1, a.err)) {
+						s_fail = 1;
+						break;
+					}
+					const bool isv = n & 1, ks = t < nkept;
+					const int y = ks ? seq * a.keep_rows + t * WT_KEYS : seq * a.cap + ((j_first + t - nkept) * WT_KEYS) % a.cap;
+					mbar_expect_tx(&full_bar[s], uint32_t(isv ? sh.v_bytes : sh.k_bytes));
+					const CUtensorMap *m = isv ? (ks ? &vsmap : &vmap) : (ks ? &ksmap : &kmap);
+					for (int c = 0; c < (isv ? vch : kch); c++)
+						tma_load_2d(stage(n) + c * WT_KEYS * 128, m, g * (isv ? a.dvp : a.dkp) + 64 * c, y, &full_bar[s]);
+					s_issued = n + 1;
+				}
+			}
+		} else if (warp == 5) {
+			if (lane == 0) {
+				const uint32_t id_s = tc_idesc_bf16(WT_KEYS, 0), id_o = tc_idesc_bf16(a.dvp, 1);
+				auto qk = [&](int t) -> bool {
+					const int n = 2 * t;
+					if (!tc_wait(&full_bar[n % sh.ns], (n / sh.ns) & 1, a.err)) return false;
+					tc_fence_after();
+					const uint32_t qa = smem_u32(smem), ka = smem_u32(stage(n));
+					for (int j = 0; j < a.dkp / 16; j++)
+						tc_mma(tmem + s_off + uint32_t((t & 1) * 64), tc_sw128_desc(qa + (j >> 2) * 128 * 128 + (j & 3) * 32, 16, 1024),
+						       tc_sw128_desc(ka + (j >> 2) * WT_KEYS * 128 + (j & 3) * 32, 16, 1024), id_s, j > 0 ? 1u : 0u);
+					tc_commit(&free_bar[n % sh.ns]);
+					tc_commit(&s_bar[t & 1]);
+					return true;
+				};
+				bool ok = tc_wait(&q_bar, 0, a.err) && qk(0);
+				for (int t = 0; t < ntile && ok; t++) {
+					// S buffer (t+1)&1 was read by the softmax of tile t-1 before it arrived on p_bar for that tile
+					if (t + 1 < ntile) ok = qk(t + 1);
+					const int n = 2 * t + 1;
+					ok = ok && tc_wait(&p_bar, t & 1, a.err) && tc_wait(&full_bar[n % sh.ns], (n / sh.ns) & 1, a.err);
+					if (!ok) break;
+					tc_fence_after();
+					const uint32_t pa = smem_u32(smem + sh.p_off), va = smem_u32(stage(n));
+					for (int j = 0; j < WT_KEYS / 16; j++)
+						tc_mma(tmem, tc_sw128_desc(pa + j * 32, 16, 1024), tc_sw128_desc(va + j * 2048, WT_KEYS * 128, 1024), id_o, (t > 0 || j > 0) ? 1u : 0u);
+					tc_commit(&free_bar[n % sh.ns]);
+					tc_commit(&pv_bar);
+				}
+				if (!ok) s_fail = 1;
+			}
+		} else {
+			const int i = i_lo + tid;  // this thread's query (rows past nq compute and are not stored)
+			const uint32_t lane_addr = uint32_t(warp * 32) << 16;
+			const float LOG2E = 1.4426950408889634f;
+			const float sc = a.scale * LOG2E;
+			const float r1 = a.r1 ? a.r1[h] : 0.0f, r2 = a.r1 ? a.r2[h] : 0.0f;
+			float m = -INFINITY, l = 0.0f;
+			// A wait that runs out leaves the warp "dead": it keeps meeting the others at the named barrier below, so
+			// that nobody waits there for good, and does nothing else.
+			bool ok = true;
+			auto wait = [&](uint64_t *bar, int parity) {
+				return __all_sync(0xffffffffu, !*(volatile int *)&s_fail && tc_wait(bar, uint32_t(parity), a.err)) != 0;
+			};
+			for (int t = 0; t < ntile; t++) {
+				const bool ks = t < nkept;
+				const int j0 = ks ? t * WT_KEYS : (j_first + t - nkept) * WT_KEYS;
+				// bias of distance i_lo - j0 - 63 + x, x = 0 .. 190: thread tid meets key c at x = tid + 63 - c
+				if (a.r1) {
+#pragma unroll
+					for (int q = 0; q < 2; q++) {
+						const int x = tid + 128 * q;
+						if (x < 191) s_bias[t & 1][x] = r1 * __log2f(1.0f + r2 * float(max(0, i_lo - j0 - 63 + x)));
+					}
+					asm volatile("bar.sync 1, 128;" ::: "memory");
+				}
+				if (ok && !wait(&s_bar[t & 1], (t >> 1) & 1)) ok = false;
+				if (!ok) {
+					s_fail = 1;
+					continue;
+				}
+				tc_fence_after();
+				uint32_t r[64];
+				{
+					uint32_t (&ra)[32] = *reinterpret_cast<uint32_t (*)[32]>(&r[0]);
+					uint32_t (&rb)[32] = *reinterpret_cast<uint32_t (*)[32]>(&r[32]);
+					tc_ld32(tmem + lane_addr + s_off + uint32_t((t & 1) * 64), ra);
+					tc_ld32(tmem + lane_addr + s_off + uint32_t((t & 1) * 64 + 32), rb);
+					asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+				}
+				const float *bias = s_bias[t & 1] + tid + 63;
+				float mx = -INFINITY;
+				// every query of the tile sees every key of it?
+				const bool whole = !ks && j0 + WT_KEYS - 1 <= i_lo && (i_lo + 127) - j0 < a.window;
+				if (whole) {
+#pragma unroll
+					for (int c = 0; c < 64; c++) {
+						float s = __uint_as_float(r[c]) * sc;
+						if (a.r1) s -= bias[-c];
+						r[c] = __float_as_uint(s);
+						mx = fmaxf(mx, s);
+					}
+				} else {
+					// the ring holds a query's window, the copy the kept tokens before it
+					const int lo = ks ? 0 : wa_first(a, i), hi = ks ? wa_kept(a, i) - 1 : i;
+#pragma unroll
+					for (int c = 0; c < 64; c++) {
+						float s = __uint_as_float(r[c]) * sc;
+						if (a.r1) s -= bias[-c];
+						s = (j0 + c >= lo && j0 + c <= hi) ? s : -INFINITY;
+						r[c] = __float_as_uint(s);
+						mx = fmaxf(mx, s);
+					}
+				}
+				// P and O may be touched once PV(t-1) is complete
+				if (t > 0 && !wait(&pv_bar, (t - 1) & 1)) {
+					ok = false;
+					s_fail = 1;
+					continue;
+				}
+				tc_fence_after();
+				const bool first = m == -INFINITY;
+				bool grow = mx > m + 8.0f || (first && mx > -INFINITY);
+				const float mn = grow ? mx : m;
+				const float corr = first ? 0.0f : exp2f(m - mn);
+				if (t > 0 && __any_sync(0xffffffffu, grow && !first)) {  // (the whole warp: TMEM accesses are warp-wide)
+					const float f = (grow && !first) ? corr : 1.0f;
+					for (int c = 0; c < a.dvp; c += 16) {
+						uint32_t o[16];
+						asm volatile(
+						    "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+						    : "=r"(o[0]), "=r"(o[1]), "=r"(o[2]), "=r"(o[3]), "=r"(o[4]), "=r"(o[5]), "=r"(o[6]), "=r"(o[7]), "=r"(o[8]), "=r"(o[9]),
+						      "=r"(o[10]), "=r"(o[11]), "=r"(o[12]), "=r"(o[13]), "=r"(o[14]), "=r"(o[15])
+						    : "r"(tmem + lane_addr + uint32_t(c))
+						    : "memory");
+						asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+#pragma unroll
+						for (int q = 0; q < 16; q++) o[q] = __float_as_uint(__uint_as_float(o[q]) * f);
+						asm volatile(
+						    "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};" ::"r"(tmem + lane_addr + uint32_t(c)),
+						    "r"(o[0]), "r"(o[1]), "r"(o[2]), "r"(o[3]), "r"(o[4]), "r"(o[5]), "r"(o[6]), "r"(o[7]), "r"(o[8]), "r"(o[9]), "r"(o[10]), "r"(o[11]),
+						    "r"(o[12]), "r"(o[13]), "r"(o[14]), "r"(o[15])
+						    : "memory");
+					}
+					asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+				}
+				l *= corr;
+				m = mn;
+				const float ms = m == -INFINITY ? 0.0f : m;
+				uint8_t *prow = smem + sh.p_off + tid * 128;
+#pragma unroll
+				for (int c8 = 0; c8 < 8; c8++) {
+					uint32_t w[4];
+#pragma unroll
+					for (int q = 0; q < 4; q++) {
+						const float p0 = exp2f(__uint_as_float(r[8 * c8 + 2 * q]) - ms), p1 = exp2f(__uint_as_float(r[8 * c8 + 2 * q + 1]) - ms);
+						l += p0 + p1;
+						w[q] = pack_bf16(p0, p1);
+					}
+					*reinterpret_cast<uint4 *>(prow + ((c8 ^ (tid & 7)) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
+				}
+				fence_proxy_async();
+				tc_fence_before();
+				__syncwarp();
+				if (lane == 0) mbar_arrive(&p_bar);
+			}
+			if (ok) ok = wait(&pv_bar, (ntile - 1) & 1);
+			if (!ok) s_fail = 1;
+			if (ok) {
+				tc_fence_after();
+				const float f = a.out_scale / l;
+				const int r = row0 + qt * 128 + tid;
+				const __nv_bfloat16 *gate = reinterpret_cast<const __nv_bfloat16 *>(a.p) + size_t(r) * a.ldp + a.p_g + h * a.dvp;
+				__nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(a.out) + size_t(r) * a.ldo + h * a.dvp;
+				for (int c = 0; c < a.dvp; c += 16) {
+					uint32_t o[16];
+					asm volatile(
+					    "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+					    : "=r"(o[0]), "=r"(o[1]), "=r"(o[2]), "=r"(o[3]), "=r"(o[4]), "=r"(o[5]), "=r"(o[6]), "=r"(o[7]), "=r"(o[8]), "=r"(o[9]), "=r"(o[10]),
+					      "=r"(o[11]), "=r"(o[12]), "=r"(o[13]), "=r"(o[14]), "=r"(o[15])
+					    : "r"(tmem + lane_addr + uint32_t(c))
+					    : "memory");
+					asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+					if (tid < nq) {
+						uint4 gv[2] = {};
+						if (a.p_g >= 0) {
+							gv[0] = *reinterpret_cast<const uint4 *>(gate + c);
+							gv[1] = *reinterpret_cast<const uint4 *>(gate + c + 8);
+						}
+						const uint32_t *gw = reinterpret_cast<const uint32_t *>(gv);
+						uint32_t w[8];
+#pragma unroll
+						for (int q = 0; q < 8; q++) {
+							float x = __uint_as_float(o[2 * q]) * f, y = __uint_as_float(o[2 * q + 1]) * f;
+							if (a.p_g >= 0) {
+								x *= 1.0f / (1.0f + __expf(-bf16_lo(gw[q])));
+								y *= 1.0f / (1.0f + __expf(-bf16_hi(gw[q])));
+							}
+							w[q] = pack_bf16(x, y);
+						}
+						*reinterpret_cast<uint4 *>(out + c) = make_uint4(w[0], w[1], w[2], w[3]);
+						*reinterpret_cast<uint4 *>(out + c + 8) = make_uint4(w[4], w[5], w[6], w[7]);
+					}
+				}
+			}
+		}
+	}
+	tc_fence_before();
+	__syncthreads();
+	if (s_fail && tid == 0) {
+		const int last = *(volatile int *)&s_issued;
+		for (int n = max(0, last - sh.ns); n < last; n++) tc_wait(&full_bar[n % sh.ns], (n / sh.ns) & 1, a.err);
+	}
+	__syncthreads();
+	tc_fence_after();
+	if (warp == 5) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(ncols));
+}
+
+// ------------------------------------------------------------------ one token per sequence
+// 256 threads; row r of the step is a segment of length 1 whose key and value are already in the cache. The run
+// `split` of WK_KEYS-key pieces is scored for all the query heads of key/value head g; the CTA that arrives last
+// merges the runs, applies the gate and writes the heads' rows.
+constexpr int WK_KEYS = 64;
+__host__ __device__ inline size_t wattn_token_smem(int per, int dkp, int dvp) {
+	return (size_t(per) * dkp + size_t(per) * WK_KEYS + size_t(8) * dvp + 2 * per + 8) * 4;
+}
+template <typename PT, typename CT, typename OT>
+__device__ void window_attn_token_cta(const WAttnArgs &a, int r, int g, int split, float *sm) {
+	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+	const int per = a.H / a.G, dkp = a.dkp, dvp = a.dvp;
+	float *q = sm, *p = q + per * dkp, *acc = p + per * WK_KEYS, *ml = acc + 8 * dvp;
+	__shared__ int s_last;
+	const int seg = a.d.row_seg[r], seq = a.d.seg_seq[seg], i = a.d.seg_pos[seg];
+	const PT *row = reinterpret_cast<const PT *>(a.p) + size_t(r) * a.ldp;
+	const CT *kc = reinterpret_cast<const CT *>(a.kc) + size_t(seq) * a.cap * a.G * dkp + g * dkp, *vc = reinterpret_cast<const CT *>(a.vc) + size_t(seq) * a.cap * a.G * dvp + g * dvp;
+	const CT *ks = reinterpret_cast<const CT *>(a.ks) + size_t(seq) * a.keep_rows * a.G * dkp + g * dkp, *vs = reinterpret_cast<const CT *>(a.vs) + size_t(seq) * a.keep_rows * a.G * dvp + g * dvp;
+	const int first = wa_first(a, i), kept = wa_kept(a, i), total = kept + i - first + 1;
+	const int pieces = (total + WK_KEYS - 1) / WK_KEYS, share = (pieces + a.nsplit - 1) / a.nsplit;
+	const int n_lo = split * share * WK_KEYS, n_hi = min(total, (split + 1) * share * WK_KEYS);
+	for (int x = tid; x < per * dkp; x += 256) q[x] = to_f32(row[a.p_q + g * per * dkp + x]) * a.scale;
+	if (tid < per) {
+		ml[2 * tid] = -INFINITY;
+		ml[2 * tid + 1] = 0.0f;
+	}
+	float *part = a.part + ((size_t(r) * a.G + g) * a.nsplit + split) * per * (dvp + 2);
+	__syncthreads();
+	constexpr int V4 = 16 / int(sizeof(CT));  // elements of a 16-byte load
+	for (int n0 = n_lo; n0 < n_hi; n0 += WK_KEYS) {
+		// scores: four lanes per key
+		{
+			const int n = n0 + (tid >> 2), sub = tid & 3;
+			const bool on = n < n_hi;
+			const int j = on ? (n < kept ? n : first + n - kept) : i;
+			const CT *k = (on && n < kept) ? ks + size_t(j) * a.G * dkp : kc + size_t(j % a.cap) * a.G * dkp;
+			for (int hh = 0; hh < per; hh += 4) {
+				float s[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+				const int nh = min(4, per - hh);
+				for (int c = sub * V4; c < dkp; c += 4 * V4) {
+					const uint4 u = *reinterpret_cast<const uint4 *>(k + c);
+					float kv[V4];
+					if (sizeof(CT) == 2) {
+						const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+						for (int e = 0; e < V4 / 2; e++) {
+							kv[2 * e] = bf16_lo(w[e]);
+							kv[2 * e + 1] = bf16_hi(w[e]);
+						}
+					} else {
+						kv[0] = __uint_as_float(u.x); kv[1] = __uint_as_float(u.y); kv[2] = __uint_as_float(u.z); kv[3] = __uint_as_float(u.w);
+					}
+#pragma unroll
+					for (int y = 0; y < 4; y++)
+						if (y < nh) {
+							const float *qh = q + (hh + y) * dkp + c;
+#pragma unroll
+							for (int e = 0; e < V4; e++) s[y] = fmaf(qh[e], kv[e], s[y]);
+						}
+				}
+#pragma unroll
+				for (int y = 0; y < 4; y++) {
+					s[y] += __shfl_xor_sync(0xffffffffu, s[y], 1);
+					s[y] += __shfl_xor_sync(0xffffffffu, s[y], 2);
+				}
+				if (sub < nh) {
+					float v = sub == 0 ? s[0] : (sub == 1 ? s[1] : (sub == 2 ? s[2] : s[3]));
+					const int h = g * per + hh + sub;
+					if (a.r1) v -= wa_bias(a.r1[h], a.r2[h], i - j);
+					p[(hh + sub) * WK_KEYS + (tid >> 2)] = on ? v : -INFINITY;
+				}
+			}
+		}
+		__syncthreads();
+		// values: a head at a time; the warps take keys, the lanes value dimensions (16 bytes each), then the warps meet
+		for (int hh = 0; hh < per; hh++) {
+			const float s0 = p[hh * WK_KEYS + lane], s1 = p[hh * WK_KEYS + 32 + lane];
+			const float mo = ml[2 * hh], mn = fmaxf(mo, warp_max(fmaxf(s0, s1)));
+			const float p0 = expf(s0 - mn), p1 = expf(s1 - mn), sum = warp_sum(p0 + p1), corr = expf(mo - mn);
+			for (int c0 = 0; c0 < dvp; c0 += 32 * V4) {
+				const int c = c0 + lane * V4;
+				float o[V4] = {};
+				for (int e = warp; e < WK_KEYS && n0 + e < n_hi; e += 8) {
+					const float pe = __shfl_sync(0xffffffffu, e < 32 ? p0 : p1, e & 31);
+					const int n = n0 + e, j = n < kept ? n : first + n - kept;
+					const CT *v = n < kept ? vs + size_t(j) * a.G * dvp : vc + size_t(j % a.cap) * a.G * dvp;
+					if (c < dvp) {
+						const uint4 u = *reinterpret_cast<const uint4 *>(v + c);
+						if (sizeof(CT) == 2) {
+							const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+							for (int z = 0; z < V4 / 2; z++) {
+								o[2 * z] = fmaf(pe, bf16_lo(w[z]), o[2 * z]);
+								o[2 * z + 1] = fmaf(pe, bf16_hi(w[z]), o[2 * z + 1]);
+							}
+						} else {
+							o[0] = fmaf(pe, __uint_as_float(u.x), o[0]); o[1] = fmaf(pe, __uint_as_float(u.y), o[1]);
+							o[2] = fmaf(pe, __uint_as_float(u.z), o[2]); o[3] = fmaf(pe, __uint_as_float(u.w), o[3]);
+						}
+					}
+				}
+				if (c < dvp)
+#pragma unroll
+					for (int z = 0; z < V4; z++) acc[warp * dvp + c + z] = o[z];
+			}
+			__syncthreads();
+			for (int c = tid; c < dvp; c += 256) {
+				float o = 0.0f;
+#pragma unroll
+				for (int w = 0; w < 8; w++) o += acc[w * dvp + c];
+				float *dst = part + hh * (dvp + 2) + c;
+				*dst = n0 == n_lo ? o : fmaf(*dst, corr, o);
+			}
+			if (tid == 0) {
+				ml[2 * hh] = mn;
+				ml[2 * hh + 1] = ml[2 * hh + 1] * corr + sum;
+			}
+			__syncthreads();
+		}
+	}
+	if (tid < per) {
+		part[tid * (dvp + 2) + dvp] = ml[2 * tid];
+		part[tid * (dvp + 2) + dvp + 1] = ml[2 * tid + 1];
+	}
+	__threadfence();
+	__syncthreads();
+	if (a.nsplit > 1) {
+		if (tid == 0) {
+			const unsigned old = atomicAdd(a.tickets + size_t(r) * a.G + g, 1u);
+			s_last = old == unsigned(a.nsplit - 1);
+			if (s_last) a.tickets[size_t(r) * a.G + g] = 0;
+		}
+		__syncthreads();
+		if (!s_last) return;
+		__threadfence();
+	}
+	const float *all = a.part + (size_t(r) * a.G + g) * a.nsplit * per * (dvp + 2);
+	for (int x = tid; x < per * dvp; x += 256) {
+		const int hh = x / dvp, c = x % dvp, h = g * per + hh;
+		float m = -INFINITY;
+		for (int s = 0; s < a.nsplit; s++) m = fmaxf(m, __ldcg(all + (size_t(s) * per + hh) * (dvp + 2) + dvp));
+		float o = 0.0f, l = 0.0f;
+		for (int s = 0; s < a.nsplit; s++) {
+			const float *ps = all + (size_t(s) * per + hh) * (dvp + 2);
+			const float ms = __ldcg(ps + dvp);
+			if (ms == -INFINITY) continue;  // a run without keys
+			const float w = expf(ms - m);
+			o = fmaf(w, __ldcg(ps + c), o);
+			l = fmaf(w, __ldcg(ps + dvp + 1), l);
+		}
+		const float gate = a.p_g >= 0 ? sigmoid_f(to_f32(row[a.p_g + h * dvp + c])) : 1.0f;
+		reinterpret_cast<OT *>(a.out)[size_t(r) * a.ldo + h * dvp + c] = from_f32<OT>(c < a.dv ? o / l * gate * a.out_scale : 0.0f);
+	}
+}
+
+}  // namespace tg

@@ -1,21 +1,16 @@
-// libtinygemma_b200: host-side engine and the extern "C" boundary declared in
-// include/tiny_gemma_b200.h. Owns the device weight store (gemma_i8.bin bytes
-// unchanged in HBM), the per-state KV caches and scratch, the launch plans and
-// the CUDA graph of one decode step.
+// The int8 Gemma-3 family: its model and state behind the C ABI of include/tiny_gemma_b200.h. Owns the device
+// weight store (gemma_i8.bin bytes unchanged in HBM), the per-state KV caches and scratch and the launch plans.
 #include <cuda_runtime.h>
 
 #include <algorithm>
-#include <atomic>
 #include <climits>
 #include <cmath>
 #include <cstdio>
-#include <cstdlib>
 #include <cstring>
 #include <ctime>
 #include <string>
 #include <vector>
 
-#include "../../include/tiny_gemma_b200.h"
 #include "kernels_decode.cuh"
 #include "kernels_mega.cuh"
 #include "kernels_persist.cuh"
@@ -23,81 +18,9 @@
 #include "kernels_attn_tc.cuh"
 #include "kernels_prefill.cuh"
 #include "kernels_sampler.cuh"
+#include "tg_internal.hpp"
 
 using namespace tg;
-
-// ===================================================================== errors
-namespace {
-
-thread_local std::string g_err;
-std::atomic<long long> g_launches{0};
-
-int fail(int code, const std::string &msg) {
-	g_err = msg;
-	return code;
-}
-
-#define TG_CUDA(call)                                                                                   \
-	do {                                                                                                \
-		cudaError_t e__ = (call);                                                                       \
-		if (e__ != cudaSuccess)                                                                         \
-			return fail(TG_ECUDA, std::string(#call) + ": " + cudaGetErrorString(e__));                 \
-	} while (0)
-
-#define TG_TRY(call)                \
-	do {                            \
-		int rc__ = (call);          \
-		if (rc__ != TG_OK) return rc__; \
-	} while (0)
-
-inline void count_launch(int n = 1) { g_launches.fetch_add(n, std::memory_order_relaxed); }
-
-int check_launch(const char *what) {
-	cudaError_t e = cudaGetLastError();
-	if (e != cudaSuccess) return fail(TG_ECUDA, std::string(what) + " launch: " + cudaGetErrorString(e));
-	return TG_OK;
-}
-
-// tunables (set through the environment for experiments; defaults are the tuned values)
-int env_int(const char *name, int dflt) {
-	const char *v = std::getenv(name);
-	return v ? std::atoi(v) : dflt;
-}
-
-int g_num_sms = 148;
-
-// cudaFuncSetAttribute is per device: "configured once" flags are kept per device index
-constexpr int TG_MAX_DEVICES = 64;
-// Launch with the programmatic-serialization attribute (see pdl_wait in tg_common.cuh): only for kernels that
-// call pdl_wait() before their first global access. TG_PDL=0 launches them as ordinary stream-ordered kernels.
-// The batched decode step switches it off for its own launches (g_pdl_scope_off): replayed from a CUDA graph the
-// step gains nothing from it (measured 3.72 ms with ordinary edges, 3.78 ms with programmatic ones at 256
-// sequences), while the eagerly launched prefill does (178 tokens: 4.00 -> 3.80 ms).
-thread_local bool g_pdl_scope_off = false;
-template <typename... KArgs, typename... Args>
-inline void launch_k(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t st, Args &&...args) {
-	static const int use_env = env_int("TG_PDL", 1);
-	const int use = use_env && !g_pdl_scope_off;
-	cudaLaunchConfig_t cfg = {};
-	cfg.gridDim = grid;
-	cfg.blockDim = block;
-	cfg.dynamicSmemBytes = smem;
-	cfg.stream = st;
-	cudaLaunchAttribute at[1];
-	at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-	at[0].val.programmaticStreamSerializationAllowed = 1;
-	cfg.attrs = at;
-	cfg.numAttrs = use ? 1 : 0;
-	cudaLaunchKernelEx(&cfg, kernel, std::forward<Args>(args)...);  // errors surface in check_launch (cudaGetLastError)
-}
-
-inline int current_device_slot() {
-	int d = 0;
-	cudaGetDevice(&d);
-	return (d >= 0 && d < TG_MAX_DEVICES) ? d : 0;
-}
-
-}  // namespace
 
 // ===================================================================== model
 struct QW {
@@ -113,9 +36,8 @@ struct LayerW {
 	bool is_local;
 };
 
-struct tg_model {
+struct GemmaModel : tg_model {
 	tg_config cfg;
-	int device = 0;
 	long weights_version = 0;  // bumped by every load
 	// layer weights re-ordered into the persistent decode kernel's per-CTA units (built on first use)
 	int8_t *dec_tiled = nullptr;
@@ -139,6 +61,10 @@ struct tg_model {
 	float gelu_min = -4.0f, gelu_max = 4.0f, gelu_eps = 0.0f;
 	int gelu_size = 0;
 	bool loaded = false;
+
+	~GemmaModel() override;
+	const char *arch() const override { return "Gemma3Int8"; }
+	int new_state(int batch, int max_pos, tg_state **out) override;
 };
 
 namespace {
@@ -152,7 +78,7 @@ size_t model_file_bytes(const tg_config &c) {
 }
 
 // transformer.hpp:99-165 read order; pointers into the device blob
-void bind_model(tg_model *m) {
+void bind_model(GemmaModel *m) {
 	const tg_config &c = m->cfg;
 	const uint8_t *p = m->blob;
 	auto take = [&](size_t n) {
@@ -199,21 +125,6 @@ bool supported_n(int N) {
 	return N == 640 || N == 262144 || N == 2048 || N == 256 || N == 1024 || N == 1152 || N == 6912;
 }
 
-int ensure_device(int device) {
-	int n = 0;
-	cudaError_t e = cudaGetDeviceCount(&n);
-	if (e != cudaSuccess || n == 0) {
-		cudaGetLastError();
-		return fail(TG_ENODEVICE, "no CUDA device available (this library has no CPU path)");
-	}
-	if (device < 0 || device >= n) return fail(TG_EINVAL, "device index out of range");
-	TG_CUDA(cudaSetDevice(device));
-	int sms = 0;
-	if (cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device) == cudaSuccess && sms > 0) g_num_sms = sms;
-	return TG_OK;
-}
-
-// ------------------------------------------------------------- matvec planning
 struct MvPlan {
 	int nsplit, kc, grid_x;
 };
@@ -288,7 +199,6 @@ int launch_mv(MvArgs a, int pro, int epi, cudaStream_t st) {
 }
 
 constexpr int MV_MAX_B = 4;
-constexpr int STEP_RANDF = 64;  // uniforms per sequence that fit the state's step block (more: a buffer of their own)
 
 // Single-wave matvec (qmatvec_cluster_kernel): a [K, N] matrix qualifies when a tile width 16 * tpr and a
 // K-split ks (= cluster size) exist with all CTAs resident at once — one per SM, and no more clusters than
@@ -395,11 +305,8 @@ struct TcScratch {
 };
 
 // ===================================================================== state
-struct tg_state {
-	tg_model *m = nullptr;
-	int B = 1;
-	int max_pos_global = 0;
-	cudaStream_t stream = nullptr;
+struct GemmaState : tg_state {
+	GemmaModel *m = nullptr;
 	// per-layer caches
 	std::vector<float *> kcache, vcache;  // [B][slots][256]
 	std::vector<int> slots;
@@ -409,8 +316,6 @@ struct tg_state {
 	float *attn_out = nullptr;         // [B][qd]
 	float *t = nullptr;                // [B][D]
 	float *act = nullptr;              // [B][I]
-	float *xnorm = nullptr;            // [B][D] final-normed hidden (parity read-back)
-	float *logits = nullptr;           // [B][V]
 	float *partial = nullptr;          // split-K scratch
 	size_t partial_floats = 0;
 	unsigned *tickets = nullptr;       // [max tiles] + [B] for attention
@@ -418,28 +323,11 @@ struct tg_state {
 	float *attn_part = nullptr;        // [B][nsplit_max][1032]
 	int attn_nsplit_local = 16, attn_nsplit_global = 64;
 	int *step_pos = nullptr, *next_pos = nullptr, *ring_base = nullptr;  // [B]
-	int *tok = nullptr;                // [B]
-	int *tok_log = nullptr;            // [log_cap][B]
 	int *force_ids = nullptr;          // [force_cap] tokens of tg_append (batch 1)
 	int force_cap = 0;
-	int log_cap = 0;
-	int *log_count = nullptr;          // [B]
-	float *randf = nullptr;            // [randf_cap][B]
-	int randf_cap = 0;
-	int randf_valid = 0;               // uniforms per sequence uploaded so far (the largest upload)
-	// One allocation holds the small per-step words, so that a step's inputs go up in ONE copy and its
-	// results come back in ONE: [err_flag, 3 pad][tok B][randf_count B][log_count B][randf STEP_RANDF x B]
-	int *step_blk = nullptr;
-	bool randf_in_blk = false;         // randf still points into step_blk (it moves out when it has to grow)
-	float *randf_blk = nullptr;        // the block's own STEP_RANDF x B uniforms
-	bool lean_randf = false;           // the next persistent launch draws from randf_blk (one-token calls)
 	// persistent kernel: its hand-off arena and grid-barrier counter are left ready by the previous launch
 	bool ps_clean = false;             // false: wipe the arena and zero the counter before the next launch
 	unsigned ps_bar_base = 0;          // arrivals at the grid barrier so far
-	int *randf_count = nullptr;        // [B]
-	int *err_flag = nullptr;
-	int *host_pin = nullptr;           // pinned staging, 64 KiB
-	bool staging_busy = false;         // an enqueued copy may still read host_pin (set by the asynchronous tg_decode)
 	// prefill scratch (grow-only)
 	float *pf = nullptr;
 	size_t pf_floats = 0;
@@ -447,12 +335,6 @@ struct tg_state {
 	int pf_ids_cap = 0;
 	// plans
 	MvPlan plan_qkv, plan_o, plan_gu, plan_dn, plan_lm;
-	// decode graph
-	cudaGraphExec_t graph = nullptr;
-	bool use_graph = true;
-	bool warmed = false;
-	int graph_launches = 0;
-	std::vector<int> host_pos;  // mirror of next_pos for call-order checks
 	// batched decode step (tensor-core GEMMs with M = batch)
 	bool batched_ok = false;
 	float *bx = nullptr, *bup = nullptr;  // [B][D] normed input, [B][I] up projection
@@ -477,16 +359,28 @@ struct tg_state {
 	float *ps_ll = nullptr;
 	size_t ps_ll_bytes = 0;
 	size_t mega_smem = 0;
+
+	~GemmaState() override;
+	int ready() override;
+	int reset() override;
+	int prefill(const int *ids, int S, float *logits_host) override;
+	int append(const int *ids, int n, float *logits_host) override;
+	int enqueue_decode_all() override;
+	int enqueue_forward() override;
+	int enqueue_sampler(float minp, float temp, bool log_tokens) override;
+	int run_steps(int n_steps, float minp, float temp) override;
+	bool lean_step() const override { return ps_ok; }
+	int report_err(int flag) override;
 };
 
 namespace {
 
-int state_alloc(tg_state *s) {
-	tg_model *m = s->m;
+int state_alloc(GemmaState *s) {
+	GemmaModel *m = s->m;
 	const tg_config &c = m->cfg;
 	const int B = s->B, D = c.hidden_size, I = c.intermediate_size, V = c.n_vocab;
 	const int qd = c.n_head * c.head_dim, kd = c.n_kv * c.head_dim;
-	TG_CUDA(cudaStreamCreateWithFlags(&s->stream, cudaStreamNonBlocking));
+	TG_TRY(s->alloc_common());
 	s->kcache.resize(c.n_layers);
 	s->vcache.resize(c.n_layers);
 	s->slots.resize(c.n_layers);
@@ -510,8 +404,6 @@ int state_alloc(tg_state *s) {
 	TG_TRY(allocf(&s->attn_out, size_t(B) * qd));
 	TG_TRY(allocf(&s->t, size_t(B) * D));
 	TG_TRY(allocf(&s->act, size_t(B) * I));
-	TG_TRY(allocf(&s->xnorm, size_t(B) * D));
-	TG_TRY(allocf(&s->logits, size_t(B) * V));
 
 	const int target = env_int("TG_MV_TARGET_CTAS", 2 * g_num_sms);
 	s->plan_qkv = plan_matvec(D, (qd + 2 * kd) / MV_TN, target);
@@ -550,25 +442,13 @@ int state_alloc(tg_state *s) {
 	TG_TRY(alloci(&s->step_pos, B));
 	TG_TRY(alloci(&s->next_pos, B));
 	TG_TRY(alloci(&s->ring_base, B));
-	TG_TRY(alloci(&s->step_blk, 4 + size_t(3 + STEP_RANDF) * B));
-	s->err_flag = s->step_blk;
-	s->tok = s->step_blk + 4;
-	s->randf_count = s->tok + B;
-	s->log_count = s->randf_count + B;
-	s->randf_blk = reinterpret_cast<float *>(s->log_count + B);
-	s->randf = s->randf_blk;
-	s->randf_cap = STEP_RANDF;
-	s->randf_in_blk = true;
-	TG_CUDA(cudaMallocHost(&s->host_pin, 64 * 1024));
-	s->host_pos.assign(B, 0);
-	s->use_graph = env_int("TG_USE_GRAPH", 1) != 0;
 	TG_CUDA(cudaStreamSynchronize(s->stream));
 	return TG_OK;
 }
 
-GeluLut make_lut(const tg_model *m) { return GeluLut{m->gelu, m->gelu_min, m->gelu_eps, m->gelu_size}; }
+GeluLut make_lut(const GemmaModel *m) { return GeluLut{m->gelu, m->gelu_min, m->gelu_eps, m->gelu_size}; }
 
-int check_ready(const tg_model *m) {
+int check_ready(const GemmaModel *m) {
 	if (!m->rope[0][0] || !m->rope[1][0] || !m->gelu)
 		return fail(TG_ESTATE, "RoPE / GeLU tables not set (tg_model_set_rope, tg_model_set_gelu_table or tg_model_build_tables)");
 	return TG_OK;
@@ -579,8 +459,8 @@ int check_ready(const tg_model *m) {
 // layer: QKV matvec (norm prologue) -> attention -> O matvec -> gate/up matvec
 // (residual+norm prologue, GeGLU epilogue) -> down matvec; then the lm_head
 // matvec with the last residual+norm prologue.
-int enqueue_decode_chunk(tg_state *s, int b0, int nb, bool with_lm_head = true) {
-	tg_model *m = s->m;
+int enqueue_decode_chunk(GemmaState *s, int b0, int nb, bool with_lm_head = true) {
+	GemmaModel *m = s->m;
 	const tg_config &c = m->cfg;
 	const int D = c.hidden_size, I = c.intermediate_size, V = c.n_vocab;
 	const int qd = c.n_head * c.head_dim, kd = c.n_kv * c.head_dim;
@@ -753,64 +633,11 @@ int enqueue_decode_chunk(tg_state *s, int b0, int nb, bool with_lm_head = true) 
 }
 
 
-int batched_setup(tg_state *s);
-int enqueue_decode_batched(tg_state *s, bool with_lm_head);
+int batched_setup(GemmaState *s);
+int enqueue_decode_batched(GemmaState *s, bool with_lm_head);
 
-
-int enqueue_decode_all(tg_state *s) {
-	if (s->batched_ok) return enqueue_decode_batched(s, true);
-	for (int b0 = 0; b0 < s->B; b0 += MV_MAX_B) TG_TRY(enqueue_decode_chunk(s, b0, std::min(MV_MAX_B, s->B - b0)));
-	return TG_OK;
-}
-
-int enqueue_decode_step(tg_state *s) {
-	// The first step of a state runs eagerly so that lazy module loading and
-	// cudaFuncSetAttribute happen outside stream capture; the graph is captured
-	// on the second step and replayed from then on.
-	if (!s->use_graph || !s->warmed) {
-		s->warmed = true;
-		return enqueue_decode_all(s);
-	}
-	if (!s->graph) {
-		cudaGraph_t g = nullptr;
-		long long before = g_launches.load();
-		TG_CUDA(cudaStreamBeginCapture(s->stream, cudaStreamCaptureModeThreadLocal));
-		int rc = enqueue_decode_all(s);
-		cudaError_t e = cudaStreamEndCapture(s->stream, &g);
-		s->graph_launches = int(g_launches.load() - before);
-		g_launches.store(before);
-		if (rc != TG_OK) {
-			if (g) cudaGraphDestroy(g);
-			return rc;
-		}
-		if (e != cudaSuccess) return fail(TG_ECUDA, std::string("cudaStreamEndCapture: ") + cudaGetErrorString(e));
-		e = cudaGraphInstantiate(&s->graph, g, 0);
-		cudaGraphDestroy(g);
-		if (e != cudaSuccess) return fail(TG_ECUDA, std::string("cudaGraphInstantiate: ") + cudaGetErrorString(e));
-	}
-	TG_CUDA(cudaGraphLaunch(s->graph, s->stream));
-	count_launch(s->graph_launches);
-	return TG_OK;
-}
 
 // ------------------------------------------------------------- persistent kernel set-up
-typedef CUresult (*PFN_encodeTiled)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *,
-                                    const cuuint64_t *, const cuuint32_t *, const cuuint32_t *, CUtensorMapInterleave,
-                                    CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-PFN_encodeTiled get_encode_fn() {
-	static PFN_encodeTiled fn = nullptr;
-	if (!fn) {
-		void *p = nullptr;
-		cudaDriverEntryPointQueryResult q;
-		if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q) == cudaSuccess &&
-		    q == cudaDriverEntryPointSuccess)
-			fn = reinterpret_cast<PFN_encodeTiled>(p);
-	}
-	return fn;
-}
-
-// 2-D uint8 map over a row-major [K, N] int8 matrix; box = TN bytes x box_rows rows, no swizzle
 int make_tmap(CUtensorMap *out, const int8_t *base, int K, int N, int TN, int box_rows, int ld = 0) {
 	PFN_encodeTiled enc = get_encode_fn();
 	if (!enc) return fail(TG_ECUDA, "cuTensorMapEncodeTiled entry point not available");
@@ -877,8 +704,8 @@ bool plan_phase(MgPhase *out, int K, const std::vector<int> &n_cols, int nmat, b
 	return best_score >= 0;
 }
 
-int mega_setup(tg_state *s) {
-	tg_model *m = s->m;
+int mega_setup(GemmaState *s) {
+	GemmaModel *m = s->m;
 	const tg_config &c = m->cfg;
 	const int D = c.hidden_size, I = c.intermediate_size, V = c.n_vocab, L = c.n_layers;
 	const int qd = c.n_head * c.head_dim, kd = c.n_kv * c.head_dim;
@@ -1032,8 +859,8 @@ int mega_setup(tg_state *s) {
 // order: for every layer the units of phase A (q|k|v column tiles x K-splits), C (O projection),
 // D (up tile followed by the gate tile of the same columns) and E (down projection), each unit a
 // contiguous [rows][TN] block, so that a CTA fetches its unit with sequential bulk copies.
-int ensure_decode_tiles(tg_state *s) {
-	tg_model *m = s->m;
+int ensure_decode_tiles(GemmaState *s) {
+	GemmaModel *m = s->m;
 	const MgArgs &a = s->mega;
 	const tg_config &c = m->cfg;
 	const int L = c.n_layers, D = c.hidden_size, I = c.intermediate_size;
@@ -1105,8 +932,8 @@ bool ps_plan(PsPhase *out, int K, int N, int nmat, int G, int max_bytes, const s
 	return best < 1e30;
 }
 
-int persist_setup(tg_state *s) {
-	tg_model *m = s->m;
+int persist_setup(GemmaState *s) {
+	GemmaModel *m = s->m;
 	const tg_config &c = m->cfg;
 	const int D = c.hidden_size, I = c.intermediate_size, V = c.n_vocab, L = c.n_layers;
 	const int qd = c.n_head * c.head_dim, kd = c.n_kv * c.head_dim;
@@ -1260,8 +1087,8 @@ int persist_setup(tg_state *s) {
 // Build (or refresh after a reload of the weights) the model's copies in the kernel's unit order:
 // per layer the units of phase A (q|k|v), C (O projection), D (up pieces followed by the gate pieces of
 // the same columns) and E (down projection), and the lm_head in ring-stage order.
-int ensure_persist_tiles(tg_state *s) {
-	tg_model *m = s->m;
+int ensure_persist_tiles(GemmaState *s) {
+	GemmaModel *m = s->m;
 	const PsArgs &a = s->ps;
 	const tg_config &c = m->cfg;
 	const int L = c.n_layers, V = c.n_vocab;
@@ -1308,8 +1135,8 @@ int ensure_persist_tiles(tg_state *s) {
 	return TG_OK;
 }
 
-int persist_launch(tg_state *s, int n_steps, int sampler, float minp, float temp, bool log_tokens, const int *force_ids = nullptr) {
-	tg_model *m = s->m;
+int persist_launch(GemmaState *s, int n_steps, int sampler, float minp, float temp, bool log_tokens, const int *force_ids = nullptr) {
+	GemmaModel *m = s->m;
 	TG_TRY(ensure_persist_tiles(s));
 	PsArgs a = s->ps;
 	a.tiled = m->ps_tiled;
@@ -1392,9 +1219,9 @@ int persist_launch(tg_state *s, int n_steps, int sampler, float minp, float temp
 }
 
 // one cooperative launch: n_steps tokens; sampler 0 none / 1 argmax / 2 min-p
-int mega_launch(tg_state *s, int n_steps, int sampler, float minp, float temp, bool log_tokens) {
+int mega_launch(GemmaState *s, int n_steps, int sampler, float minp, float temp, bool log_tokens) {
 	if (s->ps_ok) return persist_launch(s, n_steps, sampler, minp, temp, log_tokens);
-	tg_model *m = s->m;
+	GemmaModel *m = s->m;
 	TG_TRY(ensure_decode_tiles(s));
 	MgArgs a = s->mega;
 	a.tiled = m->dec_tiled;
@@ -1429,93 +1256,6 @@ int mega_launch(tg_state *s, int n_steps, int sampler, float minp, float temp, b
 	count_launch();
 	return check_launch("mega_decode");
 }
-
-SampleArgs sample_args(tg_state *s, float minp, float temp, bool log_tokens) {
-	SampleArgs a{};
-	a.logits = s->logits;
-	a.V = s->m->cfg.n_vocab;
-	a.tok_out = s->tok;
-	a.tok_log = log_tokens ? s->tok_log : nullptr;
-	a.log_count = s->log_count;
-	a.log_cap = s->log_cap;
-	a.B = s->B;
-	a.minp = minp;
-	a.temp = temp;
-	a.randf = s->randf;
-	a.randf_count = s->randf_count;
-	a.randf_cap = s->randf_cap;
-	return a;
-}
-
-int enqueue_sampler(tg_state *s, float minp, float temp, bool log_tokens) {
-	SampleArgs a = sample_args(s, minp, temp, log_tokens);
-	if (minp < 1.0f && s->mega_ok && s->B == 1 && env_int("TG_MINP_GRID", 1)) {
-		// one sequence: the row is spread over the whole GPU, sums ordered like the persistent kernel's sampler
-		TG_CUDA(cudaMemsetAsync(s->mg_bar + 8, 0, 4, s->stream));
-		unsigned *bar = s->mg_bar + 8;
-		float *part = s->mg_samp_f;
-		float *probs = s->mg_probs;
-		int *err = s->err_flag;
-		void *params[] = {&a, &bar, &part, &probs, &err};
-		TG_CUDA(cudaLaunchCooperativeKernel((void *)minp_grid_kernel, dim3(s->mega_grid), dim3(SG_THREADS), params, 0, s->stream));
-		count_launch();
-		return check_launch("minp_grid");
-	}
-	if (minp < 1.0f) {  // transformer.hpp:208,229: min-p sampling iff minp < 1
-		minp_kernel<<<s->B, SM_THREADS, 0, s->stream>>>(a);
-		count_launch();
-		return check_launch("minp");
-	}
-	launch_k(argmax_kernel, dim3(s->B), dim3(SM_THREADS), 0, s->stream, a);
-	count_launch();
-	return check_launch("argmax");
-}
-
-// the pinned staging buffer may be overwritten only when no enqueued copy still reads it
-int staging_acquire(tg_state *s) {
-	if (s->staging_busy) {
-		TG_CUDA(cudaStreamSynchronize(s->stream));
-		s->staging_busy = false;
-	}
-	return TG_OK;
-}
-
-// the error word a kernel left (read back by the caller) -> return code; clears the word on the device
-int report_err_flag(tg_state *s, int flag) {
-	if (flag) {
-		cudaMemsetAsync(s->err_flag, 0, 4, s->stream);
-		s->ps_clean = false;  // a launch that gave up leaves its hand-off words and barrier count anywhere
-		if (flag > 0xFF) {  // the persistent kernel reports where it gave up above the code
-			const int where = flag >> 8;
-			const char *what = (flag & 0xFF) == 3 ? "bulk-copy" : ((flag & 0xFF) == 4 ? "grid-barrier" : "hand-off");
-			return fail(TG_ECUDA, std::string("persistent kernel: a ") + what + " wait ran out (layer " + std::to_string(where >> 4) +
-			                          ", phase " + std::to_string(where & 15) + ")");
-		}
-		if (flag == 1) return fail(TG_EINVAL, "token id out of range");
-		if (flag == 2) return fail(TG_ESTATE, "global KV cache full (max_pos_global reached)");
-		if (flag == 6) return fail(TG_ECUDA, "tensor-core GEMM: a pipeline wait ran out");
-		if (flag == 5) return fail(TG_ECUDA, "persistent kernel: a hand-off flag wait ran out");
-		return fail(TG_ECUDA, flag == 3 ? "persistent kernel: a TMA wait ran out" : "persistent kernel: a grid barrier wait ran out");
-	}
-	return TG_OK;
-}
-
-int check_err_flag(tg_state *s) {
-	TG_CUDA(cudaMemcpyAsync(s->host_pin + 8192, s->err_flag, 4, cudaMemcpyDeviceToHost, s->stream));
-	TG_CUDA(cudaStreamSynchronize(s->stream));
-	s->staging_busy = false;
-	return report_err_flag(s, s->host_pin[8192]);
-}
-
-int ensure_log(tg_state *s, int steps) {
-	if (steps <= s->log_cap) return TG_OK;
-	if (s->tok_log) cudaFree(s->tok_log);
-	s->tok_log = nullptr;
-	TG_CUDA(cudaMalloc(&s->tok_log, size_t(steps) * s->B * 4));
-	s->log_cap = steps;
-	return TG_OK;
-}
-
 
 // K-split of the tensor-core GEMM: enough CTAs to fill the GPU, accumulation chains of at most 24
 // K-blocks (768 rows) for accuracy, as far as the partial-sum buffer allows.
@@ -1671,7 +1411,7 @@ int launch_gemm_tc(float *C, const QW &w, int M, const TcScratch &sc, cudaStream
 // For larger batches the per-token work is the prefill's: every weight matrix is read once per
 // step for all sequences by the tensor-core GEMM (M = batch), the norms run row-wise, and only
 // the attention is per sequence (each against its own cache, positions read on the device).
-int batched_setup(tg_state *s) {
+int batched_setup(GemmaState *s) {
 	const tg_config &c = s->m->cfg;
 	const int B = s->B, D = c.hidden_size, I = c.intermediate_size, V = c.n_vocab, qd = c.n_head * c.head_dim;
 	TG_CUDA(cudaMalloc(&s->bx, size_t(B) * D * 4));
@@ -1689,13 +1429,13 @@ int batched_setup(tg_state *s) {
 	return TG_OK;
 }
 
-int enqueue_decode_batched(tg_state *s, bool with_lm_head) {
+int enqueue_decode_batched(GemmaState *s, bool with_lm_head) {
 	struct PdlOff {
 		bool was = g_pdl_scope_off;
 		PdlOff() { g_pdl_scope_off = true; }
 		~PdlOff() { g_pdl_scope_off = was; }
 	} pdl_off;
-	tg_model *m = s->m;
+	GemmaModel *m = s->m;
 	const tg_config &c = m->cfg;
 	const int B = s->B, D = c.hidden_size, I = c.intermediate_size, V = c.n_vocab;
 	const int qd = c.n_head * c.head_dim;
@@ -1820,9 +1560,9 @@ int launch_gemm(float *C, const float *A, const QW &w, int M, float *partial, si
 // stacked (row = sequence * S + position): embedding, norms, GEMMs and GeGLU work on all nb * S rows at once —
 // a GEMM over 178 rows runs at a sixth of the tensor throughput of one over thousands — and only the
 // per-sequence steps (RoPE positions, cache fill, causal attention) index by sequence (blockIdx.y).
-int enqueue_prefill_seq(tg_state *s, int b, int S_seq, int nb = 1) {
+int enqueue_prefill_seq(GemmaState *s, int b, int S_seq, int nb = 1) {
 	const int S = S_seq * nb;  // rows
-	tg_model *m = s->m;
+	GemmaModel *m = s->m;
 	const tg_config &c = m->cfg;
 	const int D = c.hidden_size, I = c.intermediate_size, V = c.n_vocab;
 	const int qd = c.n_head * c.head_dim, kd = c.n_kv * c.head_dim;
@@ -2035,26 +1775,234 @@ int enqueue_prefill_seq(tg_state *s, int b, int S_seq, int nb = 1) {
 
 }  // namespace
 
-// ===================================================================== C ABI
-extern "C" {
+// ===================================================================== state behind the common entry points
+GemmaModel::~GemmaModel() {
+	GemmaModel *m = this;
+	cudaFree(m->blob);
+	cudaFree(m->dec_tiled);
+	cudaFree(m->ps_tiled);
+	cudaFree(m->ps_lm);
+	for (int i = 0; i < 2; i++)
+		for (int j = 0; j < 2; j++) cudaFree(m->rope[i][j]);
+	cudaFree(m->gelu);
+}
 
-const char *tg_last_error(void) { return g_err.c_str(); }
-const char *tg_version(void) { return "tiny-gemma_b200 0.1 (sm_100a)"; }
-
-int tg_device_count(int *count) {
-	if (!count) return fail(TG_EINVAL, "count is null");
-	int n = 0;
-	cudaError_t e = cudaGetDeviceCount(&n);
-	if (e != cudaSuccess) {
-		cudaGetLastError();
-		n = 0;
+int GemmaModel::new_state(int batch, int max_pos_global, tg_state **out) {
+	GemmaModel *m = this;
+	GemmaState *s = new GemmaState();
+	s->m = m;
+	s->model = m;
+	s->B = batch;
+	s->max_pos_global = max_pos_global;
+	int rc = state_alloc(s);
+	if (rc == TG_OK && batch >= env_int("TG_BATCH_TC_MIN", 4)) rc = batched_setup(s);
+	if (rc == TG_OK && batch == 1 && env_int("TG_MEGA", 1)) {
+		int mrc = mega_setup(s);
+		if (mrc != TG_OK) {
+			if (env_int("TG_MEGA", 1) == 2) rc = mrc;  // 2 = required
+			s->mega_ok = false;
+		} else if (env_int("TG_PERSIST", 1)) {
+			// the dp4a kernel (kernels_persist.cuh) is the batch-1 decode path; a shape it has no plan for falls back
+			// to the fp32-FMA kernel (kernels_mega.cuh), which TG_PERSIST=0 also selects
+			int prc = persist_setup(s);
+			if (prc != TG_OK) {
+				if (env_int("TG_PERSIST", 1) == 2) rc = prc;  // 2 = required
+				s->ps_ok = false;
+			}
+		}
 	}
-	*count = n;
+	if (rc != TG_OK) {
+		const std::string keep = tg_last_error();
+		tg_state_free(s);
+		return fail(rc, keep);
+	}
+	*out = s;
+	return TG_OK;
+}
+GemmaState::~GemmaState() {
+	GemmaState *s = this;
+	for (float *p : s->kcache) cudaFree(p);
+	for (float *p : s->vcache) cudaFree(p);
+	cudaFree(s->h[0]);
+	cudaFree(s->h[1]);
+	cudaFree(s->qkv);
+	cudaFree(s->attn_out);
+	cudaFree(s->t);
+	cudaFree(s->act);
+	cudaFree(s->partial);
+	cudaFree(s->tickets);
+	cudaFree(s->attn_tickets);
+	cudaFree(s->attn_part);
+	cudaFree(s->step_pos);
+	cudaFree(s->next_pos);
+	cudaFree(s->ring_base);
+	cudaFree(s->force_ids);
+	cudaFree(s->pf);
+	cudaFree(s->pf_ids);
+	cudaFree(s->bx);
+	cudaFree(s->bup);
+	cudaFree(s->btc.apack);
+	cudaFree(s->btc.partial);
+	cudaFree(s->btc.tickets);
+	cudaFree(s->d_tmaps);
+	cudaFree(s->d_layers);
+	cudaFree(s->mg_ll);
+	cudaFree(s->mg_probs);
+	cudaFree(s->mg_pe);
+	cudaFree(s->mg_samp_f);
+	cudaFree(s->mg_samp_i);
+	cudaFree(s->mg_bar);
+	cudaFree(s->mg_dbg);
+	cudaFree(s->d_pslayers);
+	cudaFree(s->ps_ll);
+	free_common();
+}
+
+int GemmaState::ready() { return check_ready(m); }
+
+int GemmaState::reset() {
+	TG_CUDA(cudaMemsetAsync(step_pos, 0, 4 * B, stream));
+	TG_CUDA(cudaMemsetAsync(next_pos, 0, 4 * B, stream));
+	TG_CUDA(cudaMemsetAsync(ring_base, 0, 4 * B, stream));
+	// the reference's caches are zero-initialised (tensor.hpp:66-74); stale rows
+	// are never read (valid_pos bounds every loop) so they are left in place
 	return TG_OK;
 }
 
+int GemmaState::prefill(const int *ids, int S, float *logits_host) {
+	GemmaState *s = this;
+	const tg_config &c = m->cfg;
+	const int D = c.hidden_size, I = c.intermediate_size, V = c.n_vocab;
+	const int qd = c.n_head * c.head_dim, kd = c.n_kv * c.head_dim;
+	if (S == 1) {
+		// a one-token prompt takes the reference's decode branch (modules.hpp:135)
+		return tg_decode(s, ids, logits_host);
+	}
+	// Batches that take the batched decode step prefill their prompts together, up to 16384 rows per pass (the
+	// scratch grows with the rows: 79 KB per row at the 1B shape); smaller batches stay one sequence per pass, so
+	// that a sequence's results do not depend on its neighbours' presence.
+	const int group = (s->batched_ok && env_int("TG_GEMM_TC", 1) && env_int("TG_PREFILL_GROUP", 1)) ? std::max(1, std::min(s->B, 16384 / S)) : 1;
+	const size_t R = size_t(group) * S;  // rows per pass
+	size_t need = R * (3 * size_t(D) + 2 * qd + 2 * kd + 2 * size_t(I));
+	size_t part = std::max(size_t(4) * R * D, size_t(1) << 22);  // split-K scratch
+	part = std::max(part, std::min(size_t(24) * R * std::max(I, qd), size_t(1) << 28));  // tensor-core GEMM partial sums (<= 1 GiB)
+	need += part;
+	need += (tc_pack_bytes(int(R), std::max(I, std::max(D, qd))) + 3) / 4 + 64;
+	need += (attn_tc_plan(S).total() + 3) / 4 + 512;  // packed q, k, v of the tensor-core attention (long prompts)
+	if (need > s->pf_floats) {
+		if (s->pf) cudaFree(s->pf);
+		s->pf = nullptr;
+		s->pf_floats = 0;
+		cudaError_t e = cudaMalloc(&s->pf, need * 4);
+		if (e != cudaSuccess) return fail(TG_ENOMEM, std::string("cudaMalloc(prefill scratch): ") + cudaGetErrorString(e));
+		s->pf_floats = need;
+	}
+	if (S * s->B > s->pf_ids_cap) {
+		if (s->pf_ids) cudaFree(s->pf_ids);
+		s->pf_ids = nullptr;
+		TG_CUDA(cudaMalloc(&s->pf_ids, size_t(S) * s->B * 4));
+		s->pf_ids_cap = S * s->B;
+	}
+	TG_CUDA(cudaMemcpyAsync(s->pf_ids, ids, size_t(S) * s->B * 4, cudaMemcpyHostToDevice, s->stream));
+	for (int b = 0; b < s->B; b += group) TG_TRY(enqueue_prefill_seq(s, b, S, std::min(group, s->B - b)));
+	// position_ptr = S; ring base per decode.hpp:98-103
+	std::vector<int> pos(s->B, S), rb(s->B, S >= c.n_pos_local ? S : 0);
+	TG_TRY(s->staging_acquire());
+	std::memcpy(s->host_pin, pos.data(), 4 * s->B);
+	std::memcpy(s->host_pin + s->B, rb.data(), 4 * s->B);
+	TG_CUDA(cudaMemcpyAsync(s->next_pos, s->host_pin, 4 * s->B, cudaMemcpyHostToDevice, s->stream));
+	TG_CUDA(cudaMemcpyAsync(s->step_pos, s->host_pin, 4 * s->B, cudaMemcpyHostToDevice, s->stream));
+	TG_CUDA(cudaMemcpyAsync(s->ring_base, s->host_pin + s->B, 4 * s->B, cudaMemcpyHostToDevice, s->stream));
+	if (logits_host)
+		TG_CUDA(cudaMemcpyAsync(logits_host, s->logits, size_t(s->B) * V * 4, cudaMemcpyDeviceToHost, s->stream));
+	TG_TRY(s->check_err_flag());
+	s->host_pos.assign(s->B, S);
+	return TG_OK;
+}
+int GemmaState::append(const int *ids, int n, float *logits_host) {
+	GemmaState *s = this;
+	if (s->ps_ok) {
+		// one launch of the persistent kernel: every step takes its token from the list instead of a sampler
+		if (s->force_cap < n) {
+			cudaFree(s->force_ids);
+			s->force_ids = nullptr;
+			TG_CUDA(cudaMalloc(&s->force_ids, size_t(n) * 4));
+			s->force_cap = n;
+		}
+		TG_CUDA(cudaMemcpyAsync(s->force_ids, ids, size_t(n) * 4, cudaMemcpyHostToDevice, s->stream));
+		TG_CUDA(cudaStreamSynchronize(s->stream));  // `ids` is the caller's pageable memory: consumed before returning
+		TG_TRY(persist_launch(s, n, 0, 2.0f, 1.0f, false, s->force_ids));
+		s->host_pos[0] += n;
+	} else {
+		for (int i = 0; i < n; i++) TG_TRY(tg_decode(s, ids + i, nullptr));
+	}
+	if (logits_host)
+		TG_CUDA(cudaMemcpyAsync(logits_host, s->logits, size_t(m->cfg.n_vocab) * 4, cudaMemcpyDeviceToHost, s->stream));
+	return s->check_err_flag();
+}
+int GemmaState::enqueue_decode_all() {
+	if (batched_ok) return enqueue_decode_batched(this, true);
+	for (int b0 = 0; b0 < B; b0 += MV_MAX_B) TG_TRY(enqueue_decode_chunk(this, b0, std::min(MV_MAX_B, B - b0)));
+	return TG_OK;
+}
+
+int GemmaState::enqueue_forward() {
+	if (mega_ok) return mega_launch(this, 1, 0, 2.0f, 1.0f, false);
+	return enqueue_decode_step();
+}
+
+int GemmaState::run_steps(int n_steps, float minp, float temp) {
+	if (mega_ok) return mega_launch(this, n_steps, minp < 1.0f ? 2 : 1, minp, temp, true);
+	return tg_state::run_steps(n_steps, minp, temp);
+}
+
+int GemmaState::enqueue_sampler(float minp, float temp, bool log_tokens) {
+	if (!(minp < 1.0f && mega_ok && B == 1 && env_int("TG_MINP_GRID", 1))) return tg_state::enqueue_sampler(minp, temp, log_tokens);
+	// one sequence: the row is spread over the whole GPU, sums ordered like the persistent kernel's sampler
+	SampleArgs a = sample_args(minp, temp, log_tokens);
+	TG_CUDA(cudaMemsetAsync(mg_bar + 8, 0, 4, stream));
+	unsigned *bar = mg_bar + 8;
+	float *part = mg_samp_f;
+	float *probs = mg_probs;
+	int *err = err_flag;
+	void *params[] = {&a, &bar, &part, &probs, &err};
+	TG_CUDA(cudaLaunchCooperativeKernel((void *)minp_grid_kernel, dim3(mega_grid), dim3(SG_THREADS), params, 0, stream));
+	count_launch();
+	return check_launch("minp_grid");
+}
+
+int GemmaState::report_err(int flag) {
+	if (!flag) return TG_OK;
+	ps_clean = false;  // a launch that gave up leaves its hand-off words and barrier count anywhere
+	if (flag > 0xFF) {  // the persistent kernel reports where it gave up above the code
+		cudaMemsetAsync(err_flag, 0, 4, stream);
+		const int where = flag >> 8;
+		const char *what = (flag & 0xFF) == 3 ? "bulk-copy" : ((flag & 0xFF) == 4 ? "grid-barrier" : "hand-off");
+		return fail(TG_ECUDA, std::string("persistent kernel: a ") + what + " wait ran out (layer " + std::to_string(where >> 4) +
+		                          ", phase " + std::to_string(where & 15) + ")");
+	}
+	if (flag >= 3 && flag <= 5) {
+		cudaMemsetAsync(err_flag, 0, 4, stream);
+		return fail(TG_ECUDA, flag == 5 ? "persistent kernel: a hand-off flag wait ran out"
+		                                : (flag == 3 ? "persistent kernel: a TMA wait ran out" : "persistent kernel: a grid barrier wait ran out"));
+	}
+	if (flag == 2) {
+		cudaMemsetAsync(err_flag, 0, 4, stream);
+		return fail(TG_ESTATE, "global KV cache full (max_pos_global reached)");
+	}
+	return tg_state::report_err(flag);
+}
+
+namespace {
+GemmaModel *as_gemma(tg_model *m) { return dynamic_cast<GemmaModel *>(m); }
+GemmaState *as_gemma(tg_state *s) { return dynamic_cast<GemmaState *>(s); }
+}  // namespace
+
+// ===================================================================== C ABI
+extern "C" {
+
 int tg_config_by_name(const char *name, tg_config *out) {
-	if (!name || !out) return fail(TG_EINVAL, "null argument");
+	if (!name || !out) return fail(TG_EINVAL, "null argument, or a handle of another family");
 	// reference config.hpp:46-48
 	if (std::strcmp(name, "270m") == 0) {
 		*out = tg_config{640, 2048, 18, 262144, 32768, 512, 256, 4, 1, 1000000.0f, 10000.0f, 6};
@@ -2068,13 +2016,13 @@ int tg_config_by_name(const char *name, tg_config *out) {
 }
 
 int tg_model_file_bytes(const tg_config *cfg, size_t *nbytes) {
-	if (!cfg || !nbytes) return fail(TG_EINVAL, "null argument");
+	if (!cfg || !nbytes) return fail(TG_EINVAL, "null argument, or a handle of another family");
 	*nbytes = model_file_bytes(*cfg);
 	return TG_OK;
 }
 
 int tg_model_create(const tg_config *cfg, int device, tg_model **out) {
-	if (!cfg || !out) return fail(TG_EINVAL, "null argument");
+	if (!cfg || !out) return fail(TG_EINVAL, "null argument, or a handle of another family");
 	const tg_config &c = *cfg;
 	if (c.head_dim != 256 || c.n_head != 4 || c.n_kv != 1)
 		return fail(TG_ESHAPE, "kernels are specialised for 4 query heads, 1 KV head, head_dim 256");
@@ -2082,9 +2030,12 @@ int tg_model_create(const tg_config *cfg, int device, tg_model **out) {
 	    !supported_n(c.intermediate_size) || c.n_vocab % 8192 != 0 || c.n_layers < 1 || c.window_pattern < 1)
 		return fail(TG_ESHAPE, "unsupported model dimensions");
 	TG_TRY(ensure_device(device));
-	tg_model *m = new tg_model();
+	GemmaModel *m = new GemmaModel();
 	m->cfg = c;
 	m->device = device;
+	m->n_vocab = c.n_vocab;
+	m->hidden_size = c.hidden_size;
+	m->n_pos = c.n_pos;
 	m->nbytes = model_file_bytes(c);
 	cudaError_t e = cudaMalloc(&m->blob, m->nbytes);
 	if (e != cudaSuccess) {
@@ -2097,22 +2048,9 @@ int tg_model_create(const tg_config *cfg, int device, tg_model **out) {
 	return TG_OK;
 }
 
-int tg_model_free(tg_model *m) {
-	if (!m) return TG_OK;
-	cudaSetDevice(m->device);
-	cudaFree(m->blob);
-	cudaFree(m->dec_tiled);
-	cudaFree(m->ps_tiled);
-	cudaFree(m->ps_lm);
-	for (int i = 0; i < 2; i++)
-		for (int j = 0; j < 2; j++) cudaFree(m->rope[i][j]);
-	cudaFree(m->gelu);
-	delete m;
-	return TG_OK;
-}
-
-int tg_model_load_memory(tg_model *m, const void *bytes, size_t nbytes) {
-	if (!m || !bytes) return fail(TG_EINVAL, "null argument");
+int tg_model_load_memory(tg_model *m_, const void *bytes, size_t nbytes) {
+	GemmaModel *m = as_gemma(m_);
+	if (!m || !bytes) return fail(TG_EINVAL, "null argument, or a handle of another family");
 	if (nbytes < m->nbytes) return fail(TG_EIO, "weights image shorter than the model needs");
 	TG_CUDA(cudaSetDevice(m->device));
 	TG_CUDA(cudaMemcpy(m->blob, bytes, m->nbytes, cudaMemcpyHostToDevice));
@@ -2121,8 +2059,9 @@ int tg_model_load_memory(tg_model *m, const void *bytes, size_t nbytes) {
 	return TG_OK;
 }
 
-int tg_model_load_file(tg_model *m, const char *path) {
-	if (!m || !path) return fail(TG_EINVAL, "null argument");
+int tg_model_load_file(tg_model *m_, const char *path) {
+	GemmaModel *m = as_gemma(m_);
+	if (!m || !path) return fail(TG_EINVAL, "null argument, or a handle of another family");
 	FILE *f = std::fopen(path, "rb");
 	if (!f) return fail(TG_EIO, "Could not open file.");
 	TG_CUDA(cudaSetDevice(m->device));
@@ -2170,7 +2109,8 @@ int tg_model_load_file(tg_model *m, const char *path) {
 	return rc;
 }
 
-int tg_model_set_rope(tg_model *m, int is_local, const float *cos_host, const float *sin_host, int n_pos) {
+int tg_model_set_rope(tg_model *m_, int is_local, const float *cos_host, const float *sin_host, int n_pos) {
+	GemmaModel *m = as_gemma(m_);
 	if (!m || !cos_host || !sin_host || n_pos <= 0) return fail(TG_EINVAL, "bad argument");
 	// the kernels read row `position` for every position a state may reach (max_pos_global <= n_pos); the
 	// reference's decode::RoPE always builds cfg.n_pos rows (decode.hpp:118-200), so a shorter table is refused
@@ -2189,7 +2129,8 @@ int tg_model_set_rope(tg_model *m, int is_local, const float *cos_host, const fl
 	return TG_OK;
 }
 
-int tg_model_set_gelu_table(tg_model *m, float mn, float mx, const float *table, int size) {
+int tg_model_set_gelu_table(tg_model *m_, float mn, float mx, const float *table, int size) {
+	GemmaModel *m = as_gemma(m_);
 	if (!m || !table || size <= 0) return fail(TG_EINVAL, "bad argument");
 	TG_CUDA(cudaSetDevice(m->device));
 	if (m->gelu) cudaFree(m->gelu);
@@ -2203,7 +2144,8 @@ int tg_model_set_gelu_table(tg_model *m, float mn, float mx, const float *table,
 	return TG_OK;
 }
 
-int tg_model_build_tables(tg_model *m, int gelu_size) {
+int tg_model_build_tables(tg_model *m_, int gelu_size) {
+	GemmaModel *m = as_gemma(m_);
 	if (!m || gelu_size <= 0) return fail(TG_EINVAL, "bad argument");
 	const tg_config &c = m->cfg;
 	const int hd = c.head_dim, half = hd / 2;
@@ -2238,397 +2180,8 @@ int tg_model_build_tables(tg_model *m, int gelu_size) {
 }
 
 // ---------------------------------------------------------------- state
-int tg_state_create(tg_model *m, int batch, int max_pos_global, tg_state **out) {
-	if (!m || !out || batch < 1 || batch > 2048) return fail(TG_EINVAL, "bad argument (batch must be 1..2048)");
-	if (max_pos_global <= 0) max_pos_global = m->cfg.n_pos;
-	if (max_pos_global > m->cfg.n_pos) return fail(TG_EINVAL, "max_pos_global exceeds n_pos");
-	TG_CUDA(cudaSetDevice(m->device));
-	tg_state *s = new tg_state();
-	s->m = m;
-	s->B = batch;
-	s->max_pos_global = max_pos_global;
-	int rc = state_alloc(s);
-	if (rc == TG_OK && batch >= env_int("TG_BATCH_TC_MIN", 4)) rc = batched_setup(s);
-	if (rc == TG_OK && batch == 1 && env_int("TG_MEGA", 1)) {
-		int mrc = mega_setup(s);
-		if (mrc != TG_OK) {
-			if (env_int("TG_MEGA", 1) == 2) rc = mrc;  // 2 = required
-			s->mega_ok = false;
-		} else if (env_int("TG_PERSIST", 1)) {
-			// the dp4a kernel (kernels_persist.cuh) is the batch-1 decode path; a shape it has no plan for falls back
-			// to the fp32-FMA kernel (kernels_mega.cuh), which TG_PERSIST=0 also selects
-			int prc = persist_setup(s);
-			if (prc != TG_OK) {
-				if (env_int("TG_PERSIST", 1) == 2) rc = prc;  // 2 = required
-				s->ps_ok = false;
-			}
-		}
-	}
-	if (rc != TG_OK) {
-		std::string keep = g_err;
-		tg_state_free(s);
-		g_err = keep;
-		return rc;
-	}
-	*out = s;
-	return TG_OK;
-}
-
-int tg_state_free(tg_state *s) {
-	if (!s) return TG_OK;
-	cudaSetDevice(s->m->device);
-	if (s->stream) cudaStreamSynchronize(s->stream);
-	if (s->graph) cudaGraphExecDestroy(s->graph);
-	for (float *p : s->kcache) cudaFree(p);
-	for (float *p : s->vcache) cudaFree(p);
-	cudaFree(s->h[0]);
-	cudaFree(s->h[1]);
-	cudaFree(s->qkv);
-	cudaFree(s->attn_out);
-	cudaFree(s->t);
-	cudaFree(s->act);
-	cudaFree(s->xnorm);
-	cudaFree(s->logits);
-	cudaFree(s->partial);
-	cudaFree(s->tickets);
-	cudaFree(s->attn_tickets);
-	cudaFree(s->attn_part);
-	cudaFree(s->step_pos);
-	cudaFree(s->next_pos);
-	cudaFree(s->ring_base);
-	cudaFree(s->tok_log);
-	cudaFree(s->force_ids);
-	if (!s->randf_in_blk) cudaFree(s->randf);
-	cudaFree(s->step_blk);  // err_flag, tok, randf_count, log_count (and the first randf)
-	cudaFree(s->pf);
-	cudaFree(s->pf_ids);
-	cudaFree(s->bx);
-	cudaFree(s->bup);
-	cudaFree(s->btc.apack);
-	cudaFree(s->btc.partial);
-	cudaFree(s->btc.tickets);
-	cudaFree(s->d_tmaps);
-	cudaFree(s->d_layers);
-	cudaFree(s->mg_ll);
-	cudaFree(s->mg_probs);
-	cudaFree(s->mg_pe);
-	cudaFree(s->mg_samp_f);
-	cudaFree(s->mg_samp_i);
-	cudaFree(s->mg_bar);
-	cudaFree(s->mg_dbg);
-	cudaFree(s->d_pslayers);
-	cudaFree(s->ps_ll);
-	if (s->host_pin) cudaFreeHost(s->host_pin);
-	if (s->stream) cudaStreamDestroy(s->stream);
-	delete s;
-	return TG_OK;
-}
-
-int tg_state_reset(tg_state *s) {
-	if (!s) return fail(TG_EINVAL, "null state");
-	TG_CUDA(cudaSetDevice(s->m->device));
-	const int B = s->B;
-	TG_CUDA(cudaMemsetAsync(s->step_pos, 0, 4 * B, s->stream));
-	TG_CUDA(cudaMemsetAsync(s->next_pos, 0, 4 * B, s->stream));
-	TG_CUDA(cudaMemsetAsync(s->ring_base, 0, 4 * B, s->stream));
-	TG_CUDA(cudaMemsetAsync(s->log_count, 0, 4 * B, s->stream));
-	TG_CUDA(cudaMemsetAsync(s->randf_count, 0, 4 * B, s->stream));
-	TG_CUDA(cudaMemsetAsync(s->err_flag, 0, 4, s->stream));
-	// the reference's caches are zero-initialised (tensor.hpp:66-74); stale rows
-	// are never read (valid_pos bounds every loop) so they are left in place
-	TG_CUDA(cudaStreamSynchronize(s->stream));
-	s->host_pos.assign(B, 0);
-	return TG_OK;
-}
-
-int tg_state_position(tg_state *s, int b, int *position) {
-	if (!s || !position || b < 0 || b >= s->B) return fail(TG_EINVAL, "bad argument");
-	*position = s->host_pos[b];
-	return TG_OK;
-}
-
-int tg_state_stream(tg_state *s, void **stream) {
-	if (!s || !stream) return fail(TG_EINVAL, "null argument");
-	*stream = (void *)s->stream;
-	return TG_OK;
-}
-
-int tg_prefill(tg_state *s, const int *ids, int S, float *logits_host) {
-	if (!s || !ids || S < 1) return fail(TG_EINVAL, "bad argument");
-	tg_model *m = s->m;
-	TG_TRY(check_ready(m));
-	const tg_config &c = m->cfg;
-	if (S > c.n_pos) return fail(TG_EINVAL, "prompt longer than n_pos");
-	if (S > s->max_pos_global) return fail(TG_EINVAL, "prompt longer than max_pos_global");
-	for (int b = 0; b < s->B; b++)
-		if (s->host_pos[b] != 0) return fail(TG_ESTATE, "prefill needs an empty KV cache (decode.hpp:78-79)");
-	TG_CUDA(cudaSetDevice(m->device));
-	const int D = c.hidden_size, I = c.intermediate_size, V = c.n_vocab;
-	const int qd = c.n_head * c.head_dim, kd = c.n_kv * c.head_dim;
-	if (S == 1) {
-		// a one-token prompt takes the reference's decode branch (modules.hpp:135)
-		TG_TRY(tg_decode(s, ids, logits_host));
-		return TG_OK;
-	}
-	// Batches that take the batched decode step prefill their prompts together, up to 16384 rows per pass (the
-	// scratch grows with the rows: 79 KB per row at the 1B shape); smaller batches stay one sequence per pass, so
-	// that a sequence's results do not depend on its neighbours' presence.
-	const int group = (s->batched_ok && env_int("TG_GEMM_TC", 1) && env_int("TG_PREFILL_GROUP", 1)) ? std::max(1, std::min(s->B, 16384 / S)) : 1;
-	const size_t R = size_t(group) * S;  // rows per pass
-	size_t need = R * (3 * size_t(D) + 2 * qd + 2 * kd + 2 * size_t(I));
-	size_t part = std::max(size_t(4) * R * D, size_t(1) << 22);  // split-K scratch
-	part = std::max(part, std::min(size_t(24) * R * std::max(I, qd), size_t(1) << 28));  // tensor-core GEMM partial sums (<= 1 GiB)
-	need += part;
-	need += (tc_pack_bytes(int(R), std::max(I, std::max(D, qd))) + 3) / 4 + 64;
-	need += (attn_tc_plan(S).total() + 3) / 4 + 512;  // packed q, k, v of the tensor-core attention (long prompts)
-	if (need > s->pf_floats) {
-		if (s->pf) cudaFree(s->pf);
-		s->pf = nullptr;
-		s->pf_floats = 0;
-		cudaError_t e = cudaMalloc(&s->pf, need * 4);
-		if (e != cudaSuccess) return fail(TG_ENOMEM, std::string("cudaMalloc(prefill scratch): ") + cudaGetErrorString(e));
-		s->pf_floats = need;
-	}
-	if (S * s->B > s->pf_ids_cap) {
-		if (s->pf_ids) cudaFree(s->pf_ids);
-		s->pf_ids = nullptr;
-		TG_CUDA(cudaMalloc(&s->pf_ids, size_t(S) * s->B * 4));
-		s->pf_ids_cap = S * s->B;
-	}
-	TG_CUDA(cudaMemcpyAsync(s->pf_ids, ids, size_t(S) * s->B * 4, cudaMemcpyHostToDevice, s->stream));
-	for (int b = 0; b < s->B; b += group) TG_TRY(enqueue_prefill_seq(s, b, S, std::min(group, s->B - b)));
-	// position_ptr = S; ring base per decode.hpp:98-103
-	std::vector<int> pos(s->B, S), rb(s->B, S >= c.n_pos_local ? S : 0);
-	TG_TRY(staging_acquire(s));
-	std::memcpy(s->host_pin, pos.data(), 4 * s->B);
-	std::memcpy(s->host_pin + s->B, rb.data(), 4 * s->B);
-	TG_CUDA(cudaMemcpyAsync(s->next_pos, s->host_pin, 4 * s->B, cudaMemcpyHostToDevice, s->stream));
-	TG_CUDA(cudaMemcpyAsync(s->step_pos, s->host_pin, 4 * s->B, cudaMemcpyHostToDevice, s->stream));
-	TG_CUDA(cudaMemcpyAsync(s->ring_base, s->host_pin + s->B, 4 * s->B, cudaMemcpyHostToDevice, s->stream));
-	if (logits_host)
-		TG_CUDA(cudaMemcpyAsync(logits_host, s->logits, size_t(s->B) * V * 4, cudaMemcpyDeviceToHost, s->stream));
-	TG_TRY(check_err_flag(s));
-	s->host_pos.assign(s->B, S);
-	return TG_OK;
-}
-
-int tg_decode(tg_state *s, const int *ids, float *logits_host) {
-	if (!s) return fail(TG_EINVAL, "null state");
-	tg_model *m = s->m;
-	TG_TRY(check_ready(m));
-	TG_CUDA(cudaSetDevice(m->device));
-	for (int b = 0; b < s->B; b++)
-		if (s->host_pos[b] >= s->max_pos_global) return fail(TG_ESTATE, "global KV cache full (max_pos_global reached)");
-	if (ids) {
-		for (int b = 0; b < s->B; b++)
-			if (ids[b] < 0 || ids[b] >= m->cfg.n_vocab) return fail(TG_EINVAL, "token id out of range");
-		TG_TRY(staging_acquire(s));
-		std::memcpy(s->host_pin, ids, 4 * s->B);
-		TG_CUDA(cudaMemcpyAsync(s->tok, s->host_pin, 4 * s->B, cudaMemcpyHostToDevice, s->stream));
-	}
-	if (s->mega_ok)
-		TG_TRY(mega_launch(s, 1, 0, 2.0f, 1.0f, false));
-	else
-		TG_TRY(enqueue_decode_step(s));
-	for (int b = 0; b < s->B; b++) s->host_pos[b] += 1;
-	s->staging_busy = s->staging_busy || ids != nullptr;  // (an earlier asynchronous call's copy may still be queued)
-	if (logits_host) {
-		TG_CUDA(cudaMemcpyAsync(logits_host, s->logits, size_t(s->B) * m->cfg.n_vocab * 4, cudaMemcpyDeviceToHost, s->stream));
-		TG_TRY(check_err_flag(s));
-	}
-	// without a host read-back the call only enqueues: the step runs while the caller prepares the sampler
-	// call, and a device-side error (a wait that ran out) is reported by the next call that synchronises
-	return TG_OK;
-}
-
-int tg_append(tg_state *s, const int *ids, int n, float *logits_host) {
-	if (!s || !ids || n < 1) return fail(TG_EINVAL, "bad argument");
-	if (s->B != 1) return fail(TG_EINVAL, "tg_append: one sequence per state");
-	tg_model *m = s->m;
-	TG_TRY(check_ready(m));
-	TG_CUDA(cudaSetDevice(m->device));
-	if (s->host_pos[0] + n > s->max_pos_global) return fail(TG_ESTATE, "global KV cache too small for the appended tokens");
-	for (int i = 0; i < n; i++)
-		if (ids[i] < 0 || ids[i] >= m->cfg.n_vocab) return fail(TG_EINVAL, "token id out of range");
-	if (s->ps_ok) {
-		// one launch of the persistent kernel: every step takes its token from the list instead of a sampler
-		if (s->force_cap < n) {
-			cudaFree(s->force_ids);
-			s->force_ids = nullptr;
-			TG_CUDA(cudaMalloc(&s->force_ids, size_t(n) * 4));
-			s->force_cap = n;
-		}
-		TG_CUDA(cudaMemcpyAsync(s->force_ids, ids, size_t(n) * 4, cudaMemcpyHostToDevice, s->stream));
-		TG_CUDA(cudaStreamSynchronize(s->stream));  // `ids` is the caller's pageable memory: consumed before returning
-		TG_TRY(persist_launch(s, n, 0, 2.0f, 1.0f, false, s->force_ids));
-		s->host_pos[0] += n;
-	} else {
-		for (int i = 0; i < n; i++) TG_TRY(tg_decode(s, ids + i, nullptr));
-	}
-	if (logits_host)
-		TG_CUDA(cudaMemcpyAsync(logits_host, s->logits, size_t(m->cfg.n_vocab) * 4, cudaMemcpyDeviceToHost, s->stream));
-	return check_err_flag(s);
-}
-
-int tg_sample_argmax(tg_state *s, int *toks_host) {
-	if (!s) return fail(TG_EINVAL, "null state");
-	TG_CUDA(cudaSetDevice(s->m->device));
-	TG_TRY(enqueue_sampler(s, 2.0f, 1.0f, false));
-	TG_CUDA(cudaMemcpyAsync(s->host_pin, s->tok, 4 * s->B, cudaMemcpyDeviceToHost, s->stream));
-	TG_TRY(check_err_flag(s));  // synchronises
-	if (toks_host) std::memcpy(toks_host, s->host_pin, 4 * s->B);
-	return TG_OK;
-}
-
-int tg_state_set_randf(tg_state *s, const float *randf_host, int n) {
-	if (!s || !randf_host || n < 1) return fail(TG_EINVAL, "bad argument");
-	TG_CUDA(cudaSetDevice(s->m->device));
-	if (n > s->randf_cap) {
-		if (s->randf && !s->randf_in_blk) cudaFree(s->randf);
-		s->randf = nullptr;
-		s->randf_in_blk = false;
-		s->randf_cap = 0;
-		TG_CUDA(cudaMalloc(&s->randf, size_t(n) * s->B * 4));
-		s->randf_cap = n;
-		// captured graphs do not hold this pointer (the sampler is launched outside the graph)
-	}
-	TG_CUDA(cudaMemcpyAsync(s->randf, randf_host, size_t(n) * s->B * 4, cudaMemcpyHostToDevice, s->stream));
-	TG_CUDA(cudaMemsetAsync(s->randf_count, 0, 4 * s->B, s->stream));
-	TG_CUDA(cudaStreamSynchronize(s->stream));
-	s->randf_valid = std::max(s->randf_valid, n);
-	return TG_OK;
-}
-
-int tg_sample_minp(tg_state *s, float minp, float temp, const float *randf_host, int *toks_host) {
-	if (!s || !randf_host) return fail(TG_EINVAL, "bad argument");
-	if (!(minp < 1.0f)) return fail(TG_EINVAL, "minp must be < 1 (the reference uses argmax otherwise, transformer.hpp:208)");
-	TG_CUDA(cudaSetDevice(s->m->device));
-	if (s->randf_cap >= 1 && size_t(s->B) * 4 <= 4096) {
-		// one uniform per sequence, staged through pinned memory: no synchronisation before the launch
-		s->randf_valid = std::max(s->randf_valid, 1);
-		float *stage = reinterpret_cast<float *>(s->host_pin + 4096);
-		std::memcpy(stage, randf_host, size_t(s->B) * 4);
-		TG_CUDA(cudaMemcpyAsync(s->randf, stage, size_t(s->B) * 4, cudaMemcpyHostToDevice, s->stream));
-		TG_CUDA(cudaMemsetAsync(s->randf_count, 0, 4 * s->B, s->stream));
-	} else {
-		TG_TRY(tg_state_set_randf(s, randf_host, 1));
-	}
-	TG_TRY(enqueue_sampler(s, minp, temp, false));
-	TG_CUDA(cudaMemcpyAsync(s->host_pin, s->tok, 4 * s->B, cudaMemcpyDeviceToHost, s->stream));
-	TG_TRY(check_err_flag(s));  // synchronises
-	if (toks_host) std::memcpy(toks_host, s->host_pin, 4 * s->B);
-	return TG_OK;
-}
-
-int tg_logits_read(tg_state *s, float *logits_host) {
-	if (!s || !logits_host) return fail(TG_EINVAL, "null argument");
-	TG_CUDA(cudaSetDevice(s->m->device));
-	TG_CUDA(cudaMemcpyAsync(logits_host, s->logits, size_t(s->B) * s->m->cfg.n_vocab * 4, cudaMemcpyDeviceToHost, s->stream));
-	TG_CUDA(cudaStreamSynchronize(s->stream));
-	return TG_OK;
-}
-
-namespace {
-// `counters_zeroed`: the caller's upload has already set log_count (and randf_count) to zero
-int generate_async(tg_state *s, int n_steps, float minp, float temp, bool counters_zeroed) {
-	TG_TRY(check_ready(s->m));
-	TG_CUDA(cudaSetDevice(s->m->device));
-	if (s->host_pos[0] + n_steps > s->max_pos_global) return fail(TG_ESTATE, "global KV cache too small for n_steps");
-	if (minp < 1.0f && s->randf_valid < n_steps) return fail(TG_ESTATE, "upload uniforms first (tg_state_set_randf)");
-	TG_TRY(ensure_log(s, n_steps));
-	if (!counters_zeroed) TG_CUDA(cudaMemsetAsync(s->log_count, 0, 4 * s->B, s->stream));
-	if (s->mega_ok) {
-		TG_TRY(mega_launch(s, n_steps, minp < 1.0f ? 2 : 1, minp, temp, true));
-	} else {
-		for (int i = 0; i < n_steps; i++) {
-			TG_TRY(enqueue_decode_step(s));
-			TG_TRY(enqueue_sampler(s, minp, temp, true));
-		}
-	}
-	for (int b = 0; b < s->B; b++) s->host_pos[b] += n_steps;
-	return TG_OK;
-}
-}  // namespace
-
-int tg_generate_async(tg_state *s, int n_steps, float minp, float temp) {
-	if (!s || n_steps < 1) return fail(TG_EINVAL, "bad argument");
-	return generate_async(s, n_steps, minp, temp, false);
-}
-
-int tg_state_tokens(tg_state *s, int n_steps, int *toks_host) {
-	if (!s || !toks_host || n_steps < 1 || n_steps > s->log_cap) return fail(TG_EINVAL, "bad argument");
-	TG_CUDA(cudaSetDevice(s->m->device));
-	TG_CUDA(cudaMemcpyAsync(toks_host, s->tok_log, size_t(n_steps) * s->B * 4, cudaMemcpyDeviceToHost, s->stream));
-	TG_TRY(check_err_flag(s));
-	return TG_OK;
-}
-
-int tg_generate(tg_state *s, const int *first_ids, int n_steps, float minp, float temp, const float *randf_host,
-                int *toks_host) {
-	if (!s || !first_ids || n_steps < 1) return fail(TG_EINVAL, "bad argument");
-	TG_CUDA(cudaSetDevice(s->m->device));
-	// Short runs (a step at a time from a host loop) go through the pinned staging buffer with one
-	// synchronisation at the end: ids and uniforms in, the launch, tokens out.
-	const size_t nbytes = size_t(n_steps) * s->B * 4;
-	const bool lean = nbytes <= 16384;
-	TG_TRY(staging_acquire(s));
-	if (minp < 1.0f && !randf_host) return fail(TG_EINVAL, "min-p sampling needs uniforms");
-	if (n_steps == 1 && s->B == 1 && s->ps_ok && env_int("TG_LEAN_STEP", 1)) {
-		// One token per call (a host loop around the sampler): the step's inputs — id, uniform, zeroed
-		// counters — lie next to each other in the state's step block and go up in ONE copy; the error word
-		// and the sampled id lie next to each other too and come back in ONE; the persistent kernel leaves
-		// its arena and barrier ready for the next launch. So the call is upload, launch, read-back, wait.
-		if (first_ids[0] < 0 || first_ids[0] >= s->m->cfg.n_vocab) return fail(TG_EINVAL, "token id out of range");
-		int *up = s->host_pin;
-		up[0] = first_ids[0];  // tok
-		up[1] = 0;             // randf_count
-		up[2] = 0;             // log_count
-		if (minp < 1.0f) {
-			std::memcpy(up + 3, randf_host, 4);
-			s->randf_valid = std::max(s->randf_valid, 1);
-		}
-		TG_CUDA(cudaMemcpyAsync(s->tok, up, minp < 1.0f ? 16 : 12, cudaMemcpyHostToDevice, s->stream));
-		s->lean_randf = true;
-		const int rc = generate_async(s, 1, minp, temp, true);
-		s->lean_randf = false;
-		if (rc) return rc;
-		int *down = s->host_pin + 8192;
-		TG_CUDA(cudaMemcpyAsync(down, s->err_flag, 20, cudaMemcpyDeviceToHost, s->stream));  // err_flag, pad, tok
-		TG_CUDA(cudaStreamSynchronize(s->stream));
-		s->staging_busy = false;
-		TG_TRY(report_err_flag(s, down[0]));
-		if (toks_host) toks_host[0] = down[4];
-		return TG_OK;
-	}
-	if (minp < 1.0f) {
-		if (lean && s->randf_cap >= n_steps) {
-			s->randf_valid = std::max(s->randf_valid, n_steps);
-			float *stage = reinterpret_cast<float *>(s->host_pin + 4096);
-			std::memcpy(stage, randf_host, nbytes);
-			TG_CUDA(cudaMemcpyAsync(s->randf, stage, nbytes, cudaMemcpyHostToDevice, s->stream));
-			TG_CUDA(cudaMemsetAsync(s->randf_count, 0, 4 * s->B, s->stream));
-		} else {
-			TG_TRY(tg_state_set_randf(s, randf_host, n_steps));
-		}
-	}
-	for (int b = 0; b < s->B; b++)
-		if (first_ids[b] < 0 || first_ids[b] >= s->m->cfg.n_vocab) return fail(TG_EINVAL, "token id out of range");
-	std::memcpy(s->host_pin, first_ids, 4 * s->B);
-	TG_CUDA(cudaMemcpyAsync(s->tok, s->host_pin, 4 * s->B, cudaMemcpyHostToDevice, s->stream));
-	TG_TRY(tg_generate_async(s, n_steps, minp, temp));
-	if (toks_host && lean) {
-		// (stream order: the ids above were consumed by their copy before this one writes the buffer)
-		TG_CUDA(cudaMemcpyAsync(s->host_pin, s->tok_log, nbytes, cudaMemcpyDeviceToHost, s->stream));
-		TG_TRY(check_err_flag(s));  // synchronises
-		std::memcpy(toks_host, s->host_pin, nbytes);
-		return TG_OK;
-	}
-	if (toks_host) return tg_state_tokens(s, n_steps, toks_host);
-	TG_CUDA(cudaStreamSynchronize(s->stream));
-	return TG_OK;
-}
-
-int tg_kv_read(tg_state *s, int b, int layer, int slot0, int nslots, float *k_host, float *v_host) {
+int tg_kv_read(tg_state *s_, int b, int layer, int slot0, int nslots, float *k_host, float *v_host) {
+	GemmaState *s = as_gemma(s_);
 	if (!s || !k_host || !v_host || b < 0 || b >= s->B || layer < 0 || layer >= s->m->cfg.n_layers)
 		return fail(TG_EINVAL, "bad argument");
 	const int slots = s->slots[layer];
@@ -2641,24 +2194,17 @@ int tg_kv_read(tg_state *s, int b, int layer, int slot0, int nslots, float *k_ho
 	return TG_OK;
 }
 
-int tg_hidden_read(tg_state *s, float *hidden_host) {
-	if (!s || !hidden_host) return fail(TG_EINVAL, "null argument");
-	TG_CUDA(cudaSetDevice(s->m->device));
-	TG_CUDA(cudaMemcpyAsync(hidden_host, s->xnorm, size_t(s->B) * s->m->cfg.hidden_size * 4, cudaMemcpyDeviceToHost, s->stream));
-	TG_CUDA(cudaStreamSynchronize(s->stream));
-	return TG_OK;
-}
-
 // ---------------------------------------------------------------- vocab-sharded lm_head support
-int tg_decode_hidden(tg_state *s, const int *ids) {
-	if (!s) return fail(TG_EINVAL, "null state");
-	tg_model *m = s->m;
+int tg_decode_hidden(tg_state *s_, const int *ids) {
+	GemmaState *s = as_gemma(s_);
+	if (!s) return fail(TG_EINVAL, "not a state of this family");
+	GemmaModel *m = s->m;
 	TG_TRY(check_ready(m));
 	TG_CUDA(cudaSetDevice(m->device));
 	for (int b = 0; b < s->B; b++)
 		if (s->host_pos[b] >= s->max_pos_global) return fail(TG_ESTATE, "global KV cache full (max_pos_global reached)");
 	if (ids) {
-		TG_TRY(staging_acquire(s));
+		TG_TRY(s->staging_acquire());
 		std::memcpy(s->host_pin, ids, 4 * s->B);
 		TG_CUDA(cudaMemcpyAsync(s->tok, s->host_pin, 4 * s->B, cudaMemcpyHostToDevice, s->stream));
 	}
@@ -2667,33 +2213,30 @@ int tg_decode_hidden(tg_state *s, const int *ids) {
 	} else {
 		for (int b0 = 0; b0 < s->B; b0 += MV_MAX_B) TG_TRY(enqueue_decode_chunk(s, b0, std::min(MV_MAX_B, s->B - b0), false));
 	}
-	if (ids) TG_TRY(check_err_flag(s));  // fed from the device: enqueue only, tg_state_check reports the error word later
+	if (ids) TG_TRY(s->check_err_flag());  // fed from the device: enqueue only, tg_state_check reports the error word later
 	for (int b = 0; b < s->B; b++) s->host_pos[b] += 1;
 	return TG_OK;
 }
 
-int tg_state_check(tg_state *s) {
-	if (!s) return fail(TG_EINVAL, "null state");
-	TG_CUDA(cudaSetDevice(s->m->device));
-	return check_err_flag(s);
-}
-
-int tg_dev_hidden_copy(tg_state *s, float *dst_dev) {
-	if (!s || !dst_dev) return fail(TG_EINVAL, "null argument");
+int tg_dev_hidden_copy(tg_state *s_, float *dst_dev) {
+	GemmaState *s = as_gemma(s_);
+	if (!s || !dst_dev) return fail(TG_EINVAL, "null argument, or a handle of another family");
 	TG_CUDA(cudaSetDevice(s->m->device));
 	TG_CUDA(cudaMemcpyAsync(dst_dev, s->xnorm, size_t(s->B) * s->m->cfg.hidden_size * 4, cudaMemcpyDeviceToDevice, s->stream));
 	return TG_OK;
 }
 
-int tg_dev_set_tokens(tg_state *s, const int *toks_dev) {
-	if (!s || !toks_dev) return fail(TG_EINVAL, "null argument");
+int tg_dev_set_tokens(tg_state *s_, const int *toks_dev) {
+	GemmaState *s = as_gemma(s_);
+	if (!s || !toks_dev) return fail(TG_EINVAL, "null argument, or a handle of another family");
 	TG_CUDA(cudaSetDevice(s->m->device));
 	TG_CUDA(cudaMemcpyAsync(s->tok, toks_dev, size_t(s->B) * 4, cudaMemcpyDeviceToDevice, s->stream));
 	return TG_OK;
 }
 
-int tg_dev_lm_head_top1(tg_model *m, const float *hidden_dev, int M, int col0, int ncols, float *max_dev, int *idx_dev,
+int tg_dev_lm_head_top1(tg_model *m_, const float *hidden_dev, int M, int col0, int ncols, float *max_dev, int *idx_dev,
                         void *stream) {
+	GemmaModel *m = as_gemma(m_);
 	if (!m || !hidden_dev || !max_dev || !idx_dev || M < 1) return fail(TG_EINVAL, "bad argument");
 	const int V = m->cfg.n_vocab, D = m->cfg.hidden_size;
 	if (col0 < 0 || ncols < MV_TN || col0 % MV_TN || ncols % MV_TN || col0 + ncols > V)
@@ -2786,7 +2329,7 @@ int tg_dev_resolve_top1(const void *cand_all_dev, int world, int M, int row0, in
 
 // ---------------------------------------------------------------- isolated ops
 int tg_dev_qmatvec(float *y, const float *x, const int8_t *w, const float *scales, int K, int N, void *stream) {
-	if (!y || !x || !w || !scales) return fail(TG_EINVAL, "null argument");
+	if (!y || !x || !w || !scales) return fail(TG_EINVAL, "null argument, or a handle of another family");
 	if (!supported_k(K)) return fail(TG_ESHAPE, "Unsupported ROW dimension: " + std::to_string(K));
 	if (!supported_n(N)) return fail(TG_ESHAPE, "Unsupported COL dimension: " + std::to_string(N));
 	// scratch for split-K, per device, grown on demand
@@ -2847,7 +2390,7 @@ constexpr size_t STATIC_TICKET_BYTES = STATIC_MAX_TILES * sizeof(unsigned);
 static __device__ __align__(256) unsigned char g_static_scratch[STATIC_TICKET_BYTES + STATIC_PARTIAL_FLOATS * sizeof(float)];
 
 int tg_dev_qmatvec_static(float *y, const float *x, const int8_t *w, const float *scales, int K, int N, void *stream) {
-	if (!y || !x || !w || !scales) return fail(TG_EINVAL, "null argument");
+	if (!y || !x || !w || !scales) return fail(TG_EINVAL, "null argument, or a handle of another family");
 	if (N > STATIC_MAX_TILES * MV_TN)
 		return fail(TG_EINVAL, "N = " + std::to_string(N) + " is beyond the static scratch maximum of " +
 		                           std::to_string(STATIC_MAX_TILES * MV_TN) + " columns");
@@ -2972,7 +2515,7 @@ struct DevBuf {
 }  // namespace
 
 int tg_qmatvec(float *y, const float *x, const int8_t *w, const float *scales, int K, int N) {
-	if (!y || !x || !w || !scales) return fail(TG_EINVAL, "null argument");
+	if (!y || !x || !w || !scales) return fail(TG_EINVAL, "null argument, or a handle of another family");
 	if (!supported_k(K)) return fail(TG_ESHAPE, "Unsupported ROW dimension: " + std::to_string(K));
 	if (!supported_n(N)) return fail(TG_ESHAPE, "Unsupported COL dimension: " + std::to_string(N));
 	TG_TRY(ensure_device(0));
@@ -3009,71 +2552,6 @@ int tg_qgemm(float *c, const float *a, const int8_t *w, const float *scales, int
 	return TG_OK;
 }
 
-int tg_argmax_logits(const float *logits, int n, int *tok) {
-	if (!logits || !tok || n < 4 || n % 4) return fail(TG_EINVAL, "bad argument (n must be a multiple of 4)");
-	TG_TRY(ensure_device(0));
-	DevBuf dl, dt, dc;
-	TG_TRY(dl.alloc(size_t(n) * 4));
-	TG_TRY(dt.alloc(4));
-	TG_TRY(dc.alloc(4));
-	TG_CUDA(cudaMemcpy(dl.p, logits, size_t(n) * 4, cudaMemcpyHostToDevice));
-	SampleArgs a{};
-	a.logits = (float *)dl.p;
-	a.V = n;
-	a.tok_out = (int *)dt.p;
-	a.B = 1;
-	argmax_kernel<<<1, SM_THREADS>>>(a);
-	count_launch();
-	TG_TRY(check_launch("argmax"));
-	TG_CUDA(cudaMemcpy(tok, dt.p, 4, cudaMemcpyDeviceToHost));
-	return TG_OK;
-}
-
-int tg_minp_logits(float *logits, int n, float minp, float temp, float randf, int *tok) {
-	if (!logits || !tok || n < MP_CHUNK || n % MP_CHUNK) return fail(TG_EINVAL, "bad argument (n must be a multiple of 8192)");
-	TG_TRY(ensure_device(0));
-	DevBuf dl, dt, dr, dc;
-	TG_TRY(dl.alloc(size_t(n) * 4));
-	TG_TRY(dt.alloc(4));
-	TG_TRY(dr.alloc(4));
-	TG_TRY(dc.alloc(4));
-	TG_CUDA(cudaMemcpy(dl.p, logits, size_t(n) * 4, cudaMemcpyHostToDevice));
-	TG_CUDA(cudaMemcpy(dr.p, &randf, 4, cudaMemcpyHostToDevice));
-	TG_CUDA(cudaMemset(dc.p, 0, 4));
-	SampleArgs a{};
-	a.logits = (float *)dl.p;
-	a.V = n;
-	a.tok_out = (int *)dt.p;
-	a.B = 1;
-	a.minp = minp;
-	a.temp = temp;
-	a.randf = (const float *)dr.p;
-	a.randf_count = (int *)dc.p;
-	a.randf_cap = 1;
-	minp_kernel<<<1, SM_THREADS>>>(a);
-	count_launch();
-	TG_TRY(check_launch("minp"));
-	TG_CUDA(cudaMemcpy(tok, dt.p, 4, cudaMemcpyDeviceToHost));
-	TG_CUDA(cudaMemcpy(logits, dl.p, size_t(n) * 4, cudaMemcpyDeviceToHost));
-	return TG_OK;
-}
-
-int tg_inverse_cdf(const float *p, int n, float cum0, float randf, int *idx, float *cum_out) {
-	if (!p || !idx || n < 1) return fail(TG_EINVAL, "bad argument");
-	TG_TRY(ensure_device(0));
-	DevBuf dp, di, dc;
-	TG_TRY(dp.alloc(size_t(n) * 4));
-	TG_TRY(di.alloc(4));
-	TG_TRY(dc.alloc(4));
-	TG_CUDA(cudaMemcpy(dp.p, p, size_t(n) * 4, cudaMemcpyHostToDevice));
-	inverse_cdf_kernel<<<1, SM_THREADS>>>((const float *)dp.p, n, cum0, randf, (int *)di.p, (float *)dc.p);
-	count_launch();
-	TG_TRY(check_launch("inverse_cdf"));
-	TG_CUDA(cudaMemcpy(idx, di.p, 4, cudaMemcpyDeviceToHost));
-	if (cum_out) TG_CUDA(cudaMemcpy(cum_out, dc.p, 4, cudaMemcpyDeviceToHost));
-	return TG_OK;
-}
-
 int tg_rmsnorm(float *x, const float *w, int rows, int dim) {
 	if (!x || !w || rows < 1 || dim < 1) return fail(TG_EINVAL, "bad argument");
 	TG_TRY(ensure_device(0));
@@ -3089,8 +2567,9 @@ int tg_rmsnorm(float *x, const float *w, int rows, int dim) {
 	return TG_OK;
 }
 
-int tg_state_phase_clocks(tg_state *s, long long *clocks_host, int cap, int *n) {
-	if (!s || !n) return fail(TG_EINVAL, "null argument");
+int tg_state_phase_clocks(tg_state *s_, long long *clocks_host, int cap, int *n) {
+	GemmaState *s = as_gemma(s_);
+	if (!s || !n) return fail(TG_EINVAL, "null argument, or a handle of another family");
 	TG_CUDA(cudaSetDevice(s->m->device));
 	if (!s->mg_dbg) {  // first call arms the recorder; later launches fill it
 		TG_CUDA(cudaMalloc(&s->mg_dbg, 4096 * sizeof(long long)));
@@ -3106,12 +2585,6 @@ int tg_state_phase_clocks(tg_state *s, long long *clocks_host, int cap, int *n) 
 	*n = k;
 	if (clocks_host) std::memcpy(clocks_host, tmp.data(), sizeof(long long) * std::min(cap >= 4096 ? 4096 : k, cap));
 	TG_CUDA(cudaMemset(s->mg_dbg, 0, 4096 * sizeof(long long)));
-	return TG_OK;
-}
-
-int tg_launch_count(int reset, long long *count) {
-	if (count) *count = g_launches.load();
-	if (reset) g_launches.store(0);
 	return TG_OK;
 }
 
