@@ -249,7 +249,8 @@ def test_sliding_window_ring_270m(capi, model_270m, ref_or_none, golden, weights
     assert rel_l2(cases.subsample(logits[0]), g["sw_last_logits"]) <= tol
     # after 8 decode steps slots 0..7 of a local layer hold the new tokens, 8.. the prompt tail
     k, _ = st.kv_read(0, 0, 10)
-    assert rel_max(k, g["sw_l0_k_first10"]) <= 1e-5
+    # (rotated by ~600 positions: tables built by another math library move a key by a few 1e-5)
+    assert rel_max(k, g["sw_l0_k_first10"]) <= (1e-5 if exact_tables else 1e-4)
     assert st.position() == int(g["sw_kv_info_l0"][0]) == 608
     st.close()
 

@@ -110,7 +110,8 @@ struct Run {
 struct HybridModel : tg_model {
 	std::string architecture;
 	int dtype = TG_BF16;
-	int D = 0, Dp = 0, taps = 1;
+	int D = 0, Dp = 0, taps = 1;  // taps of the input convolution
+	bool has_canon = false;
 	float eps = 1e-6f, softcap = 0.0f;
 	std::vector<Layer> layers;
 	std::vector<Run> runs;
@@ -220,7 +221,12 @@ struct Loader {
 		const AttnSpec &A = L.at;
 		DeltaSpec &E = L.de;
 		TG_TRY(vec(p + "norm1", D, &L.norm1));
-		if (m->taps > 1 || st.tensors.count(p + "canon1")) TG_TRY(conv({{p + "canon1", D}}, m->taps, &L.canon));
+		if (m->has_canon) {
+			TG_TRY(conv({{p + "canon1", D}}, m->taps, &L.canon));
+		} else {
+			const std::vector<float> none(D, 0.0f);
+			TG_TRY(upload(none.data(), size_t(D) * 4, reinterpret_cast<void **>(&L.canon)));
+		}
 		const SafeTensors::Tensor *q, *k, *v, *g, *o, *rq, *rk, *rv, *b, *a1, *a2, *g1, *g2, *ro;
 		TG_TRY(get(lp + "q", {A.H * A.dk, D}, &q));
 		TG_TRY(get(lp + "k", {A.G * A.dk, D}, &k));
@@ -347,7 +353,10 @@ int read_config(const json::Value &c, HybridModel *m) {
 	m->n_pos = 1 << 24;  // distances stay exact in fp32
 	m->eps = float(r.num(r.obj(&c, "norm", "model"), "eps", "norm"));
 	m->softcap = float(r.num(&c, "logit_softcap", "model", false, 0.0));
-	if (const json::Value *cn = c.find("canon")) m->taps = r.size(cn, "taps", "canon");
+	if (const json::Value *cn = c.find("canon")) {
+		m->has_canon = true;
+		m->taps = r.size(cn, "taps", "canon");
+	}
 	const json::Value *ls = c.find("layers");
 	if (!ls || ls->kind != json::Value::ARRAY || ls->items.empty()) return fail(TG_EINVAL, "config.json: no layers");
 	for (const auto &l : ls->items) {

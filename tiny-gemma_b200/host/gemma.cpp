@@ -4,6 +4,8 @@
 //   gemma --weights_path W --model_size 270m|1B --prompt "..." --n_dec N [--minp P] --temp T
 //         --chat_format 0|1 --terminate_on_eos 0|1 [--tokenizer_path weights/tokenizer_gemma3.bin] [--seed S]
 //
+// --weights_path may also name a model folder (config.json + model.safetensors); --model_size is then the number
+// format, bfloat16 or float32, and --tokenizer_path a tokenizer of that model's vocabulary.
 // Every option is "--name value"; minp >= 1 (the default 2.0) selects greedy decoding. --seed (not in the
 // reference, which seeds from std::random_device) makes a sampled run repeatable.
 #include <cstdio>
@@ -67,8 +69,8 @@ int main(int argc, char **argv) {
 	app.strings = {{"weights_path", &weights_path}, {"model_size", &model_size}, {"prompt", &prompt}, {"tokenizer_path", &tokenizer_path}};
 	app.ints = {{"n_dec", &n_decode}, {"chat_format", &chat_format}, {"terminate_on_eos", &terminate_on_eos}, {"seed", &seed}};
 	app.floats = {{"minp", &minp}, {"temp", &temp}};
-	opt("weights_path", "File path for model weights.");
-	opt("model_size", "Model size to load.");
+	opt("weights_path", "File path for model weights, or a model folder.");
+	opt("model_size", "Model size to load (270m, 1B), or the number format of a model folder (bfloat16, float32).");
 	opt("prompt", "The prompt.");
 	opt("n_dec", "Number of tokens to generate.");
 	opt("minp", "Minp sampler, defaults to greedy sampling if `minp >= 1`.");
@@ -85,11 +87,16 @@ int main(int argc, char **argv) {
 		return 1;
 	}
 	try {
-		gemma::Config config = gemma::CONFIG_MAP.at(model_size);
-		gemma::Transformer t(config);
-		gemma::read_weights(&t, weights_path.c_str());
+		std::unique_ptr<gemma::Transformer> model;
+		if (model_size == "bfloat16" || model_size == "float32") {
+			model.reset(new gemma::Transformer(weights_path, model_size == "float32" ? TG_F32 : TG_BF16, 0));
+		} else {
+			model.reset(new gemma::Transformer(gemma::CONFIG_MAP.at(model_size)));
+			gemma::read_weights(model.get(), weights_path.c_str());
+		}
+		gemma::Transformer &t = *model;
 		printf("Weights loaded!\n");
-		sentencepiece::Tokenizer tokenizer(tokenizer_path, constants::bos_id, constants::eos_id, constants::vocab, bool(chat_format));
+		sentencepiece::Tokenizer tokenizer(tokenizer_path, constants::bos_id, constants::eos_id, size_t(t.cfg.n_vocab), bool(chat_format));
 		const unsigned useed = unsigned(seed);
 		auto generations = gemma::generate(prompt, n_decode, &tokenizer, &t, minp, temp, bool(terminate_on_eos), seed >= 0 ? &useed : nullptr);
 		const int n_generated_tokens = std::get<0>(generations);

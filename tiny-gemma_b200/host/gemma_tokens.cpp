@@ -5,6 +5,7 @@
 //   sampler -> n_decode x (forward_decode + sampler) -> print ids and tok/s.
 //
 //   gemma_tokens <weights.bin> <270m|1B> <ids.txt> <n_decode> [minp temp seed] [--device-loop]
+//   gemma_tokens <model folder> <bfloat16|float32> <ids.txt> <n_decode> ...   (config.json + model.safetensors)
 // ids.txt: whitespace-separated prompt token ids. minp >= 1 (default 2.0, as
 // gemma.cpp:13) selects greedy decoding.
 #include <chrono>
@@ -15,7 +16,7 @@
 
 int main(int argc, char **argv) {
 	if (argc < 5) {
-		std::fprintf(stderr, "usage: %s weights.bin 270m|1B ids.txt n_decode [minp temp seed] [--device-loop]\n", argv[0]);
+		std::fprintf(stderr, "usage: %s weights.bin 270m|1B ids.txt n_decode [minp temp seed] [--device-loop]\n       %s model_folder bfloat16|float32 ids.txt n_decode [minp temp seed] [--device-loop]\n", argv[0], argv[0]);
 		return 2;
 	}
 	try {
@@ -26,9 +27,15 @@ int main(int argc, char **argv) {
 		const unsigned seed = argc > 7 ? unsigned(std::atol(argv[7])) : 0u;
 		const bool device_loop = argc > 8 && std::string(argv[8]) == "--device-loop";
 
-		config::Config cfg = config::CONFIG_MAP.at(size);  // unknown size -> std::out_of_range, as gemma.cpp:38
-		gemma::Transformer t(cfg);
-		gemma::read_weights(&t, weights.c_str());
+		std::unique_ptr<gemma::Transformer> model;
+		if (size == "bfloat16" || size == "float32") {
+			model.reset(new gemma::Transformer(weights, size == "float32" ? TG_F32 : TG_BF16, 0));
+		} else {
+			model.reset(new gemma::Transformer(config::CONFIG_MAP.at(size)));  // unknown size -> std::out_of_range, as gemma.cpp:38
+			gemma::read_weights(model.get(), weights.c_str());
+		}
+		gemma::Transformer &t = *model;
+		config::Config &cfg = t.cfg;
 
 		std::vector<int> ids;
 		{
@@ -51,10 +58,8 @@ int main(int argc, char **argv) {
 
 		gemma::forward_prefill(&o, &tokens, &t, &d, &rope, &rope_sw, &table);
 		tensor::tokens tok(1, 1);
-		if (minp < 1)
-			ops::minp_logits(&tok, &o, minp, temp, unif(gen));
-		else
-			ops::argmax_logits(&tok, &o);
+		auto sample = [&] { gemma::detail::sample(&tok, &o, &t, &d, minp, temp, minp < 1 ? unif(gen) : 0.0f); };
+		sample();
 		auto t1 = std::chrono::high_resolution_clock::now();
 
 		std::vector<int> out{tok.data[0]};
@@ -64,10 +69,7 @@ int main(int argc, char **argv) {
 		} else {
 			for (int step = 0; step < n_decode; step++) {
 				gemma::forward_decode(&o, &tok, &t, &d, &rope, &rope_sw, ids.size() + step, &table);
-				if (minp < 1)
-					ops::minp_logits(&tok, &o, minp, temp, unif(gen));
-				else
-					ops::argmax_logits(&tok, &o);
+				sample();
 				out.push_back(tok.data[0]);
 			}
 		}

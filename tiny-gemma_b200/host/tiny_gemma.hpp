@@ -213,6 +213,14 @@ struct Transformer {  // transformer.hpp:22-47
 		            cfg.rope_theta_local, cfg.window_pattern};
 		tg_detail::check(tg_model_create(&k, device, &gpu));
 	}
+	// a model folder (config.json + model.safetensors); config.json names the architecture. dtype: TG_BF16 or TG_F32.
+	// Of `cfg` only n_vocab and hidden_size mean something then: tables (RoPE, GeLU) are not inputs of such a model.
+	bool opened = false;
+	Transformer(const std::string &folder, int dtype, int device) : cfg(0, 0, 0, 0, 0, 0, 0, 0, 0, 0.0f, 0.0f, 0), opened(true) {
+		tg_detail::check(tg_model_open(folder.c_str(), device, dtype, &gpu));
+		tg_detail::check(tg_model_vocab(gpu, &cfg.n_vocab));
+		tg_detail::check(tg_model_hidden_size(gpu, &cfg.hidden_size));
+	}
 	Transformer(const Transformer &) = delete;
 	Transformer &operator=(const Transformer &) = delete;
 	~Transformer() { tg_model_free(gpu); }
@@ -223,7 +231,7 @@ inline void read_weights(Transformer *t, const char *file) { tg_detail::check(tg
 
 namespace detail {
 inline void ensure(Transformer *t, decode::DecodeState *d, decode::RoPE *r, decode::RoPE *r_sw, GeLUTable *table) {
-	if (t->tables_from[0] != r || t->tables_from[1] != r_sw || t->tables_from[2] != table) {
+	if (!t->opened && (t->tables_from[0] != r || t->tables_from[1] != r_sw || t->tables_from[2] != table)) {
 		tg_detail::check(tg_model_set_rope(t->gpu, 0, r->freqs_cos.data.get(), r->freqs_sin.data.get(), r->max_pos));
 		tg_detail::check(tg_model_set_rope(t->gpu, 1, r_sw->freqs_cos.data.get(), r_sw->freqs_sin.data.get(), r_sw->max_pos));
 		tg_detail::check(tg_model_set_gelu_table(t->gpu, table->min, table->max, table->table.get(), int(table->table_size)));
@@ -232,6 +240,16 @@ inline void ensure(Transformer *t, decode::DecodeState *d, decode::RoPE *r, deco
 		t->tables_from[2] = table;
 	}
 	if (!d->gpu) tg_detail::check(tg_state_create(t->gpu, d->batch, d->cfg.n_pos, &d->gpu));
+}
+// the token after the prompt, from the logits a forward call has just left
+inline void sample(tensor::tokens *tok, tensor::activation *o, Transformer *t, decode::DecodeState *d, float minp, float temp, float u) {
+	if (t->opened) {  // any vocabulary size: on the device
+		tg_detail::check(minp < 1 ? tg_sample_minp(d->gpu, minp, temp, &u, tok->data.get()) : tg_sample_argmax(d->gpu, tok->data.get()));
+	} else if (minp < 1) {
+		ops_detail::minp(tok, o, minp, temp, u);
+	} else {
+		ops_detail::argmax(tok, o);
+	}
 }
 }  // namespace detail
 
@@ -298,10 +316,7 @@ inline std::tuple<int, std::string, float, float> generate(std::string prompt, i
 	tensor::activation o(1, 1, t->cfg.n_vocab);
 	forward_prefill(&o, &tokens, t, &d, &rope, &rope_sw, &table);
 	tensor::tokens tokens_decode(1, 1);
-	if (minp < 1)
-		ops_detail::minp(&tokens_decode, &o, minp, temp, unif(gen));
-	else
-		ops_detail::argmax(&tokens_decode, &o);
+	detail::sample(&tokens_decode, &o, t, &d, minp, temp, minp < 1 ? unif(gen) : 0.0f);
 	int prev_token = ids[ids.size() - 1];
 	std::cout << tokenizer->decode(tokens_decode.data[0], prev_token) << std::flush;
 	prev_token = tokens_decode.data[0];
