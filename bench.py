@@ -39,6 +39,9 @@ over ranks / max time over ranks.
 Other modes (one JSON line each, 1 GPU):
     python bench.py --phase-clocks [--greedy]   where a decoded token's time goes (in-kernel recorder)
     python bench.py --batched-step --batch B    the batched step alone, from an empty cache
+    python bench.py --nabelix [--model 270m|1B|3B] [--no-extras]
+                                                prefill and decode throughput of the Nabelix design (bf16, random
+                                                weights) beside int8 Gemma-3 of the same width, depth and vocabulary
 """
 
 from __future__ import annotations
@@ -814,6 +817,128 @@ def run_phase_clocks(args):
     return 0
 
 
+# ------------------------------------------------------------------ Nabelix
+def nabelix_work(cfg):
+    """per layer-run sums: bf16 weight bytes, matrix-product FLOPs per token, attention FLOPs per (query, key) pair,
+    delta-rule FLOPs per token, fp32 state bytes, cache bytes per key"""
+    w = dict(weight_bytes=0.0, gemm_flops=0.0, attn_flops=0.0, delta_flops=0.0, state_bytes=0.0, key_bytes=0.0)
+    synth = importlib.import_module("tiny-gemma_b200.synth")
+    for name, shape in synth.nabelix_shapes(cfg):
+        if name == "embed" or len(shape) == 1 or name.endswith(("conv", "canon1")):
+            continue
+        w["weight_bytes"] += 2.0 * shape[0] * shape[1]
+        w["gemm_flops"] += 2.0 * shape[0] * shape[1]
+    for sp in cfg["layers"]:
+        lf, rt = sp["mixer"]["left"], sp["mixer"]["right"]
+        w["attn_flops"] += 2.0 * lf["heads"] * (lf["dim"] + lf["vdim"])
+        w["key_bytes"] += 2.0 * lf["kv_heads"] * (lf["dim"] + lf["vdim"])
+        w["delta_flops"] += 8.0 * rt["heads"] * rt["dim"] * rt["vdim"]
+        w["state_bytes"] += 4.0 * rt["heads"] * rt["dim"] * rt["vdim"]
+    w["head_bytes"] = w["head_flops"] = 2.0 * cfg["vocab"] * cfg["width"]
+    return w
+
+
+def run_nabelix(args):
+    """One JSON line. Weights exceed the L2 (0.6 to 4 GB), so nothing is flushed between iterations. Device times from
+    CUDA events on the state's stream; a prefill's includes the upload of its token ids."""
+    import torch
+
+    if not torch.cuda.is_available():
+        print(json.dumps({"error": "no CUDA device: this benchmark has no CPU path"}), flush=True)
+        return 1
+    importlib.import_module("tiny-gemma_b200.build").build()
+    capi = importlib.import_module("tiny-gemma_b200.capi")
+    synth = importlib.import_module("tiny-gemma_b200.synth")
+    hbm, src = measured_peaks()
+    tf = measured_tensor_peak()
+    sizes = [args.model] if args.no_extras or args.model == "3B" else ["270m", "1B", "3B"]
+    lens = [args.prompt_len] if args.no_extras else [178, 1024, 4096, 16384]
+    steps = args.steps if args.no_extras else 256
+
+    def timed(st, fn, reps):
+        ev = [(torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)) for _ in range(reps)]
+        stream = torch.cuda.ExternalStream(st.stream())
+        out = []
+        for a, b in ev:
+            st.reset()
+            torch.cuda.synchronize()
+            fn[0]()
+            a.record(stream)
+            fn[1]()
+            b.record(stream)
+            torch.cuda.synchronize()
+            out.append(a.elapsed_time(b))
+        return float(np.median(out[1 if reps > 1 else 0:]))
+
+    def measure(model, vocab):
+        res = {"prefill": [], "decode": []}
+        rng = np.random.default_rng(1)
+        for S in lens:
+            st = model.state(1, S + 8)
+            ids = rng.integers(0, vocab, S).astype(np.int32)
+            st.prefill(ids[None], want_logits=False)
+            st.reset()
+            ms = timed(st, (lambda: None, lambda: st.prefill(ids[None], want_logits=False)), 1 if args.repeats == 1 else 6)
+            res["prefill"].append((S, ms))
+            st.close()
+        for B, pos in ([(1, args.prompt_len)] if args.no_extras else [(1, 178), (1, 4096), (4, 178), (32, 178), (256, 178)]):
+            st = model.state(B, pos + steps + 16)
+            ids = np.stack([rng.integers(0, vocab, pos).astype(np.int32) for _ in range(B)])
+
+            def before():
+                st.prefill(ids, want_logits=False)
+                st.sample_argmax()
+                st.generate_async(4)
+
+            ms = timed(st, (before, lambda: st.generate_async(steps)), 1 if args.repeats == 1 else 3)
+            res["decode"].append((B, pos, ms / steps))
+            st.check()
+            st.close()
+        return res
+
+    clocks = ClockSampler(0)
+    clocks.start()
+    rows = []
+    for name in sizes:
+        cfg = synth.nabelix_config(name)
+        w = nabelix_work(cfg)
+        folder = synth.write_random_nabelix(os.path.join(CACHE, "tg_nabelix_%s" % name), cfg)
+        t0 = time.perf_counter()
+        model = capi.Model.open(folder)
+        load_s = time.perf_counter() - t0
+        capi.launch_count(reset=True)
+        r = measure(model, cfg["vocab"])
+        rec = {"size": name, "width": cfg["width"], "ff": cfg["layers"][0]["mlp"]["ff"], "layers": len(cfg["layers"]), "vocab": cfg["vocab"],
+               "weight_gb": (w["weight_bytes"] + w["head_bytes"]) / 1e9, "load_s": load_s, "gpu_launches": capi.launch_count(), "prefill": [], "decode": []}
+        win = cfg["layers"][0]["mixer"]["left"]["mask"]["size"] + cfg["layers"][0]["mixer"]["left"]["mask"]["keep_first"]
+        for S, ms in r["prefill"]:
+            pairs = sum(min(i + 1, win) for i in range(S))
+            fl = S * w["gemm_flops"] + w["head_flops"] + pairs * w["attn_flops"]
+            rec["prefill"].append({"tokens": S, "ms": ms, "tok_s": S / ms * 1e3, "tflops": fl / ms / 1e9, "of_measured_tensor": fl / ms / 1e9 / tf})
+        for B, pos, ms in r["decode"]:
+            keys = min(pos + steps / 2, win)
+            by = w["weight_bytes"] + w["head_bytes"] + B * (2 * w["state_bytes"] + keys * w["key_bytes"])
+            rec["decode"].append({"batch": B, "position": pos, "ms_per_step": ms, "tok_s": B / ms * 1e3, "gbs": by / ms / 1e6, "of_measured_hbm": by / ms / 1e6 / hbm})
+        model.close()
+        if not args.no_extras and name in synth.CONFIGS:
+            gm = capi.Model(name).load_file(synth.write_random_model(os.path.join(CACHE, "tg_%s_s%d.bin" % (name, WEIGHT_SEED)), name, WEIGHT_SEED))
+            gm.build_tables(1024)
+            r = measure(gm, gm.vocab)
+            c = synth.CONFIGS[name]
+            per = c.n_layers * 2.0 * c.hidden_size * (2 * c.q_dim + 2 * c.kv_dim + 3 * c.intermediate_size)
+            rec["gemma_int8"] = {
+                "prefill": [{"tokens": S, "ms": ms, "tok_s": S / ms * 1e3,
+                             "of_measured_tensor": (S * per + 2.0 * c.hidden_size * c.n_vocab) / ms / 1e9 / tf} for S, ms in r["prefill"]],
+                "decode": [{"batch": B, "position": pos, "ms_per_step": ms, "tok_s": B / ms * 1e3,
+                            "of_measured_hbm": (algorithmic_bytes_per_token(c, []) + B * (algorithmic_bytes_per_token(c, [pos + steps // 2]) - algorithmic_bytes_per_token(c, [])))
+                            / ms / 1e6 / hbm} for B, pos, ms in r["decode"]]}
+            gm.close()
+        rows.append(rec)
+    print(json.dumps({"mode": "nabelix", "dtype": "bf16", "data": "synthetic (random weights and token ids)", "steps": steps,
+                      "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": src}, "clocks": clocks.stop(), "sizes": rows}), flush=True)
+    return 0
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -822,8 +947,8 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--batch", type=int, default=1, help="total independent sequences (greedy); >1 selects the batched step")
     ap.add_argument("--no-extras", action="store_true", help="skip the matvec sweep and the CPU baseline sample")
-    ap.add_argument("--model", default=MODEL, choices=["270m", "1B"],
-                    help="architecture; 1B is the benchmark configuration, 270m is the small case used for profiling")
+    ap.add_argument("--model", default=MODEL, choices=["270m", "1B", "3B"],
+                    help="architecture (3B: only with --nabelix); 1B is the benchmark configuration, 270m is the small case used for profiling")
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN,
                     help="prompt tokens; 178 is the benchmark configuration, 16384 the long-context one "
                          "(use --no-extras: the CPU baseline sample would prefill the same prompt)")
@@ -833,7 +958,12 @@ def main():
     ap.add_argument("--phase-clocks", action="store_true", help="per-section timing of one decoded token (in-kernel recorder)")
     ap.add_argument("--greedy", action="store_true", help="with --phase-clocks: argmax instead of the min-p sampler")
     ap.add_argument("--batched-step", action="store_true", help="time the batched step alone (--batch sequences, empty cache)")
+    ap.add_argument("--nabelix", action="store_true", help="throughput of the Nabelix design; with --no-extras only --model at --prompt-len")
     args = ap.parse_args()
+    if args.model == "3B" and not args.nabelix:
+        ap.error("--model 3B needs --nabelix")
+    if args.nabelix:
+        return run_nabelix(args)
     globals()["MODEL"] = args.model
     globals()["PROMPT_LEN"] = args.prompt_len
     if args.impl == "reference":

@@ -192,3 +192,120 @@ def mt19937_uniforms(n: int, seed: int) -> np.ndarray:
     out = words.astype(np.float32) * np.float32(2.0**-32)
     out[out >= np.float32(1.0)] = np.nextafter(np.float32(1.0), np.float32(0.0))
     return out.astype(np.float32)
+
+
+# ------------------------------------------------------------------ Nabelix model folders
+def nabelix_config(name: str) -> dict:
+    """config.json of layers that resemble a real model's: the widths, feed-forward sizes, depths and vocabularies of
+    the Gemma-3 sizes above (a few more weights per layer than theirs), and a wider one"""
+    #          width    ff layers  vocab  left heads/kv  right heads
+    sizes = {"270m": (640, 2048, 18, 262144, 4, 1, 4),
+             "1B": (1152, 6912, 26, 262144, 8, 2, 4),
+             "3B": (2560, 9216, 24, 65536, 20, 4, 20)}
+    width, ff, n, vocab, h, g, r = sizes[name]
+    layer = {"type": "parallel", "mlp": {"kind": "dense", "ff": ff},
+             "mixer": {"left_scale": 1.0, "right_scale": 1.0,
+                       "left": {"heads": h, "kv_heads": g, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                "mask": {"size": 512, "keep_first": 4}},
+                       "right": {"heads": r, "kv_heads": r, "dim": 128, "vdim": 128, "conv": 4}}}
+    return {"architecture": "Nabelix", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "canon": {"taps": 4},
+            "logit_softcap": 30.0, "layers": [layer] * n}
+
+
+NABELIX_RANK = 128  # inner size of the two low-rank projections
+
+
+def nabelix_shapes(cfg: dict):
+    """(tensor name, shape) of every tensor of a Nabelix model"""
+    D, taps = cfg["width"], cfg["canon"]["taps"]
+    yield "embed", (cfg["vocab"], D)
+    for i, sp in enumerate(cfg["layers"]):
+        p, lf, rt = "l%d." % i, sp["mixer"]["left"], sp["mixer"]["right"]
+        yield p + "norm1", (D,)
+        yield p + "canon1", (D, taps)
+        m = p + "mix.left."
+        for n, rows in (("q", lf["heads"] * lf["dim"]), ("k", lf["kv_heads"] * lf["dim"]), ("v", lf["kv_heads"] * lf["vdim"]),
+                        ("g", lf["heads"] * lf["vdim"])):
+            yield m + n, (rows, D)
+        yield m + "r1", (lf["heads"],)
+        yield m + "r2", (lf["heads"],)
+        yield m + "o", (D, lf["heads"] * lf["vdim"])
+        m = p + "mix.right."
+        kc, vc = rt["kv_heads"] * rt["dim"], rt["heads"] * rt["vdim"]
+        for n, rows in (("q", kc), ("k", kc), ("v", vc)):
+            yield m + n, (rows, D)
+            yield m + n + ".conv", (rows, rt["conv"])
+        yield m + "b", (rt["heads"], D)
+        yield m + "A_log", (rt["heads"],)
+        yield m + "dt_bias", (rt["heads"] * rt["dim"],)
+        yield m + "norm", (rt["vdim"],)
+        yield m + "a1", (NABELIX_RANK, D)
+        yield m + "a2", (rt["heads"] * rt["dim"], NABELIX_RANK)
+        yield m + "g1", (NABELIX_RANK, D)
+        yield m + "g2", (vc, NABELIX_RANK)
+        yield m + "o", (D, vc)
+        if sp["mlp"]:
+            yield p + "norm2", (D,)
+            yield p + "mlp.gate", (sp["mlp"]["ff"], D)
+            yield p + "mlp.up", (sp["mlp"]["ff"], D)
+            yield p + "mlp.down", (D, sp["mlp"]["ff"])
+    yield "final.norm", (D,)
+
+
+def write_random_nabelix(folder: str, cfg: dict, seed: int = 0) -> str:
+    """config.json and model.safetensors with seeded random bfloat16 weights. Matrices are N(0, 1/columns), cut from one
+    block of random numbers at random offsets (drawing billions of them would take minutes)."""
+    import json
+
+    done = os.path.join(folder, "model.safetensors")
+    text = json.dumps(cfg)
+    try:
+        with open(os.path.join(folder, "config.json")) as f:
+            if f.read() == text and os.path.exists(done):
+                return folder
+    except OSError:
+        pass
+    os.makedirs(folder, exist_ok=True)
+    if os.path.exists(done):
+        os.unlink(done)
+    g = np.random.default_rng(seed)
+    block = g.standard_normal(1 << 24, dtype=np.float32)
+    shapes = list(nabelix_shapes(cfg))
+    head, at = {}, 0
+    for name, shape in shapes:
+        n = 2 * int(np.prod(shape))
+        head[name] = {"dtype": "BF16", "shape": list(shape), "data_offsets": [at, at + n]}
+        at += n
+    h = json.dumps(head).encode()
+    h += b" " * (-len(h) % 8)
+
+    def bf16(x):
+        b = np.ascontiguousarray(x, np.float32).view(np.uint32)
+        return ((b + np.uint32(0x7FFF) + ((b >> np.uint32(16)) & np.uint32(1))) >> np.uint32(16)).astype("<u2")
+
+    scaled = {}
+    part = done + ".part"
+    with open(part, "wb") as f:
+        f.write(len(h).to_bytes(8, "little") + h)
+        for name, shape in shapes:
+            n = int(np.prod(shape))
+            if len(shape) == 1:
+                leaf = name.rsplit(".", 1)[-1]
+                x = {"A_log": g.uniform(-3, 0, n), "dt_bias": g.uniform(-4, 0, n), "r1": g.uniform(0.1, 1, n), "r2": g.uniform(0.1, 1, n)}.get(
+                    leaf, 1.0 + 0.1 * g.standard_normal(n))
+                f.write(bf16(x).tobytes())
+                continue
+            k = shape[1]
+            if k not in scaled:
+                scaled[k] = bf16(block * np.float32(k ** -0.5))
+            src = scaled[k]
+            o = int(g.integers(0, src.size))
+            while n:
+                c = min(n, src.size - o)
+                f.write(src[o:o + c].tobytes())
+                n -= c
+                o = 0
+    os.replace(part, done)
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        f.write(text)
+    return folder
