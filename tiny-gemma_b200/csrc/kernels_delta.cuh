@@ -16,6 +16,7 @@
 // registers; delta_out_kernel norms and gates the result.
 #pragma once
 #include "kernels_rowwise.cuh"
+#include "tc_common.cuh"
 
 namespace tg {
 
@@ -45,10 +46,9 @@ struct DeltaArgs {
 	int lda2, ldg2;
 	// block quantities, DKP = dk rounded up to 32, 64, 128 or 256
 	int dkp;
-	float *bW, *bQ, *bK;   // [blocks][H][DB][dkp]
-	float *bD;             // [blocks][H][dkp]
-	float *bV;             // [blocks][H][DB][dv]
-	float *bM;             // [blocks][H][DB][DB]
+	float *blk;            // [blocks][H]: W, Q, K [DB][dkp], D [dkp], M [DB][DB] (delta_block_floats)
+	float *bV;             // [blocks][H][DB][dv]: T V
+	int *err;
 	float *o;              // [R][H*dv] raw read-outs
 };
 
@@ -199,12 +199,14 @@ __device__ void delta_token_cta(const DeltaArgs &a, int r, int h, float *sm) {
 // ------------------------------------------------------------------ blocks of a portion
 __host__ __device__ inline int delta_block_base(int seg_row, int seg) { return seg_row / DB + seg; }
 
+__host__ __device__ constexpr size_t delta_block_floats(int dkp) { return size_t(3) * DB * dkp + dkp + DB * DB; }
+
 // smem floats: k, q, g, p [DB][dkp], v [DB][dv], A, M, T [DB][DB], beta [DB]
 __host__ __device__ inline size_t delta_block_smem(int dkp, int dv) { return (size_t(3) * DB * dkp + size_t(DB) * dv + 3 * DB * DB + DB) * 4; }
 
 // grid (blocks of the longest segment, H, segments), 256 threads
 template <typename PT>
-__global__ void __launch_bounds__(256) delta_block_kernel(DeltaArgs a) {
+__global__ void __launch_bounds__(256, 3) delta_block_kernel(DeltaArgs a) {
 	pdl_trigger();
 	pdl_wait();
 	extern __shared__ float db_sm[];
@@ -222,21 +224,33 @@ __global__ void __launch_bounds__(256) delta_block_kernel(DeltaArgs a) {
 	      *sb = sT + DB * DB;
 	// q, k, g, v, beta; tokens past the end change nothing (g = 1, everything else 0)
 	const float ea = expf(a.A_log[h]);
+	for (int i = tid; i < 2 * dkp + dv; i += 256) {  // a thread walks a channel down the block's tokens
+		const int kind = i < dkp ? 0 : (i < 2 * dkp ? 1 : 2), c = kind == 0 ? i : (kind == 1 ? i - dkp : i - 2 * dkp);
+		float *dst = (kind == 0 ? sq : (kind == 1 ? sk : sv)) + c;
+		const int ld = kind == 2 ? dv : dkp;
+		if (kind < 2 && c >= dk) {
+			for (int t = 0; t < DB; t++) dst[t * ld] = 0.0f;
+			continue;
+		}
+		const int ch = kind == 0 ? kh * dk + c : (kind == 1 ? (a.KH + kh) * dk + c : 2 * a.KH * dk + h * dv + c);
+		if (a.taps <= 4) {
+			float x[DB + 3], w[4];
+#pragma unroll
+			for (int j = 0; j < 4; j++) w[j] = j >= 4 - a.taps ? a.cw[size_t(j - (4 - a.taps)) * C + ch] : 0.0f;
+#pragma unroll
+			for (int j = 0; j < DB + 3; j++) x[j] = j - 3 < n && 3 - j < a.taps ? delta_conv_in<PT>(a, row0, pos, hr, C, t0 + j - 3, ch) : 0.0f;
+#pragma unroll
+			for (int t = 0; t < DB; t++) {
+				const float y = fmaf(w[3], x[t + 3], fmaf(w[2], x[t + 2], fmaf(w[1], x[t + 1], w[0] * x[t])));
+				dst[t * ld] = t < n ? __fdividef(y, 1.0f + __expf(-y)) : 0.0f;
+			}
+		} else {
+			for (int t = 0; t < DB; t++) dst[t * ld] = t < n ? delta_conv<PT>(a, row0, pos, hr, C, t0 + t, ch) : 0.0f;
+		}
+	}
 	for (int i = tid; i < DB * dkp; i += 256) {
 		const int t = i / dkp, c = i % dkp;
-		float k = 0.0f, q = 0.0f, g = 1.0f;
-		if (t < n && c < dk) {
-			q = delta_conv<PT>(a, row0, pos, hr, C, t0 + t, kh * dk + c);
-			k = delta_conv<PT>(a, row0, pos, hr, C, t0 + t, (a.KH + kh) * dk + c);
-			g = expf(-ea * softplus_f(a.z[size_t(row0 + t0 + t) * a.ldz + h * dk + c] + a.dt_bias[h * dk + c]));
-		}
-		sk[i] = k;
-		sq[i] = q;
-		sg[i] = g;
-	}
-	for (int i = tid; i < DB * dv; i += 256) {
-		const int t = i / dv, c = i % dv;
-		sv[i] = t < n ? delta_conv<PT>(a, row0, pos, hr, C, t0 + t, 2 * a.KH * dk + h * dv + c) : 0.0f;
+		sg[i] = t < n && c < dk ? expf(-ea * softplus_f(a.z[size_t(row0 + t0 + t) * a.ldz + h * dk + c] + a.dt_bias[h * dk + c])) : 1.0f;
 	}
 	if (tid < DB) sb[tid] = tid < n ? sigmoid_f(to_f32(reinterpret_cast<const PT *>(a.p)[size_t(row0 + t0 + tid) * a.ldp + a.p_b + h])) : 0.0f;
 	if (t0 + DB >= len) {  // the segment's last block
@@ -261,30 +275,45 @@ __global__ void __launch_bounds__(256) delta_block_kernel(DeltaArgs a) {
 		}
 	}
 	__syncthreads();
-	// A and M, column s: p = k_s decayed step by step. A warp takes the columns s = warp and 15 - warp (17 steps in
-	// all for every warp), a lane the channels lane, lane + 32, ...
-	for (int half = 0; half < 2; half++) {
-		const int s = half ? DB - 1 - warp : warp;
-		float p[8];
+	// A and M, columns s1 = warp and s2 = 15 - warp: p = k_s decayed step by step. A lane takes the channels lane,
+	// lane + 32, ...; the four sums of a step are reduced together.
+	{
+		const int s1 = warp, s2 = DB - 1 - warp;
+		float p1[8], p2[8];
 #pragma unroll
-		for (int j = 0; j < 8; j++) p[j] = lane + 32 * j < dkp ? sk[s * dkp + lane + 32 * j] : 0.0f;
-		for (int t = 0; t < s; t++)
-			if (lane == 0) sA[t * DB + s] = sM[t * DB + s] = 0.0f;
-		for (int t = s; t < DB; t++) {
-			float xa = 0.0f, xm = 0.0f;
+		for (int j = 0; j < 8; j++) {
+			p1[j] = lane + 32 * j < dkp ? sk[s1 * dkp + lane + 32 * j] : 0.0f;
+			p2[j] = lane + 32 * j < dkp ? sk[s2 * dkp + lane + 32 * j] : 0.0f;
+		}
+		for (int t = 0; t < DB; t++) {
+			float xa = 0.0f, xm = 0.0f, ya = 0.0f, ym = 0.0f;  // columns s1 (x) and s2 (y) of A and M
+			if (t >= s1) {
 #pragma unroll
-			for (int j = 0; j < 8; j++)
-				if (lane + 32 * j < dkp) {
-					const int i = t * dkp + lane + 32 * j;
-					if (t > s) p[j] *= sg[i];
-					xa = fmaf(sk[i], p[j], xa);
-					xm = fmaf(sq[i], p[j], xm);
-				}
-			xa = warp_sum(xa);
-			xm = warp_sum(xm);
-			if (lane == 0) {
-				sA[t * DB + s] = t > s ? xa : 0.0f;
-				sM[t * DB + s] = xm;
+				for (int j = 0; j < 8; j++)
+					if (32 * j < dkp) {
+						const int i = t * dkp + lane + 32 * j;
+						const float k = sk[i], q = sq[i], g = sg[i];
+						if (t > s1) p1[j] *= g;
+						xa = fmaf(k, p1[j], xa);
+						xm = fmaf(q, p1[j], xm);
+						if (t >= s2) {
+							if (t > s2) p2[j] *= g;
+							ya = fmaf(k, p2[j], ya);
+							ym = fmaf(q, p2[j], ym);
+						}
+					}
+				const bool hi = lane & 16, mid = lane & 8;
+				const float a1 = (hi ? ya : xa) + __shfl_xor_sync(0xffffffffu, hi ? xa : ya, 16), m1 = (hi ? ym : xm) + __shfl_xor_sync(0xffffffffu, hi ? xm : ym, 16);
+				float v = (mid ? m1 : a1) + __shfl_xor_sync(0xffffffffu, mid ? a1 : m1, 8);
+				v += __shfl_xor_sync(0xffffffffu, v, 4);
+				v += __shfl_xor_sync(0xffffffffu, v, 2);
+				v += __shfl_xor_sync(0xffffffffu, v, 1);
+				xa = v;  // lanes 0, 8, 16, 24: A s1, M s1, A s2, M s2
+			}
+			if ((lane & 7) == 0) {
+				const int s = lane & 16 ? s2 : s1;
+				const bool isM = lane & 8;
+				(isM ? sM : sA)[t * DB + s] = (isM ? t >= s : t > s) ? xa : 0.0f;
 			}
 		}
 	}
@@ -301,7 +330,8 @@ __global__ void __launch_bounds__(256) delta_block_kernel(DeltaArgs a) {
 			sT[t * DB + tid] = x[t];
 		}
 	}
-	if (tid >= 64 && tid < 64 + DB * DB / 4) reinterpret_cast<float4 *>(a.bM + bh * DB * DB)[tid - 64] = reinterpret_cast<float4 *>(sM)[tid - 64];
+	float *gW = a.blk + bh * delta_block_floats(dkp), *gQ = gW + DB * dkp, *gK = gQ + DB * dkp, *gD = gK + DB * dkp, *gM = gD + dkp;
+	if (tid >= 64 && tid < 64 + DB * DB / 4) reinterpret_cast<float4 *>(gM)[tid - 64] = reinterpret_cast<float4 *>(sM)[tid - 64];
 	// per channel: D_t k_t, D_t q_t, and the suffix products
 	for (int c = tid; c < dkp; c += 256) {
 		float D = 1.0f, suf[DB];
@@ -312,18 +342,18 @@ __global__ void __launch_bounds__(256) delta_block_kernel(DeltaArgs a) {
 		for (int t = 0; t < DB; t++) {
 			const float k = sk[t * dkp + c];
 			D *= sg[t * dkp + c];
-			a.bK[(bh * DB + t) * dkp + c] = suf[t] * k;
-			a.bQ[(bh * DB + t) * dkp + c] = D * sq[t * dkp + c];
+			gK[t * dkp + c] = suf[t] * k;
+			gQ[t * dkp + c] = D * sq[t * dkp + c];
 			sk[t * dkp + c] = D * k;
 		}
-		a.bD[bh * dkp + c] = D;
+		gD[c] = D;
 	}
 	__syncthreads();
 	// W = T Kt and T V
 	for (int c = tid; c < dkp + dv; c += 256) {
 		const float *src = c < dkp ? sk + c : sv + (c - dkp);
 		const int ld = c < dkp ? dkp : dv;
-		float *dst = c < dkp ? a.bW + bh * DB * dkp + c : a.bV + bh * DB * dv + (c - dkp);
+		float *dst = c < dkp ? gW + c : a.bV + bh * DB * dv + (c - dkp);
 		float x[DB];
 #pragma unroll
 		for (int t = 0; t < DB; t++) x[t] = src[t * ld];
@@ -338,147 +368,207 @@ __global__ void __launch_bounds__(256) delta_block_kernel(DeltaArgs a) {
 }
 
 // ------------------------------------------------------------------ carrying the state through the blocks
-// grid (column groups of 16, H, segments), 128 threads = 4 warps of 4 columns. A lane holds RPL rows of one column:
-// rows 4 (lane & 7) + 32 j + {0..3}; the eight lanes of a column meet by butterflies.
-template <int RPL>
-__global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a) {
+// grid (column groups of 4 NC, H, segments), one warp per CTA. A lane holds RPL rows of NC columns: rows
+// 4 (lane & 7) + 32 j + {0..3} of columns 4 NC x + (lane >> 3) + 4 i; the eight lanes of a column meet by butterflies.
+// The chain over the blocks is sequential, so a CTA is kept as short as possible: the block quantities of a
+// (block, head) are one bulk copy, `stages` of them in flight, and the products run on packed fp32 pairs. Every lane
+// reads every block quantity of its rows from shared memory once per NC columns; that read rate is what bounds an SM.
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+	float2 d;
+	asm("fma.rn.f32x2 %0, %1, %2, %3;"
+	    : "=l"(reinterpret_cast<unsigned long long &>(d))
+	    : "l"(reinterpret_cast<const unsigned long long &>(a)), "l"(reinterpret_cast<const unsigned long long &>(b)), "l"(reinterpret_cast<const unsigned long long &>(c)));
+	return d;
+}
+// (volatile: the loads stay where they are written, ahead of their use)
+__device__ __forceinline__ float4 ds_ld4(const float *p) {
+	float4 v;
+	asm volatile("ld.shared.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(smem_u32(p)) : "memory");
+	return v;
+}
+// acc[16] per lane -> the sums over the 8 lanes of a column for tokens 2 rl, 2 rl + 1
+__device__ __forceinline__ float2 delta_reduce(const float (&acc)[DB], int rl) {
+	float r1[8], r2[4];
+	const bool h4 = rl & 4, h2 = rl & 2, h1 = rl & 1;
+#pragma unroll
+	for (int i = 0; i < 8; i++) r1[i] = (h4 ? acc[8 + i] : acc[i]) + __shfl_xor_sync(0xffffffffu, h4 ? acc[i] : acc[8 + i], 4);
+#pragma unroll
+	for (int i = 0; i < 4; i++) r2[i] = (h2 ? r1[4 + i] : r1[i]) + __shfl_xor_sync(0xffffffffu, h2 ? r1[i] : r1[4 + i], 2);
+	float2 o;
+	o.x = (h1 ? r2[2] : r2[0]) + __shfl_xor_sync(0xffffffffu, h1 ? r2[0] : r2[2], 1);
+	o.y = (h1 ? r2[3] : r2[1]) + __shfl_xor_sync(0xffffffffu, h1 ? r2[1] : r2[3], 1);
+	return o;
+}
+constexpr int DS_MAX_STAGES = 4;
+template <int RPL, int NC> size_t delta_scan_smem(int stages) { return (size_t(stages) * delta_block_floats(8 * RPL) + 4 * NC * 20) * 4; }
+
+template <int RPL, int NC>
+__global__ void __launch_bounds__(32) delta_scan_kernel(DeltaArgs a, int stages) {
 	pdl_trigger();
-	pdl_wait();
 	constexpr int DKP = 8 * RPL;
-	constexpr int STAGE = 3 * DB * DKP + DKP + DB * DB + DB * 16;  // W, Q, K, D, M, V columns
-	extern __shared__ __align__(16) float ds_sm[];
-	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-	const int h = blockIdx.y, seg = blockIdx.z, c0 = blockIdx.x * 16;
+	constexpr size_t BF = delta_block_floats(DKP);
+	extern __shared__ __align__(128) float ds_sm[];
+	__shared__ uint64_t full_bar[DS_MAX_STAGES];
+	const int lane = threadIdx.x;
+	const int h = blockIdx.y, seg = blockIdx.z, rl = lane & 7, cl = lane >> 3;
+	float *su = ds_sm + size_t(stages) * BF;  // [4 NC columns][20]
+	if (lane == 0) {
+		for (int i = 0; i < stages; i++) mbar_init(&full_bar[i], 1);
+		asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+	}
+	__syncwarp();
+	pdl_wait();
 	const int len = a.d.seg_len[seg], row0 = a.d.seg_row[seg], pos = a.d.seg_pos[seg], seq = a.d.seg_seq[seg];
 	const int nb = (len + DB - 1) / DB, dk = a.dk, dv = a.dv;
-	const int rl = lane & 7, c = c0 + warp * 4 + (lane >> 3);
-	const bool on = c < dv;
 	const size_t blk0 = delta_block_base(row0, seg);
-	float S[RPL];
+	auto fetch = [&](int b) {
+		if (lane == 0) {
+			fence_proxy_async();
+			mbar_expect_tx(&full_bar[b % stages], uint32_t(BF * 4));
+			asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(ds_sm + size_t(b % stages) * BF)),
+			             "l"(a.blk + ((blk0 + b) * a.H + h) * BF), "r"(uint32_t(BF * 4)), "r"(smem_u32(&full_bar[b % stages]))
+			             : "memory");
+		}
+	};
+	int issued = min(stages - 1, nb);
+	for (int b = 0; b < issued; b++) fetch(b);
+	int col[NC];
+	float2 S[NC][RPL / 2];
 	float *Sg = a.S + (size_t(seq) * a.H + h) * dk * dv;
 #pragma unroll
-	for (int j = 0; j < RPL; j++) {
-		const int i = 4 * rl + 32 * (j >> 2) + (j & 3);
-		S[j] = (on && pos > 0 && i < dk) ? Sg[size_t(i) * dv + c] : 0.0f;
+	for (int x = 0; x < NC; x++) {
+		col[x] = (blockIdx.x * NC + x) * 4 + cl;
+#pragma unroll
+		for (int j = 0; j < RPL / 2; j++) {
+			const int i = 4 * rl + 32 * (j >> 1) + 2 * (j & 1);
+			S[x][j].x = (pos > 0 && col[x] < dv && i < dk) ? Sg[size_t(i) * dv + col[x]] : 0.0f;
+			S[x][j].y = (pos > 0 && col[x] < dv && i + 1 < dk) ? Sg[size_t(i + 1) * dv + col[x]] : 0.0f;
+		}
 	}
-	auto fetch = [&](int b) {
-		float *st = ds_sm + (b & 1) * STAGE;
-		const size_t bh = (blk0 + b) * a.H + h;
-		auto cp = [&](float *dst, const float *src, int n4) {
-			for (int i = tid; i < n4; i += 128)
-				asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(uint32_t(__cvta_generic_to_shared(dst + 4 * i))), "l"(src + 4 * i) : "memory");
-		};
-		cp(st, a.bW + bh * DB * DKP, DB * DKP / 4);
-		cp(st + DB * DKP, a.bQ + bh * DB * DKP, DB * DKP / 4);
-		cp(st + 2 * DB * DKP, a.bK + bh * DB * DKP, DB * DKP / 4);
-		cp(st + 3 * DB * DKP, a.bD + bh * DKP, DKP / 4);
-		cp(st + 3 * DB * DKP + DKP, a.bM + bh * DB * DB, DB * DB / 4);
-		float *v = st + 3 * DB * DKP + DKP + DB * DB;
-		for (int i = tid; i < DB * 16; i += 128) {
-			const int t = i >> 4, cc = c0 + (i & 15);
-			if (cc < dv)
-				asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(uint32_t(__cvta_generic_to_shared(v + i))), "l"(a.bV + (bh * DB + t) * dv + cc) : "memory");
-			else
-				v[i] = 0.0f;
-		}
-		asm volatile("cp.async.commit_group;" ::: "memory");
+	float2 v[NC];
+	auto load_v = [&](int b) {
+		const float *vb = a.bV + ((blk0 + b) * a.H + h) * DB * dv + size_t(2 * rl) * dv;
+#pragma unroll
+		for (int x = 0; x < NC; x++) v[x] = col[x] < dv ? make_float2(vb[col[x]], vb[dv + col[x]]) : make_float2(0.0f, 0.0f);
 	};
-	fetch(0);
+	load_v(0);
 	for (int b = 0; b < nb; b++) {
-		if (b + 1 < nb) {
-			fetch(b + 1);
-			asm volatile("cp.async.wait_group 1;" ::: "memory");
-		} else {
-			asm volatile("cp.async.wait_group 0;" ::: "memory");
+		if (issued < nb) fetch(issued++);
+		if (!__all_sync(0xffffffffu, tc_wait(&full_bar[b % stages], (b / stages) & 1, a.err))) {
+			for (int q = b + 1; q < issued; q++) tc_wait(&full_bar[q % stages], (q / stages) & 1, a.err);  // copies in flight land first
+			break;
 		}
-		__syncthreads();
-		const float *st = ds_sm + (b & 1) * STAGE;
-		const float *sW = st, *sQ = st + DB * DKP, *sK = st + 2 * DB * DKP, *sD = st + 3 * DB * DKP, *sM = sD + DKP, *sV = sM + DB * DB;
-		// dots of every token's W and Q with this column of S: acc[t] = W_t . S, acc[16 + t] = Q_t . S
-		float acc[2 * DB];
+		const float *sW = ds_sm + size_t(b % stages) * BF, *sD = sW + 3 * DB * DKP, *sM = sD + DKP;
+		// W, Q and K are read as one stream of groups of TG token rows, a group ahead of its use: a warp alone on its
+		// scheduler has nobody else to hide the latency of shared memory
+		constexpr int TG = RPL >= 32 ? 2 : 4, GR = DB / TG;
+		float4 cur[TG][RPL / 4], nxt[TG][RPL / 4];
+		auto rows = [&](int g, float4 (&w)[TG][RPL / 4]) {  // g: 0 .. 3 GR - 1 (W, Q and K lie one after the other)
 #pragma unroll
-		for (int t = 0; t < DB; t++) {
-			float x = 0.0f, y = 0.0f;
+			for (int t = 0; t < TG; t++)
 #pragma unroll
-			for (int j = 0; j < RPL / 4; j++) {
-				const float4 w = *reinterpret_cast<const float4 *>(sW + t * DKP + 4 * rl + 32 * j);
-				const float4 q = *reinterpret_cast<const float4 *>(sQ + t * DKP + 4 * rl + 32 * j);
-				x = fmaf(w.x, S[4 * j], x); x = fmaf(w.y, S[4 * j + 1], x); x = fmaf(w.z, S[4 * j + 2], x); x = fmaf(w.w, S[4 * j + 3], x);
-				y = fmaf(q.x, S[4 * j], y); y = fmaf(q.y, S[4 * j + 1], y); y = fmaf(q.z, S[4 * j + 2], y); y = fmaf(q.w, S[4 * j + 3], y);
-			}
-			acc[t] = x;
-			acc[DB + t] = y;
+				for (int j = 0; j < RPL / 4; j++) w[t][j] = ds_ld4(sW + (g * TG + t) * DKP + 4 * rl + 32 * j);
+		};
+		float acc[NC][DB];
+		auto dots = [&](int g) {
+#pragma unroll
+			for (int t = 0; t < TG; t++)
+#pragma unroll
+				for (int x = 0; x < NC; x++) {
+					float2 s = make_float2(0.0f, 0.0f);
+#pragma unroll
+					for (int j = 0; j < RPL / 4; j++) {
+						s = fma2(make_float2(cur[t][j].x, cur[t][j].y), S[x][2 * j], s);
+						s = fma2(make_float2(cur[t][j].z, cur[t][j].w), S[x][2 * j + 1], s);
+					}
+					acc[x][(g % GR) * TG + t] = s.x + s.y;
+				}
+		};
+		auto shift = [&] {
+#pragma unroll
+			for (int t = 0; t < TG; t++)
+#pragma unroll
+				for (int j = 0; j < RPL / 4; j++) cur[t][j] = nxt[t][j];
+		};
+		rows(0, cur);
+#pragma unroll
+		for (int g = 0; g < GR; g++) {
+			rows(g + 1, nxt);
+			dots(g);
+			shift();
 		}
-		// reduce over the 8 lanes of the column; lane rl ends with tokens 2 rl, 2 rl + 1 of both
-		float w2[2], q2[2];
-		{
-			float r1[DB];
-			const bool hi4 = rl & 4;
 #pragma unroll
-			for (int i = 0; i < 8; i++) {  // tokens (hi4 ? 8 + i : i)
-				const float sw = hi4 ? acc[i] : acc[8 + i], kw = hi4 ? acc[8 + i] : acc[i];
-				const float sq = hi4 ? acc[DB + i] : acc[DB + 8 + i], kq = hi4 ? acc[DB + 8 + i] : acc[DB + i];
-				r1[i] = kw + __shfl_xor_sync(0xffffffffu, sw, 4);
-				r1[8 + i] = kq + __shfl_xor_sync(0xffffffffu, sq, 4);
-			}
-			float r2[8];
-			const bool hi2 = rl & 2;
-#pragma unroll
-			for (int i = 0; i < 4; i++) {
-				const float sw = hi2 ? r1[i] : r1[4 + i], kw = hi2 ? r1[4 + i] : r1[i];
-				const float sq = hi2 ? r1[8 + i] : r1[12 + i], kq = hi2 ? r1[12 + i] : r1[8 + i];
-				r2[i] = kw + __shfl_xor_sync(0xffffffffu, sw, 2);
-				r2[4 + i] = kq + __shfl_xor_sync(0xffffffffu, sq, 2);
-			}
-			const bool hi1 = rl & 1;
-#pragma unroll
-			for (int i = 0; i < 2; i++) {
-				const float sw = hi1 ? r2[i] : r2[2 + i], kw = hi1 ? r2[2 + i] : r2[i];
-				const float sq = hi1 ? r2[4 + i] : r2[6 + i], kq = hi1 ? r2[6 + i] : r2[4 + i];
-				w2[i] = kw + __shfl_xor_sync(0xffffffffu, sw, 1);
-				q2[i] = kq + __shfl_xor_sync(0xffffffffu, sq, 1);
-			}
+		for (int x = 0; x < NC; x++) {
+			const float2 dw = delta_reduce(acc[x], rl);
+			*reinterpret_cast<float2 *>(su + (4 * x + cl) * 20 + 2 * rl) = make_float2(v[x].x - dw.x, v[x].y - dw.y);
 		}
-		const int vc = warp * 4 + (lane >> 3);
-		float u2[2];
-		u2[0] = sV[(2 * rl) * 16 + vc] - w2[0];
-		u2[1] = sV[(2 * rl + 1) * 16 + vc] - w2[1];
-		// every lane needs all of the column's u
-		float u[DB];
+		if (b + 1 < nb) load_v(b + 1);
+		float2 dq[NC];
 #pragma unroll
-		for (int t = 0; t < DB; t++) u[t] = __shfl_sync(0xffffffffu, u2[t & 1], (lane & 24) + (t >> 1));
-		if (on) {
+		for (int g = GR; g < 2 * GR; g++) {
+			rows(g + 1, nxt);
+			dots(g);
+			shift();
+		}
 #pragma unroll
-			for (int i = 0; i < 2; i++) {
-				const int t = 2 * rl + i;
-				float o = q2[i];
+		for (int x = 0; x < NC; x++) dq[x] = delta_reduce(acc[x], rl);
+		__syncwarp();
+		const float4 *m0 = reinterpret_cast<const float4 *>(sM + 2 * rl * DB);
 #pragma unroll
-				for (int s = 0; s < DB; s++) o = fmaf(sM[t * DB + s], u[s], o);  // (zero above the diagonal)
-				if (b * DB + t < len) a.o[size_t(row0 + b * DB + t) * a.H * dv + h * dv + c] = o;
+		for (int x = 0; x < NC; x++) {
+			float u[DB];
+#pragma unroll
+			for (int i = 0; i < 4; i++) *reinterpret_cast<float4 *>(&u[4 * i]) = *reinterpret_cast<const float4 *>(su + (4 * x + cl) * 20 + 4 * i);
+			float2 o = dq[x];
+#pragma unroll
+			for (int i = 0; i < 4; i++) {  // (M is zero above the diagonal)
+				const float4 p = m0[i], q = m0[4 + i];
+				o.x = fmaf(p.x, u[4 * i], o.x); o.x = fmaf(p.y, u[4 * i + 1], o.x); o.x = fmaf(p.z, u[4 * i + 2], o.x); o.x = fmaf(p.w, u[4 * i + 3], o.x);
+				o.y = fmaf(q.x, u[4 * i], o.y); o.y = fmaf(q.y, u[4 * i + 1], o.y); o.y = fmaf(q.z, u[4 * i + 2], o.y); o.y = fmaf(q.w, u[4 * i + 3], o.y);
+			}
+			const int t = b * DB + 2 * rl;
+			if (col[x] < dv) {
+				float *dst = a.o + size_t(row0 + t) * a.H * dv + h * dv + col[x];
+				if (t < len) dst[0] = o.x;
+				if (t + 1 < len) dst[size_t(a.H) * dv] = o.y;
 			}
 		}
 #pragma unroll
 		for (int j = 0; j < RPL / 4; j++) {
 			const float4 g = *reinterpret_cast<const float4 *>(sD + 4 * rl + 32 * j);
-			S[4 * j] *= g.x; S[4 * j + 1] *= g.y; S[4 * j + 2] *= g.z; S[4 * j + 3] *= g.w;
+#pragma unroll
+			for (int x = 0; x < NC; x++) {
+				S[x][2 * j].x *= g.x; S[x][2 * j].y *= g.y;
+				S[x][2 * j + 1].x *= g.z; S[x][2 * j + 1].y *= g.w;
+			}
 		}
 #pragma unroll
-		for (int t = 0; t < DB; t++)
+		for (int g = 2 * GR; g < 3 * GR; g++) {
+			if (g + 1 < 3 * GR) rows(g + 1, nxt);
 #pragma unroll
-			for (int j = 0; j < RPL / 4; j++) {
-				const float4 k = *reinterpret_cast<const float4 *>(sK + t * DKP + 4 * rl + 32 * j);
-				S[4 * j] = fmaf(k.x, u[t], S[4 * j]); S[4 * j + 1] = fmaf(k.y, u[t], S[4 * j + 1]);
-				S[4 * j + 2] = fmaf(k.z, u[t], S[4 * j + 2]); S[4 * j + 3] = fmaf(k.w, u[t], S[4 * j + 3]);
-			}
-		__syncthreads();
+			for (int t = 0; t < TG; t++)
+#pragma unroll
+				for (int x = 0; x < NC; x++) {
+					const float u = su[(4 * x + cl) * 20 + (g - 2 * GR) * TG + t];
+#pragma unroll
+					for (int j = 0; j < RPL / 4; j++) {
+						S[x][2 * j] = fma2(make_float2(cur[t][j].x, cur[t][j].y), make_float2(u, u), S[x][2 * j]);
+						S[x][2 * j + 1] = fma2(make_float2(cur[t][j].z, cur[t][j].w), make_float2(u, u), S[x][2 * j + 1]);
+					}
+				}
+			if (g + 1 < 3 * GR) shift();
+		}
+		__syncwarp();
 	}
 #pragma unroll
-	for (int j = 0; j < RPL; j++) {
-		const int i = 4 * rl + 32 * (j >> 2) + (j & 3);
-		if (on && i < dk) Sg[size_t(i) * dv + c] = S[j];
-	}
+	for (int x = 0; x < NC; x++)
+#pragma unroll
+		for (int j = 0; j < RPL / 2; j++) {
+			const int i = 4 * rl + 32 * (j >> 1) + 2 * (j & 1);
+			if (col[x] < dv && i < dk) Sg[size_t(i) * dv + col[x]] = S[x][j].x;
+			if (col[x] < dv && i + 1 < dk) Sg[size_t(i + 1) * dv + col[x]] = S[x][j].y;
+		}
 }
-template <int RPL> constexpr size_t delta_scan_smem() { return size_t(2) * (3 * DB * 8 * RPL + 8 * RPL + DB * DB + DB * 16) * 4; }
 
 // out = rms_norm(o) * norm * sigmoid(gz) * out_scale: a warp per (row, head)
 template <typename OT>

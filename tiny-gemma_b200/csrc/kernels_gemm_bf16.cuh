@@ -181,6 +181,19 @@ __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 		int n = 0;
 		for (int t = blockIdx.x; t < tiles && !*(volatile int *)&s_fail; t += gridDim.x, n++) {
 			const int buf = n & 1;
+			// the residual values of a block of 32 columns are requested one block ahead (and the first before the
+			// accumulator is complete)
+			float4 res[8];
+			auto request = [&](int c) {
+				const int rr0 = (t % a.m_tiles) * GB_BM + quad * 32, col = (t / a.m_tiles) * BN + c * 32 + (lane & 7) * 4;
+#pragma unroll
+				for (int i = 0; i < 8; i++) {
+					const int row = rr0 + 4 * i + (lane >> 3);
+					res[i] = (c < BN / 32 && row < a.M && col < a.N) ? *reinterpret_cast<const float4 *>(reinterpret_cast<const float *>(a.C) + size_t(row) * a.ldc + col)
+					                                               : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+				}
+			};
+			if (EPI == GEMM_ADD) request(0);
 			if (!tc_wait(&acc_full[buf], (n >> 1) & 1, a.err)) {
 				s_fail = 1;
 				break;
@@ -227,6 +240,12 @@ __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 						}
 					} else {
 						const int cc = (lane & 7) * 4;
+						float4 add[8];
+						if (EPI == GEMM_ADD) {
+#pragma unroll
+							for (int i = 0; i < 8; i++) add[i] = res[i];
+							request(c + 1);
+						}
 #pragma unroll
 						for (int i = 0; i < 8; i++) {
 							const int rr = 4 * i + (lane >> 3);
@@ -234,8 +253,7 @@ __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 								float4 v = *reinterpret_cast<const float4 *>(stg + rr * 36 + cc);
 								float4 *dst = reinterpret_cast<float4 *>(reinterpret_cast<float *>(a.C) + size_t(r0 + rr) * a.ldc + col + cc);
 								if (EPI == GEMM_ADD) {
-									const float4 x = *dst;
-									v.x += x.x; v.y += x.y; v.z += x.z; v.w += x.w;
+									v.x += add[i].x; v.y += add[i].y; v.z += add[i].z; v.w += add[i].w;
 								}
 								if (EPI == GEMM_LOGITS) {
 									v.x = col + cc < a.N ? soft_cap(v.x, a.cap) : -INFINITY;

@@ -114,35 +114,55 @@ static __global__ void __launch_bounds__(128) window_attn_kernel(WAttnArgs a, in
 }
 
 // ------------------------------------------------------------------ portions, tensor cores
-// Warps 0-3: softmax, a thread per query row. Warp 4: TMA (Q once, then K and V tiles of 64 keys through one ring).
-// Warp 5: issues the MMAs in the order QK(t+1), PV(t), with S double-buffered in TMEM. P goes through shared memory
-// (one buffer: P(t+1) waits for PV(t)); O stays in TMEM and is rescaled there only when a row's running maximum has
-// grown by more than 8 (powers of two), the sums staying exact for any reference maximum.
-constexpr int WT_THREADS = 192, WT_KEYS = 64;
+// Warps 0-7: softmax, two threads per query row (32 keys of a tile each; they exchange their maxima through shared
+// memory). Warp 8: TMA (Q once, then K and V tiles of 64 keys through one ring). Warp 9: issues the MMAs in the order QK(t+1), PV(t), with S double-buffered in TMEM, so that the softmax of a tile
+// runs under the MMAs of its neighbours (and two CTAs share an SM where their tiles fit). P replaces S in TMEM, as the
+// bf16 operand of PV; O stays in TMEM and is rescaled there only when a row's running maximum has grown by more than 8
+// (powers of two), the sums staying exact for any reference maximum. The distance bias within the window is a table in shared memory
+// (lanes of consecutive queries read consecutive words); kept tokens, and windows the table does not reach, evaluate it.
+constexpr int WT_THREADS = 320, WT_KEYS = 64, WT_TABLE = 2304;
+// D += A B with A in TMEM (row = lane, two bf16 per 32-bit column)
+__device__ __forceinline__ void tc_mma_ta(uint32_t d_tmem, uint32_t a_tmem, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+	asm volatile(
+	    "{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
+	    "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}" ::"r"(d_tmem),
+	    "r"(a_tmem), "l"(bdesc), "r"(idesc), "r"(accumulate)
+	    : "memory");
+}
+// 16 columns of this warp's 32 TMEM lanes, complete on return
+__device__ __forceinline__ void wt_ld16(uint32_t taddr, uint32_t (&o)[16]) {
+	asm volatile(
+	    "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+	    : "=r"(o[0]), "=r"(o[1]), "=r"(o[2]), "=r"(o[3]), "=r"(o[4]), "=r"(o[5]), "=r"(o[6]), "=r"(o[7]), "=r"(o[8]), "=r"(o[9]), "=r"(o[10]), "=r"(o[11]),
+	      "=r"(o[12]), "=r"(o[13]), "=r"(o[14]), "=r"(o[15])
+	    : "r"(taddr)
+	    : "memory");
+	asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+}
+__device__ __forceinline__ float ex2_f(float x) {
+	float y;
+	asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+	return y;
+}
 struct WtShape {
-	int q_bytes, k_bytes, v_bytes, stage, ns, p_off, total;
+	int q_bytes, k_bytes, v_bytes, stage, ns, table, total;  // table: entries of the bias table (0: none)
 };
 __host__ __device__ inline int wt_chunks(int d) { return (d + 63) / 64; }
-__host__ __device__ inline WtShape wt_shape(int dkp, int dvp) {
+__host__ __device__ inline WtShape wt_shape(int dkp, int dvp, int window) {
 	WtShape s;
 	s.q_bytes = wt_chunks(dkp) * 128 * 128;
 	s.k_bytes = wt_chunks(dkp) * WT_KEYS * 128;
 	s.v_bytes = wt_chunks(dvp) * WT_KEYS * 128;
 	s.stage = s.k_bytes > s.v_bytes ? s.k_bytes : s.v_bytes;
-	const int p = 128 * 128;
-	// two CTAs per SM where three stages allow it, else as deep as one CTA's shared memory goes (at most 4)
-	s.ns = 3;
-	if (s.q_bytes + p + 3 * s.stage + 1024 > 110 * 1024) {
-		s.ns = 4;
-		while (s.ns > 2 && s.q_bytes + p + s.ns * s.stage + 1024 > 220 * 1024) s.ns--;
-	}
-	s.p_off = s.q_bytes + s.ns * s.stage;
-	s.total = s.p_off + p + 1024;
+	s.ns = 4;  // two CTAs per SM where four stages allow it; fewer stages only where one CTA's shared memory ends
+	s.table = window + 256 <= WT_TABLE ? window + 256 : 0;
+	while (s.ns > 2 && s.q_bytes + s.ns * s.stage + 4 * s.table + 1024 > 220 * 1024) s.ns--;
+	s.total = s.q_bytes + s.ns * s.stage + 4 * s.table + 1024;
 	return s;
 }
-__host__ __device__ inline int wt_tmem_cols(int dvp) { return dvp <= 128 ? 256 : 512; }  // O, then two S buffers of 64
+__host__ __device__ inline int wt_tmem_cols(int dvp) { return dvp <= 128 ? 256 : 512; }  // O, then two S (and P) buffers of 64
 
-static __global__ void __launch_bounds__(WT_THREADS) window_attn_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap kmap,
+static __global__ void __launch_bounds__(WT_THREADS, 2) window_attn_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap kmap,
                                                                            const __grid_constant__ CUtensorMap vmap, const __grid_constant__ CUtensorMap ksmap,
                                                                            const __grid_constant__ CUtensorMap vsmap, WAttnArgs a) {
 	pdl_trigger();
@@ -151,9 +171,9 @@ static __global__ void __launch_bounds__(WT_THREADS) window_attn_tc_kernel(const
 	__shared__ uint64_t q_bar, full_bar[4], free_bar[4], s_bar[2], p_bar, pv_bar;
 	__shared__ uint32_t tmem_base_s;
 	__shared__ int s_fail, s_issued;
-	__shared__ float s_bias[2][192];
+	__shared__ float s_max[2][2][128];  // [tile parity][half of the row][row]
 	const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-	const WtShape sh = wt_shape(a.dkp, a.dvp);
+	const WtShape sh = wt_shape(a.dkp, a.dvp, a.window);
 	const int ncols = wt_tmem_cols(a.dvp);
 	if (tid == 0) {
 		mbar_init(&q_bar, 1);
@@ -163,13 +183,13 @@ static __global__ void __launch_bounds__(WT_THREADS) window_attn_tc_kernel(const
 		}
 		mbar_init(&s_bar[0], 1);
 		mbar_init(&s_bar[1], 1);
-		mbar_init(&p_bar, 4);
+		mbar_init(&p_bar, 8);
 		mbar_init(&pv_bar, 1);
 		s_fail = 0;
 		s_issued = 0;
 		asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
 	}
-	if (warp == 5) {
+	if (warp == 9) {
 		asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_base_s)), "r"(ncols) : "memory");
 		asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
 	}
@@ -193,7 +213,7 @@ static __global__ void __launch_bounds__(WT_THREADS) window_attn_tc_kernel(const
 		const int kch = wt_chunks(a.dkp), vch = wt_chunks(a.dvp);
 		auto stage = [&](int n) { return smem + sh.q_bytes + (n % sh.ns) * sh.stage; };
 
-		if (warp == 4) {
+		if (warp == 8) {
 			if (lane == 0) {
 				mbar_expect_tx(&q_bar, uint32_t(sh.q_bytes));
 				for (int c = 0; c < kch; c++) tma_load_2d(smem + c * 128 * 128, &qmap, a.p_q + h * a.dkp + 64 * c, row0 + qt * 128, &q_bar);
@@ -213,7 +233,7 @@ static __global__ void __launch_bounds__(WT_THREADS) window_attn_tc_kernel(const
 					s_issued = n + 1;
 				}
 			}
-		} else if (warp == 5) {
+		} else if (warp == 9) {
 			if (lane == 0) {
 				const uint32_t id_s = tc_idesc_bf16(WT_KEYS, 0), id_o = tc_idesc_bf16(a.dvp, 1);
 				auto qk = [&](int t) -> bool {
@@ -236,22 +256,28 @@ static __global__ void __launch_bounds__(WT_THREADS) window_attn_tc_kernel(const
 					ok = ok && tc_wait(&p_bar, t & 1, a.err) && tc_wait(&full_bar[n % sh.ns], (n / sh.ns) & 1, a.err);
 					if (!ok) break;
 					tc_fence_after();
-					const uint32_t pa = smem_u32(smem + sh.p_off), va = smem_u32(stage(n));
+					const uint32_t va = smem_u32(stage(n)), pt = tmem + s_off + uint32_t((t & 1) * 64);
 					for (int j = 0; j < WT_KEYS / 16; j++)
-						tc_mma(tmem, tc_sw128_desc(pa + j * 32, 16, 1024), tc_sw128_desc(va + j * 2048, WT_KEYS * 128, 1024), id_o, (t > 0 || j > 0) ? 1u : 0u);
+						tc_mma_ta(tmem, pt + uint32_t(j * 8), tc_sw128_desc(va + j * 2048, WT_KEYS * 128, 1024), id_o, (t > 0 || j > 0) ? 1u : 0u);
 					tc_commit(&free_bar[n % sh.ns]);
 					tc_commit(&pv_bar);
 				}
 				if (!ok) s_fail = 1;
 			}
 		} else {
-			const int i = i_lo + tid;  // this thread's query (rows past nq compute and are not stored)
-			const uint32_t lane_addr = uint32_t(warp * 32) << 16;
+			const int row = tid & 127, half = tid >> 7, quad = warp & 3;
+			const int i = i_lo + row;  // this thread's query (rows past nq compute and are not stored)
+			const uint32_t lane_addr = uint32_t(quad * 32) << 16, s_col = s_off + uint32_t(half * 32), p_col = s_off + uint32_t(half * 16);
 			const float LOG2E = 1.4426950408889634f;
 			const float sc = a.scale * LOG2E;
 			const float r1 = a.r1 ? a.r1[h] : 0.0f, r2 = a.r1 ? a.r2[h] : 0.0f;
+			// minus the bias (in powers of two) of distance x - 64
+			float *tab = reinterpret_cast<float *>(smem + sh.q_bytes + sh.ns * sh.stage);
+			if (a.r1)
+				for (int x = tid; x < sh.table; x += 256) tab[x] = -r1 * __log2f(1.0f + r2 * float(max(0, x - 64)));
+			asm volatile("bar.sync 1, 256;" ::: "memory");
 			float m = -INFINITY, l = 0.0f;
-			// A wait that runs out leaves the warp "dead": it keeps meeting the others at the named barrier below, so
+			// A wait that runs out leaves the warp "dead": it keeps meeting its partner at the named barriers below, so
 			// that nobody waits there for good, and does nothing else.
 			bool ok = true;
 			auto wait = [&](uint64_t *bar, int parity) {
@@ -259,76 +285,57 @@ static __global__ void __launch_bounds__(WT_THREADS) window_attn_tc_kernel(const
 			};
 			for (int t = 0; t < ntile; t++) {
 				const bool ks = t < nkept;
-				const int j0 = ks ? t * WT_KEYS : (j_first + t - nkept) * WT_KEYS;
-				// bias of distance i_lo - j0 - 63 + x, x = 0 .. 190: thread tid meets key c at x = tid + 63 - c
-				if (a.r1) {
-#pragma unroll
-					for (int q = 0; q < 2; q++) {
-						const int x = tid + 128 * q;
-						if (x < 191) s_bias[t & 1][x] = r1 * __log2f(1.0f + r2 * float(max(0, i_lo - j0 - 63 + x)));
-					}
-					asm volatile("bar.sync 1, 128;" ::: "memory");
-				}
+				const int j0 = (ks ? t * WT_KEYS : (j_first + t - nkept) * WT_KEYS) + half * 32;  // first key of this thread's half
+				float r[32];
+				float mx = -INFINITY;
 				if (ok && !wait(&s_bar[t & 1], (t >> 1) & 1)) ok = false;
+				if (ok) {
+					tc_fence_after();
+					uint32_t ra[32];
+					tc_ld32(tmem + lane_addr + s_col + uint32_t((t & 1) * 64), ra);
+					asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+					if (!a.r1) {
+#pragma unroll
+						for (int c = 0; c < 32; c++) r[c] = __uint_as_float(ra[c]) * sc;
+					} else if (!ks && sh.table) {
+						const float *nb = tab + (i - j0 + 64);
+#pragma unroll
+						for (int c = 0; c < 32; c++) r[c] = fmaf(__uint_as_float(ra[c]), sc, nb[-c]);
+					} else {
+#pragma unroll
+						for (int c = 0; c < 32; c++) r[c] = fmaf(__uint_as_float(ra[c]), sc, -r1 * __log2f(1.0f + r2 * float(max(0, i - j0 - c))));
+					}
+					// unless every query of the tile sees every key of it: the ring holds a query's window, the copy the
+					// kept tokens before it
+					if (ks || j0 + 31 > i_lo || (i_lo + 127) - j0 >= a.window) {
+						const int lo = (ks ? 0 : wa_first(a, i)) - j0, hi = (ks ? wa_kept(a, i) - 1 : i) - j0;
+#pragma unroll
+						for (int c = 0; c < 32; c++) r[c] = (c >= lo && c <= hi) ? r[c] : -INFINITY;
+					}
+					float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+					for (int c = 0; c < 32; c++) mx4[c & 3] = fmaxf(mx4[c & 3], r[c]);
+					mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+				}
+				s_max[t & 1][half][row] = mx;
+				asm volatile("bar.sync %0, 64;" ::"r"(2 + quad) : "memory");
+				mx = fmaxf(mx, s_max[t & 1][half ^ 1][row]);
+				// P and O may be touched once PV(t-1) is complete
+				if (ok && t > 0 && !wait(&pv_bar, (t - 1) & 1)) ok = false;
 				if (!ok) {
 					s_fail = 1;
 					continue;
 				}
 				tc_fence_after();
-				uint32_t r[64];
-				{
-					uint32_t (&ra)[32] = *reinterpret_cast<uint32_t (*)[32]>(&r[0]);
-					uint32_t (&rb)[32] = *reinterpret_cast<uint32_t (*)[32]>(&r[32]);
-					tc_ld32(tmem + lane_addr + s_off + uint32_t((t & 1) * 64), ra);
-					tc_ld32(tmem + lane_addr + s_off + uint32_t((t & 1) * 64 + 32), rb);
-					asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-				}
-				const float *bias = s_bias[t & 1] + tid + 63;
-				float mx = -INFINITY;
-				// every query of the tile sees every key of it?
-				const bool whole = !ks && j0 + WT_KEYS - 1 <= i_lo && (i_lo + 127) - j0 < a.window;
-				if (whole) {
-#pragma unroll
-					for (int c = 0; c < 64; c++) {
-						float s = __uint_as_float(r[c]) * sc;
-						if (a.r1) s -= bias[-c];
-						r[c] = __float_as_uint(s);
-						mx = fmaxf(mx, s);
-					}
-				} else {
-					// the ring holds a query's window, the copy the kept tokens before it
-					const int lo = ks ? 0 : wa_first(a, i), hi = ks ? wa_kept(a, i) - 1 : i;
-#pragma unroll
-					for (int c = 0; c < 64; c++) {
-						float s = __uint_as_float(r[c]) * sc;
-						if (a.r1) s -= bias[-c];
-						s = (j0 + c >= lo && j0 + c <= hi) ? s : -INFINITY;
-						r[c] = __float_as_uint(s);
-						mx = fmaxf(mx, s);
-					}
-				}
-				// P and O may be touched once PV(t-1) is complete
-				if (t > 0 && !wait(&pv_bar, (t - 1) & 1)) {
-					ok = false;
-					s_fail = 1;
-					continue;
-				}
-				tc_fence_after();
 				const bool first = m == -INFINITY;
-				bool grow = mx > m + 8.0f || (first && mx > -INFINITY);
+				const bool grow = mx > m + 8.0f || (first && mx > -INFINITY);
 				const float mn = grow ? mx : m;
-				const float corr = first ? 0.0f : exp2f(m - mn);
+				const float corr = first ? 0.0f : ex2_f(m - mn);
 				if (t > 0 && __any_sync(0xffffffffu, grow && !first)) {  // (the whole warp: TMEM accesses are warp-wide)
 					const float f = (grow && !first) ? corr : 1.0f;
-					for (int c = 0; c < a.dvp; c += 16) {
+					for (int c = 16 * half; c < a.dvp; c += 32) {
 						uint32_t o[16];
-						asm volatile(
-						    "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
-						    : "=r"(o[0]), "=r"(o[1]), "=r"(o[2]), "=r"(o[3]), "=r"(o[4]), "=r"(o[5]), "=r"(o[6]), "=r"(o[7]), "=r"(o[8]), "=r"(o[9]),
-						      "=r"(o[10]), "=r"(o[11]), "=r"(o[12]), "=r"(o[13]), "=r"(o[14]), "=r"(o[15])
-						    : "r"(tmem + lane_addr + uint32_t(c))
-						    : "memory");
-						asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+						wt_ld16(tmem + lane_addr + uint32_t(c), o);
 #pragma unroll
 						for (int q = 0; q < 16; q++) o[q] = __float_as_uint(__uint_as_float(o[q]) * f);
 						asm volatile(
@@ -342,46 +349,47 @@ static __global__ void __launch_bounds__(WT_THREADS) window_attn_tc_kernel(const
 				l *= corr;
 				m = mn;
 				const float ms = m == -INFINITY ? 0.0f : m;
-				uint8_t *prow = smem + sh.p_off + tid * 128;
+				uint32_t w[16];
+				float l4[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
-				for (int c8 = 0; c8 < 8; c8++) {
-					uint32_t w[4];
-#pragma unroll
-					for (int q = 0; q < 4; q++) {
-						const float p0 = exp2f(__uint_as_float(r[8 * c8 + 2 * q]) - ms), p1 = exp2f(__uint_as_float(r[8 * c8 + 2 * q + 1]) - ms);
-						l += p0 + p1;
-						w[q] = pack_bf16(p0, p1);
-					}
-					*reinterpret_cast<uint4 *>(prow + ((c8 ^ (tid & 7)) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
+				for (int c = 0; c < 16; c++) {
+					const float p0 = ex2_f(r[2 * c] - ms), p1 = ex2_f(r[2 * c + 1] - ms);
+					l4[c & 3] += p0 + p1;
+					w[c] = pack_bf16(p0, p1);
 				}
-				fence_proxy_async();
+				l += (l4[0] + l4[1]) + (l4[2] + l4[3]);
+				// both halves of a row's S have been read (the exchange above), so P may replace it
+				asm volatile(
+				    "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};" ::"r"(tmem + lane_addr + p_col +
+				                                                                                                           uint32_t((t & 1) * 64)),
+				    "r"(w[0]), "r"(w[1]), "r"(w[2]), "r"(w[3]), "r"(w[4]), "r"(w[5]), "r"(w[6]), "r"(w[7]), "r"(w[8]), "r"(w[9]), "r"(w[10]), "r"(w[11]), "r"(w[12]),
+				    "r"(w[13]), "r"(w[14]), "r"(w[15])
+				    : "memory");
+				asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
 				tc_fence_before();
 				__syncwarp();
 				if (lane == 0) mbar_arrive(&p_bar);
 			}
 			if (ok) ok = wait(&pv_bar, (ntile - 1) & 1);
 			if (!ok) s_fail = 1;
+			s_max[ntile & 1][half][row] = l;
+			asm volatile("bar.sync %0, 64;" ::"r"(2 + quad) : "memory");
+			l += s_max[ntile & 1][half ^ 1][row];
 			if (ok) {
 				tc_fence_after();
 				const float f = a.out_scale / l;
-				const int r = row0 + qt * 128 + tid;
-				const __nv_bfloat16 *gate = reinterpret_cast<const __nv_bfloat16 *>(a.p) + size_t(r) * a.ldp + a.p_g + h * a.dvp;
-				__nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(a.out) + size_t(r) * a.ldo + h * a.dvp;
-				for (int c = 0; c < a.dvp; c += 16) {
+				const int rr = row0 + qt * 128 + row;
+				const __nv_bfloat16 *gate = reinterpret_cast<const __nv_bfloat16 *>(a.p) + size_t(rr) * a.ldp + a.p_g + h * a.dvp;
+				__nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(a.out) + size_t(rr) * a.ldo + h * a.dvp;
+				for (int c = 16 * half; c < a.dvp; c += 32) {
+					uint4 gv[2] = {};
+					if (a.p_g >= 0 && row < nq) {
+						gv[0] = *reinterpret_cast<const uint4 *>(gate + c);
+						gv[1] = *reinterpret_cast<const uint4 *>(gate + c + 8);
+					}
 					uint32_t o[16];
-					asm volatile(
-					    "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
-					    : "=r"(o[0]), "=r"(o[1]), "=r"(o[2]), "=r"(o[3]), "=r"(o[4]), "=r"(o[5]), "=r"(o[6]), "=r"(o[7]), "=r"(o[8]), "=r"(o[9]), "=r"(o[10]),
-					      "=r"(o[11]), "=r"(o[12]), "=r"(o[13]), "=r"(o[14]), "=r"(o[15])
-					    : "r"(tmem + lane_addr + uint32_t(c))
-					    : "memory");
-					asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-					if (tid < nq) {
-						uint4 gv[2] = {};
-						if (a.p_g >= 0) {
-							gv[0] = *reinterpret_cast<const uint4 *>(gate + c);
-							gv[1] = *reinterpret_cast<const uint4 *>(gate + c + 8);
-						}
+					wt_ld16(tmem + lane_addr + uint32_t(c), o);
+					if (row < nq) {
 						const uint32_t *gw = reinterpret_cast<const uint32_t *>(gv);
 						uint32_t w[8];
 #pragma unroll
@@ -408,7 +416,7 @@ static __global__ void __launch_bounds__(WT_THREADS) window_attn_tc_kernel(const
 	}
 	__syncthreads();
 	tc_fence_after();
-	if (warp == 5) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(ncols));
+	if (warp == 9) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(ncols));
 }
 
 // ------------------------------------------------------------------ one token per sequence

@@ -458,7 +458,7 @@ struct HybridState : tg_state {
 	int ldx = 0;
 	void *h = nullptr, *P = nullptr, *O = nullptr, *act = nullptr;   // bf16, or fp32 in a 32-bit state
 	float *P32 = nullptr, *O32 = nullptr, *act32 = nullptr;          // the few-row pipeline's, always fp32
-	float *z = nullptr, *gz = nullptr, *o_raw = nullptr, *bW = nullptr, *bQ = nullptr, *bK = nullptr, *bD = nullptr, *bV = nullptr, *bM = nullptr;
+	float *z = nullptr, *gz = nullptr, *o_raw = nullptr, *blk = nullptr, *bV = nullptr;
 	float *part = nullptr;
 	unsigned *tickets = nullptr;
 	int nsplit_cap = 1;
@@ -546,7 +546,7 @@ template <typename K> int allow_smem(K kernel, size_t bytes) {
 	return TG_OK;
 }
 
-// rows x columns of a tile: fewest waves, weighted by how well a tile shape keeps the tensor pipe busy
+// columns of a tile: waves x measured time of a K-block (a tile is bound by what it reads from the L2)
 int pick_bn(int m_tiles, int N) {
 	static const int forced = env_int("TG_GEMM_BN", 0);
 	if (forced) return forced;
@@ -554,7 +554,7 @@ int pick_bn(int m_tiles, int N) {
 	double cost = 1e30;
 	for (int bn : {256, 128, 64}) {
 		const int tiles = m_tiles * ((N + bn - 1) / bn);
-		const double c = double((tiles + g_num_sms - 1) / g_num_sms) * (bn == 256 ? 256.0 : (bn == 128 ? 150.0 : 100.0));
+		const double c = double((tiles + g_num_sms - 1) / g_num_sms) * (bn == 256 ? 1.0 : (bn == 128 ? 0.79 : 0.6));
 		if (c < cost) {
 			cost = c;
 			best = bn;
@@ -638,7 +638,7 @@ int HybridState::alloc() {
 	const size_t es = f32 ? 4 : 2;
 	ldx = round_up(D, 8);
 	int ldp = 8, kc = 8, ffp = 16, hz = 1, hv = 1;
-	size_t blkK = 1, blkD = 1, blkV = 1, blkM = 1, partn = 1;
+	size_t blkn = 1, blkV = 1, partn = 1;
 	int gmax = 1;
 	for (const Layer &L : m->layers) {
 		ldp = std::max(ldp, L.ldp);
@@ -646,10 +646,8 @@ int HybridState::alloc() {
 		ffp = std::max(ffp, L.ffp);
 		hz = std::max(hz, round_up(L.de.H * L.de.dk, 4));
 		hv = std::max(hv, round_up(L.de.H * L.de.dv, 4));
-		blkK = std::max(blkK, size_t(L.de.H) * DB * L.de.dkp());
-		blkD = std::max(blkD, size_t(L.de.H) * L.de.dkp());
+		blkn = std::max(blkn, size_t(L.de.H) * delta_block_floats(L.de.dkp()));
 		blkV = std::max(blkV, size_t(L.de.H) * DB * L.de.dv);
-		blkM = std::max(blkM, size_t(L.de.H) * DB * DB);
 		partn = std::max(partn, size_t(L.at.H) * (L.at.dvp + 2));
 		gmax = std::max(gmax, L.at.G);
 	}
@@ -666,12 +664,8 @@ int HybridState::alloc() {
 	TG_TRY(take(&gz, size_t(R) * hv));
 	TG_TRY(take(&o_raw, size_t(R) * hv));
 	const size_t nb = size_t(R) / DB + B + 1;
-	TG_TRY(take(&bW, nb * blkK));
-	TG_TRY(take(&bQ, nb * blkK));
-	TG_TRY(take(&bK, nb * blkK));
-	TG_TRY(take(&bD, nb * blkD));
+	TG_TRY(take(&blk, nb * blkn));
 	TG_TRY(take(&bV, nb * blkV));
-	TG_TRY(take(&bM, nb * blkM));
 	nsplit_cap = std::max(1, std::min(TOKEN_SPLITS, 2 * g_num_sms / B));
 	TG_TRY(take(&part, size_t(B) * nsplit_cap * partn));
 	TG_TRY(take(&tickets, size_t(B) * gmax));
@@ -926,12 +920,9 @@ DeltaArgs HybridState::delta_args(const StepDesc &d, int run, const void *p, int
 	a.lda2 = L.a2.ld;
 	a.ldg2 = L.g2.ld;
 	a.dkp = L.de.dkp();
-	a.bW = bW;
-	a.bQ = bQ;
-	a.bK = bK;
-	a.bD = bD;
+	a.blk = blk;
 	a.bV = bV;
-	a.bM = bM;
+	a.err = err_flag;
 	a.o = o_raw;
 	return a;
 }
@@ -945,11 +936,27 @@ template <typename PT, typename CT, typename OT> int launch_token_mix(const WAtt
 	count_launch();
 	return check_launch("hybrid_token_mix");
 }
-template <int RPL> int launch_scan(const DeltaArgs &a, int nseg, cudaStream_t st) {
-	TG_TRY(allow_smem(delta_scan_kernel<RPL>, delta_scan_smem<RPL>()));
-	launch_k(delta_scan_kernel<RPL>, dim3((a.dv + 15) / 16, a.H, nseg), dim3(128), delta_scan_smem<RPL>(), st, a);
+template <int RPL, int NC> int launch_scan_nc(const DeltaArgs &a, int nseg, cudaStream_t st) {
+	const int groups = (a.dv + 4 * NC - 1) / (4 * NC);
+	// few CTAs: deep prefetch; many: more of them per SM
+	int stages = (long long)groups * a.H * nseg <= 2 * g_num_sms ? 4 : 2;
+	while (stages > 2 && delta_scan_smem<RPL, NC>(stages) > 200 * 1024) stages--;
+	const size_t smem = delta_scan_smem<RPL, NC>(stages);
+	auto kernel = delta_scan_kernel<RPL, NC>;
+	TG_TRY(allow_smem(kernel, smem));
+	launch_k(kernel, dim3(groups, a.H, nseg), dim3(32), smem, st, a, stages);
 	count_launch();
 	return check_launch("delta_scan");
+}
+// columns per lane: one while a warp per SM holds all of them, more (fewer shared-memory reads per column) beyond
+template <int RPL> int launch_scan(const DeltaArgs &a, int nseg, cudaStream_t st) {
+	static const int forced = env_int("TG_SCAN_COLS", 0);
+	const long long cols = (long long)a.dv * a.H * nseg;
+	const int nc = forced ? forced : (cols <= 4 * g_num_sms ? 1 : (cols <= 16 * g_num_sms || RPL > 16 ? 2 : 4));
+	if (nc == 1) return launch_scan_nc<RPL, 1>(a, nseg, st);
+	if constexpr (RPL <= 16)
+		if (nc == 4) return launch_scan_nc<RPL, 4>(a, nseg, st);
+	return launch_scan_nc<RPL, 2>(a, nseg, st);
 }
 template <typename PT> int launch_delta(const DeltaArgs &a, int R, int nseg, int max_len, cudaStream_t st) {
 	const size_t smem = delta_block_smem(a.dkp, a.dv);
@@ -969,15 +976,23 @@ template <typename PT> int launch_delta(const DeltaArgs &a, int R, int nseg, int
 }
 template <typename PT> int launch_ln_conv(void *out, int ldo, const float *x, int ldx, const float *w, const float *cw, float *hist, const StepDesc &d, int R,
                                           int D, int taps, float eps, cudaStream_t st) {
-	const dim3 grid((R + LC_ROWS - 1) / LC_ROWS);
-	if (taps <= 4) launch_k(ln_conv_kernel<PT, 4>, grid, dim3(256), 0, st, static_cast<PT *>(out), ldo, x, ldx, w, cw, hist, d, R, D, taps, eps);
-	else launch_k(ln_conv_kernel<PT, 16>, grid, dim3(256), 0, st, static_cast<PT *>(out), ldo, x, ldx, w, cw, hist, d, R, D, taps, eps);
+	int rows = LC_ROWS;
+	while (rows > 1 && ln_conv_smem(rows, taps, D) > 100 * 1024) rows /= 2;
+	const size_t smem = ln_conv_smem(rows, taps, D);
+	const dim3 grid((R + rows - 1) / rows);
+	if (taps <= 4) {
+		TG_TRY(allow_smem(ln_conv_kernel<PT, 4>, smem));
+		launch_k(ln_conv_kernel<PT, 4>, grid, dim3(256), smem, st, static_cast<PT *>(out), ldo, x, ldx, w, cw, hist, d, R, D, taps, eps, rows);
+	} else {
+		TG_TRY(allow_smem(ln_conv_kernel<PT, 16>, smem));
+		launch_k(ln_conv_kernel<PT, 16>, grid, dim3(256), smem, st, static_cast<PT *>(out), ldo, x, ldx, w, cw, hist, d, R, D, taps, eps, rows);
+	}
 	count_launch();
 	return check_launch("ln_conv");
 }
 template <typename PT> int launch_ln(void *out, int ldo, const float *x, int ldx, const float *w, const int *rows, int n, int D, float eps, float *out32,
                                      cudaStream_t st) {
-	launch_k(layer_norm_kernel<PT>, dim3((n + 7) / 8), dim3(256), 0, st, static_cast<PT *>(out), ldo, x, ldx, w, rows, n, D, eps, out32);
+	launch_k(layer_norm_kernel<PT>, dim3(n), dim3(128), 0, st, static_cast<PT *>(out), ldo, x, ldx, w, rows, n, D, eps, out32);
 	count_launch();
 	return check_launch("layer_norm");
 }
@@ -1079,7 +1094,7 @@ int HybridState::run_layers(const StepDesc &d, int R, int nseg, int max_len) {
 			} else {
 				static const int use_tc = env_int("TG_WATTN_TC", 1);
 				if (!f32 && use_tc && wa.dkp <= 256 && wa.dvp <= 256) {
-					const WtShape sh = wt_shape(wa.dkp, wa.dvp);
+					const WtShape sh = wt_shape(wa.dkp, wa.dvp, wa.window);
 					TG_TRY(allow_smem(window_attn_tc_kernel, sh.total));
 					launch_k(window_attn_tc_kernel, dim3((max_len + 127) / 128, wa.H, nseg), dim3(WT_THREADS), size_t(sh.total), stream, pmap[li], c.kmap, c.vmap,
 					         c.ksmap, c.vsmap, wa);
