@@ -368,11 +368,11 @@ __global__ void __launch_bounds__(256, 3) delta_block_kernel(DeltaArgs a) {
 }
 
 // ------------------------------------------------------------------ carrying the state through the blocks
-// grid (column groups of 4 NC, H, segments), one warp per CTA. A lane holds RPL rows of NC columns: rows
-// 4 (lane & 7) + 32 j + {0..3} of columns 4 NC x + (lane >> 3) + 4 i; the eight lanes of a column meet by butterflies.
-// The chain over the blocks is sequential, so a CTA is kept as short as possible: the block quantities of a
-// (block, head) are one bulk copy, `stages` of them in flight, and the products run on packed fp32 pairs. Every lane
-// reads every block quantity of its rows from shared memory once per NC columns; that read rate is what bounds an SM.
+// grid (column groups of 4 NC, H, segments), NW warps. The CTA holds 4 NC columns of S in registers: warp w rows
+// 8 RPL w .. , a lane RPL of them (4 (lane & 7) + 32 j + {0..3}) of columns 4 NC x + (lane >> 3) + 4 i. The chain over
+// the blocks is sequential and a block is a few hundred instructions per warp, so what counts is its latency: the block
+// quantities of a (block, head) are one bulk copy, `stages` of them in flight; rows are read from shared memory a group
+// ahead of their use; the products run on packed fp32 pairs; and the warps meet at one barrier per block.
 __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
 	float2 d;
 	asm("fma.rn.f32x2 %0, %1, %2, %3;"
@@ -400,29 +400,35 @@ __device__ __forceinline__ float2 delta_reduce(const float (&acc)[DB], int rl) {
 	return o;
 }
 constexpr int DS_MAX_STAGES = 4;
-template <int RPL, int NC> size_t delta_scan_smem(int stages) { return (size_t(stages) * delta_block_floats(8 * RPL) + 4 * NC * 20) * 4; }
+template <int RPL, int NW, int NC> size_t delta_scan_smem(int stages) {
+	return (size_t(stages) * delta_block_floats(8 * RPL * NW) + size_t(5) * NW * 4 * NC * 20) * 4;
+}
 
-template <int RPL, int NC>
-__global__ void __launch_bounds__(32) delta_scan_kernel(DeltaArgs a, int stages) {
+template <int RPL, int NW, int NC>
+__global__ void __launch_bounds__(32 * NW) delta_scan_kernel(DeltaArgs a, int stages) {
 	pdl_trigger();
-	constexpr int DKP = 8 * RPL;
+	constexpr int DKP = 8 * RPL * NW, COLS = 4 * NC;
 	constexpr size_t BF = delta_block_floats(DKP);
 	extern __shared__ __align__(128) float ds_sm[];
 	__shared__ uint64_t full_bar[DS_MAX_STAGES];
-	const int lane = threadIdx.x;
+	__shared__ int s_fail;
+	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
 	const int h = blockIdx.y, seg = blockIdx.z, rl = lane & 7, cl = lane >> 3;
-	float *su = ds_sm + size_t(stages) * BF;  // [4 NC columns][20]
-	if (lane == 0) {
+	float *pw = ds_sm + size_t(stages) * BF;          // [2][NW][COLS][20] partial W dots
+	float *pq = pw + 2 * NW * COLS * 20;              // the same of Q
+	float *su = pq + 2 * NW * COLS * 20 + warp * COLS * 20;  // this warp's copy of u [COLS][20]
+	if (tid == 0) {
 		for (int i = 0; i < stages; i++) mbar_init(&full_bar[i], 1);
+		s_fail = 0;
 		asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
 	}
-	__syncwarp();
+	__syncthreads();
 	pdl_wait();
 	const int len = a.d.seg_len[seg], row0 = a.d.seg_row[seg], pos = a.d.seg_pos[seg], seq = a.d.seg_seq[seg];
 	const int nb = (len + DB - 1) / DB, dk = a.dk, dv = a.dv;
 	const size_t blk0 = delta_block_base(row0, seg);
 	auto fetch = [&](int b) {
-		if (lane == 0) {
+		if (tid == 0) {
 			fence_proxy_async();
 			mbar_expect_tx(&full_bar[b % stages], uint32_t(BF * 4));
 			asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(ds_sm + size_t(b % stages) * BF)),
@@ -435,12 +441,13 @@ __global__ void __launch_bounds__(32) delta_scan_kernel(DeltaArgs a, int stages)
 	int col[NC];
 	float2 S[NC][RPL / 2];
 	float *Sg = a.S + (size_t(seq) * a.H + h) * dk * dv;
+	const int r_base = warp * 8 * RPL + 4 * rl;
 #pragma unroll
 	for (int x = 0; x < NC; x++) {
 		col[x] = (blockIdx.x * NC + x) * 4 + cl;
 #pragma unroll
 		for (int j = 0; j < RPL / 2; j++) {
-			const int i = 4 * rl + 32 * (j >> 1) + 2 * (j & 1);
+			const int i = r_base + 32 * (j >> 1) + 2 * (j & 1);
 			S[x][j].x = (pos > 0 && col[x] < dv && i < dk) ? Sg[size_t(i) * dv + col[x]] : 0.0f;
 			S[x][j].y = (pos > 0 && col[x] < dv && i + 1 < dk) ? Sg[size_t(i + 1) * dv + col[x]] : 0.0f;
 		}
@@ -453,21 +460,17 @@ __global__ void __launch_bounds__(32) delta_scan_kernel(DeltaArgs a, int stages)
 	};
 	load_v(0);
 	for (int b = 0; b < nb; b++) {
-		if (issued < nb) fetch(issued++);
-		if (!__all_sync(0xffffffffu, tc_wait(&full_bar[b % stages], (b / stages) & 1, a.err))) {
-			for (int q = b + 1; q < issued; q++) tc_wait(&full_bar[q % stages], (q / stages) & 1, a.err);  // copies in flight land first
-			break;
-		}
+		const int par = b & 1;
+		if (!tc_wait(&full_bar[b % stages], (b / stages) & 1, a.err)) s_fail = 1;
 		const float *sW = ds_sm + size_t(b % stages) * BF, *sD = sW + 3 * DB * DKP, *sM = sD + DKP;
-		// W, Q and K are read as one stream of groups of TG token rows, a group ahead of its use: a warp alone on its
-		// scheduler has nobody else to hide the latency of shared memory
-		constexpr int TG = RPL >= 32 ? 2 : 4, GR = DB / TG;
+		// W, Q and K are read as one stream of groups of TG token rows, a group ahead of its use
+		constexpr int TG = RPL >= 8 ? 4 : 8, GR = DB / TG;
 		float4 cur[TG][RPL / 4], nxt[TG][RPL / 4];
 		auto rows = [&](int g, float4 (&w)[TG][RPL / 4]) {  // g: 0 .. 3 GR - 1 (W, Q and K lie one after the other)
 #pragma unroll
 			for (int t = 0; t < TG; t++)
 #pragma unroll
-				for (int j = 0; j < RPL / 4; j++) w[t][j] = ds_ld4(sW + (g * TG + t) * DKP + 4 * rl + 32 * j);
+				for (int j = 0; j < RPL / 4; j++) w[t][j] = ds_ld4(sW + (g * TG + t) * DKP + r_base + 32 * j);
 		};
 		float acc[NC][DB];
 		auto dots = [&](int g) {
@@ -492,50 +495,39 @@ __global__ void __launch_bounds__(32) delta_scan_kernel(DeltaArgs a, int stages)
 		};
 		rows(0, cur);
 #pragma unroll
-		for (int g = 0; g < GR; g++) {
+		for (int g = 0; g < 2 * GR; g++) {
 			rows(g + 1, nxt);
 			dots(g);
 			shift();
+			if (g == GR - 1 || g == 2 * GR - 1) {
+				float *dst = (g == GR - 1 ? pw : pq) + (par * NW + warp) * COLS * 20;
+#pragma unroll
+				for (int x = 0; x < NC; x++) *reinterpret_cast<float2 *>(dst + (4 * x + cl) * 20 + 2 * rl) = delta_reduce(acc[x], rl);
+			}
 		}
+		if (NW > 1) __syncthreads();
+		else __syncwarp();
+		if (*(volatile int *)&s_fail) {
+			for (int q = b + 1; q < issued; q++) tc_wait(&full_bar[q % stages], (q / stages) & 1, a.err);  // copies in flight land first
+			break;
+		}
+		if (issued < nb) fetch(issued++);  // (every warp is past the block that used this stage)
 #pragma unroll
 		for (int x = 0; x < NC; x++) {
-			const float2 dw = delta_reduce(acc[x], rl);
-			*reinterpret_cast<float2 *>(su + (4 * x + cl) * 20 + 2 * rl) = make_float2(v[x].x - dw.x, v[x].y - dw.y);
+			float2 u = v[x];
+#pragma unroll
+			for (int w = 0; w < NW; w++) {
+				const float2 d = *reinterpret_cast<const float2 *>(pw + ((par * NW + w) * COLS + 4 * x + cl) * 20 + 2 * rl);
+				u.x -= d.x;
+				u.y -= d.y;
+			}
+			*reinterpret_cast<float2 *>(su + (4 * x + cl) * 20 + 2 * rl) = u;
 		}
 		if (b + 1 < nb) load_v(b + 1);
-		float2 dq[NC];
-#pragma unroll
-		for (int g = GR; g < 2 * GR; g++) {
-			rows(g + 1, nxt);
-			dots(g);
-			shift();
-		}
-#pragma unroll
-		for (int x = 0; x < NC; x++) dq[x] = delta_reduce(acc[x], rl);
 		__syncwarp();
-		const float4 *m0 = reinterpret_cast<const float4 *>(sM + 2 * rl * DB);
-#pragma unroll
-		for (int x = 0; x < NC; x++) {
-			float u[DB];
-#pragma unroll
-			for (int i = 0; i < 4; i++) *reinterpret_cast<float4 *>(&u[4 * i]) = *reinterpret_cast<const float4 *>(su + (4 * x + cl) * 20 + 4 * i);
-			float2 o = dq[x];
-#pragma unroll
-			for (int i = 0; i < 4; i++) {  // (M is zero above the diagonal)
-				const float4 p = m0[i], q = m0[4 + i];
-				o.x = fmaf(p.x, u[4 * i], o.x); o.x = fmaf(p.y, u[4 * i + 1], o.x); o.x = fmaf(p.z, u[4 * i + 2], o.x); o.x = fmaf(p.w, u[4 * i + 3], o.x);
-				o.y = fmaf(q.x, u[4 * i], o.y); o.y = fmaf(q.y, u[4 * i + 1], o.y); o.y = fmaf(q.z, u[4 * i + 2], o.y); o.y = fmaf(q.w, u[4 * i + 3], o.y);
-			}
-			const int t = b * DB + 2 * rl;
-			if (col[x] < dv) {
-				float *dst = a.o + size_t(row0 + t) * a.H * dv + h * dv + col[x];
-				if (t < len) dst[0] = o.x;
-				if (t + 1 < len) dst[size_t(a.H) * dv] = o.y;
-			}
-		}
 #pragma unroll
 		for (int j = 0; j < RPL / 4; j++) {
-			const float4 g = *reinterpret_cast<const float4 *>(sD + 4 * rl + 32 * j);
+			const float4 g = *reinterpret_cast<const float4 *>(sD + r_base + 32 * j);
 #pragma unroll
 			for (int x = 0; x < NC; x++) {
 				S[x][2 * j].x *= g.x; S[x][2 * j].y *= g.y;
@@ -546,25 +538,46 @@ __global__ void __launch_bounds__(32) delta_scan_kernel(DeltaArgs a, int stages)
 		for (int g = 2 * GR; g < 3 * GR; g++) {
 			if (g + 1 < 3 * GR) rows(g + 1, nxt);
 #pragma unroll
-			for (int t = 0; t < TG; t++)
+			for (int x = 0; x < NC; x++) {
+				float u[TG];
 #pragma unroll
-				for (int x = 0; x < NC; x++) {
-					const float u = su[(4 * x + cl) * 20 + (g - 2 * GR) * TG + t];
+				for (int t = 0; t < TG; t += 4) *reinterpret_cast<float4 *>(&u[t]) = *reinterpret_cast<const float4 *>(su + (4 * x + cl) * 20 + (g - 2 * GR) * TG + t);
+#pragma unroll
+				for (int t = 0; t < TG; t++)
 #pragma unroll
 					for (int j = 0; j < RPL / 4; j++) {
-						S[x][2 * j] = fma2(make_float2(cur[t][j].x, cur[t][j].y), make_float2(u, u), S[x][2 * j]);
-						S[x][2 * j + 1] = fma2(make_float2(cur[t][j].z, cur[t][j].w), make_float2(u, u), S[x][2 * j + 1]);
+						S[x][2 * j] = fma2(make_float2(cur[t][j].x, cur[t][j].y), make_float2(u[t], u[t]), S[x][2 * j]);
+						S[x][2 * j + 1] = fma2(make_float2(cur[t][j].z, cur[t][j].w), make_float2(u[t], u[t]), S[x][2 * j + 1]);
 					}
-				}
+			}
 			if (g + 1 < 3 * GR) shift();
 		}
-		__syncwarp();
+		// read-outs: the warps share the 16 tokens; two lanes per (token, column), each half of the sum over s
+#pragma unroll
+		for (int e = 0; e < 4 * NC / NW + (4 * NC % NW != 0); e++) {
+			const int item = (e * NW + warp) * 16 + (lane >> 1), half = lane & 1;  // 16 items per warp and round
+			const int t = item / COLS, c = item % COLS;
+			if (item < DB * COLS) {
+				float o = 0.0f;
+#pragma unroll
+				for (int i = 0; i < 2; i++) {  // (M is zero above the diagonal)
+					const float4 m = *reinterpret_cast<const float4 *>(sM + t * DB + 8 * half + 4 * i), u = *reinterpret_cast<const float4 *>(su + c * 20 + 8 * half + 4 * i);
+					o = fmaf(m.x, u.x, o); o = fmaf(m.y, u.y, o); o = fmaf(m.z, u.z, o); o = fmaf(m.w, u.w, o);
+				}
+#pragma unroll
+				for (int w = 0; w < NW; w++)
+					if ((w & 1) == half || NW == 1) o += NW == 1 && half ? 0.0f : pq[((par * NW + w) * COLS + c) * 20 + t];
+				o += __shfl_xor_sync(0xffffffffu, o, 1);
+				const int gc = blockIdx.x * COLS + c;
+				if (half == 0 && gc < dv && b * DB + t < len) a.o[size_t(row0 + b * DB + t) * a.H * dv + h * dv + gc] = o;
+			}
+		}
 	}
 #pragma unroll
 	for (int x = 0; x < NC; x++)
 #pragma unroll
 		for (int j = 0; j < RPL / 2; j++) {
-			const int i = 4 * rl + 32 * (j >> 1) + 2 * (j & 1);
+			const int i = r_base + 32 * (j >> 1) + 2 * (j & 1);
 			if (col[x] < dv && i < dk) Sg[size_t(i) * dv + col[x]] = S[x][j].x;
 			if (col[x] < dv && i + 1 < dk) Sg[size_t(i + 1) * dv + col[x]] = S[x][j].y;
 		}

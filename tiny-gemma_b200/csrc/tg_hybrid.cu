@@ -936,27 +936,26 @@ template <typename PT, typename CT, typename OT> int launch_token_mix(const WAtt
 	count_launch();
 	return check_launch("hybrid_token_mix");
 }
-template <int RPL, int NC> int launch_scan_nc(const DeltaArgs &a, int nseg, cudaStream_t st) {
+template <int RPL, int NW, int NC> int launch_scan_nc(const DeltaArgs &a, int nseg, cudaStream_t st) {
 	const int groups = (a.dv + 4 * NC - 1) / (4 * NC);
 	// few CTAs: deep prefetch; many: more of them per SM
 	int stages = (long long)groups * a.H * nseg <= 2 * g_num_sms ? 4 : 2;
-	while (stages > 2 && delta_scan_smem<RPL, NC>(stages) > 200 * 1024) stages--;
-	const size_t smem = delta_scan_smem<RPL, NC>(stages);
-	auto kernel = delta_scan_kernel<RPL, NC>;
+	while (stages > 2 && delta_scan_smem<RPL, NW, NC>(stages) > 200 * 1024) stages--;
+	const size_t smem = delta_scan_smem<RPL, NW, NC>(stages);
+	auto kernel = delta_scan_kernel<RPL, NW, NC>;
 	TG_TRY(allow_smem(kernel, smem));
-	launch_k(kernel, dim3(groups, a.H, nseg), dim3(32), smem, st, a, stages);
+	launch_k(kernel, dim3(groups, a.H, nseg), dim3(32 * NW), smem, st, a, stages);
 	count_launch();
 	return check_launch("delta_scan");
 }
-// columns per lane: one while a warp per SM holds all of them, more (fewer shared-memory reads per column) beyond
-template <int RPL> int launch_scan(const DeltaArgs &a, int nseg, cudaStream_t st) {
+// columns per lane: one while every SM gets at most one CTA, more (fewer shared-memory reads per column) beyond
+template <int RPL, int NW> int launch_scan(const DeltaArgs &a, int nseg, cudaStream_t st) {
 	static const int forced = env_int("TG_SCAN_COLS", 0);
 	const long long cols = (long long)a.dv * a.H * nseg;
-	const int nc = forced ? forced : (cols <= 4 * g_num_sms ? 1 : (cols <= 16 * g_num_sms || RPL > 16 ? 2 : 4));
-	if (nc == 1) return launch_scan_nc<RPL, 1>(a, nseg, st);
-	if constexpr (RPL <= 16)
-		if (nc == 4) return launch_scan_nc<RPL, 4>(a, nseg, st);
-	return launch_scan_nc<RPL, 2>(a, nseg, st);
+	const int nc = forced ? forced : (cols <= 4 * g_num_sms ? 1 : (cols <= 16 * g_num_sms ? 2 : 4));
+	if (nc == 1) return launch_scan_nc<RPL, NW, 1>(a, nseg, st);
+	if (nc == 2) return launch_scan_nc<RPL, NW, 2>(a, nseg, st);
+	return launch_scan_nc<RPL, NW, 4>(a, nseg, st);
 }
 template <typename PT> int launch_delta(const DeltaArgs &a, int R, int nseg, int max_len, cudaStream_t st) {
 	const size_t smem = delta_block_smem(a.dkp, a.dv);
@@ -965,10 +964,10 @@ template <typename PT> int launch_delta(const DeltaArgs &a, int R, int nseg, int
 	count_launch();
 	TG_TRY(check_launch("delta_block"));
 	switch (a.dkp) {
-		case 32: TG_TRY(launch_scan<4>(a, nseg, st)); break;
-		case 64: TG_TRY(launch_scan<8>(a, nseg, st)); break;
-		case 128: TG_TRY(launch_scan<16>(a, nseg, st)); break;
-		default: TG_TRY(launch_scan<32>(a, nseg, st)); break;
+		case 32: TG_TRY((launch_scan<4, 1>(a, nseg, st))); break;
+		case 64: TG_TRY((launch_scan<4, 2>(a, nseg, st))); break;
+		case 128: TG_TRY((launch_scan<4, 4>(a, nseg, st))); break;
+		default: TG_TRY((launch_scan<8, 4>(a, nseg, st))); break;
 	}
 	launch_k(delta_out_kernel<PT>, dim3((R * a.H + 7) / 8), dim3(256), 0, st, a, R);
 	count_launch();
