@@ -881,7 +881,7 @@ def run_nabelix(args):
             ms = timed(st, (lambda: None, lambda: st.prefill(ids[None], want_logits=False)), 1 if args.repeats == 1 else 6)
             res["prefill"].append((S, ms))
             st.close()
-        for B, pos in ([(1, args.prompt_len)] if args.no_extras else [(1, 178), (1, 4096), (4, 178), (32, 178), (256, 178)]):
+        for B, pos in ([(args.batch, args.prompt_len)] if args.no_extras else [(1, 178), (1, 4096), (4, 178), (32, 178), (256, 178)]):
             st = model.state(B, pos + steps + 16)
             ids = np.stack([rng.integers(0, vocab, pos).astype(np.int32) for _ in range(B)])
 
@@ -958,7 +958,7 @@ def main():
     ap.add_argument("--phase-clocks", action="store_true", help="per-section timing of one decoded token (in-kernel recorder)")
     ap.add_argument("--greedy", action="store_true", help="with --phase-clocks: argmax instead of the min-p sampler")
     ap.add_argument("--batched-step", action="store_true", help="time the batched step alone (--batch sequences, empty cache)")
-    ap.add_argument("--nabelix", action="store_true", help="throughput of the Nabelix design; with --no-extras only --model at --prompt-len")
+    ap.add_argument("--nabelix", action="store_true", help="throughput of the Nabelix design; with --no-extras only --model at --prompt-len and --batch")
     args = ap.parse_args()
     if args.model == "3B" and not args.nabelix:
         ap.error("--model 3B needs --nabelix")

@@ -370,6 +370,23 @@ static __global__ void __launch_bounds__(WT_THREADS, 2) window_attn_tc_kernel(co
 				__syncwarp();
 				if (lane == 0) mbar_arrive(&p_bar);
 			}
+			// the gate of the first 128 columns is requested before the last products are awaited
+			const int rr = row0 + qt * 128 + row;
+			const bool gated = a.p_g >= 0 && row < nq;
+			const __nv_bfloat16 *gate = reinterpret_cast<const __nv_bfloat16 *>(a.p) + size_t(rr) * a.ldp + a.p_g + h * a.dvp;
+			uint4 gv[4][2];
+			auto load_gate = [&](int c0) {
+#pragma unroll
+				for (int e = 0; e < 4; e++) {
+					const int c = c0 + 32 * e;
+					gv[e][0] = gv[e][1] = make_uint4(0, 0, 0, 0);
+					if (gated && c < a.dvp) {
+						gv[e][0] = *reinterpret_cast<const uint4 *>(gate + c);
+						gv[e][1] = *reinterpret_cast<const uint4 *>(gate + c + 8);
+					}
+				}
+			};
+			load_gate(16 * half);
 			if (ok) ok = wait(&pv_bar, (ntile - 1) & 1);
 			if (!ok) s_fail = 1;
 			s_max[ntile & 1][half][row] = l;
@@ -378,31 +395,30 @@ static __global__ void __launch_bounds__(WT_THREADS, 2) window_attn_tc_kernel(co
 			if (ok) {
 				tc_fence_after();
 				const float f = a.out_scale / l;
-				const int rr = row0 + qt * 128 + row;
-				const __nv_bfloat16 *gate = reinterpret_cast<const __nv_bfloat16 *>(a.p) + size_t(rr) * a.ldp + a.p_g + h * a.dvp;
 				__nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(a.out) + size_t(rr) * a.ldo + h * a.dvp;
-				for (int c = 16 * half; c < a.dvp; c += 32) {
-					uint4 gv[2] = {};
-					if (a.p_g >= 0 && row < nq) {
-						gv[0] = *reinterpret_cast<const uint4 *>(gate + c);
-						gv[1] = *reinterpret_cast<const uint4 *>(gate + c + 8);
-					}
-					uint32_t o[16];
-					wt_ld16(tmem + lane_addr + uint32_t(c), o);
-					if (row < nq) {
-						const uint32_t *gw = reinterpret_cast<const uint32_t *>(gv);
-						uint32_t w[8];
+				for (int c0 = 16 * half; c0 < a.dvp; c0 += 128) {
+					if (c0 >= 128) load_gate(c0);
 #pragma unroll
-						for (int q = 0; q < 8; q++) {
-							float x = __uint_as_float(o[2 * q]) * f, y = __uint_as_float(o[2 * q + 1]) * f;
-							if (a.p_g >= 0) {
-								x *= 1.0f / (1.0f + __expf(-bf16_lo(gw[q])));
-								y *= 1.0f / (1.0f + __expf(-bf16_hi(gw[q])));
+					for (int e = 0; e < 4; e++) {
+						const int c = c0 + 32 * e;
+						if (c >= a.dvp) break;
+						uint32_t o[16];
+						wt_ld16(tmem + lane_addr + uint32_t(c), o);
+						if (row < nq) {
+							const uint32_t gw[8] = {gv[e][0].x, gv[e][0].y, gv[e][0].z, gv[e][0].w, gv[e][1].x, gv[e][1].y, gv[e][1].z, gv[e][1].w};
+							uint32_t w[8];
+#pragma unroll
+							for (int q = 0; q < 8; q++) {
+								float x = __uint_as_float(o[2 * q]) * f, y = __uint_as_float(o[2 * q + 1]) * f;
+								if (a.p_g >= 0) {
+									x *= __fdividef(1.0f, 1.0f + __expf(-bf16_lo(gw[q])));
+									y *= __fdividef(1.0f, 1.0f + __expf(-bf16_hi(gw[q])));
+								}
+								w[q] = pack_bf16(x, y);
 							}
-							w[q] = pack_bf16(x, y);
+							*reinterpret_cast<uint4 *>(out + c) = make_uint4(w[0], w[1], w[2], w[3]);
+							*reinterpret_cast<uint4 *>(out + c + 8) = make_uint4(w[4], w[5], w[6], w[7]);
 						}
-						*reinterpret_cast<uint4 *>(out + c) = make_uint4(w[0], w[1], w[2], w[3]);
-						*reinterpret_cast<uint4 *>(out + c + 8) = make_uint4(w[4], w[5], w[6], w[7]);
 					}
 				}
 			}
