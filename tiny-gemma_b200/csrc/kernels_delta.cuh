@@ -77,20 +77,35 @@ __device__ __forceinline__ void delta_hist_save(const DeltaArgs &a, int row0, in
 // smem: q[dk] k[dk] g[dk] v[dv] gate[dv] part[nparts*2*dv] red[32]. 256 threads. Row r of the step is a segment of
 // length 1.
 __host__ __device__ inline int delta_token_parts(int dv) { return dv >= 256 ? 1 : 256 / dv; }
+// the state of a head held in registers between its two uses: 16 rows of 4 columns per thread
+__host__ __device__ inline bool delta_token_in_regs(int dk, int dv) { return dk <= 128 && dv <= 128 && dv % 4 == 0; }
 __host__ __device__ inline size_t delta_token_smem(int dk, int dv) {
-	return (size_t(3) * dk + 2 * size_t(dv) + size_t(delta_token_parts(dv)) * 2 * dv + 64) * 4;
+	const int parts = delta_token_in_regs(dk, dv) ? 8 : delta_token_parts(dv);
+	return (size_t(3) * dk + 2 * size_t(dv) + size_t(parts) * 2 * dv + 64) * 4;
 }
 template <typename PT, typename OT>
 __device__ void delta_token_cta(const DeltaArgs &a, int r, int h, float *sm) {
 	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
 	const int dk = a.dk, dv = a.dv, per = a.H / a.KH, kh = h / per, C = 2 * a.KH * dk + a.H * dv;
 	float *sq = sm, *sk = sq + dk, *sg = sk + dk, *sv = sg + dk, *sgate = sv + dv, *part = sgate + dv;
-	float *red = part + delta_token_parts(dv) * 2 * dv;
+	const bool in_regs = delta_token_in_regs(dk, dv);
+	float *red = part + (in_regs ? 8 : delta_token_parts(dv)) * 2 * dv;
 	const int seg = a.d.row_seg[r], seq = a.d.seg_seq[seg], pos = a.d.seg_pos[seg], par = a.d.seg_par[seg];
 	float *hb = a.hist + size_t(seq) * 2 * (a.taps - 1) * C;
 	const float *hr = hb + size_t(par) * (a.taps - 1) * C;
 	float *hw = hb + size_t(par ^ 1) * (a.taps - 1) * C;
 	const PT *prow = reinterpret_cast<const PT *>(a.p) + size_t(r) * a.ldp;
+	// the state: with in_regs a lane owns four columns of the rows warp, warp + 8, ...; requested first
+	float *S = a.S + (size_t(seq) * a.H + h) * dk * dv;
+	const bool fresh = pos == 0;
+	float4 st[16];
+	if (in_regs) {
+#pragma unroll
+		for (int e = 0; e < 16; e++) {
+			const int i = warp + 8 * e;
+			st[e] = !fresh && i < dk && 4 * lane < dv ? *reinterpret_cast<const float4 *>(S + size_t(i) * dv + 4 * lane) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+		}
+	}
 	// convolutions
 	for (int i = tid; i < 2 * dk + dv; i += 256) {
 		if (i < dk) sq[i] = delta_conv<PT>(a, r, pos, hr, C, 0, kh * dk + i);
@@ -142,13 +157,55 @@ __device__ void delta_token_cta(const DeltaArgs &a, int r, int h, float *sm) {
 		if (lane == 0) red[33] = s;
 	}
 	const float beta = sigmoid_f(to_f32(prow[a.p_b + h]));
-	// the state: a thread owns a column (and one of `np` runs of rows)
-	float *S = a.S + (size_t(seq) * a.H + h) * dk * dv;
-	const int np = delta_token_parts(dv);
-	const bool fresh = pos == 0;
 	float ss = 0.0f;
 	__syncthreads();
-	for (int c0 = 0; c0 < dv; c0 += 256 / np) {
+	if (in_regs) {
+		float4 xk = make_float4(0.0f, 0.0f, 0.0f, 0.0f), xq = xk;
+#pragma unroll
+		for (int e = 0; e < 16; e++) {
+			const int i = warp + 8 * e;
+			if (i < dk) {
+				const float gi = sg[i], ki = sk[i], qi = sq[i];
+				st[e].x *= gi; st[e].y *= gi; st[e].z *= gi; st[e].w *= gi;
+				xk.x = fmaf(st[e].x, ki, xk.x); xk.y = fmaf(st[e].y, ki, xk.y); xk.z = fmaf(st[e].z, ki, xk.z); xk.w = fmaf(st[e].w, ki, xk.w);
+				xq.x = fmaf(st[e].x, qi, xq.x); xq.y = fmaf(st[e].y, qi, xq.y); xq.z = fmaf(st[e].z, qi, xq.z); xq.w = fmaf(st[e].w, qi, xq.w);
+			}
+		}
+		if (4 * lane < dv) {
+			float *pk = part + (warp * 2) * dv + 4 * lane, *pq = part + (warp * 2 + 1) * dv + 4 * lane;
+			pk[0] = xk.x; pk[1] = xk.y; pk[2] = xk.z; pk[3] = xk.w;
+			pq[0] = xq.x; pq[1] = xq.y; pq[2] = xq.z; pq[3] = xq.w;
+		}
+		__syncthreads();
+		if (tid < dv) {  // u into sv, the read-out times the gate into sgate
+			float k = 0.0f, q = 0.0f;
+#pragma unroll
+			for (int w = 0; w < 8; w++) {
+				k += part[(w * 2) * dv + tid];
+				q += part[(w * 2 + 1) * dv + tid];
+			}
+			const float u = beta * (sv[tid] - k), o = fmaf(u, red[33], q);
+			sv[tid] = u;
+			ss = o * o;
+			sgate[tid] *= o;
+		}
+		__syncthreads();
+		if (4 * lane < dv) {
+			const float u0 = sv[4 * lane], u1 = sv[4 * lane + 1], u2 = sv[4 * lane + 2], u3 = sv[4 * lane + 3];
+#pragma unroll
+			for (int e = 0; e < 16; e++) {
+				const int i = warp + 8 * e;
+				if (i < dk) {
+					const float ki = sk[i];
+					*reinterpret_cast<float4 *>(S + size_t(i) * dv + 4 * lane) =
+					    make_float4(fmaf(ki, u0, st[e].x), fmaf(ki, u1, st[e].y), fmaf(ki, u2, st[e].z), fmaf(ki, u3, st[e].w));
+				}
+			}
+		}
+	}
+	// any other size: a thread owns a column (and one of `np` runs of rows) and reads it twice
+	const int np = delta_token_parts(dv);
+	for (int c0 = in_regs ? dv : 0; c0 < dv; c0 += 256 / np) {
 		const int c = c0 + tid % (256 / np), pt = tid / (256 / np);
 		const bool on = c < dv && pt < np;
 		const int rows = (dk + np - 1) / np, i0 = pt * rows, i1 = min(dk, i0 + rows);

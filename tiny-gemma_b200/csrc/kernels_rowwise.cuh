@@ -142,7 +142,7 @@ __global__ void __launch_bounds__(256) ln_conv_kernel(OT *out, int ldo, const fl
 	if (threadIdx.x < nr) seg_s[threadIdx.x] = d.row_seg[r0 + threadIdx.x];
 	for (int i = warp; i < nr + H; i += 8) {  // rows r0 - H .. r0 + nr - 1
 		const int r = r0 - H + i;
-		if (r < 0) continue;
+		if (r < 0 || (i < H && d.row_seg[r] != d.row_seg[r0])) continue;  // (another segment's rows are not in any window)
 		const float *xr = x + size_t(r) * ldx;
 		float *n = lc_sm + size_t(i) * ld;
 		float s = 0.0f;

@@ -436,18 +436,28 @@ static __global__ void __launch_bounds__(WT_THREADS, 2) window_attn_tc_kernel(co
 }
 
 // ------------------------------------------------------------------ one token per sequence
-// 256 threads; row r of the step is a segment of length 1 whose key and value are already in the cache. The run
-// `split` of WK_KEYS-key pieces is scored for all the query heads of key/value head g; the CTA that arrives last
-// merges the runs, applies the gate and writes the heads' rows.
-constexpr int WK_KEYS = 64;
+// 256 threads; row r of the step is a segment of length 1 whose key and value are already in the cache. The CTA scores
+// its run of keys for up to WK_HEADS query heads of key/value head g at a time, in pieces of WK_KEYS; the CTA that
+// arrives last merges the runs, applies the gate and writes the heads' rows.
+constexpr int WK_KEYS = 64, WK_HEADS = 4;
 __host__ __device__ inline size_t wattn_token_smem(int per, int dkp, int dvp) {
-	return (size_t(per) * dkp + size_t(per) * WK_KEYS + size_t(8) * dvp + 2 * per + 8) * 4;
+	return (size_t(per) * dkp + size_t(WK_HEADS) * WK_KEYS + size_t(8) * WK_HEADS * (dvp < 256 ? dvp : 256) + 3 * WK_HEADS + 8) * 4;
+}
+// 16 bytes of a cache row -> floats
+__device__ __forceinline__ void wk_unpack(const uint4 &u, float (&f)[8]) {
+	f[0] = bf16_lo(u.x); f[1] = bf16_hi(u.x); f[2] = bf16_lo(u.y); f[3] = bf16_hi(u.y);
+	f[4] = bf16_lo(u.z); f[5] = bf16_hi(u.z); f[6] = bf16_lo(u.w); f[7] = bf16_hi(u.w);
+}
+__device__ __forceinline__ void wk_unpack(const uint4 &u, float (&f)[4]) {
+	f[0] = __uint_as_float(u.x); f[1] = __uint_as_float(u.y); f[2] = __uint_as_float(u.z); f[3] = __uint_as_float(u.w);
 }
 template <typename PT, typename CT, typename OT>
 __device__ void window_attn_token_cta(const WAttnArgs &a, int r, int g, int split, float *sm) {
 	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
 	const int per = a.H / a.G, dkp = a.dkp, dvp = a.dvp;
-	float *q = sm, *p = q + per * dkp, *acc = p + per * WK_KEYS, *ml = acc + 8 * dvp;
+	constexpr int V4 = 16 / int(sizeof(CT));                 // elements of a 16-byte load
+	const int cw = dvp < 32 * V4 ? dvp : 32 * V4;            // value columns of a pass
+	float *q = sm, *p = q + per * dkp, *acc = p + WK_HEADS * WK_KEYS, *ml = acc + 8 * WK_HEADS * (dvp < 256 ? dvp : 256), *cr = ml + 2 * WK_HEADS;
 	__shared__ int s_last;
 	const int seg = a.d.row_seg[r], seq = a.d.seg_seq[seg], i = a.d.seg_pos[seg];
 	const PT *row = reinterpret_cast<const PT *>(a.p) + size_t(r) * a.ldp;
@@ -457,107 +467,118 @@ __device__ void window_attn_token_cta(const WAttnArgs &a, int r, int g, int spli
 	const int pieces = (total + WK_KEYS - 1) / WK_KEYS, share = (pieces + a.nsplit - 1) / a.nsplit;
 	const int n_lo = split * share * WK_KEYS, n_hi = min(total, (split + 1) * share * WK_KEYS);
 	for (int x = tid; x < per * dkp; x += 256) q[x] = to_f32(row[a.p_q + g * per * dkp + x]) * a.scale;
-	if (tid < per) {
-		ml[2 * tid] = -INFINITY;
-		ml[2 * tid + 1] = 0.0f;
-	}
 	float *part = a.part + ((size_t(r) * a.G + g) * a.nsplit + split) * per * (dvp + 2);
-	__syncthreads();
-	constexpr int V4 = 16 / int(sizeof(CT));  // elements of a 16-byte load
-	for (int n0 = n_lo; n0 < n_hi; n0 += WK_KEYS) {
-		// scores: four lanes per key
-		{
-			const int n = n0 + (tid >> 2), sub = tid & 3;
-			const bool on = n < n_hi;
-			const int j = on ? (n < kept ? n : first + n - kept) : i;
-			const CT *k = (on && n < kept) ? ks + size_t(j) * a.G * dkp : kc + size_t(j % a.cap) * a.G * dkp;
-			for (int hh = 0; hh < per; hh += 4) {
-				float s[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-				const int nh = min(4, per - hh);
-				for (int c = sub * V4; c < dkp; c += 4 * V4) {
-					const uint4 u = *reinterpret_cast<const uint4 *>(k + c);
-					float kv[V4];
-					if (sizeof(CT) == 2) {
-						const uint32_t w[4] = {u.x, u.y, u.z, u.w};
-#pragma unroll
-						for (int e = 0; e < V4 / 2; e++) {
-							kv[2 * e] = bf16_lo(w[e]);
-							kv[2 * e + 1] = bf16_hi(w[e]);
-						}
-					} else {
-						kv[0] = __uint_as_float(u.x); kv[1] = __uint_as_float(u.y); kv[2] = __uint_as_float(u.z); kv[3] = __uint_as_float(u.w);
-					}
-#pragma unroll
-					for (int y = 0; y < 4; y++)
-						if (y < nh) {
-							const float *qh = q + (hh + y) * dkp + c;
-#pragma unroll
-							for (int e = 0; e < V4; e++) s[y] = fmaf(qh[e], kv[e], s[y]);
-						}
-				}
-#pragma unroll
-				for (int y = 0; y < 4; y++) {
-					s[y] += __shfl_xor_sync(0xffffffffu, s[y], 1);
-					s[y] += __shfl_xor_sync(0xffffffffu, s[y], 2);
-				}
-				if (sub < nh) {
-					float v = sub == 0 ? s[0] : (sub == 1 ? s[1] : (sub == 2 ? s[2] : s[3]));
-					const int h = g * per + hh + sub;
-					if (a.r1) v -= wa_bias(a.r1[h], a.r2[h], i - j);
-					p[(hh + sub) * WK_KEYS + (tid >> 2)] = on ? v : -INFINITY;
-				}
+	// lanes of a value row (a power of two), value rows a warp reads at once
+	int lpk = 1;
+	while (lpk * V4 < cw) lpk *= 2;
+	const int kpw = 32 / lpk, vsub = lane / lpk, vcol = (lane % lpk) * V4;
+	for (int h0 = 0; h0 < per; h0 += WK_HEADS) {
+		const int nh = min(WK_HEADS, per - h0);
+		for (int c0 = 0; c0 < dvp; c0 += cw) {  // (more than one pass only for very wide values: scores are formed again)
+			float o[WK_HEADS][V4] = {};
+			__syncthreads();
+			if (tid < WK_HEADS) {
+				ml[2 * tid] = -INFINITY;
+				ml[2 * tid + 1] = 0.0f;
 			}
-		}
-		__syncthreads();
-		// values: a head at a time; the warps take keys, the lanes value dimensions (16 bytes each), then the warps meet
-		for (int hh = 0; hh < per; hh++) {
-			const float s0 = p[hh * WK_KEYS + lane], s1 = p[hh * WK_KEYS + 32 + lane];
-			const float mo = ml[2 * hh], mn = fmaxf(mo, warp_max(fmaxf(s0, s1)));
-			const float p0 = expf(s0 - mn), p1 = expf(s1 - mn), sum = warp_sum(p0 + p1), corr = expf(mo - mn);
-			for (int c0 = 0; c0 < dvp; c0 += 32 * V4) {
-				const int c = c0 + lane * V4;
-				float o[V4] = {};
-				for (int e = warp; e < WK_KEYS && n0 + e < n_hi; e += 8) {
-					const float pe = __shfl_sync(0xffffffffu, e < 32 ? p0 : p1, e & 31);
-					const int n = n0 + e, j = n < kept ? n : first + n - kept;
-					const CT *v = n < kept ? vs + size_t(j) * a.G * dvp : vc + size_t(j % a.cap) * a.G * dvp;
-					if (c < dvp) {
-						const uint4 u = *reinterpret_cast<const uint4 *>(v + c);
-						if (sizeof(CT) == 2) {
-							const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+			__syncthreads();
+			for (int n0 = n_lo; n0 < n_hi; n0 += WK_KEYS) {
+				{  // scores: four lanes per key
+					const int n = n0 + (tid >> 2), sub = tid & 3;
+					const bool on = n < n_hi;
+					const int j = on ? (n < kept ? n : first + n - kept) : i;
+					const CT *k = (on && n < kept) ? ks + size_t(j) * a.G * dkp : kc + size_t(j % a.cap) * a.G * dkp;
+					float s[WK_HEADS] = {};
+#pragma unroll 4
+					for (int c = sub * V4; c < dkp; c += 4 * V4) {
+						float kv[V4];
+						wk_unpack(*reinterpret_cast<const uint4 *>(k + c), kv);
 #pragma unroll
-							for (int z = 0; z < V4 / 2; z++) {
-								o[2 * z] = fmaf(pe, bf16_lo(w[z]), o[2 * z]);
-								o[2 * z + 1] = fmaf(pe, bf16_hi(w[z]), o[2 * z + 1]);
+						for (int y = 0; y < WK_HEADS; y++)
+							if (y < nh) {
+								const float4 *qh = reinterpret_cast<const float4 *>(q + (h0 + y) * dkp + c);
+#pragma unroll
+								for (int e = 0; e < V4 / 4; e++) {
+									const float4 w = qh[e];
+									s[y] = fmaf(w.x, kv[4 * e], fmaf(w.y, kv[4 * e + 1], fmaf(w.z, kv[4 * e + 2], fmaf(w.w, kv[4 * e + 3], s[y]))));
+								}
 							}
-						} else {
-							o[0] = fmaf(pe, __uint_as_float(u.x), o[0]); o[1] = fmaf(pe, __uint_as_float(u.y), o[1]);
-							o[2] = fmaf(pe, __uint_as_float(u.z), o[2]); o[3] = fmaf(pe, __uint_as_float(u.w), o[3]);
-						}
+					}
+#pragma unroll
+					for (int y = 0; y < WK_HEADS; y++) {
+						s[y] += __shfl_xor_sync(0xffffffffu, s[y], 1);
+						s[y] += __shfl_xor_sync(0xffffffffu, s[y], 2);
+					}
+					if (sub < nh) {
+						float v = sub == 0 ? s[0] : (sub == 1 ? s[1] : (sub == 2 ? s[2] : s[3]));
+						const int h = g * per + h0 + sub;
+						if (a.r1) v -= wa_bias(a.r1[h], a.r2[h], i - j);
+						p[sub * WK_KEYS + (tid >> 2)] = on ? v : -INFINITY;
 					}
 				}
-				if (c < dvp)
+				__syncthreads();
+				if (warp < nh) {  // a warp per head: running maximum, weights, sum
+					const float s0 = p[warp * WK_KEYS + lane], s1 = p[warp * WK_KEYS + 32 + lane];
+					const float mo = ml[2 * warp], mn = fmaxf(mo, warp_max(fmaxf(s0, s1)));
+					const float p0 = expf(s0 - mn), p1 = expf(s1 - mn), sum = warp_sum(p0 + p1), corr = expf(mo - mn);
+					p[warp * WK_KEYS + lane] = p0;
+					p[warp * WK_KEYS + 32 + lane] = p1;
+					if (lane == 0) {
+						cr[warp] = corr;
+						ml[2 * warp + 1] = ml[2 * warp + 1] * corr + sum;
+						ml[2 * warp] = mn;
+					}
+				}
+				__syncthreads();
 #pragma unroll
-					for (int z = 0; z < V4; z++) acc[warp * dvp + c + z] = o[z];
-			}
-			__syncthreads();
-			for (int c = tid; c < dvp; c += 256) {
-				float o = 0.0f;
+				for (int y = 0; y < WK_HEADS; y++) {
+					const float corr = y < nh ? cr[y] : 0.0f;
 #pragma unroll
-				for (int w = 0; w < 8; w++) o += acc[w * dvp + c];
-				float *dst = part + hh * (dvp + 2) + c;
-				*dst = n0 == n_lo ? o : fmaf(*dst, corr, o);
+					for (int z = 0; z < V4; z++) o[y][z] *= corr;
+				}
+				const int c = c0 + vcol;
+				if (vcol < cw && c < dvp) {
+#pragma unroll 4
+					for (int e = warp * kpw + vsub; e < WK_KEYS; e += 8 * kpw) {
+						const int n = n0 + e;
+						if (n >= n_hi) break;
+						const int j = n < kept ? n : first + n - kept;
+						const CT *v = n < kept ? vs + size_t(j) * a.G * dvp : vc + size_t(j % a.cap) * a.G * dvp;
+						float vv[V4];
+						wk_unpack(*reinterpret_cast<const uint4 *>(v + c), vv);
+#pragma unroll
+						for (int y = 0; y < WK_HEADS; y++)
+							if (y < nh) {
+								const float pe = p[y * WK_KEYS + e];
+#pragma unroll
+								for (int z = 0; z < V4; z++) o[y][z] = fmaf(pe, vv[z], o[y][z]);
+							}
+					}
+				}
 			}
-			if (tid == 0) {
-				ml[2 * hh] = mn;
-				ml[2 * hh + 1] = ml[2 * hh + 1] * corr + sum;
-			}
+			// the warp's value rows meet by shuffles, the warps in shared memory
+#pragma unroll
+			for (int y = 0; y < WK_HEADS; y++)
+#pragma unroll
+				for (int z = 0; z < V4; z++) {
+					float v = o[y][z];
+					for (int d = lpk; d < 32; d *= 2) v += __shfl_xor_sync(0xffffffffu, v, d);
+					if (y < nh && vsub == 0 && vcol < cw && c0 + vcol < dvp) acc[(warp * WK_HEADS + y) * cw + vcol + z] = v;
+				}
 			__syncthreads();
+			for (int x = tid; x < nh * cw; x += 256) {
+				const int y = x / cw, c = x % cw;
+				if (c0 + c >= dvp) continue;
+				float v = 0.0f;
+#pragma unroll
+				for (int w = 0; w < 8; w++) v += acc[(w * WK_HEADS + y) * cw + c];
+				part[(h0 + y) * (dvp + 2) + c0 + c] = v;
+			}
+			if (tid < nh) {
+				part[(h0 + tid) * (dvp + 2) + dvp] = ml[2 * tid];
+				part[(h0 + tid) * (dvp + 2) + dvp + 1] = ml[2 * tid + 1];
+			}
 		}
-	}
-	if (tid < per) {
-		part[tid * (dvp + 2) + dvp] = ml[2 * tid];
-		part[tid * (dvp + 2) + dvp + 1] = ml[2 * tid + 1];
 	}
 	__threadfence();
 	__syncthreads();

@@ -976,6 +976,7 @@ template <typename PT> int launch_delta(const DeltaArgs &a, int R, int nseg, int
 template <typename PT> int launch_ln_conv(void *out, int ldo, const float *x, int ldx, const float *w, const float *cw, float *hist, const StepDesc &d, int R,
                                           int D, int taps, float eps, cudaStream_t st) {
 	int rows = LC_ROWS;
+	while (rows > 1 && R < rows * 2 * g_num_sms) rows /= 2;
 	while (rows > 1 && ln_conv_smem(rows, taps, D) > 100 * 1024) rows /= 2;
 	const size_t smem = ln_conv_smem(rows, taps, D);
 	const dim3 grid((R + rows - 1) / rows);
