@@ -230,6 +230,24 @@ def test_lockstep_decode_in_batches(capi, folder, dtype):
     m.close()
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_large_batch_of_equal_requests(capi, folder, dtype):
+    """150 sequences, several pieces of keys per CTA: every row has the same bits, and they are the plain result"""
+    path, cfg, W = folder("real_heads")
+    toks, B = N.tokens(cfg, 190, 31), 150
+    want = Ref.get("real_heads", cfg, W, toks)[0]
+    m = capi.Model.open(path, dtype)
+    st = m.state(B, 200)
+    for b0 in range(0, B, 50):
+        st.step([(b, toks[:150], []) for b in range(b0, b0 + 50)])
+    for i in range(150, 190):
+        got = st.decode(np.full(B, toks[i]))
+        assert np.array_equal(got, np.broadcast_to(got[0], got.shape)), (i, np.nonzero((got != got[0]).any(1))[0])
+        close(got[0], want[i], dtype)
+    st.close()
+    m.close()
+
+
 # ------------------------------------------------------------------ edges
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("window,keep", [(24, 3), (64, 1), (65, 64), (130, 70), (7, 0)])

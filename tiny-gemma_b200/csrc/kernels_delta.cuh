@@ -74,14 +74,14 @@ __device__ __forceinline__ void delta_hist_save(const DeltaArgs &a, int row0, in
 }
 
 // ------------------------------------------------------------------ one token
-// smem: q[dk] k[dk] g[dk] v[dv] gate[dv] part[nparts*2*dv] red[32]. 256 threads. Row r of the step is a segment of
+// smem: q[dk] k[dk] g[dk] v[dv] gate[dv] part[nparts*2*dv] red[64] low-rank inputs[ra + rg]. 256 threads. Row r of the step is a segment of
 // length 1.
 __host__ __device__ inline int delta_token_parts(int dv) { return dv >= 256 ? 1 : 256 / dv; }
 // the state of a head held in registers between its two uses: 16 rows of 4 columns per thread
 __host__ __device__ inline bool delta_token_in_regs(int dk, int dv) { return dk <= 128 && dv <= 128 && dv % 4 == 0; }
-__host__ __device__ inline size_t delta_token_smem(int dk, int dv) {
+__host__ __device__ inline size_t delta_token_smem(int dk, int dv, int ra, int rg) {
 	const int parts = delta_token_in_regs(dk, dv) ? 8 : delta_token_parts(dv);
-	return (size_t(3) * dk + 2 * size_t(dv) + size_t(parts) * 2 * dv + 64) * 4;
+	return (size_t(3) * dk + 2 * size_t(dv) + size_t(parts) * 2 * dv + 64 + ra + rg) * 4;
 }
 template <typename PT, typename OT>
 __device__ void delta_token_cta(const DeltaArgs &a, int r, int h, float *sm) {
@@ -106,25 +106,45 @@ __device__ void delta_token_cta(const DeltaArgs &a, int r, int h, float *sm) {
 			st[e] = !fresh && i < dk && 4 * lane < dv ? *reinterpret_cast<const float4 *>(S + size_t(i) * dv + 4 * lane) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 		}
 	}
+	float *lr = red + 64;
+	for (int i = tid; i < a.ra + a.rg; i += 256) lr[i] = to_f32(prow[i < a.ra ? a.p_a1 + i : a.p_g1 + i - a.ra]);
 	// convolutions
 	for (int i = tid; i < 2 * dk + dv; i += 256) {
-		if (i < dk) sq[i] = delta_conv<PT>(a, r, pos, hr, C, 0, kh * dk + i);
-		else if (i < 2 * dk) sk[i - dk] = delta_conv<PT>(a, r, pos, hr, C, 0, (a.KH + kh) * dk + i - dk);
-		else sv[i - 2 * dk] = delta_conv<PT>(a, r, pos, hr, C, 0, 2 * a.KH * dk + h * dv + i - 2 * dk);
+		const int ch = i < dk ? kh * dk + i : (i < 2 * dk ? (a.KH + kh) * dk + i - dk : 2 * a.KH * dk + h * dv + i - 2 * dk);
+		float y;
+		if (a.taps <= 4) {  // all loads in flight together
+			float w[4], x[4];
+#pragma unroll
+			for (int j = 0; j < 4; j++) {
+				w[j] = j >= 4 - a.taps ? a.cw[size_t(j - (4 - a.taps)) * C + ch] : 0.0f;
+				x[j] = j >= 4 - a.taps ? delta_conv_in<PT>(a, r, pos, hr, C, j - 3, ch) : 0.0f;
+			}
+			y = silu_f(fmaf(w[3], x[3], fmaf(w[2], x[2], fmaf(w[1], x[1], w[0] * x[0]))));
+		} else {
+			y = delta_conv<PT>(a, r, pos, hr, C, 0, ch);
+		}
+		(i < dk ? sq[i] : (i < 2 * dk ? sk[i - dk] : sv[i - 2 * dk])) = y;
 	}
-	// low-rank second stages: eight lanes per output
+	__syncthreads();
+	// low-rank second stages: eight lanes per output, 16 bytes of its row per lane and round
 	{
 		const float ea = expf(a.A_log[h]);
 		const int sub = lane & 7;
+#pragma unroll 4
 		for (int o0 = 0; o0 < dk + dv; o0 += 32) {
 			const int o = o0 + warp * 4 + (lane >> 3);
+			const bool first = o < dk;
+			const __nv_bfloat16 *w = first ? a.a2 + size_t(h * dk + o) * a.lda2 : a.g2 + size_t(h * dv + o - dk) * a.ldg2;
+			const float *x = first ? lr : lr + a.ra;
+			const int n = o < dk + dv ? (first ? a.ra : a.rg) : 0;
 			float s = 0.0f;
-			if (o < dk) {
-				const __nv_bfloat16 *w = a.a2 + size_t(h * dk + o) * a.lda2;
-				for (int j = sub; j < a.ra; j += 8) s = fmaf(__bfloat162float(w[j]), to_f32(prow[a.p_a1 + j]), s);
-			} else if (o < dk + dv) {
-				const __nv_bfloat16 *w = a.g2 + size_t(h * dv + o - dk) * a.ldg2;
-				for (int j = sub; j < a.rg; j += 8) s = fmaf(__bfloat162float(w[j]), to_f32(prow[a.p_g1 + j]), s);
+#pragma unroll 2
+			for (int j = 8 * sub; j < n; j += 64) {
+				const uint4 u = *reinterpret_cast<const uint4 *>(w + j);
+				s = fmaf(bf16_lo(u.x), x[j], s); s = fmaf(bf16_hi(u.x), x[j + 1], s);
+				s = fmaf(bf16_lo(u.y), x[j + 2], s); s = fmaf(bf16_hi(u.y), x[j + 3], s);
+				s = fmaf(bf16_lo(u.z), x[j + 4], s); s = fmaf(bf16_hi(u.z), x[j + 5], s);
+				s = fmaf(bf16_lo(u.w), x[j + 6], s); s = fmaf(bf16_hi(u.w), x[j + 7], s);
 			}
 			s += __shfl_xor_sync(0xffffffffu, s, 1);
 			s += __shfl_xor_sync(0xffffffffu, s, 2);

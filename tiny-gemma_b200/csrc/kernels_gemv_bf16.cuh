@@ -45,7 +45,7 @@ struct GemvArgs {
 constexpr int GV_THREADS = 256;
 __host__ __device__ inline int gv_k8(int K) { return (K + 7) / 8; }
 template <int R, int NR> __host__ __device__ constexpr int gv_red_floats() { return 2 * 8 * NR * R; }
-template <int R, int NR> size_t gv_smem(int K) { return (size_t(R) * 8 * gv_k8(K) + gv_red_floats<R, NR>() + 32) * 4; }
+template <int R, int NR> size_t gv_smem(int K, int pro) { return ((size_t(R) + pro) * 8 * gv_k8(K) + gv_red_floats<R, NR>() + 32) * 4; }
 
 __device__ __forceinline__ float gv_block_sum(float v, float *red) {
 	v = warp_sum(v);
@@ -67,6 +67,7 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 	float *xs = gv_sm;                                   // [R][two halves of 8 k][K8] float4
 	float *red = gv_sm + size_t(R) * 8 * K8;             // [2][row set][KS][NR][R]
 	float *bred = red + gv_red_floats<R, NR>();
+	float *wn = bred + 32, *hc = wn + 8 * K8;            // norm weight (x its factor in the convolution); history's share
 	constexpr int SETS = 8 / KS, GROUP = SETS * NR;      // weight rows per CTA and group
 	const int set = warp / KS, ks = warp % KS;
 	const int n_out = EPI == GV_GEGLU ? a.N / 2 : (EPI == GV_LOGITS ? a.ldo : a.N);
@@ -96,6 +97,10 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 	};
 	uint4 cur[NR], nxt[NR];
 	load(blockIdx.x, 0, cur);
+	if (PRO != GV_VEC) {  // (weights too: nobody's output)
+#pragma unroll 4
+		for (int k = tid; k < a.D; k += GV_THREADS) wn[k] = PRO == GV_LN_CONV ? fmaf(a.cw[size_t(a.taps - 1) * a.D + k], a.w[k], a.w[k]) : a.w[k];
+	}
 	pdl_wait();
 
 	// ---------------------------------------------------------------- prologue: activations into shared memory
@@ -116,10 +121,31 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 				tok = 0;
 			}
 		}
+		const int H = PRO == GV_LN_CONV ? a.taps - 1 : 0;
+		const float *hr = nullptr;
+		float *hw = nullptr;
+		int pos = 0;
+		if (PRO == GV_LN_CONV) {
+			pos = a.d.seg_pos[seg];
+			float *hb = a.hist + size_t(a.d.seg_seq[seg]) * 2 * H * a.D;
+			hr = hb + size_t(a.d.seg_par[seg]) * H * a.D;
+			hw = hb + size_t(a.d.seg_par[seg] ^ 1) * H * a.D;
+		}
 		float s = 0.0f;
+#pragma unroll 2
 		for (int k = tid; k < a.D; k += GV_THREADS) {
 			float v = a.embed_mode == 1 ? 0.0f : a.x[size_t(r) * a.ldx + k];
 			if (a.embed_mode) v += __bfloat162float(a.embed[size_t(tok) * a.lde + k]);
+			if (PRO == GV_LN_CONV) {
+				float c = 0.0f;
+#pragma unroll 3
+				for (int j = 0; j < H; j++) {
+					const float u = pos - H + j >= 0 ? hr[size_t(j) * a.D + k] : 0.0f;
+					c = fmaf(a.cw[size_t(j) * a.D + k], u, c);
+					if (blockIdx.x == 0 && j > 0) hw[size_t(j - 1) * a.D + k] = u;
+				}
+				hc[k] = c;
+			}
 			xr[xi(k)] = v;
 			s += v;
 		}
@@ -130,31 +156,14 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 			q = fmaf(c, c, q);
 		}
 		const float rstd = 1.0f / sqrtf(gv_block_sum(q, bred) / float(a.D) + a.eps);
-		const int H = a.taps - 1;
-		float *hb = nullptr;
-		const float *hr = nullptr;
-		float *hw = nullptr;
-		int pos = 0;
-		if (PRO == GV_LN_CONV) {
-			pos = a.d.seg_pos[seg];
-			hb = a.hist + size_t(a.d.seg_seq[seg]) * 2 * H * a.D;
-			hr = hb + size_t(a.d.seg_par[seg]) * H * a.D;
-			hw = hb + size_t(a.d.seg_par[seg] ^ 1) * H * a.D;
-		}
 		for (int k = tid; k < 8 * K8; k += GV_THREADS) {
 			float y = 0.0f;
 			if (k < a.D) {
-				const float n = (xr[xi(k)] - mean) * rstd * a.w[k];
-				y = n;
+				const float n = (xr[xi(k)] - mean) * rstd;
+				y = n * wn[k];
 				if (PRO == GV_LN_CONV) {
-					float c = 0.0f;
-					for (int j = 0; j < H; j++) {
-						const float v = pos - H + j >= 0 ? hr[size_t(j) * a.D + k] : 0.0f;
-						c = fmaf(a.cw[size_t(j) * a.D + k], v, c);
-						if (blockIdx.x == 0 && j > 0) hw[size_t(j - 1) * a.D + k] = v;
-					}
-					y += fmaf(a.cw[size_t(H) * a.D + k], n, c);
-					if (blockIdx.x == 0 && H > 0) hw[size_t(H - 1) * a.D + k] = n;
+					y += hc[k];
+					if (blockIdx.x == 0 && H > 0) hw[size_t(H - 1) * a.D + k] = n * a.w[k];
 				}
 				if (a.norm_out && blockIdx.x == 0) a.norm_out[size_t(r) * a.D + k] = y;
 			}

@@ -555,6 +555,7 @@ __device__ void window_attn_token_cta(const WAttnArgs &a, int r, int g, int spli
 							}
 					}
 				}
+				__syncthreads();  // (p and cr are written again by the next piece)
 			}
 			// the warp's value rows meet by shuffles, the warps in shared memory
 #pragma unroll

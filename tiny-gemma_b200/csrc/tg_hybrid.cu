@@ -590,7 +590,7 @@ template <int EPI> int launch_gemm_f32(const float *A, int lda, const Lin &w, co
 }
 
 template <int R, int NR, int KS, int PRO, int EPI> int launch_gemv(const GemvArgs &g, cudaStream_t st) {
-	const size_t smem = gv_smem<R, NR>(g.K);
+	const size_t smem = gv_smem<R, NR>(g.K, PRO);
 	auto kernel = gemv_bf16_kernel<R, NR, KS, PRO, EPI>;
 	TG_TRY(allow_smem(kernel, smem));
 	int occ = 1;
@@ -929,7 +929,7 @@ DeltaArgs HybridState::delta_args(const StepDesc &d, int run, const void *p, int
 
 namespace {
 template <typename PT, typename CT, typename OT> int launch_token_mix(const WAttnArgs &w, const DeltaArgs &d, int R, cudaStream_t st) {
-	const size_t smem = std::max(wattn_token_smem(w.H / w.G, w.dkp, w.dvp), delta_token_smem(d.dk, d.dv));
+	const size_t smem = std::max(wattn_token_smem(w.H / w.G, w.dkp, w.dvp), delta_token_smem(d.dk, d.dv, d.ra, d.rg));
 	auto kernel = hybrid_token_mix_kernel<PT, CT, OT>;
 	TG_TRY(allow_smem(kernel, smem));
 	launch_k(kernel, dim3(w.G * w.nsplit + d.H, R), dim3(256), smem, st, w, d);
