@@ -286,7 +286,7 @@ template <typename PT>
 __global__ void __launch_bounds__(256, 3) delta_block_kernel(DeltaArgs a) {
 	pdl_trigger();
 	pdl_wait();
-	extern __shared__ float db_sm[];
+	extern __shared__ __align__(16) float db_sm[];
 	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
 	const int blk = blockIdx.x, h = blockIdx.y, seg = blockIdx.z;
 	const int len = a.d.seg_len[seg], t0 = blk * DB;
@@ -436,9 +436,12 @@ __global__ void __launch_bounds__(256, 3) delta_block_kernel(DeltaArgs a) {
 		for (int t = 0; t < DB; t++) x[t] = src[t * ld];
 #pragma unroll
 		for (int t = 0; t < DB; t++) {
-			float s = 0.0f;
+			float s = 0.0f;  // (T is zero above the diagonal)
 #pragma unroll
-			for (int j = 0; j <= t; j++) s = fmaf(sT[t * DB + j], x[j], s);
+			for (int j = 0; j <= t; j += 4) {
+				const float4 w = *reinterpret_cast<const float4 *>(sT + t * DB + j);
+				s = fmaf(w.x, x[j], fmaf(w.y, x[j + 1], fmaf(w.z, x[j + 2], fmaf(w.w, x[j + 3], s))));
+			}
 			dst[size_t(t) * ld] = s;
 		}
 	}

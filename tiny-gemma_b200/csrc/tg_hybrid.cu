@@ -952,7 +952,7 @@ template <int RPL, int NW, int NC> int launch_scan_nc(const DeltaArgs &a, int ns
 template <int RPL, int NW> int launch_scan(const DeltaArgs &a, int nseg, cudaStream_t st) {
 	static const int forced = env_int("TG_SCAN_COLS", 0);
 	const long long cols = (long long)a.dv * a.H * nseg;
-	const int nc = forced ? forced : (cols <= 4 * g_num_sms ? 1 : (cols <= 16 * g_num_sms ? 2 : 4));
+	const int nc = forced ? forced : (cols <= 4 * g_num_sms ? 1 : (cols <= 40 * g_num_sms ? 2 : 4));
 	if (nc == 1) return launch_scan_nc<RPL, NW, 1>(a, nseg, st);
 	if (nc == 2) return launch_scan_nc<RPL, NW, 2>(a, nseg, st);
 	return launch_scan_nc<RPL, NW, 4>(a, nseg, st);
@@ -977,7 +977,7 @@ template <typename PT> int launch_ln_conv(void *out, int ldo, const float *x, in
                                           int D, int taps, float eps, cudaStream_t st) {
 	int rows = LC_ROWS;
 	while (rows > 1 && R < rows * 2 * g_num_sms) rows /= 2;
-	while (rows > 1 && ln_conv_smem(rows, taps, D) > 100 * 1024) rows /= 2;
+	while (rows > 1 && ln_conv_smem(rows, taps, D) > 112 * 1024) rows /= 2;
 	const size_t smem = ln_conv_smem(rows, taps, D);
 	const dim3 grid((R + rows - 1) / rows);
 	if (taps <= 4) {
