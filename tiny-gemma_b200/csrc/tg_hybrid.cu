@@ -373,7 +373,7 @@ int read_config(const json::Value &c, HybridModel *m) {
 		L.at.scale = float(r.num(a, "scale", "left"));
 		const json::Value *mk = r.obj(a, "mask", "left");
 		L.at.window = r.size(mk, "size", "mask");
-		L.at.keep = r.size(mk, "keep_first", "mask", 0);
+		if (mk && mk->find("keep_first")) L.at.keep = r.size(mk, "keep_first", "mask", 0);
 		L.at.dkp = round_up(L.at.dk, 16);
 		L.at.dvp = round_up(L.at.dv, 16);
 		L.de.H = r.size(d, "heads", "right");
