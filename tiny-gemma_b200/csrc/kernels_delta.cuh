@@ -301,33 +301,47 @@ __global__ void __launch_bounds__(256, 3) delta_block_kernel(DeltaArgs a) {
 	      *sb = sT + DB * DB;
 	// q, k, g, v, beta; tokens past the end change nothing (g = 1, everything else 0)
 	const float ea = expf(a.A_log[h]);
-	for (int i = tid; i < 2 * dkp + dv; i += 256) {  // a thread walks a channel down the block's tokens
-		const int kind = i < dkp ? 0 : (i < 2 * dkp ? 1 : 2), c = kind == 0 ? i : (kind == 1 ? i - dkp : i - 2 * dkp);
-		float *dst = (kind == 0 ? sq : (kind == 1 ? sk : sv)) + c;
+	constexpr int HB = DB / 2;  // a thread walks a channel down half of the block's tokens
+	for (int i = tid; i < 2 * (2 * dkp + dv); i += 256) {
+		const int part = i >= 2 * dkp + dv, f = part * HB, e = i - part * (2 * dkp + dv);
+		const int kind = e < dkp ? 0 : (e < 2 * dkp ? 1 : 2), c = kind == 0 ? e : (kind == 1 ? e - dkp : e - 2 * dkp);
 		const int ld = kind == 2 ? dv : dkp;
+		float *dst = (kind == 0 ? sq : (kind == 1 ? sk : sv)) + f * ld + c;
 		if (kind < 2 && c >= dk) {
-			for (int t = 0; t < DB; t++) dst[t * ld] = 0.0f;
+			for (int t = 0; t < HB; t++) dst[t * ld] = 0.0f;
 			continue;
 		}
 		const int ch = kind == 0 ? kh * dk + c : (kind == 1 ? (a.KH + kh) * dk + c : 2 * a.KH * dk + h * dv + c);
 		if (a.taps <= 4) {
-			float x[DB + 3], w[4];
+			float x[HB + 3], w[4];
 #pragma unroll
 			for (int j = 0; j < 4; j++) w[j] = j >= 4 - a.taps ? a.cw[size_t(j - (4 - a.taps)) * C + ch] : 0.0f;
+			const int tf = t0 + f - 3;
+			if (tf >= 0) {  // no history: plain rows (those past the segment's end are not used)
+				const PT *px = reinterpret_cast<const PT *>(a.p) + size_t(row0 + tf) * a.ldp + a.p_conv + ch;
 #pragma unroll
-			for (int j = 0; j < DB + 3; j++) x[j] = j - 3 < n && 3 - j < a.taps ? delta_conv_in<PT>(a, row0, pos, hr, C, t0 + j - 3, ch) : 0.0f;
+				for (int j = 0; j < HB + 3; j++) x[j] = f + j - 3 < n ? to_f32(px[size_t(j) * a.ldp]) : 0.0f;
+			} else {
 #pragma unroll
-			for (int t = 0; t < DB; t++) {
+				for (int j = 0; j < HB + 3; j++) x[j] = f + j - 3 < n && 3 - j < a.taps ? delta_conv_in<PT>(a, row0, pos, hr, C, tf + j, ch) : 0.0f;
+			}
+#pragma unroll
+			for (int t = 0; t < HB; t++) {
 				const float y = fmaf(w[3], x[t + 3], fmaf(w[2], x[t + 2], fmaf(w[1], x[t + 1], w[0] * x[t])));
-				dst[t * ld] = t < n ? __fdividef(y, 1.0f + __expf(-y)) : 0.0f;
+				dst[t * ld] = f + t < n ? __fdividef(y, 1.0f + __expf(-y)) : 0.0f;
 			}
 		} else {
-			for (int t = 0; t < DB; t++) dst[t * ld] = t < n ? delta_conv<PT>(a, row0, pos, hr, C, t0 + t, ch) : 0.0f;
+			for (int t = 0; t < HB; t++) dst[t * ld] = f + t < n ? delta_conv<PT>(a, row0, pos, hr, C, t0 + f + t, ch) : 0.0f;
 		}
 	}
-	for (int i = tid; i < DB * dkp; i += 256) {
-		const int t = i / dkp, c = i % dkp;
-		sg[i] = t < n && c < dk ? expf(-ea * softplus_f(a.z[size_t(row0 + t0 + t) * a.ldz + h * dk + c] + a.dt_bias[h * dk + c])) : 1.0f;
+	for (int i = tid; i < 2 * dkp; i += 256) {
+		const int part = i >= dkp, f = part * HB, c = i - part * dkp;
+		const float bias = c < dk ? a.dt_bias[h * dk + c] : 0.0f;
+		float zv[HB];
+#pragma unroll
+		for (int t = 0; t < HB; t++) zv[t] = f + t < n && c < dk ? a.z[size_t(row0 + t0 + f + t) * a.ldz + h * dk + c] : 0.0f;
+#pragma unroll
+		for (int t = 0; t < HB; t++) sg[(f + t) * dkp + c] = f + t < n && c < dk ? expf(-ea * softplus_f(zv[t] + bias)) : 1.0f;
 	}
 	if (tid < DB) sb[tid] = tid < n ? sigmoid_f(to_f32(reinterpret_cast<const PT *>(a.p)[size_t(row0 + t0 + tid) * a.ldp + a.p_b + h])) : 0.0f;
 	if (t0 + DB >= len) {  // the segment's last block
