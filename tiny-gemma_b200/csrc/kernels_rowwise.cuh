@@ -126,96 +126,124 @@ __global__ void __launch_bounds__(128) layer_norm_kernel(OT *out, int ldo, const
 // meets the current row). The taps - 1 normed rows before a segment come from hist[seq][par], and the segment's
 // last ones (or, in a shorter segment, the older ones that still matter) are left in hist[seq][par ^ 1], oldest
 // first. hist: [B][2][taps-1][D]. Rows before a sequence's start count as zero, whatever hist holds.
-// One CTA per `rows` (<= LC_ROWS) consecutive rows: its warps norm these rows and the taps - 1 before them into shared
-// memory, then a thread walks its channels down the rows with the window in registers.
-constexpr int LC_ROWS = 8;
-__host__ __device__ inline size_t ln_conv_smem(int rows, int taps, int D) { return size_t(rows + taps - 1) * ((D + 3) & ~3) * 4; }
-template <typename OT, int MT>
-__global__ void __launch_bounds__(256) ln_conv_kernel(OT *out, int ldo, const float *x, int ldx, const float *w, const float *cw, float *hist,
-                                                      StepDesc d, int R, int D, int taps, float eps, int rows) {
+// Two kernels: mean and 1/sqrt(var + eps) of every row, then a walk down the rows with the window in registers, four
+// channels per thread, LC_ROWS rows per CTA (the rows before them are normed again, not exchanged).
+static __global__ void __launch_bounds__(128) ln_stats_kernel(float2 *stats, const float *x, int ldx, int D, float eps) {
 	pdl_trigger();
 	pdl_wait();
-	extern __shared__ __align__(16) float lc_sm[];
-	__shared__ int seg_s[LC_ROWS];
-	const int r0 = blockIdx.x * rows, nr = min(rows, R - r0), H = taps - 1, ld = (D + 3) & ~3;
-	const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-	if (threadIdx.x < nr) seg_s[threadIdx.x] = d.row_seg[r0 + threadIdx.x];
-	for (int i = warp; i < nr + H; i += 8) {  // rows r0 - H .. r0 + nr - 1
-		const int r = r0 - H + i;
-		if (r < 0 || (i < H && d.row_seg[r] != d.row_seg[r0])) continue;  // (another segment's rows are not in any window)
-		const float *xr = x + size_t(r) * ldx;
-		float *n = lc_sm + size_t(i) * ld;
-		float s = 0.0f;
-#pragma unroll 8
-		for (int c = 4 * lane; c < D; c += 128) {  // (columns D .. ldx - 1 of x are zero)
-			const float4 v = *reinterpret_cast<const float4 *>(xr + c);
-			*reinterpret_cast<float4 *>(n + c) = v;
-			s += (v.x + v.y) + (v.z + v.w);
-		}
-		const float mean = warp_sum(s) / float(D);
-		float q = 0.0f;
-#pragma unroll 4
-		for (int c = 4 * lane; c < D; c += 128) {
-			const float4 v = *reinterpret_cast<const float4 *>(n + c);
-			const float a0 = v.x - mean, a1 = c + 1 < D ? v.y - mean : 0.0f, a2 = c + 2 < D ? v.z - mean : 0.0f, a3 = c + 3 < D ? v.w - mean : 0.0f;
-			q = fmaf(a0, a0, fmaf(a1, a1, fmaf(a2, a2, fmaf(a3, a3, q))));
-		}
-		const float f = 1.0f / sqrtf(warp_sum(q) / float(D) + eps);
-#pragma unroll 4
-		for (int c = lane; c < D; c += 32) n[c] = (n[c] - mean) * f * w[c];
-	}
-	__syncthreads();
-	for (int c = threadIdx.x; c < ldo; c += 256) {
-		if (c >= D) {
-			for (int i = 0; i < nr; i++) out[size_t(r0 + i) * ldo + c] = from_f32<OT>(0.0f);
-			continue;
-		}
-		float cf[MT], win[MT];  // win[MT-1] is the current row; taps are right-aligned
+	__shared__ float red[4];
+	const int tid = threadIdx.x;
+	const float *xr = x + size_t(blockIdx.x) * ldx;
+	float mean, q = 0.0f, s = 0.0f;
+	if (D <= 4096 && D % 4 == 0) {
+		float4 v[8];
 #pragma unroll
-		for (int j = 0; j < MT; j++) cf[j] = j >= MT - taps ? cw[size_t(j - (MT - taps)) * D + c] : 0.0f;
-		int seg = -1, row0 = 0, len = 0;
-		float *hw = nullptr;
-		for (int i = 0; i < nr; i++) {
-			const int r = r0 + i;
+		for (int j = 0; j < 8; j++) {
+			const int c = 4 * (tid + 128 * j);
+			v[j] = c < D ? *reinterpret_cast<const float4 *>(xr + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+			s += (v[j].x + v[j].y) + (v[j].z + v[j].w);
+		}
+		mean = cta_sum<4>(s, red) / float(D);
+#pragma unroll
+		for (int j = 0; j < 8; j++)
+			if (4 * (tid + 128 * j) < D) {
+				v[j].x -= mean; v[j].y -= mean; v[j].z -= mean; v[j].w -= mean;
+				q = fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, fmaf(v[j].z, v[j].z, fmaf(v[j].w, v[j].w, q))));
+			}
+	} else {
+		for (int c = tid; c < D; c += 128) s += xr[c];
+		mean = cta_sum<4>(s, red) / float(D);
+		for (int c = tid; c < D; c += 128) q = fmaf(xr[c] - mean, xr[c] - mean, q);
+	}
+	q = cta_sum<4>(q, red);
+	if (tid == 0) stats[blockIdx.x] = make_float2(mean, 1.0f / sqrtf(q / float(D) + eps));
+}
+
+// grid (ceil(R / rows), ceil(ldo / 512)); rows <= LC_ROWS; ldx and ldo multiples of 4
+constexpr int LC_ROWS = 16;
+template <typename OT, int MT>
+__global__ void __launch_bounds__(128) ln_conv_kernel(OT *out, int ldo, const float *x, int ldx, const float2 *stats, const float *w, const float *cw,
+                                                      float *hist, StepDesc d, int R, int D, int taps, int rows) {
+	pdl_trigger();
+	pdl_wait();
+	__shared__ float2 st[LC_ROWS + MT];
+	__shared__ int seg_s[LC_ROWS];
+	const int r0 = blockIdx.x * rows, nr = min(rows, R - r0), H = taps - 1, tid = threadIdx.x;
+	if (tid < nr) seg_s[tid] = d.row_seg[r0 + tid];
+	if (tid < nr + H && r0 - H + tid >= 0) st[tid] = stats[r0 - H + tid];
+	__syncthreads();
+	const int c = 4 * (blockIdx.y * 128 + tid);
+	if (c >= ldo) return;
+	if (c >= D) {
+		for (int i = 0; i < nr; i++) store4<OT>(out + size_t(r0 + i) * ldo + c, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
+		return;
+	}
+	auto get = [&](const float *p) {  // four consecutive channels of an unpadded row
+		return make_float4(p[0], c + 1 < D ? p[1] : 0.0f, c + 2 < D ? p[2] : 0.0f, c + 3 < D ? p[3] : 0.0f);
+	};
+	auto put = [&](float *p, const float4 &v) {
+		p[0] = v.x;
+		if (c + 1 < D) p[1] = v.y;
+		if (c + 2 < D) p[2] = v.z;
+		if (c + 3 < D) p[3] = v.w;
+	};
+	auto norm = [&](const float4 &v, const float2 &t, const float4 &g) {
+		return make_float4((v.x - t.x) * t.y * g.x, (v.y - t.x) * t.y * g.y, (v.z - t.x) * t.y * g.z, (v.w - t.x) * t.y * g.w);
+	};
+	const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f), wc = get(w + c);
+	float4 cf[MT], win[MT];  // win[MT-1] is the current row; taps are right-aligned
+#pragma unroll
+	for (int j = 0; j < MT; j++) cf[j] = j >= MT - taps ? get(cw + size_t(j - (MT - taps)) * D + c) : zero;
+	int seg = -1, row0 = 0, len = 0;
+	float *hw = nullptr;
+	for (int i0 = 0; i0 < nr; i0 += 4) {
+		float4 xv[4];
+#pragma unroll
+		for (int u = 0; u < 4; u++) xv[u] = i0 + u < nr ? *reinterpret_cast<const float4 *>(x + size_t(r0 + i0 + u) * ldx + c) : zero;
+#pragma unroll
+		for (int u = 0; u < 4; u++) {
+			const int i = i0 + u, r = r0 + i;
+			if (i >= nr) break;
 			if (seg_s[i] != seg) {
 				seg = seg_s[i];
 				row0 = d.seg_row[seg];
 				len = d.seg_len[seg];
 				const int pos = d.seg_pos[seg];
-				float *hb = hist + size_t(d.seg_seq[seg]) * 2 * H * D;
+				float *hb = hist + size_t(d.seg_seq[seg]) * 2 * H * D + c;
 				const float *hr = hb + size_t(d.seg_par[seg]) * H * D;
 				hw = hb + size_t(d.seg_par[seg] ^ 1) * H * D;
 				const int t = r - row0;
 #pragma unroll
 				for (int j = 0; j < MT; j++) {  // slot j of the window before row t: time t - (MT - j)
 					const int back = MT - j, tt = t - back;
-					float v = 0.0f;
+					win[j] = zero;
 					if (back <= H) {
 						if (tt >= 0)
-							v = lc_sm[size_t(i + H - back) * ld + c];
+							win[j] = norm(*reinterpret_cast<const float4 *>(x + size_t(r - back) * ldx + c), st[i + H - back], wc);
 						else if (pos + tt >= 0)
-							v = hr[size_t(H + tt) * D + c];
+							win[j] = get(hr + size_t(H + tt) * D);
 					}
-					win[j] = v;
 				}
 				if (t == 0)  // history rows that lie before this segment and stay relevant
 					for (int q = 0; q < H; q++) {
 						const int tt = len - H + q;
-						if (tt < 0) hw[size_t(q) * D + c] = pos + tt >= 0 ? hr[size_t(H + tt) * D + c] : 0.0f;
+						if (tt < 0) put(hw + size_t(q) * D, pos + tt >= 0 ? get(hr + size_t(H + tt) * D) : zero);
 					}
 			}
-			const float nv = lc_sm[size_t(i + H) * ld + c];
-			float y = 0.0f;
+			const float4 nv = norm(xv[u], st[i + H], wc);
+			float4 y = nv;
 #pragma unroll
-			for (int j = 0; j < MT - 1; j++) {
-				win[j] = win[j + 1];
-				y = fmaf(cf[j], win[j], y);
+			for (int j = 0; j < MT; j++) {
+				win[j] = j + 1 < MT ? win[j + 1] : nv;
+				y.x = fmaf(cf[j].x, win[j].x, y.x); y.y = fmaf(cf[j].y, win[j].y, y.y);
+				y.z = fmaf(cf[j].z, win[j].z, y.z); y.w = fmaf(cf[j].w, win[j].w, y.w);
 			}
-			win[MT - 1] = nv;
-			y = fmaf(cf[MT - 1], nv, y);
-			out[size_t(r) * ldo + c] = from_f32<OT>(nv + y);
+			if (c + 1 >= D) y.y = 0.0f;
+			if (c + 2 >= D) y.z = 0.0f;
+			if (c + 3 >= D) y.w = 0.0f;
+			store4<OT>(out + size_t(r) * ldo + c, y);
 			const int q = (r - row0) - (len - H);
-			if (q >= 0) hw[size_t(q) * D + c] = nv;
+			if (q >= 0) put(hw + size_t(q) * D, nv);
 		}
 	}
 }

@@ -456,6 +456,7 @@ struct HybridState : tg_state {
 	// activations of a pass
 	float *x = nullptr;
 	int ldx = 0;
+	float2 *stats = nullptr;          // mean and 1/deviation of the rows
 	void *h = nullptr, *P = nullptr, *O = nullptr, *act = nullptr;   // bf16, or fp32 in a 32-bit state
 	float *P32 = nullptr, *O32 = nullptr, *act32 = nullptr;          // the few-row pipeline's, always fp32
 	float *z = nullptr, *gz = nullptr, *o_raw = nullptr, *blk = nullptr, *bV = nullptr;
@@ -652,6 +653,7 @@ int HybridState::alloc() {
 		gmax = std::max(gmax, L.at.G);
 	}
 	TG_TRY(take(&x, size_t(R) * ldx));
+	TG_TRY(take(&stats, R));
 	TG_TRY(take_act(&h, size_t(R) * m->Dp));
 	TG_TRY(take_act(&P, size_t(R) * ldp));
 	TG_TRY(take_act(&O, size_t(R) * kc));
@@ -973,20 +975,17 @@ template <typename PT> int launch_delta(const DeltaArgs &a, int R, int nseg, int
 	count_launch();
 	return check_launch("delta_out");
 }
-template <typename PT> int launch_ln_conv(void *out, int ldo, const float *x, int ldx, const float *w, const float *cw, float *hist, const StepDesc &d, int R,
-                                          int D, int taps, float eps, cudaStream_t st) {
+template <typename PT> int launch_ln_conv(void *out, int ldo, const float *x, int ldx, float2 *stats, const float *w, const float *cw, float *hist,
+                                          const StepDesc &d, int R, int D, int taps, float eps, cudaStream_t st) {
+	launch_k(ln_stats_kernel, dim3(R), dim3(128), 0, st, stats, x, ldx, D, eps);
+	count_launch();
+	TG_TRY(check_launch("ln_stats"));
+	const int cols = (ldo + 511) / 512;
 	int rows = LC_ROWS;
-	while (rows > 1 && R < rows * 2 * g_num_sms) rows /= 2;
-	while (rows > 1 && ln_conv_smem(rows, taps, D) > 112 * 1024) rows /= 2;
-	const size_t smem = ln_conv_smem(rows, taps, D);
-	const dim3 grid((R + rows - 1) / rows);
-	if (taps <= 4) {
-		TG_TRY(allow_smem(ln_conv_kernel<PT, 4>, smem));
-		launch_k(ln_conv_kernel<PT, 4>, grid, dim3(256), smem, st, static_cast<PT *>(out), ldo, x, ldx, w, cw, hist, d, R, D, taps, eps, rows);
-	} else {
-		TG_TRY(allow_smem(ln_conv_kernel<PT, 16>, smem));
-		launch_k(ln_conv_kernel<PT, 16>, grid, dim3(256), smem, st, static_cast<PT *>(out), ldo, x, ldx, w, cw, hist, d, R, D, taps, eps, rows);
-	}
+	while (rows > 1 && (R + rows - 1) / rows * cols < 4 * g_num_sms) rows /= 2;
+	const dim3 grid((R + rows - 1) / rows, cols);
+	if (taps <= 4) launch_k(ln_conv_kernel<PT, 4>, grid, dim3(128), 0, st, static_cast<PT *>(out), ldo, x, ldx, stats, w, cw, hist, d, R, D, taps, rows);
+	else launch_k(ln_conv_kernel<PT, 16>, grid, dim3(128), 0, st, static_cast<PT *>(out), ldo, x, ldx, stats, w, cw, hist, d, R, D, taps, rows);
 	count_launch();
 	return check_launch("ln_conv");
 }
@@ -1076,8 +1075,8 @@ int HybridState::run_layers(const StepDesc &d, int R, int nseg, int max_len) {
 			}
 		} else {
 			if (m->runs[run].add_embed) TG_TRY(embed_rows(1));
-			if (f32) TG_TRY(launch_ln_conv<float>(h, m->Dp, x, ldx, L.norm1, L.canon, c.canon, d, R, D, m->taps, m->eps, stream));
-			else TG_TRY(launch_ln_conv<bf16>(h, m->Dp, x, ldx, L.norm1, L.canon, c.canon, d, R, D, m->taps, m->eps, stream));
+			if (f32) TG_TRY(launch_ln_conv<float>(h, m->Dp, x, ldx, stats, L.norm1, L.canon, c.canon, d, R, D, m->taps, m->eps, stream));
+			else TG_TRY(launch_ln_conv<bf16>(h, m->Dp, x, ldx, stats, L.norm1, L.canon, c.canon, d, R, D, m->taps, m->eps, stream));
 			TG_TRY(gemm(GEMM_STORE, h, m->Dp, &hmap, L.proj, R, P, L.ldp));
 			WAttnArgs wa = attn_args(d, int(run), P, L.ldp, O, L.kc);
 			const DeltaArgs da = delta_args(d, int(run), P, L.ldp, O, L.kc);
