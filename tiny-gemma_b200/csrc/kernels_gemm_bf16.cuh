@@ -6,8 +6,9 @@
 //                         accumulator back, so a tile's epilogue runs under the next tile's products.
 //   gemm_f32_kernel       A fp32: CUDA cores, fp32 FMA (the weights are exact in fp32).
 //
-// The epilogue is a parameter of both: store, add to the residual stream, gated GELU over interleaved
-// gate / up columns, soft-capped logits.
+// The epilogue is a parameter of both: store, add to the residual stream, gated activation over interleaved
+// gate / up columns, soft-capped logits. Trailing columns of a product (gates of a recurrence, router logits) may go to
+// an fp32 buffer of their own. Grouped products (GRP): every tile of 128 rows has weights of its own (an expert's).
 #pragma once
 #include "tc_common.cuh"
 
@@ -17,8 +18,15 @@ enum GemmEpi {
 	GEMM_STORE = 0,   // C = v                                   (C has the type of the activations)
 	GEMM_STORE32 = 1, // C = v, fp32
 	GEMM_ADD = 2,     // C += v, fp32 (the residual stream)
-	GEMM_GEGLU = 3,   // columns come as blocks of 16 gate, 16 up: C[16 columns] = gelu_tanh(gate) * up
+	GEMM_GLU = 3,     // columns come as blocks of 16 gate, 16 up: C[16 columns] = glu(gate, up)
 	GEMM_LOGITS = 4,  // C = cap * tanh(v / cap) (cap = 0: v), fp32; columns N .. ldc-1 are set to -inf
+};
+
+// Gated activations
+enum GluAct {
+	GLU_GELU = 0,   // gelu_tanh(g) u
+	GLU_SILU = 1,   // g sigmoid(g) u
+	GLU_CLAMP = 2,  // g' sigmoid(1.702 g') (u' + 1), g' = min(g, limit), u' = u within +- limit
 };
 
 struct GemmArgs {
@@ -28,11 +36,25 @@ struct GemmArgs {
 	float cap;
 	int m_tiles, n_tiles;
 	int *err;
+	int act;                 // GEMM_GLU
+	float limit;
+	int n32;                 // columns n32 .. N-1 (n32 a multiple of 8, of 32 for GEMM_GLU) are stored to C32 as fp32
+	float *C32;
+	int ld32;
+	const int *tile_expert;  // GRP: [row tiles] expert of a tile; its weights are rows expert * N ..
+	const int *n_row_tiles;  // GRP: row tiles of this step
 };
 
 __device__ __forceinline__ float gelu_tanh(float z) {
 	const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
 	return 0.5f * z * (1.0f + tanhf(u));
+}
+__device__ __forceinline__ float glu(int act, float limit, float g, float u) {
+	if (act == GLU_GELU) return gelu_tanh(g) * u;
+	if (act == GLU_SILU) return g / (1.0f + expf(-g)) * u;
+	g = fminf(g, limit);
+	u = fminf(fmaxf(u, -limit), limit);
+	return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
 }
 __device__ __forceinline__ float soft_cap(float v, float cap) { return cap > 0.0f ? cap * tanhf(v / cap) : v; }
 __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
@@ -73,7 +95,7 @@ __device__ __forceinline__ uint32_t tc_idesc_bf16(int n, int b_mn) {
 	return (1u << 4) | (1u << 7) | (1u << 10) | (uint32_t(b_mn) << 16) | (uint32_t(n >> 3) << 17) | (uint32_t(GB_BM >> 4) << 24);
 }
 
-template <int BN, int EPI>
+template <int BN, int EPI, bool GRP = false>
 __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap amap,
                                                                      const __grid_constant__ CUtensorMap wmap, GemmArgs a) {
 	using SH = GbShape<BN>;
@@ -86,7 +108,13 @@ __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 	__shared__ int s_fail, s_issued;
 	const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 	const int k_blocks = (a.K + GB_BK - 1) / GB_BK;
+	if (GRP) {
+		pdl_wait();
+		a.m_tiles = *a.n_row_tiles;
+	}
 	const int tiles = a.m_tiles * a.n_tiles;
+	// first weight row of a tile
+	auto w_row = [&](int t) { return (t / a.m_tiles) * BN + (GRP ? a.tile_expert[t % a.m_tiles] * a.N : 0); };
 	if (tid == 0) {
 		for (int s = 0; s < NS; s++) {
 			mbar_init(&full_bar[s], 1);
@@ -120,13 +148,13 @@ __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 				ahead = min(NS, k_blocks);
 				for (int s = 0; s < ahead; s++) {
 					mbar_expect_tx(&full_bar[s], SH::STAGE);
-					tma_load_2d(smem + s * SH::STAGE + SH::A_BYTES, &wmap, s * GB_BK, (first / a.m_tiles) * BN, &full_bar[s]);
+					tma_load_2d(smem + s * SH::STAGE + SH::A_BYTES, &wmap, s * GB_BK, w_row(first), &full_bar[s]);
 				}
 			}
 			pdl_wait();
 			int it = 0;
 			for (int t = first; t < tiles && !*(volatile int *)&s_fail; t += gridDim.x) {
-				const int m0 = (t % a.m_tiles) * GB_BM, n0 = (t / a.m_tiles) * BN;
+				const int m0 = (t % a.m_tiles) * GB_BM, n0 = w_row(t);
 				for (int kb = 0; kb < k_blocks; kb++, it++) {
 					const int s = it % NS, use = it / NS;
 					if (use > 0 && !tc_wait(&free_bar[s], (use - 1) & 1, a.err)) {
@@ -209,14 +237,15 @@ __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 				tc_ld32(taddr + uint32_t(c * 32), r);
 				asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 				const int col = n0 + c * 32;
-				if constexpr (EPI == GEMM_GEGLU) {
+				const bool tail = (EPI == GEMM_GLU || EPI == GEMM_STORE) && a.C32 && col >= a.n32;
+				if (EPI == GEMM_GLU && !tail) {
 					const int row = r0 + lane;
 					if (row < a.M) {
 						uint32_t o[8];
 #pragma unroll
 						for (int i = 0; i < 8; i++)
-							o[i] = pack_bf16(gelu_tanh(__uint_as_float(r[2 * i])) * __uint_as_float(r[16 + 2 * i]),
-							                 gelu_tanh(__uint_as_float(r[2 * i + 1])) * __uint_as_float(r[17 + 2 * i]));
+							o[i] = pack_bf16(glu(a.act, a.limit, __uint_as_float(r[2 * i]), __uint_as_float(r[16 + 2 * i])),
+							                 glu(a.act, a.limit, __uint_as_float(r[2 * i + 1]), __uint_as_float(r[17 + 2 * i])));
 						uint4 *dst = reinterpret_cast<uint4 *>(reinterpret_cast<__nv_bfloat16 *>(a.C) + size_t(row) * a.ldc + col / 2);
 						dst[0] = make_uint4(o[0], o[1], o[2], o[3]);
 						dst[1] = make_uint4(o[4], o[5], o[6], o[7]);
@@ -227,14 +256,19 @@ __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 					for (int i = 0; i < 8; i++)
 						*reinterpret_cast<uint4 *>(stg + lane * 36 + 4 * i) = make_uint4(r[4 * i], r[4 * i + 1], r[4 * i + 2], r[4 * i + 3]);
 					__syncwarp();
-					if (EPI == GEMM_STORE) {
+					if (EPI == GEMM_STORE || EPI == GEMM_GLU) {
 						const int cc = (lane & 3) * 8;
 #pragma unroll
 						for (int i = 0; i < 4; i++) {
 							const int rr = 8 * i + (lane >> 2);
 							if (r0 + rr < a.M && col + cc < a.N) {
 								const float4 u = *reinterpret_cast<const float4 *>(stg + rr * 36 + cc), v = *reinterpret_cast<const float4 *>(stg + rr * 36 + cc + 4);
-								*reinterpret_cast<uint4 *>(reinterpret_cast<__nv_bfloat16 *>(a.C) + size_t(r0 + rr) * a.ldc + col + cc) =
+								if (a.C32 && col + cc >= a.n32) {
+									float4 *dst = reinterpret_cast<float4 *>(a.C32 + size_t(r0 + rr) * a.ld32 + col + cc - a.n32);
+									dst[0] = u;
+									dst[1] = v;
+								} else
+									*reinterpret_cast<uint4 *>(reinterpret_cast<__nv_bfloat16 *>(a.C) + size_t(r0 + rr) * a.ldc + col + cc) =
 								    make_uint4(pack_bf16(u.x, u.y), pack_bf16(u.z, u.w), pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
 							}
 						}
@@ -286,12 +320,16 @@ __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 
 // ------------------------------------------------------------------ fp32 activations
 constexpr int GF_T = 64, GF_K = 16;
-template <int EPI>
+template <int EPI, bool GRP = false>
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const float *A, int lda, const __nv_bfloat16 *W, int ldw, GemmArgs a) {
 	pdl_trigger();
 	pdl_wait();
 	__shared__ float sa[GF_K][GF_T + 4], sw[GF_K][GF_T + 4];
 	const int tid = threadIdx.x, m0 = blockIdx.y * GF_T, n0 = blockIdx.x * GF_T;
+	if (GRP) {
+		if (m0 / GB_BM >= *a.n_row_tiles) return;
+		W += size_t(a.tile_expert[m0 / GB_BM]) * a.N * ldw;
+	}
 	const int tx = tid & 15, ty = tid >> 4;
 	float acc[4][4] = {};
 	for (int k0 = 0; k0 < a.K; k0 += GF_K) {
@@ -321,10 +359,17 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float *A, int lda, 
 	for (int i = 0; i < 4; i++) {
 		const int row = m0 + ty + 16 * i;
 		if (row >= a.M) continue;
-		if constexpr (EPI == GEMM_GEGLU) {  // columns n0 + tx + 16 j: j = 0, 2 gate, j = 1, 3 the up values beside them
+		if constexpr (EPI == GEMM_GLU) {  // columns n0 + tx + 16 j: j = 0, 2 gate, j = 1, 3 the up values beside them
 #pragma unroll
-			for (int j = 0; j < 4; j += 2)
-				if (n0 + 16 * j < a.N) C[size_t(row) * a.ldc + (n0 + 16 * j) / 2 + tx] = gelu_tanh(acc[i][j]) * acc[i][j + 1];
+			for (int j = 0; j < 4; j += 2) {
+				const int col = n0 + 16 * j + tx;
+				if (a.C32 && n0 + 16 * j >= a.n32) {
+					if (col < a.N) a.C32[size_t(row) * a.ld32 + col - a.n32] = acc[i][j];
+					if (col + 16 < a.N) a.C32[size_t(row) * a.ld32 + col + 16 - a.n32] = acc[i][j + 1];
+				} else if (n0 + 16 * j < a.N) {
+					C[size_t(row) * a.ldc + (n0 + 16 * j) / 2 + tx] = glu(a.act, a.limit, acc[i][j], acc[i][j + 1]);
+				}
+			}
 		} else {
 #pragma unroll
 			for (int j = 0; j < 4; j++) {
@@ -332,6 +377,8 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float *A, int lda, 
 				float *dst = C + size_t(row) * a.ldc + col;
 				if (EPI == GEMM_LOGITS) {
 					if (col < a.ldc) *dst = col < a.N ? soft_cap(acc[i][j], a.cap) : -INFINITY;
+				} else if (EPI == GEMM_STORE && a.C32 && col >= a.n32) {
+					if (col < a.N) a.C32[size_t(row) * a.ld32 + col - a.n32] = acc[i][j];
 				} else if (col < a.N) {
 					*dst = EPI == GEMM_ADD ? *dst + acc[i][j] : acc[i][j];
 				}

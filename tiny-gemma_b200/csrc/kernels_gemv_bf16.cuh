@@ -1,7 +1,10 @@
 // Matrix-vector products with bfloat16 weights [N][K] for a few rows (decoding): HBM bound. Activations stay fp32.
-// The norm (and input convolution) that precedes a product is its prologue, what follows it is its epilogue, so a
-// layer is five launches: [norm + conv -> projections -> cache], token mixing, [output projection + residual],
-// [norm -> gate|up -> gated GELU], [down + residual].
+// The norm (and input convolution) that precedes a product is its prologue, what follows it is its epilogue. A layer
+// whose feed-forward follows its mixer is five launches: [norm + conv -> projections -> cache], token mixing, [output
+// projection + residual], [norm -> gate|up -> gated activation], [down + residual]. A layer whose feed-forward stands
+// beside its mixer is three (GV_FRONT, token mixing, GV_MIX): [norm + shift -> projections, gate|up -> gated activation,
+// router], token mixing beside the chosen experts' gate|up (kernels_moe.cuh), [read-out norm and gate -> output
+// projection, down, the experts' down + residual].
 //
 // A CTA of 8 warps walks groups of output rows: a warp owns NR rows of the group (or, with KS > 1, the KS warps of a
 // row set share its K range), a lane 8 consecutive k of every 256. The next 16-byte weight words are requested before
@@ -12,8 +15,10 @@
 
 namespace tg {
 
-enum GemvPro { GV_VEC = 0, GV_LN = 1, GV_LN_CONV = 2 };
-enum GemvEpi { GV_PROJ = 0, GV_ADD = 1, GV_GEGLU = 2, GV_LOGITS = 3 };
+enum GemvPro { GV_VEC = 0, GV_LN = 1, GV_LN_CONV = 2, GV_MIX = 3 };
+enum GemvEpi { GV_PROJ = 0, GV_ADD = 1, GV_GLU = 2, GV_LOGITS = 3, GV_FRONT = 4 };
+// what GV_MIX does to a mixer's raw read-out
+enum MixNorm { MIX_NONE = 0, MIX_GATE_NORM = 1 /* norm(o silu(z)) w */, MIX_NORM_GATE = 2 /* norm(o) w sigmoid(z) */ };
 
 struct GemvArgs {
 	StepDesc d;
@@ -40,12 +45,35 @@ struct GemvArgs {
 	void *kc, *vc, *ks, *vs;
 	int cap_rows, keep, keep_rows, cache_f32;
 	int *err;
+	int rms;                   // the norm takes off no mean
+	float embed_scale;
+	int act;                   // gated activation
+	float limit;
+	// GV_FRONT: weight rows are [n_proj of the projections][2 n_glu gate | up][n_route router rows]; the projections read
+	// the convolved norm, the others the plain one. Projection columns from n32 on go to out32.
+	int n_proj, n32, n_glu, n_route;
+	float *out32;
+	int ld32;
+	float *glu_out, *route_out;
+	int ld_glu, ld_route;
+	// GV_MIX: columns 0 .. mix_n-1 of vec are a raw read-out, `parts` equal parts of it normed
+	int mix_norm, mix_n, parts;
+	const float *gate;         // [R][ldg]
+	int ldg;
+	// chosen experts: activations [R][top][n_ex], their weights and ids [R][top], down projections [experts][N][ld_ex]
+	const float *ex_act, *ex_w;
+	const int *ex_id;
+	int top, n_ex, ld_ex;
+	const __nv_bfloat16 *ex_W;
 };
 
 constexpr int GV_THREADS = 256;
 __host__ __device__ inline int gv_k8(int K) { return (K + 7) / 8; }
 template <int R, int NR> __host__ __device__ constexpr int gv_red_floats() { return 2 * 8 * NR * R; }
-template <int R, int NR> size_t gv_smem(int K, int pro) { return ((size_t(R) + pro) * 8 * gv_k8(K) + gv_red_floats<R, NR>() + 32) * 4; }
+template <int R, int NR> size_t gv_smem(int K, int pro, int epi, int parts, int ex) {
+	const size_t rows = epi == GV_FRONT ? 2 * R : R, extra = pro == GV_MIX ? 0 : pro;
+	return ((rows + extra) * 8 * gv_k8(K) + gv_red_floats<R, NR>() + 32 + (pro == GV_MIX ? size_t(R) * ((parts + 3) / 4 * 4 + ex) : 0)) * 4;
+}
 
 __device__ __forceinline__ float gv_block_sum(float v, float *red) {
 	v = warp_sum(v);
@@ -68,16 +96,31 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 	float *red = gv_sm + size_t(R) * 8 * K8;             // [2][row set][KS][NR][R]
 	float *bred = red + gv_red_floats<R, NR>();
 	float *wn = bred + 32, *hc = wn + 8 * K8;            // norm weight (x its factor in the convolution); history's share
+	float *xp = hc + 8 * K8;                             // GV_FRONT: the plain norms, laid out as xs
+	float *prt = bred + 32, *xe = prt + (PRO == GV_MIX ? R * ((a.parts + 3) / 4 * 4) : 0);  // GV_MIX: 1 / deviation of the parts; experts' activations
 	constexpr int SETS = 8 / KS, GROUP = SETS * NR;      // weight rows per CTA and group
 	const int set = warp / KS, ks = warp % KS;
-	const int n_out = EPI == GV_GEGLU ? a.N / 2 : (EPI == GV_LOGITS ? a.ldo : a.N);
-	constexpr int OUTS = EPI == GV_GEGLU ? GROUP / 2 : GROUP;  // outputs per group
-	const int groups = (n_out + OUTS - 1) / OUTS;
+	const int n_out = EPI == GV_GLU ? a.N / 2 : (EPI == GV_LOGITS ? a.ldo : a.N);
+	constexpr int OUTS = EPI == GV_GLU ? GROUP / 2 : GROUP;  // outputs per group
+	const int gp = EPI == GV_FRONT ? (a.n_proj + GROUP - 1) / GROUP : 0, gg = EPI == GV_FRONT ? gp + (a.n_glu + GROUP / 2 - 1) / (GROUP / 2) : 0;
+	const int groups = EPI == GV_FRONT ? gg + (a.n_route + GROUP - 1) / GROUP : (n_out + OUTS - 1) / OUTS;
 	const int nit = (K8 + 32 * KS - 1) / (32 * KS);
 
 	// weight row i (of NR) of this warp in a group
 	auto wrow = [&](int grp, int i) -> int {
-		if (EPI == GV_GEGLU) {
+		if (EPI == GV_FRONT) {
+			if (grp < gp) {
+				const int n = grp * GROUP + set * NR + i;
+				return n < a.n_proj ? n : a.N;
+			}
+			if (grp < gg) {
+				const int o = (grp - gp) * (GROUP / 2) + set * (NR / 2) + (i >> 1);
+				return o < a.n_glu ? a.n_proj + (o >> 4) * 32 + (o & 15) + (i & 1) * 16 : a.N;
+			}
+			const int n = (grp - gg) * GROUP + set * NR + i;
+			return n < a.n_route ? a.n_proj + 2 * a.n_glu + n : a.N;
+		}
+		if (EPI == GV_GLU) {
 			const int o = grp * OUTS + set * (NR / 2) + (i >> 1);
 			return (o >> 4) * 32 + (o & 15) + (i & 1) * 16;
 		}
@@ -97,7 +140,7 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 	};
 	uint4 cur[NR], nxt[NR];
 	load(blockIdx.x, 0, cur);
-	if (PRO != GV_VEC) {  // (weights too: nobody's output)
+	if (PRO == GV_LN || PRO == GV_LN_CONV) {  // (weights too: nobody's output)
 #pragma unroll 4
 		for (int k = tid; k < a.D; k += GV_THREADS) wn[k] = PRO == GV_LN_CONV ? fmaf(a.cw[size_t(a.taps - 1) * a.D + k], a.w[k], a.w[k]) : a.w[k];
 	}
@@ -110,6 +153,32 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 		float *xr = xs + size_t(r) * 8 * K8;
 		if (PRO == GV_VEC) {
 			for (int k = tid; k < 8 * K8; k += GV_THREADS) xr[xi(k)] = k < a.K ? a.vec[size_t(r) * a.ldv + k] : 0.0f;
+			continue;
+		}
+		if (PRO == GV_MIX) {
+			const float *gate = a.gate + size_t(r) * a.ldg;
+			for (int k = tid; k < 8 * K8; k += GV_THREADS) {
+				float v = k < a.K ? a.vec[size_t(r) * a.ldv + k] : 0.0f;
+				if (a.mix_norm == MIX_GATE_NORM && k < a.mix_n) v *= silu_f(gate[k]);
+				xr[xi(k)] = v;
+			}
+			for (int k = tid; k < a.top * a.n_ex; k += GV_THREADS)
+				xe[r * a.top * a.n_ex + k] = a.ex_act[size_t(r) * a.top * a.n_ex + k] * a.ex_w[r * a.top + k / a.n_ex];
+			if (a.mix_norm == MIX_NONE) continue;
+			__syncthreads();
+			const int width = a.mix_n / a.parts;
+			for (int p = warp; p < a.parts; p += 8) {
+				float q = 0.0f;
+				for (int k = p * width + lane; k < (p + 1) * width; k += 32) q = fmaf(xr[xi(k)], xr[xi(k)], q);
+				q = warp_sum(q);
+				if (lane == 0) prt[r * a.parts + p] = 1.0f / sqrtf(q / float(width) + a.eps);
+			}
+			__syncthreads();
+			for (int k = tid; k < a.mix_n; k += GV_THREADS) {
+				float v = xr[xi(k)] * prt[r * a.parts + k / width] * a.w[k];
+				if (a.mix_norm == MIX_NORM_GATE) v *= sigmoid_f(gate[k]);
+				xr[xi(k)] = v;
+			}
 			continue;
 		}
 		const int seg = a.d.row_seg[r];
@@ -135,7 +204,7 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 #pragma unroll 2
 		for (int k = tid; k < a.D; k += GV_THREADS) {
 			float v = a.embed_mode == 1 ? 0.0f : a.x[size_t(r) * a.ldx + k];
-			if (a.embed_mode) v += __bfloat162float(a.embed[size_t(tok) * a.lde + k]);
+			if (a.embed_mode) v += a.embed_scale * __bfloat162float(a.embed[size_t(tok) * a.lde + k]);
 			if (PRO == GV_LN_CONV) {
 				float c = 0.0f;
 #pragma unroll 3
@@ -149,7 +218,7 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 			xr[xi(k)] = v;
 			s += v;
 		}
-		const float mean = gv_block_sum(s, bred) / float(a.D);
+		const float mean = a.rms ? 0.0f : gv_block_sum(s, bred) / float(a.D);
 		float q = 0.0f;
 		for (int k = tid; k < a.D; k += GV_THREADS) {
 			const float c = xr[xi(k)] - mean;
@@ -158,14 +227,20 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 		const float rstd = 1.0f / sqrtf(gv_block_sum(q, bred) / float(a.D) + a.eps);
 		for (int k = tid; k < 8 * K8; k += GV_THREADS) {
 			float y = 0.0f;
+			if (EPI == GV_FRONT) xp[size_t(r) * 8 * K8 + xi(k)] = 0.0f;
 			if (k < a.D) {
 				const float n = (xr[xi(k)] - mean) * rstd;
 				y = n * wn[k];
+				if (EPI == GV_FRONT) {
+					const float plain = n * a.w[k];
+					xp[size_t(r) * 8 * K8 + xi(k)] = plain;
+					if (a.norm_out && blockIdx.x == 0) a.norm_out[size_t(r) * a.D + k] = plain;
+				}
 				if (PRO == GV_LN_CONV) {
 					y += hc[k];
 					if (blockIdx.x == 0 && H > 0) hw[size_t(H - 1) * a.D + k] = n * a.w[k];
 				}
-				if (a.norm_out && blockIdx.x == 0) a.norm_out[size_t(r) * a.D + k] = y;
+				if (EPI != GV_FRONT && a.norm_out && blockIdx.x == 0) a.norm_out[size_t(r) * a.D + k] = y;
 			}
 			xr[xi(k)] = y;
 		}
@@ -176,6 +251,7 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 	int flip = 0;
 	for (int grp = blockIdx.x; grp < groups; grp += gridDim.x, flip ^= 1) {
 		float acc[R][NR] = {};
+		const float *xg = EPI == GV_FRONT && grp >= gp ? xp : xs;
 		for (int it = 0; it < nit; it++) {
 			if (it + 1 < nit) load(grp, it + 1, nxt);
 			else load(grp + gridDim.x, 0, nxt);
@@ -183,8 +259,8 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 			if (k8 < K8) {
 #pragma unroll
 				for (int r = 0; r < R; r++) {
-					const float4 x0 = *reinterpret_cast<const float4 *>(xs + size_t(r) * 8 * K8 + 4 * k8);
-					const float4 x1 = *reinterpret_cast<const float4 *>(xs + size_t(r) * 8 * K8 + 4 * K8 + 4 * k8);
+					const float4 x0 = *reinterpret_cast<const float4 *>(xg + size_t(r) * 8 * K8 + 4 * k8);
+					const float4 x1 = *reinterpret_cast<const float4 *>(xg + size_t(r) * 8 * K8 + 4 * K8 + 4 * k8);
 #pragma unroll
 					for (int i = 0; i < NR; i++) {
 						float s = acc[r][i];
@@ -201,6 +277,32 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 			}
 #pragma unroll
 			for (int i = 0; i < NR; i++) cur[i] = nxt[i];
+		}
+		if (PRO == GV_MIX && a.top) {  // each row's own experts: 16 bytes of (expert, k) per lane
+			const int e8 = a.n_ex / 8, n0 = grp * GROUP + set * NR;
+#pragma unroll
+			for (int r = 0; r < R; r++) {
+				const float *xv = xe + r * a.top * a.n_ex;
+#pragma unroll 2
+				for (int j = ks * 32 + lane; j < a.top * e8; j += 32 * KS) {
+					const __nv_bfloat16 *w = a.ex_W + size_t(a.ex_id[r * a.top + j / e8]) * a.N * a.ld_ex + 8 * (j % e8);
+					const float4 x0 = *reinterpret_cast<const float4 *>(xv + 8 * j), x1 = *reinterpret_cast<const float4 *>(xv + 8 * j + 4);
+#pragma unroll
+					for (int i = 0; i < NR; i++) {
+						if (n0 + i >= a.N) break;
+						const int4 v = ld_stream_int4(w + size_t(n0 + i) * a.ld_ex);
+						float s = acc[r][i];
+						s = fmaf(bf16_lo(v.x), x0.x, s);
+						s = fmaf(bf16_hi(v.x), x0.y, s);
+						s = fmaf(bf16_lo(v.y), x0.z, s);
+						s = fmaf(bf16_hi(v.y), x0.w, s);
+						s = fmaf(bf16_lo(v.z), x1.x, s);
+						s = fmaf(bf16_hi(v.z), x1.y, s);
+						s = fmaf(bf16_lo(v.w), x1.z, s);
+						acc[r][i] = fmaf(bf16_hi(v.w), x1.w, s);
+					}
+				}
+			}
 		}
 		float *rb = red + flip * 8 * NR * R;
 #pragma unroll
@@ -220,16 +322,28 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 				for (int q = 0; q < KS; q++) v += rb[((st * KS + q) * NR + i) * R + r];
 				return v;
 			};
-			if (n < n_out) {
+			if (EPI == GV_FRONT) {
+				if (grp < gp) {
+					const float v = sum(o / NR, o % NR);
+					if (n < a.n32) a.out[size_t(r) * a.ldo + n] = v;
+					else if (n < a.n_proj) a.out32[size_t(r) * a.ld32 + n - a.n32] = v;
+				} else if (grp < gg) {
+					const int st = o / (NR / 2), i = (o % (NR / 2)) * 2, c = (grp - gp) * (GROUP / 2) + o;
+					if (o < GROUP / 2 && c < a.n_glu) a.glu_out[size_t(r) * a.ld_glu + c] = glu(a.act, a.limit, sum(st, i), sum(st, i + 1));
+				} else {
+					const int c = (grp - gg) * GROUP + o;
+					if (c < a.n_route) a.route_out[size_t(r) * a.ld_route + c] = sum(o / NR, o % NR);
+				}
+			} else if (n < n_out) {
 				float *dst = a.out + size_t(r) * a.ldo + n;
-				if (EPI == GV_GEGLU) {
+				if (EPI == GV_GLU) {
 					const int st = o / (NR / 2), i = (o % (NR / 2)) * 2;
-					*dst = gelu_tanh(sum(st, i)) * sum(st, i + 1);
+					*dst = glu(a.act, a.limit, sum(st, i), sum(st, i + 1));
 				} else {
 					const float v = sum(o / NR, o % NR);
 					if (EPI == GV_ADD) {
 						float b = a.embed_mode == 1 ? 0.0f : *dst;
-						if (a.embed_mode) b += __bfloat162float(a.embed[size_t(min(max(a.d.tok[r], 0), a.V - 1)) * a.lde + n]);
+						if (a.embed_mode) b += a.embed_scale * __bfloat162float(a.embed[size_t(min(max(a.d.tok[r], 0), a.V - 1)) * a.lde + n]);
 						*dst = b + v;
 					} else if (EPI == GV_LOGITS) {
 						*dst = n < a.N ? soft_cap(v, a.cap) : -INFINITY;

@@ -1,4 +1,5 @@
-// Row-wise kernels over the tokens of one step: embedding, layer norm, layer norm with the input convolution.
+// Row-wise kernels over the tokens of one step: embedding, layer / RMS norm, norm with the input convolution (of which
+// the token shift h + (h' - h) s is the two-tap case), rotation tables.
 #pragma once
 #include <cuda_bf16.h>
 
@@ -31,8 +32,8 @@ __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 
-// x[r] = embed[tok[r]], or x[r] += embed[tok[r]] (another pass through a looped block)
-static __global__ void __launch_bounds__(256) embed_rows_kernel(float *x, int ldx, const __nv_bfloat16 *embed, int lde, StepDesc d, int D, int V,
+// x[r] = scale embed[tok[r]], or x[r] += that (another pass through a looped block)
+static __global__ void __launch_bounds__(256) embed_rows_kernel(float *x, int ldx, const __nv_bfloat16 *embed, int lde, float scale, StepDesc d, int D, int V,
                                                                 int add, int *err) {
 	pdl_trigger();
 	pdl_wait();
@@ -43,7 +44,7 @@ static __global__ void __launch_bounds__(256) embed_rows_kernel(float *x, int ld
 		tok = 0;
 	}
 	for (int i = threadIdx.x; i < D; i += 256) {
-		const float e = __bfloat162float(embed[size_t(tok) * lde + i]);
+		const float e = scale * __bfloat162float(embed[size_t(tok) * lde + i]);
 		float *p = x + size_t(r) * ldx + i;
 		*p = add ? *p + e : e;
 	}
@@ -67,11 +68,11 @@ template <> __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16 
 	*reinterpret_cast<uint2 *>(p) = *reinterpret_cast<const uint2 *>(q);
 }
 
-// out[i] = layer_norm(x[row(i)]) for i < n; row(i) = rows ? rows[i] : i. Columns D .. ldo-1 become 0 (operand padding).
+// out[i] = norm(x[row(i)]) for i < n; row(i) = rows ? rows[i] : i; rms: no mean is taken off. Columns D .. ldo-1 become 0 (operand padding).
 // One CTA of 128 threads per row, the row in registers while it fits (D <= 4096, D % 4 == 0; ldx, ldo multiples of 4).
 template <typename OT>
-__global__ void __launch_bounds__(128) layer_norm_kernel(OT *out, int ldo, const float *x, int ldx, const float *w, const int *rows, int n, int D, float eps,
-                                                         float *out32) {
+__global__ void __launch_bounds__(128) row_norm_kernel(OT *out, int ldo, const float *x, int ldx, const float *w, const int *rows, int n, int D, float eps,
+                                                       int rms, float *out32) {
 	pdl_trigger();
 	pdl_wait();
 	__shared__ float red[4];
@@ -87,7 +88,7 @@ __global__ void __launch_bounds__(128) layer_norm_kernel(OT *out, int ldo, const
 			v[j] = c < D ? *reinterpret_cast<const float4 *>(xr + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 			s += (v[j].x + v[j].y) + (v[j].z + v[j].w);
 		}
-		const float mean = cta_sum<4>(s, red) / float(D);
+		const float mean = rms ? 0.0f : cta_sum<4>(s, red) / float(D);
 		float q = 0.0f;
 #pragma unroll
 		for (int j = 0; j < 8; j++)
@@ -112,7 +113,7 @@ __global__ void __launch_bounds__(128) layer_norm_kernel(OT *out, int ldo, const
 	}
 	float s = 0.0f, q = 0.0f;
 	for (int c = tid; c < D; c += 128) s += xr[c];
-	const float mean = cta_sum<4>(s, red) / float(D);
+	const float mean = rms ? 0.0f : cta_sum<4>(s, red) / float(D);
 	for (int c = tid; c < D; c += 128) q = fmaf(xr[c] - mean, xr[c] - mean, q);
 	const float f = 1.0f / sqrtf(cta_sum<4>(q, red) / float(D) + eps);
 	for (int c = tid; c < ldo; c += 128) {
@@ -122,18 +123,38 @@ __global__ void __launch_bounds__(128) layer_norm_kernel(OT *out, int ldo, const
 	}
 }
 
-// h = n + conv(n), n = layer_norm(x): the causal convolution over time on each channel (taps at cw[j][D], the last one
+// h = n + conv(n), n = norm(x): the causal convolution over time on each channel (taps at cw[j][D], the last one
 // meets the current row). The taps - 1 normed rows before a segment come from hist[seq][par], and the segment's
 // last ones (or, in a shorter segment, the older ones that still matter) are left in hist[seq][par ^ 1], oldest
 // first. hist: [B][2][taps-1][D]. Rows before a sequence's start count as zero, whatever hist holds.
-// Two kernels: mean and 1/sqrt(var + eps) of every row, then a walk down the rows with the window in registers, four
+// Two kernels: mean (0 for an RMS norm) and 1/deviation of every row, then a walk down the rows with the window in registers, four
 // channels per thread, LC_ROWS rows per CTA (the rows before them are normed again, not exchanged).
-static __global__ void __launch_bounds__(128) ln_stats_kernel(float2 *stats, const float *x, int ldx, int D, float eps) {
+// The statistics kernel may first add what the chosen experts of the preceding layer put out (`add`): the row is read
+// here anyway.
+template <typename YT> struct ExpertSum {
+	const YT *y;        // [slots][ldy] outputs of the experts, or null
+	int ldy, top;
+	const int *slot;    // [R][top]
+	const float *w;     // [R][top]
+	int *zero;          // counters that the next layer's routing finds at zero, or null
+	int n_zero;
+};
+__device__ __forceinline__ float4 load4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16 *p) {
+	const uint2 u = *reinterpret_cast<const uint2 *>(p);
+	return make_float4(bf16_lo(u.x), bf16_hi(u.x), bf16_lo(u.y), bf16_hi(u.y));
+}
+template <typename YT>
+__global__ void __launch_bounds__(128) row_stats_kernel(float2 *stats, float *x, int ldx, int D, float eps, int rms, ExpertSum<YT> add) {
 	pdl_trigger();
 	pdl_wait();
 	__shared__ float red[4];
 	const int tid = threadIdx.x;
-	const float *xr = x + size_t(blockIdx.x) * ldx;
+	float *xr = x + size_t(blockIdx.x) * ldx;
+	const int *slot = add.slot + size_t(blockIdx.x) * add.top;
+	const float *wt = add.w + size_t(blockIdx.x) * add.top;
+	if (add.zero && blockIdx.x == 0)
+		for (int i = tid; i < add.n_zero; i += 128) add.zero[i] = 0;
 	float mean, q = 0.0f, s = 0.0f;
 	if (D <= 4096 && D % 4 == 0) {
 		float4 v[8];
@@ -141,9 +162,27 @@ static __global__ void __launch_bounds__(128) ln_stats_kernel(float2 *stats, con
 		for (int j = 0; j < 8; j++) {
 			const int c = 4 * (tid + 128 * j);
 			v[j] = c < D ? *reinterpret_cast<const float4 *>(xr + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-			s += (v[j].x + v[j].y) + (v[j].z + v[j].w);
 		}
-		mean = cta_sum<4>(s, red) / float(D);
+		if (add.y) {
+			for (int e = 0; e < add.top; e++) {
+				const YT *y = add.y + size_t(slot[e]) * add.ldy;
+				const float w = wt[e];
+#pragma unroll
+				for (int j = 0; j < 8; j++) {
+					const int c = 4 * (tid + 128 * j);
+					if (c < D) {
+						const float4 u = load4(y + c);
+						v[j].x = fmaf(w, u.x, v[j].x); v[j].y = fmaf(w, u.y, v[j].y); v[j].z = fmaf(w, u.z, v[j].z); v[j].w = fmaf(w, u.w, v[j].w);
+					}
+				}
+			}
+#pragma unroll
+			for (int j = 0; j < 8; j++)
+				if (4 * (tid + 128 * j) < D) *reinterpret_cast<float4 *>(xr + 4 * (tid + 128 * j)) = v[j];
+		}
+#pragma unroll
+		for (int j = 0; j < 8; j++) s += (v[j].x + v[j].y) + (v[j].z + v[j].w);
+		mean = rms ? 0.0f : cta_sum<4>(s, red) / float(D);
 #pragma unroll
 		for (int j = 0; j < 8; j++)
 			if (4 * (tid + 128 * j) < D) {
@@ -151,18 +190,26 @@ static __global__ void __launch_bounds__(128) ln_stats_kernel(float2 *stats, con
 				q = fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, fmaf(v[j].z, v[j].z, fmaf(v[j].w, v[j].w, q))));
 			}
 	} else {
-		for (int c = tid; c < D; c += 128) s += xr[c];
-		mean = cta_sum<4>(s, red) / float(D);
+		for (int c = tid; c < D; c += 128) {
+			float v = xr[c];
+			if (add.y) {
+				for (int e = 0; e < add.top; e++) v = fmaf(wt[e], to_f32(add.y[size_t(slot[e]) * add.ldy + c]), v);
+				xr[c] = v;
+			}
+			s += v;
+		}
+		mean = rms ? 0.0f : cta_sum<4>(s, red) / float(D);
 		for (int c = tid; c < D; c += 128) q = fmaf(xr[c] - mean, xr[c] - mean, q);
 	}
 	q = cta_sum<4>(q, red);
 	if (tid == 0) stats[blockIdx.x] = make_float2(mean, 1.0f / sqrtf(q / float(D) + eps));
 }
 
-// grid (ceil(R / rows), ceil(ldo / 512)); rows <= LC_ROWS; ldx and ldo multiples of 4
+// grid (ceil(R / rows), ceil(ldo / 512)); rows <= LC_ROWS; ldx and ldo multiples of 4. `plain`, if not null, gets n itself
+// (for what reads the norm without the convolution), rows of ldo too.
 constexpr int LC_ROWS = 16;
 template <typename OT, int MT>
-__global__ void __launch_bounds__(128) ln_conv_kernel(OT *out, int ldo, const float *x, int ldx, const float2 *stats, const float *w, const float *cw,
+__global__ void __launch_bounds__(128) norm_conv_kernel(OT *out, OT *plain, int ldo, const float *x, int ldx, const float2 *stats, const float *w, const float *cw,
                                                       float *hist, StepDesc d, int R, int D, int taps, int rows) {
 	pdl_trigger();
 	pdl_wait();
@@ -175,7 +222,10 @@ __global__ void __launch_bounds__(128) ln_conv_kernel(OT *out, int ldo, const fl
 	const int c = 4 * (blockIdx.y * 128 + tid);
 	if (c >= ldo) return;
 	if (c >= D) {
-		for (int i = 0; i < nr; i++) store4<OT>(out + size_t(r0 + i) * ldo + c, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
+		for (int i = 0; i < nr; i++) {
+			store4<OT>(out + size_t(r0 + i) * ldo + c, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
+			if (plain) store4<OT>(plain + size_t(r0 + i) * ldo + c, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
+		}
 		return;
 	}
 	auto get = [&](const float *p) {  // four consecutive channels of an unpadded row
@@ -242,9 +292,34 @@ __global__ void __launch_bounds__(128) ln_conv_kernel(OT *out, int ldo, const fl
 			if (c + 2 >= D) y.z = 0.0f;
 			if (c + 3 >= D) y.w = 0.0f;
 			store4<OT>(out + size_t(r) * ldo + c, y);
+			if (plain) store4<OT>(plain + size_t(r) * ldo + c, make_float4(nv.x, c + 1 < D ? nv.y : 0.0f, c + 2 < D ? nv.z : 0.0f, c + 3 < D ? nv.w : 0.0f));
 			const int q = (r - row0) - (len - H);
 			if (q >= 0) put(hw + size_t(q) * D, nv);
 		}
+	}
+}
+
+// ------------------------------------------------------------------ rotation
+// cs[rot][row][i] = (cos, sin) of position x frequency i, times the rotation's factor. The angle is formed and reduced
+// in double, so it is exact to fp32 rounding at any position. grid (R, rotations)
+struct RopeTable {
+	const double *freq;   // [rotations][half]
+	const float *factor;  // [rotations]
+	float2 *cs;           // [rotations][rows][half]
+	int rows, half;
+};
+static __global__ void __launch_bounds__(128) rope_table_kernel(RopeTable t, StepDesc d) {
+	pdl_trigger();
+	pdl_wait();
+	const int r = blockIdx.x, rot = blockIdx.y, seg = d.row_seg[r];
+	const double p = double(d.seg_pos[seg] + r - d.seg_row[seg]);
+	const float m = t.factor[rot];
+	for (int i = threadIdx.x; i < t.half; i += 128) {
+		double a = p * t.freq[size_t(rot) * t.half + i];
+		a -= 6.283185307179586 * rint(a * 0.15915494309189535);
+		float s, c;
+		sincosf(float(a), &s, &c);
+		t.cs[(size_t(rot) * t.rows + r) * t.half + i] = make_float2(c * m, s * m);
 	}
 }
 

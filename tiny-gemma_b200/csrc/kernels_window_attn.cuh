@@ -1,14 +1,18 @@
 // Causal attention over a sliding window plus the first tokens of a sequence, with an optional per-head distance
 // bias taken off the scores:
 //     score(i, j) = scale * q_i . k_j - r1 ln(1 + r2 (i - j)),     j <= i and (i - j < window or j < keep_first)
-// No rotation; grouped key/value heads; an optional sigmoid output gate.
+// or, instead of the first tokens, pooled blocks: for each block of `pool` tokens that lies wholly before the window one
+// row, the mean of the block's cached keys and of its values. Grouped key/value heads; an optional sigmoid output gate;
+// optional rotation of q and k and norm of v, applied between the projections and the cache.
 //
 // Cache of one layer run, per sequence: a ring of `cap` rows (slot = position mod cap; cap is a multiple of 64 and at
-// least window + rows of a step) and, because the ring forgets them, a copy of the first keep_first rows. A query
-// takes keys within its window from the ring and the others from the copy, so no key is met twice.
+// least window + rows of a step) and, because the ring forgets them, a second store: a copy of the first keep_first rows,
+// or the pooled rows (block b at row b, written when its last token arrives). A query takes keys within its window from
+// the ring and the others from the second store, so no key is met twice.
 // Rows hold G heads one after the other, each padded to a multiple of 16 elements (dkp, dvp) with zeros.
 //
 //   kv_append_kernel        rows of a step -> cache
+//   kv_transform_kernel     the same with rotation, value norm and pooling
 //   window_attn_kernel      portions, CUDA cores: any sizes, fp32 or bf16
 //   window_attn_tc_kernel   portions, bf16 on tcgen05 (dkp, dvp <= 256): 128 queries of one head per CTA
 //   window_attn_token_cta   one token per sequence: a CTA per (sequence, key/value head, run of keys)
@@ -23,12 +27,19 @@ struct WAttnArgs {
 	int H, G, dk, dv, dkp, dvp;
 	float scale;
 	int window, keep;      // keep: first tokens that stay visible
+	int pool;              // tokens of a pooled block (0: none; then keep = 0)
+	int rot;               // rotated dimensions of q and k, pair (c, c + rot/2) (0: none)
+	const float2 *cs;      // [R][ld_cs] cos and sin of the rows' positions
+	int ld_cs;
+	int vnorm;             // values are divided by their root mean square
+	float eps;
+	int append;            // one token per sequence: the token's key and value still have to be put into the cache
 	const float *r1, *r2;  // [H] or null
 	const void *p;         // projections, rows of ldp: q at p_q, k at p_k, v at p_v, gate at p_g (-1: none)
 	int ldp, p_q, p_k, p_v, p_g;
 	void *kc, *vc;         // [B][cap][G*dkp], [B][cap][G*dvp]
-	void *ks, *vs;         // [B][keep_rows][G*dkp], ...: the first tokens
-	int cap, keep_rows;    // keep_rows: keep rounded up to a multiple of 64 (0 if keep = 0)
+	void *ks, *vs;         // [B][keep_rows][G*dkp], ...: the first tokens, or the pooled blocks
+	int cap, keep_rows;    // keep_rows: rows of the second store, a multiple of 64
 	void *out;             // [R] rows of ldo, head h at h*dvp
 	int ldo;
 	float out_scale;
@@ -56,9 +67,75 @@ static __global__ void __launch_bounds__(256) kv_append_kernel(WAttnArgs a) {
 	}
 }
 
+// element c of a rotated head
+template <typename PT> __device__ __forceinline__ float wa_rotated(const WAttnArgs &a, const PT *head, const float2 *cs, int c) {
+	const float u = to_f32(head[c]);
+	const int half = a.rot >> 1;
+	if (c >= a.rot) return u;
+	if (c < half) return u * cs[c].x - to_f32(head[c + half]) * cs[c].y;
+	return u * cs[c - half].x + to_f32(head[c - half]) * cs[c - half].y;
+}
+// the mean of block b of the ring -> row b of the second store; NT threads, this one is number t
+template <typename CT, int NT> __device__ __forceinline__ void wa_pool_block(const WAttnArgs &a, int seq, int g, int b, int t) {
+	const int nk = a.G * a.dkp, nv = a.G * a.dvp;
+	for (int c = t; c < a.dkp + a.dvp; c += NT) {
+		const bool isk = c < a.dkp;
+		const int n = isk ? nk : nv, col = isk ? g * a.dkp + c : g * a.dvp + c - a.dkp;
+		const CT *ring = reinterpret_cast<const CT *>(isk ? a.kc : a.vc) + size_t(seq) * a.cap * n + col;
+		float s = 0.0f;
+#pragma unroll 4
+		for (int j = 0; j < a.pool; j++) s += to_f32(ring[size_t((b * a.pool + j) % a.cap) * n]);
+		reinterpret_cast<CT *>(isk ? a.ks : a.vs)[(size_t(seq) * a.keep_rows + b) * n + col] = from_f32<CT>(s / float(a.pool));
+	}
+}
+// Portions: rotates q in place, puts rotated keys and normed values into the ring, and pools the blocks that the step
+// completes. A CTA owns `unit` positions (a multiple of `pool`, counted from the sequence's start) of a key/value head, so
+// that what a block needs is either its own or an earlier step's. grid (units of the longest segment + 1, G, segments)
+template <typename PT, typename CT>
+static __global__ void __launch_bounds__(256) kv_transform_kernel(WAttnArgs a, int unit) {
+	pdl_trigger();
+	pdl_wait();
+	const int seg = blockIdx.z, g = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+	const int pos = a.d.seg_pos[seg], len = a.d.seg_len[seg], row0 = a.d.seg_row[seg], seq = a.d.seg_seq[seg];
+	const int u0 = (pos / unit + int(blockIdx.x)) * unit;
+	if (u0 >= pos + len) return;
+	const int lo = max(pos, u0), hi = min(pos + len, u0 + unit), per = a.H / a.G, half = a.rot >> 1;
+	const int nk = a.G * a.dkp, nv = a.G * a.dvp;
+	for (int i = lo + warp; i < hi; i += 8) {
+		const int r = row0 + i - pos;
+		PT *row = const_cast<PT *>(reinterpret_cast<const PT *>(a.p)) + size_t(r) * a.ldp;
+		const float2 *cs = a.cs + size_t(r) * a.ld_cs;
+		for (int x = lane; x < per * half; x += 32) {
+			const int c = x % half;
+			PT *q = row + a.p_q + (g * per + x / half) * a.dkp + c;
+			const float u = to_f32(q[0]), v = to_f32(q[half]);
+			q[0] = from_f32<PT>(u * cs[c].x - v * cs[c].y);
+			q[half] = from_f32<PT>(v * cs[c].x + u * cs[c].y);
+		}
+		const size_t slot = size_t(seq) * a.cap + i % a.cap;
+		CT *kd = reinterpret_cast<CT *>(a.kc) + slot * nk + g * a.dkp, *vd = reinterpret_cast<CT *>(a.vc) + slot * nv + g * a.dvp;
+		const PT *ks = row + a.p_k + g * a.dkp, *vs = row + a.p_v + g * a.dvp;
+		for (int c = lane; c < a.dkp; c += 32) kd[c] = from_f32<CT>(wa_rotated(a, ks, cs, c));
+		float f = 1.0f;
+		if (a.vnorm) {
+			float s = 0.0f;
+			for (int c = lane; c < a.dv; c += 32) s = fmaf(to_f32(vs[c]), to_f32(vs[c]), s);
+			f = 1.0f / sqrtf(warp_sum(s) / float(a.dv) + a.eps);
+		}
+		for (int c = lane; c < a.dvp; c += 32) vd[c] = from_f32<CT>(to_f32(vs[c]) * f);
+	}
+	if (!a.pool) return;
+	__syncthreads();
+	for (int b = u0 / a.pool; (b + 1) * a.pool <= hi; b++)
+		if ((b + 1) * a.pool > pos) wa_pool_block<CT, 256>(a, seq, g, b, tid);
+}
+
 // number of keys a query at position i sees, and key number n -> position
 __device__ __forceinline__ int wa_first(const WAttnArgs &a, int i) { return max(0, i - a.window + 1); }      // first window position
-__device__ __forceinline__ int wa_kept(const WAttnArgs &a, int i) { return min(a.keep, wa_first(a, i)); }    // kept tokens outside the window
+// rows of the second store that it sees: kept tokens outside the window, or blocks whose last token has left it
+__device__ __forceinline__ int wa_kept(const WAttnArgs &a, int i) {
+	return a.pool ? max(0, (i - a.window + 1) / a.pool) : min(a.keep, wa_first(a, i));
+}
 __device__ __forceinline__ float wa_bias(float r1, float r2, int dist) { return r1 * log1pf(r2 * float(dist)); }
 
 // ------------------------------------------------------------------ portions, CUDA cores
@@ -148,14 +225,14 @@ struct WtShape {
 	int q_bytes, k_bytes, v_bytes, stage, ns, table, total;  // table: entries of the bias table (0: none)
 };
 __host__ __device__ inline int wt_chunks(int d) { return (d + 63) / 64; }
-__host__ __device__ inline WtShape wt_shape(int dkp, int dvp, int window) {
+__host__ __device__ inline WtShape wt_shape(int dkp, int dvp, int window, bool bias) {
 	WtShape s;
 	s.q_bytes = wt_chunks(dkp) * 128 * 128;
 	s.k_bytes = wt_chunks(dkp) * WT_KEYS * 128;
 	s.v_bytes = wt_chunks(dvp) * WT_KEYS * 128;
 	s.stage = s.k_bytes > s.v_bytes ? s.k_bytes : s.v_bytes;
 	s.ns = 4;  // two CTAs per SM where four stages allow it; fewer stages only where one CTA's shared memory ends
-	s.table = window + 256 <= WT_TABLE ? window + 256 : 0;
+	s.table = bias && window + 256 <= WT_TABLE ? window + 256 : 0;
 	while (s.ns > 2 && s.q_bytes + s.ns * s.stage + 4 * s.table + 1024 > 220 * 1024) s.ns--;
 	s.total = s.q_bytes + s.ns * s.stage + 4 * s.table + 1024;
 	return s;
@@ -173,7 +250,7 @@ static __global__ void __launch_bounds__(WT_THREADS, 2) window_attn_tc_kernel(co
 	__shared__ int s_fail, s_issued;
 	__shared__ float s_max[2][2][128];  // [tile parity][half of the row][row]
 	const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-	const WtShape sh = wt_shape(a.dkp, a.dvp, a.window);
+	const WtShape sh = wt_shape(a.dkp, a.dvp, a.window, a.r1 != nullptr);
 	const int ncols = wt_tmem_cols(a.dvp);
 	if (tid == 0) {
 		mbar_init(&q_bar, 1);
@@ -436,7 +513,8 @@ static __global__ void __launch_bounds__(WT_THREADS, 2) window_attn_tc_kernel(co
 }
 
 // ------------------------------------------------------------------ one token per sequence
-// 256 threads; row r of the step is a segment of length 1 whose key and value are already in the cache. The CTA scores
+// 256 threads; row r of the step is a segment of length 1 whose key and value are already in the cache (or are put there
+// first, rotated, normed and pooled, by the CTA whose run ends with them: `append`). The CTA scores
 // its run of keys for up to WK_HEADS query heads of key/value head g at a time, in pieces of WK_KEYS; the CTA that
 // arrives last merges the runs, applies the gate and writes the heads' rows.
 constexpr int WK_KEYS = 64, WK_HEADS = 4;
@@ -466,7 +544,27 @@ __device__ void window_attn_token_cta(const WAttnArgs &a, int r, int g, int spli
 	const int first = wa_first(a, i), kept = wa_kept(a, i), total = kept + i - first + 1;
 	const int pieces = (total + WK_KEYS - 1) / WK_KEYS, share = (pieces + a.nsplit - 1) / a.nsplit;
 	const int n_lo = split * share * WK_KEYS, n_hi = min(total, (split + 1) * share * WK_KEYS);
-	for (int x = tid; x < per * dkp; x += 256) q[x] = to_f32(row[a.p_q + g * per * dkp + x]) * a.scale;
+	if (a.rot) {
+		const float2 *cs = a.cs + size_t(r) * a.ld_cs;
+		for (int x = tid; x < per * dkp; x += 256) q[x] = wa_rotated(a, row + a.p_q + (g * per + x / dkp) * dkp, cs, x % dkp) * a.scale;
+	} else {
+		for (int x = tid; x < per * dkp; x += 256) q[x] = to_f32(row[a.p_q + g * per * dkp + x]) * a.scale;
+	}
+	if (a.append && n_lo < total && n_hi == total) {  // (the whole CTA)
+		const float2 *cs = a.cs + size_t(r) * a.ld_cs;
+		CT *kd = const_cast<CT *>(kc) + size_t(i % a.cap) * a.G * dkp, *vd = const_cast<CT *>(vc) + size_t(i % a.cap) * a.G * dvp;
+		const PT *kp = row + a.p_k + g * dkp, *vp = row + a.p_v + g * dvp;
+		float f = 1.0f;
+		if (a.vnorm) {  // (every warp for itself)
+			float s = 0.0f;
+			for (int c = lane; c < a.dv; c += 32) s = fmaf(to_f32(vp[c]), to_f32(vp[c]), s);
+			f = 1.0f / sqrtf(warp_sum(s) / float(a.dv) + a.eps);
+		}
+		for (int c = tid; c < dkp; c += 256) kd[c] = from_f32<CT>(wa_rotated(a, kp, cs, c));
+		for (int c = tid; c < dvp; c += 256) vd[c] = from_f32<CT>(to_f32(vp[c]) * f);
+		__syncthreads();
+		if (a.pool && (i + 1) % a.pool == 0) wa_pool_block<CT, 256>(a, seq, g, i / a.pool, tid);
+	}
 	float *part = a.part + ((size_t(r) * a.G + g) * a.nsplit + split) * per * (dvp + 2);
 	// lanes of a value row (a power of two), value rows a warp reads at once
 	int lpk = 1;

@@ -1,12 +1,8 @@
-// Layered decoders read from a model folder, bf16 weights: the family of "Nabelix" (config.json names the layers and
-// every size and constant). A layer is
-//     x <- x + mixer(conv(norm1(x)));   x <- x + ff(norm2(x))
-// with layer norms, a causal input convolution, and the "parallel" mixer: windowed attention with kept first tokens
-// and a distance bias beside a gated delta rule, both reading the same input. A block of layers may run several
-// times in a row (a loop), every pass with a cache of its own.
+// States and steps of the layered decoders (hybrid_model.hpp says which designs and what a layer is made of).
 //
 // Two pipelines compute a step; both use the same caches and states:
-//   up to 4 rows, one token per sequence: five launches per layer (kernels_gemv_bf16.cuh, hybrid_token_mix_kernel)
+//   up to 4 rows, one token per sequence: matrix-vector products with the norms as prologues (kernels_gemv_bf16.cuh), five
+//     launches per layer whose feed-forward follows its mixer, three where it stands beside it
 //   anything else: tensor-core (or fp32) matrix products over all rows of the step
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
@@ -18,20 +14,19 @@
 #include <cstring>
 #include <memory>
 
+#include "hybrid_model.hpp"
 #include "kernels_delta.cuh"
 #include "kernels_gemm_bf16.cuh"
 #include "kernels_gemv_bf16.cuh"
+#include "kernels_moe.cuh"
+#include "kernels_recurrent.cuh"
 #include "kernels_rowwise.cuh"
 #include "kernels_window_attn.cuh"
-#include "model_dir.hpp"
 #include "tg_internal.hpp"
 
 using namespace tg;
-typedef __nv_bfloat16 bf16;
 
 namespace {
-
-int round_up(int x, int m) { return (x + m - 1) / m * m; }
 
 // One token per sequence: the attention of every (sequence, key/value head, run of keys) and the delta rule of every
 // (sequence, head) in one launch. grid (G * nsplit + delta heads, rows)
@@ -48,6 +43,18 @@ __global__ void __launch_bounds__(256) hybrid_token_mix_kernel(WAttnArgs w, Delt
 		window_attn_token_cta<PT, CT, OT>(w, blockIdx.y, (blockIdx.x - d.H) / w.nsplit, (blockIdx.x - d.H) % w.nsplit, mix_sm);
 }
 
+// One token per sequence, the feed-forward beside the mixer: the mixer's CTAs, then (few rows) those of the row's chosen
+// experts. grid (mixer CTAs + experts' CTAs, rows)
+template <typename PT, typename CT, typename OT, bool ATTN> __global__ void __launch_bounds__(256) beside_token_mix_kernel(WAttnArgs w, LinArgs l, MoeArgs e, int n_mix) {
+	pdl_trigger();
+	pdl_wait();
+	extern __shared__ __align__(16) float mix_sm[];
+	const int x = blockIdx.x;
+	if (x >= n_mix) expert_token_cta(e, blockIdx.y, x - n_mix, mix_sm);
+	else if (ATTN) window_attn_token_cta<PT, CT, OT>(w, blockIdx.y, x / w.nsplit, x % w.nsplit, mix_sm);
+	else lin_token_cta<PT>(l, blockIdx.y, x, mix_sm);
+}
+
 // positions and history parities of the lock-step decode after a token
 __global__ void hybrid_advance_kernel(int *pos, int *par, int n) {
 	pdl_trigger();
@@ -59,385 +66,6 @@ __global__ void hybrid_advance_kernel(int *pos, int *par, int n) {
 	}
 }
 
-// A linear layer: weights [N][ld] bf16 with K used columns (padded with zeros to a multiple of 8).
-struct Lin {
-	const bf16 *W = nullptr;
-	int N = 0, K = 0, ld = 0;
-	CUtensorMap map[3];  // boxes of 64, 128 and 256 rows
-};
-
-int make_map(CUtensorMap *out, const void *base, size_t rows, int cols, int ld, int box_rows) {
-	PFN_encodeTiled enc = get_encode_fn();
-	if (!enc) return fail(TG_ECUDA, "cuTensorMapEncodeTiled is not available");
-	cuuint64_t dims[2] = {cuuint64_t(cols), cuuint64_t(rows)};
-	cuuint64_t strides[1] = {cuuint64_t(ld) * 2};
-	cuuint32_t box[2] = {64, cuuint32_t(box_rows)}, es[2] = {1, 1};
-	CUresult r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void *>(base), dims, strides, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
-	                 CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-	if (r != CUDA_SUCCESS) return fail(TG_ECUDA, "cuTensorMapEncodeTiled failed (" + std::to_string(int(r)) + ")");
-	return TG_OK;
-}
-
-// ------------------------------------------------------------------ what config.json says
-struct AttnSpec {
-	int H = 0, G = 0, dk = 0, dv = 0, dkp = 0, dvp = 0;
-	float scale = 0.0f;
-	int window = 0, keep = 0;
-};
-struct DeltaSpec {
-	int H = 0, KH = 0, dk = 0, dv = 0, taps = 0, ra = 0, rg = 0;
-	int channels() const { return 2 * KH * dk + H * dv; }
-	int dkp() const { return dk <= 32 ? 32 : (dk <= 64 ? 64 : (dk <= 128 ? 128 : 256)); }
-};
-struct Layer {
-	AttnSpec at;
-	DeltaSpec de;
-	float left_scale = 1.0f, right_scale = 1.0f;
-	int ff = 0, ffp = 0;  // 0: no feed-forward
-	// columns of a projection row
-	int p_q, p_k, p_v, p_g, p_a1, p_g1, p_conv, p_b, ldp;
-	int o_col, kc;        // columns of a mixed row: attention heads at 0, delta heads at o_col; kc in all
-	float *norm1, *norm2 = nullptr, *canon = nullptr, *r1, *r2, *conv, *A_log, *dt_bias, *rnorm;
-	Lin proj, a2, g2, out, gu, down;
-};
-struct Run {
-	int layer;
-	bool add_embed;  // another pass through the loop begins here
-};
-
-}  // namespace
-
-struct HybridModel : tg_model {
-	std::string architecture;
-	int dtype = TG_BF16;
-	int D = 0, Dp = 0, taps = 1;  // taps of the input convolution
-	bool has_canon = false;
-	float eps = 1e-6f, softcap = 0.0f;
-	std::vector<Layer> layers;
-	std::vector<Run> runs;
-	Lin embed;
-	float *final_norm = nullptr;
-	std::vector<void *> mem;
-
-	~HybridModel() override {
-		for (void *p : mem) cudaFree(p);
-	}
-	const char *arch() const override { return architecture.c_str(); }
-	int new_state(int batch, int max_pos, tg_state **out) override;
-};
-
-namespace {
-
-// ------------------------------------------------------------------ loading
-struct Loader {
-	HybridModel *m;
-	SafeTensors st;
-
-	int get(const std::string &name, std::vector<long long> shape, const SafeTensors::Tensor **out) {
-		auto it = st.tensors.find(name);
-		if (it == st.tensors.end()) return fail(TG_EIO, "model.safetensors has no tensor " + name);
-		const auto &t = it->second;
-		if (t.dtype != "BF16" && t.dtype != "F32") return fail(TG_EINVAL, name + ": dtype " + t.dtype + " is not supported");
-		bool ok = t.shape.size() == shape.size();
-		for (size_t i = 0; ok && i < shape.size(); i++) ok = shape[i] < 0 || t.shape[i] == shape[i];
-		if (!ok) {
-			std::string got, want;
-			for (long long d : t.shape) got += (got.empty() ? "" : ", ") + std::to_string(d);
-			for (long long d : shape) want += (want.empty() ? "" : ", ") + (d < 0 ? std::string("*") : std::to_string(d));
-			return fail(TG_ESHAPE, name + ": shape [" + got + "], expected [" + want + "]");
-		}
-		*out = &t;
-		return TG_OK;
-	}
-	int upload(const void *host, size_t bytes, void **dev) {
-		if (cudaMalloc(dev, std::max<size_t>(bytes, 16)) != cudaSuccess) {
-			cudaGetLastError();
-			return fail(TG_ENOMEM, "cudaMalloc(weights)");
-		}
-		m->mem.push_back(*dev);
-		TG_CUDA(cudaMemcpy(*dev, host, bytes, cudaMemcpyHostToDevice));
-		return TG_OK;
-	}
-	int vec(const std::string &name, int n, float **dev) {
-		const SafeTensors::Tensor *t;
-		TG_TRY(get(name, {n}, &t));
-		std::vector<float> h(n);
-		for (int i = 0; i < n; i++) h[i] = t->at(i);
-		return upload(h.data(), size_t(n) * 4, reinterpret_cast<void **>(dev));
-	}
-	// a matrix under construction on the host
-	struct Host {
-		int rows, ld;
-		std::vector<uint16_t> v;
-		Host(int r, int l) : rows(r), ld(l), v(size_t(r) * l, 0) {}
-	};
-	static uint16_t to16(const SafeTensors::Tensor &t, size_t i) {
-		if (t.dtype == "BF16") {
-			uint16_t h;
-			std::memcpy(&h, t.data + 2 * i, 2);
-			return h;
-		}
-		uint32_t b;
-		std::memcpy(&b, t.data + 4 * i, 4);
-		return uint16_t((b + 0x7FFF + ((b >> 16) & 1)) >> 16);
-	}
-	// rows [r0, r0 + n) and columns [c0, c0 + k) of t -> dst rows d0.., columns e0..
-	static void put(Host &h, int d0, int e0, const SafeTensors::Tensor &t, size_t r0, int n, size_t c0, int k) {
-		const size_t cols = size_t(t.shape[1]);
-		for (int i = 0; i < n; i++) {
-			uint16_t *dst = h.v.data() + size_t(d0 + i) * h.ld + e0;
-			const size_t src = (r0 + i) * cols + c0;
-			if (t.dtype == "BF16") std::memcpy(dst, t.data + 2 * src, 2 * size_t(k));
-			else
-				for (int j = 0; j < k; j++) dst[j] = to16(t, src + j);
-		}
-	}
-	int linear(const Host &h, Lin *l) {
-		l->N = h.rows;
-		l->K = l->ld = h.ld;
-		TG_TRY(upload(h.v.data(), h.v.size() * 2, reinterpret_cast<void **>(const_cast<bf16 **>(&l->W))));
-		for (int i = 0; i < 3; i++) TG_TRY(make_map(&l->map[i], l->W, l->N, l->K, l->ld, 64 << i));
-		return TG_OK;
-	}
-	// [taps][channels] fp32 from [channels, taps] tensors laid one after the other
-	int conv(const std::vector<std::pair<std::string, int>> &parts, int taps, float **dev) {
-		int n = 0, c0 = 0;
-		for (const auto &p : parts) n += p.second;
-		std::vector<float> h(size_t(taps) * n);
-		for (const auto &p : parts) {
-			const SafeTensors::Tensor *t;
-			TG_TRY(get(p.first, {p.second, taps}, &t));
-			for (int c = 0; c < p.second; c++)
-				for (int j = 0; j < taps; j++) h[size_t(j) * n + c0 + c] = t->at(size_t(c) * taps + j);
-			c0 += p.second;
-		}
-		return upload(h.data(), h.size() * 4, reinterpret_cast<void **>(dev));
-	}
-
-	int layer(int i) {
-		Layer &L = m->layers[i];
-		const int D = m->D, Dp = m->Dp;
-		const std::string p = "l" + std::to_string(i) + ".", lp = p + "mix.left.", rp = p + "mix.right.";
-		const AttnSpec &A = L.at;
-		DeltaSpec &E = L.de;
-		TG_TRY(vec(p + "norm1", D, &L.norm1));
-		if (m->has_canon) {
-			TG_TRY(conv({{p + "canon1", D}}, m->taps, &L.canon));
-		} else {
-			const std::vector<float> none(D, 0.0f);
-			TG_TRY(upload(none.data(), size_t(D) * 4, reinterpret_cast<void **>(&L.canon)));
-		}
-		const SafeTensors::Tensor *q, *k, *v, *g, *o, *rq, *rk, *rv, *b, *a1, *a2, *g1, *g2, *ro;
-		TG_TRY(get(lp + "q", {A.H * A.dk, D}, &q));
-		TG_TRY(get(lp + "k", {A.G * A.dk, D}, &k));
-		TG_TRY(get(lp + "v", {A.G * A.dv, D}, &v));
-		TG_TRY(get(lp + "g", {A.H * A.dv, D}, &g));
-		TG_TRY(get(lp + "o", {D, A.H * A.dv}, &o));
-		TG_TRY(vec(lp + "r1", A.H, &L.r1));
-		TG_TRY(vec(lp + "r2", A.H, &L.r2));
-		TG_TRY(get(rp + "q", {E.KH * E.dk, D}, &rq));
-		TG_TRY(get(rp + "k", {E.KH * E.dk, D}, &rk));
-		TG_TRY(get(rp + "v", {E.H * E.dv, D}, &rv));
-		TG_TRY(get(rp + "b", {E.H, D}, &b));
-		TG_TRY(get(rp + "a1", {-1, D}, &a1));
-		TG_TRY(get(rp + "g1", {-1, D}, &g1));
-		const int ra = int(a1->shape[0]), rg = int(g1->shape[0]);
-		TG_TRY(get(rp + "a2", {E.H * E.dk, ra}, &a2));
-		TG_TRY(get(rp + "g2", {E.H * E.dv, rg}, &g2));
-		TG_TRY(get(rp + "o", {D, E.H * E.dv}, &ro));
-		TG_TRY(vec(rp + "A_log", E.H, &L.A_log));
-		TG_TRY(vec(rp + "dt_bias", E.H * E.dk, &L.dt_bias));
-		TG_TRY(vec(rp + "norm", E.dv, &L.rnorm));
-		TG_TRY(conv({{rp + "q.conv", E.KH * E.dk}, {rp + "k.conv", E.KH * E.dk}, {rp + "v.conv", E.H * E.dv}}, E.taps, &L.conv));
-		E.ra = round_up(ra, 8);
-		E.rg = round_up(rg, 8);
-		// the projections, one matrix: heads of the attention padded to multiples of 16 columns
-		int n = 0;
-		auto place = [&](int w) {
-			const int at = n;
-			n += w;
-			return at;
-		};
-		L.p_q = place(A.H * A.dkp);
-		L.p_k = place(A.G * A.dkp);
-		L.p_v = place(A.G * A.dvp);
-		L.p_g = place(A.H * A.dvp);
-		L.p_a1 = place(E.ra);
-		L.p_g1 = place(E.rg);
-		L.p_conv = place(E.channels());
-		L.p_b = place(E.H);
-		L.ldp = round_up(n, 8);
-		{
-			Host h(L.ldp, Dp);
-			for (int x = 0; x < A.H; x++) put(h, L.p_q + x * A.dkp, 0, *q, size_t(x) * A.dk, A.dk, 0, D);
-			for (int x = 0; x < A.G; x++) put(h, L.p_k + x * A.dkp, 0, *k, size_t(x) * A.dk, A.dk, 0, D);
-			for (int x = 0; x < A.G; x++) put(h, L.p_v + x * A.dvp, 0, *v, size_t(x) * A.dv, A.dv, 0, D);
-			for (int x = 0; x < A.H; x++) put(h, L.p_g + x * A.dvp, 0, *g, size_t(x) * A.dv, A.dv, 0, D);
-			put(h, L.p_a1, 0, *a1, 0, ra, 0, D);
-			put(h, L.p_g1, 0, *g1, 0, rg, 0, D);
-			put(h, L.p_conv, 0, *rq, 0, E.KH * E.dk, 0, D);
-			put(h, L.p_conv + E.KH * E.dk, 0, *rk, 0, E.KH * E.dk, 0, D);
-			put(h, L.p_conv + 2 * E.KH * E.dk, 0, *rv, 0, E.H * E.dv, 0, D);
-			put(h, L.p_b, 0, *b, 0, E.H, 0, D);
-			TG_TRY(linear(h, &L.proj));
-		}
-		{
-			Host h(E.H * E.dk, E.ra);
-			put(h, 0, 0, *a2, 0, E.H * E.dk, 0, ra);
-			TG_TRY(linear(h, &L.a2));
-		}
-		{
-			Host h(E.H * E.dv, E.rg);
-			put(h, 0, 0, *g2, 0, E.H * E.dv, 0, rg);
-			TG_TRY(linear(h, &L.g2));
-		}
-		// both output projections side by side
-		L.o_col = A.H * A.dvp;
-		L.kc = round_up(L.o_col + E.H * E.dv, 8);
-		{
-			Host h(D, L.kc);
-			for (int x = 0; x < A.H; x++) put(h, 0, x * A.dvp, *o, 0, D, size_t(x) * A.dv, A.dv);
-			put(h, 0, L.o_col, *ro, 0, D, 0, E.H * E.dv);
-			TG_TRY(linear(h, &L.out));
-		}
-		if (L.ff) {
-			const SafeTensors::Tensor *ga, *up, *dn;
-			TG_TRY(vec(p + "norm2", D, &L.norm2));
-			TG_TRY(get(p + "mlp.gate", {L.ff, D}, &ga));
-			TG_TRY(get(p + "mlp.up", {L.ff, D}, &up));
-			TG_TRY(get(p + "mlp.down", {D, L.ff}, &dn));
-			{
-				Host h(2 * L.ffp, Dp);  // blocks of 16 gate rows, 16 up rows
-				for (int x = 0; x < L.ff; x += 16) {
-					const int c = std::min(16, L.ff - x);
-					put(h, 2 * x, 0, *ga, x, c, 0, D);
-					put(h, 2 * x + 16, 0, *up, x, c, 0, D);
-				}
-				TG_TRY(linear(h, &L.gu));
-			}
-			Host h(D, L.ffp);
-			put(h, 0, 0, *dn, 0, D, 0, L.ff);
-			TG_TRY(linear(h, &L.down));
-		}
-		return TG_OK;
-	}
-};
-
-// config.json -> the model's layer list. Every size and constant comes from here (or from a tensor's shape).
-struct ConfigReader {
-	std::string err;
-	double num(const json::Value *o, const char *key, const char *where, bool need = true, double dflt = 0.0) {
-		const json::Value *v = o ? o->find(key) : nullptr;
-		if (v && v->kind == json::Value::NUMBER) return v->num;
-		if ((need || v) && err.empty()) err = std::string("config.json: ") + where + "." + key + " is not a number";
-		return dflt;
-	}
-	int size(const json::Value *o, const char *key, const char *where, int lo = 1) {
-		const double d = num(o, key, where);
-		if (err.empty() && (d < lo || d > 1e9 || d != std::floor(d))) err = std::string("config.json: ") + where + "." + key + " is out of range";
-		return err.empty() ? int(d) : lo;
-	}
-	const json::Value *obj(const json::Value *o, const char *key, const char *where) {
-		const json::Value *v = o ? o->find(key) : nullptr;
-		if ((!v || v->kind != json::Value::OBJECT) && err.empty()) err = std::string("config.json: ") + where + "." + key + " is missing";
-		return v;
-	}
-};
-
-int read_config(const json::Value &c, HybridModel *m) {
-	ConfigReader r;
-	m->D = r.size(&c, "width", "model");
-	m->hidden_size = m->D;
-	m->Dp = round_up(m->D, 8);
-	m->n_vocab = r.size(&c, "vocab", "model");
-	m->n_pos = 1 << 24;  // distances stay exact in fp32
-	m->eps = float(r.num(r.obj(&c, "norm", "model"), "eps", "norm"));
-	m->softcap = float(r.num(&c, "logit_softcap", "model", false, 0.0));
-	if (const json::Value *cn = c.find("canon")) {
-		m->has_canon = true;
-		m->taps = r.size(cn, "taps", "canon");
-	}
-	const json::Value *ls = c.find("layers");
-	if (!ls || ls->kind != json::Value::ARRAY || ls->items.empty()) return fail(TG_EINVAL, "config.json: no layers");
-	for (const auto &l : ls->items) {
-		Layer L;
-		const json::Value *ty = l.find("type");
-		if (!ty || ty->str != "parallel") return fail(TG_EINVAL, "config.json: unknown layer type" + (ty ? " " + ty->str : std::string()));
-		const json::Value *mx = r.obj(&l, "mixer", "layer"), *a = r.obj(mx, "left", "mixer"), *d = r.obj(mx, "right", "mixer");
-		L.left_scale = float(r.num(mx, "left_scale", "mixer"));
-		L.right_scale = float(r.num(mx, "right_scale", "mixer"));
-		L.at.H = r.size(a, "heads", "left");
-		L.at.G = r.size(a, "kv_heads", "left");
-		L.at.dk = r.size(a, "dim", "left");
-		L.at.dv = r.size(a, "vdim", "left");
-		L.at.scale = float(r.num(a, "scale", "left"));
-		const json::Value *mk = r.obj(a, "mask", "left");
-		L.at.window = r.size(mk, "size", "mask");
-		if (mk && mk->find("keep_first")) L.at.keep = r.size(mk, "keep_first", "mask", 0);
-		L.at.dkp = round_up(L.at.dk, 16);
-		L.at.dvp = round_up(L.at.dv, 16);
-		L.de.H = r.size(d, "heads", "right");
-		L.de.KH = r.size(d, "kv_heads", "right");
-		L.de.dk = r.size(d, "dim", "right");
-		L.de.dv = r.size(d, "vdim", "right");
-		L.de.taps = r.size(d, "conv", "right");
-		const json::Value *ff = l.find("mlp");
-		if (ff) {
-			const json::Value *kd = ff->find("kind");
-			if (!kd || kd->str != "dense") return fail(TG_EINVAL, "config.json: unknown kind of feed-forward");
-			L.ff = r.size(ff, "ff", "mlp");
-			L.ffp = round_up(L.ff, 16);
-		}
-		if (!r.err.empty()) return fail(TG_EINVAL, r.err);
-		if (L.at.H % L.at.G || L.de.H % L.de.KH) return fail(TG_ESHAPE, "config.json: heads are not a multiple of kv_heads");
-		if (L.de.dk > 256) return fail(TG_ESHAPE, "delta rule: key sizes above 256 are not supported");
-		m->layers.push_back(L);
-	}
-	const int n = int(m->layers.size());
-	int start = 0, stop = 0, times = 1;
-	if (const json::Value *lp = c.find("loop")) {
-		start = r.size(lp, "start", "loop", 0);
-		stop = r.size(lp, "stop", "loop", 0);
-		times = r.size(lp, "times", "loop", 1);
-		if (r.err.empty() && (start > stop || stop > n)) return fail(TG_EINVAL, "config.json: loop lies outside the layers");
-	}
-	if (!r.err.empty()) return fail(TG_EINVAL, r.err);
-	if (m->taps > 16) return fail(TG_ESHAPE, "input convolutions of more than 16 taps are not supported");
-	for (int i = 0; i < start; i++) m->runs.push_back({i, false});
-	for (int t = 0; t < times; t++)
-		for (int i = start; i < stop; i++) m->runs.push_back({i, t > 0 && i == start});
-	for (int i = std::max(start, stop); i < n; i++) m->runs.push_back({i, false});
-	return TG_OK;
-}
-
-int open_hybrid(const char *dir, int device, int dtype, tg_model **out) {
-	json::Value cfg;
-	std::string err;
-	if (!json::parse_file(std::string(dir) + "/config.json", &cfg, &err)) return fail(TG_EIO, err);
-	std::unique_ptr<HybridModel> m(new HybridModel());
-	m->architecture = cfg.find("architecture")->str;
-	m->device = device;
-	m->dtype = dtype;
-	TG_TRY(read_config(cfg, m.get()));
-	Loader ld;
-	ld.m = m.get();
-	if (!ld.st.open(std::string(dir) + "/model.safetensors", &err)) return fail(TG_EIO, err);
-	TG_TRY(ensure_device(device));
-	const SafeTensors::Tensor *e;
-	TG_TRY(ld.get("embed", {m->n_vocab, m->D}, &e));
-	{
-		Loader::Host h(m->n_vocab, m->Dp);
-		Loader::put(h, 0, 0, *e, 0, m->n_vocab, 0, m->D);
-		TG_TRY(ld.linear(h, &m->embed));
-	}
-	TG_TRY(ld.vec("final.norm", m->D, &m->final_norm));
-	for (size_t i = 0; i < m->layers.size(); i++) TG_TRY(ld.layer(int(i)));
-	*out = m.release();
-	return TG_OK;
-}
-
-RegisterArch reg_nabelix("Nabelix", open_hybrid);
-
 }  // namespace
 
 // ===================================================================== state
@@ -448,7 +76,7 @@ struct HybridState : tg_state {
 	struct RunCache {
 		void *kc = nullptr, *vc = nullptr, *ks = nullptr, *vs = nullptr;
 		int cap = 0, keep_rows = 0;
-		float *canon = nullptr, *conv = nullptr, *S = nullptr;
+		float *canon = nullptr, *conv = nullptr, *S = nullptr, *n = nullptr, *mx = nullptr;  // n, mx: LIN_MLSTM
 		CUtensorMap kmap, vmap, ksmap, vsmap;
 	};
 	std::vector<RunCache> cache;
@@ -457,14 +85,22 @@ struct HybridState : tg_state {
 	float *x = nullptr;
 	int ldx = 0;
 	float2 *stats = nullptr;          // mean and 1/deviation of the rows
-	void *h = nullptr, *P = nullptr, *O = nullptr, *act = nullptr;   // bf16, or fp32 in a 32-bit state
-	float *P32 = nullptr, *O32 = nullptr, *act32 = nullptr;          // the few-row pipeline's, always fp32
+	void *h = nullptr, *hp = nullptr, *P = nullptr, *O = nullptr, *act = nullptr;  // bf16, or fp32 in a 32-bit state; hp: h before the shift
+	float *T32 = nullptr;                                            // fp32 columns of the projections
+	float2 *cs = nullptr;                                            // rotations of the rows' positions
+	float *P32 = nullptr, *O32 = nullptr, *act32 = nullptr, *h32 = nullptr, *ex32 = nullptr;  // the few-row pipeline's, always fp32
 	float *z = nullptr, *gz = nullptr, *o_raw = nullptr, *blk = nullptr, *bV = nullptr;
+	void *xc = nullptr;               // convolved inputs of a recurrence
+	LinArgs lin{};                    // the recurrences' buffers
+	bool lin_tc = false;              // ... of the tensor-core path are there
+	MoeArgs moe{};                    // routing buffers
+	float *RL = nullptr;              // router logits
+	void *xg = nullptr, *xa = nullptr, *xy = nullptr;  // gathered rows, experts' activations, experts' outputs
 	float *part = nullptr;
 	unsigned *tickets = nullptr;
 	int nsplit_cap = 1;
-	CUtensorMap hmap;                 // h as an operand
-	std::vector<CUtensorMap> pmap, omap, amap, a1map, g1map;  // per layer
+	CUtensorMap hmap, hpmap, xgmap;   // h, hp and xg as operands
+	std::vector<CUtensorMap> pmap, omap, amap, a1map, g1map, xcmap, xamap, shmap, slmap;  // per layer
 	float *wl = nullptr;              // logits of wanted rows
 	int wl_rows = 0;
 	void *hn = nullptr;               // their normed rows
@@ -502,10 +138,29 @@ struct HybridState : tg_state {
 	StepDesc lockstep_desc() const;
 	int run_layers(const StepDesc &d, int R, int nseg, int max_len);
 	int score_rows(const int *rows_dev, int n, float *out, float *norm_out);
-	int gemm(int epi, const void *A, int lda, const CUtensorMap *amap_, const Lin &w, int M, void *C, int ldc, float cap = 0.0f);
+	struct GemmOpt {
+		float cap = 0.0f, limit = 0.0f;
+		int act = GLU_GELU, n32 = 0, ld32 = 0;
+		float *C32 = nullptr;
+		bool grouped = false;   // by expert: M is the most rows there can be, est the likely row tiles
+		int est = 0;
+	};
+	int gemm(int epi, const void *A, int lda, const CUtensorMap *amap_, const Lin &w, int M, void *C, int ldc, const GemmOpt &o);
+	int gemm(int epi, const void *A, int lda, const CUtensorMap *amap_, const Lin &w, int M, void *C, int ldc) { return gemm(epi, A, lda, amap_, w, M, C, ldc, GemmOpt()); }
 	int gemv(int pro, int epi, GemvArgs g, int R);
 	WAttnArgs attn_args(const StepDesc &d, int run, const void *p, int ldp, void *out, int ldo);
 	DeltaArgs delta_args(const StepDesc &d, int run, const void *p, int ldp, void *out, int ldo);
+	LinArgs lin_args(const StepDesc &d, int run, const void *p);
+	MoeArgs moe_args(const Layer &L);
+	int moe_rows(const Layer &L, int rows) const { return (rows * L.ff.top / GB_BM + L.ff.experts) * GB_BM; }
+	int few_layer(const StepDesc &d, int run, int R);
+	int rows_layer(const StepDesc &d, int run, int R, int nseg, int max_len);
+	int beside_few_layer(const StepDesc &d, int run, int R);
+	int beside_rows_layer(const StepDesc &d, int run, int R, int nseg, int max_len, int pending);
+	int norm_in(const StepDesc &d, int run, int R, int pending);  // norm1 and what follows it; first adds layer `pending`'s experts (-1: none)
+	int add_experts(int layer, int R);
+	int attn_rows(const WAttnArgs &wa, int run, int R, int nseg, int max_len);
+	int token_splits(const WAttnArgs &wa, int fill) const;
 
 	struct Entry {
 		int seq, count, done;
@@ -539,6 +194,7 @@ struct HybridState : tg_state {
 namespace {
 constexpr int FEW_ROWS = 4;  // rows of the matrix-vector pipeline
 constexpr int TOKEN_SPLITS = 32;
+constexpr int LIN_SCAN_MAX = 8;  // portions up to this long go through a recurrence token by token
 
 template <typename K> int allow_smem(K kernel, size_t bytes) {
 	if (bytes <= 48 * 1024) return TG_OK;
@@ -564,41 +220,44 @@ int pick_bn(int m_tiles, int N) {
 	return best;
 }
 
-template <int BN, int EPI> int launch_gemm_tc(const CUtensorMap &am, const CUtensorMap &wm, const GemmArgs &a, cudaStream_t st) {
+template <int BN, int EPI, bool GRP> int launch_gemm_tc(const CUtensorMap &am, const CUtensorMap &wm, const GemmArgs &a, cudaStream_t st) {
 	static bool done[TG_MAX_DEVICES] = {};
 	bool &d = done[current_device_slot()];
+	auto kernel = gemm_bf16_tc_kernel<BN, EPI, GRP>;
 	if (!d) {
-		TG_TRY(allow_smem(gemm_bf16_tc_kernel<BN, EPI>, GbShape<BN>::SMEM));
+		TG_TRY(allow_smem(kernel, GbShape<BN>::SMEM));
 		d = true;
 	}
-	launch_k(gemm_bf16_tc_kernel<BN, EPI>, dim3(std::min(g_num_sms, a.m_tiles * a.n_tiles)), dim3(GB_THREADS), size_t(GbShape<BN>::SMEM), st, am, wm, a);
+	launch_k(kernel, dim3(std::min(g_num_sms, a.m_tiles * a.n_tiles)), dim3(GB_THREADS), size_t(GbShape<BN>::SMEM), st, am, wm, a);
 	count_launch();
 	return check_launch("gemm_bf16_tc");
 }
-template <int EPI> int launch_gemm(const CUtensorMap &am, const Lin &w, GemmArgs a, cudaStream_t st) {
+// est: row tiles that a grouped product is likely to have
+template <int EPI, bool GRP = false> int launch_gemm(const CUtensorMap &am, const Lin &w, GemmArgs a, cudaStream_t st, int est = 0) {
 	a.m_tiles = (a.M + GB_BM - 1) / GB_BM;
-	const int cols = EPI == GEMM_LOGITS ? a.ldc : a.N, bn = pick_bn(a.m_tiles, cols);
+	const int cols = EPI == GEMM_LOGITS ? a.ldc : a.N, bn = pick_bn(est ? est : a.m_tiles, cols);
 	a.n_tiles = (cols + bn - 1) / bn;
-	if (bn == 256) return launch_gemm_tc<256, EPI>(am, w.map[2], a, st);
-	if (bn == 128) return launch_gemm_tc<128, EPI>(am, w.map[1], a, st);
-	return launch_gemm_tc<64, EPI>(am, w.map[0], a, st);
+	if (bn == 256) return launch_gemm_tc<256, EPI, GRP>(am, w.map[2], a, st);
+	if (bn == 128) return launch_gemm_tc<128, EPI, GRP>(am, w.map[1], a, st);
+	return launch_gemm_tc<64, EPI, GRP>(am, w.map[0], a, st);
 }
-template <int EPI> int launch_gemm_f32(const float *A, int lda, const Lin &w, const GemmArgs &a, cudaStream_t st) {
+template <int EPI, bool GRP = false> int launch_gemm_f32(const float *A, int lda, const Lin &w, const GemmArgs &a, cudaStream_t st) {
 	const int cols = EPI == GEMM_LOGITS ? a.ldc : a.N;
-	launch_k(gemm_f32_kernel<EPI>, dim3((cols + GF_T - 1) / GF_T, (a.M + GF_T - 1) / GF_T), dim3(256), 0, st, A, lda, w.W, w.ld, a);
+	launch_k(gemm_f32_kernel<EPI, GRP>, dim3((cols + GF_T - 1) / GF_T, (a.M + GF_T - 1) / GF_T), dim3(256), 0, st, A, lda, w.W, w.ld, a);
 	count_launch();
 	return check_launch("gemm_f32");
 }
 
 template <int R, int NR, int KS, int PRO, int EPI> int launch_gemv(const GemvArgs &g, cudaStream_t st) {
-	const size_t smem = gv_smem<R, NR>(g.K, PRO);
+	const size_t smem = gv_smem<R, NR>(g.K, PRO, EPI, g.parts, g.top * g.n_ex);
 	auto kernel = gemv_bf16_kernel<R, NR, KS, PRO, EPI>;
 	TG_TRY(allow_smem(kernel, smem));
 	int occ = 1;
 	TG_CUDA(cudaOccupancyMaxActiveBlocksPerMultiprocessor(&occ, kernel, GV_THREADS, smem));
-	const int outs = (8 / KS) * NR / (EPI == GV_GEGLU ? 2 : 1);
-	const int n_out = EPI == GV_GEGLU ? g.N / 2 : (EPI == GV_LOGITS ? g.ldo : g.N);
-	const int groups = (n_out + outs - 1) / outs;
+	const int outs = (8 / KS) * NR / (EPI == GV_GLU ? 2 : 1);
+	const int n_out = EPI == GV_GLU ? g.N / 2 : (EPI == GV_LOGITS ? g.ldo : g.N);
+	auto per = [](int n, int m) { return (n + m - 1) / m; };
+	const int groups = EPI == GV_FRONT ? per(g.n_proj, outs) + per(g.n_glu, outs / 2) + per(g.n_route, outs) : per(n_out, outs);
 	launch_k(kernel, dim3(std::min(groups, std::max(1, occ) * g_num_sms)), dim3(GV_THREADS), smem, st, g);
 	count_launch();
 	return check_launch("gemv_bf16");
@@ -606,7 +265,9 @@ template <int R, int NR, int KS, int PRO, int EPI> int launch_gemv(const GemvArg
 template <int R> int launch_gemv_r(int pro, int epi, const GemvArgs &g, cudaStream_t st) {
 	if (pro == GV_LN_CONV && epi == GV_PROJ) return launch_gemv<R, 4, 2, GV_LN_CONV, GV_PROJ>(g, st);
 	if (pro == GV_VEC && epi == GV_ADD) return launch_gemv<R, 4, 8, GV_VEC, GV_ADD>(g, st);
-	if (pro == GV_LN && epi == GV_GEGLU) return launch_gemv<R, 4, 2, GV_LN, GV_GEGLU>(g, st);
+	if (pro == GV_LN && epi == GV_GLU) return launch_gemv<R, 4, 2, GV_LN, GV_GLU>(g, st);
+	if (pro == GV_LN_CONV && epi == GV_FRONT) return launch_gemv<R, 4, 2, GV_LN_CONV, GV_FRONT>(g, st);
+	if (pro == GV_MIX && epi == GV_ADD) return launch_gemv<R, 4, 8, GV_MIX, GV_ADD>(g, st);
 	if (pro == GV_LN && epi == GV_LOGITS) return launch_gemv<R, 4, 2, GV_LN, GV_LOGITS>(g, st);
 	return fail(TG_EINVAL, "gemv: no such combination");
 }
@@ -638,36 +299,98 @@ int HybridState::alloc() {
 	const int R = max_rows;
 	const size_t es = f32 ? 4 : 2;
 	ldx = round_up(D, 8);
-	int ldp = 8, kc = 8, ffp = 16, hz = 1, hv = 1;
-	size_t blkn = 1, blkV = 1, partn = 1;
+	int ldp = 8, kc = 8, ffp = 16, hz = 1, hv = 1, tail = 0, xcn = 0, inner = 0, half = m->rot_half;
+	size_t blkn = 0, blkV = 0, partn = 1;
 	int gmax = 1;
+	bool beside = false;
+	size_t linS = 0, linSp = 0, linN = 0;  // per chunk: state rows x columns (two paddings), key vectors
+	int linH = 0, top = 0, experts = 0, slots = 0, effp = 0, exf = 0;
 	for (const Layer &L : m->layers) {
 		ldp = std::max(ldp, L.ldp);
-		kc = std::max(kc, L.kc);
-		ffp = std::max(ffp, L.ffp);
-		hz = std::max(hz, round_up(L.de.H * L.de.dk, 4));
-		hv = std::max(hv, round_up(L.de.H * L.de.dv, 4));
-		blkn = std::max(blkn, size_t(L.de.H) * delta_block_floats(L.de.dkp()));
-		blkV = std::max(blkV, size_t(L.de.H) * DB * L.de.dv);
-		partn = std::max(partn, size_t(L.at.H) * (L.at.dvp + 2));
-		gmax = std::max(gmax, L.at.G);
+		kc = std::max(kc, L.kcat);
+		ffp = std::max(ffp, L.ff.ffp);
+		tail = std::max(tail, L.tail());
+		beside = beside || L.beside;
+		if (L.de.H) {
+			hz = std::max(hz, round_up(L.de.H * L.de.dk, 4));
+			hv = std::max(hv, round_up(L.de.H * L.de.dv, 4));
+			blkn = std::max(blkn, size_t(L.de.H) * delta_block_floats(L.de.dkp()));
+			blkV = std::max(blkV, size_t(L.de.H) * DB * L.de.dv);
+		}
+		if (L.at.H) {
+			partn = std::max(partn, size_t(L.at.H) * (L.at.dvp + 2));
+			gmax = std::max(gmax, L.at.G);
+		}
+		if (L.li.H) {
+			const LinSpec &li = L.li;
+			inner = std::max(inner, round_up(li.H * li.vd, 4));
+			linH = std::max(linH, li.H);
+			if (li.kind == LIN_SSM) xcn = std::max(xcn, li.xc_cols());
+			if (li.Np <= 256) {
+				linS = std::max(linS, size_t(li.H) * li.N * li.vdp);
+				linSp = std::max(linSp, size_t(li.H) * li.Np * li.vdp);
+				linN = std::max(linN, size_t(li.H) * li.N);
+			}
+		}
+		if (L.ff.experts) {
+			top = std::max(top, L.ff.top);
+			experts = std::max(experts, round_up(L.ff.experts, 8));
+			slots = std::max(slots, moe_rows(L, R));
+			effp = std::max(effp, L.ff.effp);
+			exf = std::max(exf, L.ff.top * L.ff.effp);
+		}
 	}
 	TG_TRY(take(&x, size_t(R) * ldx));
 	TG_TRY(take(&stats, R));
 	TG_TRY(take_act(&h, size_t(R) * m->Dp));
 	TG_TRY(take_act(&P, size_t(R) * ldp));
 	TG_TRY(take_act(&O, size_t(R) * kc));
-	TG_TRY(take_act(&act, size_t(R) * ffp));
+	if (beside) TG_TRY(take_act(&hp, size_t(R) * m->Dp));
+	else TG_TRY(take_act(&act, size_t(R) * ffp));
+	TG_TRY(take(&T32, size_t(R) * tail));
+	if (half) TG_TRY(take(&cs, size_t(R) * m->rots.size() * half));
 	const int F = std::min(FEW_ROWS, B);
 	TG_TRY(take(&P32, size_t(F) * ldp));
 	TG_TRY(take(&O32, size_t(F) * kc));
 	TG_TRY(take(&act32, size_t(F) * ffp));
-	TG_TRY(take(&z, size_t(R) * hz));
-	TG_TRY(take(&gz, size_t(R) * hv));
-	TG_TRY(take(&o_raw, size_t(R) * hv));
-	const size_t nb = size_t(R) / DB + B + 1;
-	TG_TRY(take(&blk, nb * blkn));
-	TG_TRY(take(&bV, nb * blkV));
+	TG_TRY(take(&h32, size_t(F) * D));
+	TG_TRY(take(&ex32, size_t(F) * exf));
+	TG_TRY(take(&o_raw, size_t(R) * std::max(hv, inner)));
+	if (blkn) {
+		TG_TRY(take(&z, size_t(R) * hz));
+		TG_TRY(take(&gz, size_t(R) * hv));
+		const size_t nb = size_t(R) / DB + B + 1;
+		TG_TRY(take(&blk, nb * blkn));
+		TG_TRY(take(&bV, nb * blkV));
+	}
+	if (linH) {
+		if (xcn) TG_TRY(take_act(&xc, size_t(R) * xcn));
+		TG_TRY(take(&lin.la, size_t(R) * linH));
+		TG_TRY(take(&lin.b, size_t(R) * linH));
+		TG_TRY(take(&lin.em, size_t(R) * linH));
+	}
+	const size_t nchunk = size_t(R) / LC + B + 1;
+	lin_tc = !f32 && linS && env_int("TG_LIN_TC", 1);
+	if (lin_tc) {
+		TG_TRY(take(&lin.dS, nchunk * linS));
+		TG_TRY(take(&lin.Sh, nchunk * linSp));
+		TG_TRY(take(&lin.Sl, nchunk * linSp));
+		TG_TRY(take(&lin.dn, nchunk * linN));
+		TG_TRY(take(&lin.n0, nchunk * linN));
+		TG_TRY(take(&lin.tot, nchunk * linH));
+	}
+	if (experts) {
+		TG_TRY(take(&RL, size_t(R) * experts));
+		TG_TRY(take(&moe.id, size_t(R) * top));
+		TG_TRY(take(&moe.w, size_t(R) * top));
+		TG_TRY(take(&moe.place, size_t(R) * top));
+		TG_TRY(take(&moe.count, experts));
+		TG_TRY(take(&moe.tile_expert, slots / GB_BM));
+		TG_TRY(take(&moe.n_tiles, 1));
+		TG_TRY(take_act(&xg, size_t(slots) * m->Dp));
+		TG_TRY(take_act(&xa, size_t(slots) * effp));
+		TG_TRY(take_act(&xy, size_t(slots) * ldx));
+	}
 	nsplit_cap = std::max(1, std::min(TOKEN_SPLITS, 2 * g_num_sms / B));
 	TG_TRY(take(&part, size_t(B) * nsplit_cap * partn));
 	TG_TRY(take(&tickets, size_t(B) * gmax));
@@ -677,8 +400,24 @@ int HybridState::alloc() {
 		const Layer &L = m->layers[m->runs[i].layer];
 		const AttnSpec &A = L.at;
 		RunCache &c = cache[i];
-		c.cap = round_up(int(std::min<long long>(max_pos_global, (long long)A.window + max_seq_rows)), 64);
-		c.keep_rows = round_up(std::min(A.keep, max_pos_global), 64);
+		if (m->taps > 1) TG_TRY(take(&c.canon, size_t(B) * 2 * (m->taps - 1) * D));
+		if (L.de.H) {
+			TG_TRY(take(&c.conv, size_t(B) * 2 * (L.de.taps - 1) * L.de.channels()));
+			TG_TRY(take(&c.S, size_t(B) * L.de.H * L.de.dk * L.de.dv));
+		}
+		if (L.li.H) {
+			TG_TRY(take(&c.S, size_t(B) * L.li.H * L.li.N * L.li.vdp));
+			if (L.li.kind == LIN_SSM) {
+				TG_TRY(take(&c.conv, size_t(B) * 2 * (L.li.taps - 1) * L.li.channels()));
+			} else {
+				TG_TRY(take(&c.n, size_t(B) * 2 * L.li.H * L.li.N));
+				TG_TRY(take(&c.mx, size_t(B) * 2 * L.li.H));
+			}
+		}
+		if (!A.H) continue;
+		// (a pooled block is formed from the ring, so the ring reaches back a whole block)
+		c.cap = round_up(int(std::min<long long>(max_pos_global, (long long)std::max(A.window, A.pool) + max_seq_rows)), 64);
+		c.keep_rows = round_up(A.pool ? max_pos_global / A.pool : std::min(A.keep, max_pos_global), 64);
 		uint8_t *q;
 		auto rows = [&](void **p, size_t n, int w) -> int {
 			TG_TRY(take(&q, size_t(B) * n * w * es));
@@ -689,13 +428,10 @@ int HybridState::alloc() {
 		TG_TRY(rows(&c.vc, c.cap, A.G * A.dvp));
 		TG_TRY(rows(&c.ks, c.keep_rows, A.G * A.dkp));
 		TG_TRY(rows(&c.vs, c.keep_rows, A.G * A.dvp));
-		TG_TRY(take(&c.canon, size_t(B) * 2 * (m->taps - 1) * D));
-		TG_TRY(take(&c.conv, size_t(B) * 2 * (L.de.taps - 1) * L.de.channels()));
-		TG_TRY(take(&c.S, size_t(B) * L.de.H * L.de.dk * L.de.dv));
 		if (!f32) {
 			TG_TRY(make_map(&c.kmap, c.kc, size_t(B) * c.cap, A.G * A.dkp, A.G * A.dkp, WT_KEYS));
 			TG_TRY(make_map(&c.vmap, c.vc, size_t(B) * c.cap, A.G * A.dvp, A.G * A.dvp, WT_KEYS));
-			c.ksmap = c.kmap;  // (not used without kept tokens)
+			c.ksmap = c.kmap;  // (not used without a second store)
 			c.vsmap = c.vmap;
 			if (c.keep_rows) {
 				TG_TRY(make_map(&c.ksmap, c.ks, size_t(B) * c.keep_rows, A.G * A.dkp, A.G * A.dkp, WT_KEYS));
@@ -713,15 +449,26 @@ int HybridState::alloc() {
 		TG_TRY(make_map(&hmap, h, R, m->Dp, m->Dp, GB_BM));
 		TG_TRY(make_map(&hnmap, hn, std::max(wl_rows, B), m->Dp, m->Dp, GB_BM));
 		const size_t n = m->layers.size();
-		for (auto *v : {&pmap, &omap, &amap, &a1map, &g1map}) v->resize(n);
+		if (beside) TG_TRY(make_map(&hpmap, hp, R, m->Dp, m->Dp, GB_BM));
+		if (experts) TG_TRY(make_map(&xgmap, xg, slots, m->Dp, m->Dp, GB_BM));
+		for (auto *v : {&pmap, &omap, &amap, &a1map, &g1map, &xcmap, &xamap, &shmap, &slmap}) v->resize(n);
 		for (size_t i = 0; i < n; i++) {
 			const Layer &L = m->layers[i];
 			const bf16 *p = static_cast<const bf16 *>(P);
 			TG_TRY(make_map(&pmap[i], P, R, L.ldp, L.ldp, 128));
-			TG_TRY(make_map(&omap[i], O, R, L.kc, L.kc, GB_BM));
-			if (L.ff) TG_TRY(make_map(&amap[i], act, R, L.ffp, L.ffp, GB_BM));
-			TG_TRY(make_map(&a1map[i], p + L.p_a1, R, L.de.ra, L.ldp, GB_BM));
-			TG_TRY(make_map(&g1map[i], p + L.p_g1, R, L.de.rg, L.ldp, GB_BM));
+			TG_TRY(make_map(&omap[i], O, R, L.kcat, L.kcat, GB_BM));
+			if (!L.beside && L.ff.ff) TG_TRY(make_map(&amap[i], act, R, L.ff.ffp, L.ff.ffp, GB_BM));
+			if (L.de.H) {
+				TG_TRY(make_map(&a1map[i], p + L.p_a1, R, L.de.ra, L.ldp, GB_BM));
+				TG_TRY(make_map(&g1map[i], p + L.p_g1, R, L.de.rg, L.ldp, GB_BM));
+			}
+			const LinSpec &li = L.li;
+			if (li.kind == LIN_SSM) TG_TRY(make_map(&xcmap[i], xc, R, li.xc_cols(), li.xc_cols(), LC));
+			if (lin_tc && li.H && li.Np <= 256) {
+				TG_TRY(make_map(&shmap[i], lin.Sh, nchunk * li.H * li.Np, li.vdp, li.vdp, li.Np));
+				TG_TRY(make_map(&slmap[i], lin.Sl, nchunk * li.H * li.Np, li.vdp, li.vdp, li.Np));
+			}
+			if (L.ff.experts) TG_TRY(make_map(&xamap[i], xa, moe_rows(L, R), L.ff.effp, L.ff.effp, GB_BM));
 		}
 	}
 	// descriptors
@@ -798,38 +545,49 @@ int HybridState::trace_read(float *x_host, size_t cap_floats, int *runs, int *to
 }
 
 // ------------------------------------------------------------------ pieces of a step
-int HybridState::gemm(int epi, const void *A, int lda, const CUtensorMap *am, const Lin &w, int M, void *C, int ldc, float cap) {
+int HybridState::gemm(int epi, const void *A, int lda, const CUtensorMap *am, const Lin &w, int M, void *C, int ldc, const GemmOpt &o) {
 	GemmArgs a{};
 	a.M = M;
 	a.N = w.N;
 	a.K = w.K;
 	a.C = C;
 	a.ldc = ldc;
-	a.cap = cap;
+	a.cap = o.cap;
 	a.err = err_flag;
+	a.act = o.act;
+	a.limit = o.limit;
+	a.n32 = o.n32;
+	a.C32 = o.C32;
+	a.ld32 = o.ld32;
+	a.tile_expert = moe.tile_expert;
+	a.n_row_tiles = moe.n_tiles;
 	if (f32) {
 		const float *Af = static_cast<const float *>(A);
 		switch (epi) {
 			case GEMM_ADD: return launch_gemm_f32<GEMM_ADD>(Af, lda, w, a, stream);
-			case GEMM_GEGLU: return launch_gemm_f32<GEMM_GEGLU>(Af, lda, w, a, stream);
+			case GEMM_GLU: return o.grouped ? launch_gemm_f32<GEMM_GLU, true>(Af, lda, w, a, stream) : launch_gemm_f32<GEMM_GLU>(Af, lda, w, a, stream);
 			case GEMM_LOGITS: return launch_gemm_f32<GEMM_LOGITS>(Af, lda, w, a, stream);
-			default: return launch_gemm_f32<GEMM_STORE>(Af, lda, w, a, stream);
+			default: return o.grouped ? launch_gemm_f32<GEMM_STORE, true>(Af, lda, w, a, stream) : launch_gemm_f32<GEMM_STORE>(Af, lda, w, a, stream);
 		}
 	}
+	if (o.grouped) return epi == GEMM_GLU ? launch_gemm<GEMM_GLU, true>(*am, w, a, stream, o.est) : launch_gemm<GEMM_STORE, true>(*am, w, a, stream, o.est);
 	switch (epi) {
 		case GEMM_STORE: return launch_gemm<GEMM_STORE>(*am, w, a, stream);
 		case GEMM_STORE32: return launch_gemm<GEMM_STORE32>(*am, w, a, stream);
 		case GEMM_ADD: return launch_gemm<GEMM_ADD>(*am, w, a, stream);
-		case GEMM_GEGLU: return launch_gemm<GEMM_GEGLU>(*am, w, a, stream);
+		case GEMM_GLU: return launch_gemm<GEMM_GLU>(*am, w, a, stream);
 		default: return launch_gemm<GEMM_LOGITS>(*am, w, a, stream);
 	}
 }
 
 int HybridState::gemv(int pro, int epi, GemvArgs g, int R) {
 	g.err = err_flag;
+	g.rms = m->rms;
+	g.embed_scale = m->embed_scale;
 	// (rows whose activations do not fit shared memory together go in smaller groups)
 	int most = R >= 4 ? 4 : (R >= 2 ? 2 : 1);
-	while (most > 1 && size_t(most) * 8 * gv_k8(g.K) * 4 > 160 * 1024) most /= 2;
+	const size_t row_floats = size_t(epi == GV_FRONT ? 2 : 1) * 8 * gv_k8(g.K) + (pro == GV_MIX ? g.top * g.n_ex : 0);
+	while (most > 1 && most * row_floats * 4 > 160 * 1024) most /= 2;
 	for (int r = 0; r < R;) {
 		int n = most;
 		while (n > R - r) n /= 2;
@@ -839,6 +597,15 @@ int HybridState::gemv(int pro, int epi, GemvArgs g, int R) {
 		if (s.vec) s.vec += size_t(r) * g.ldv;
 		if (s.x) s.x += size_t(r) * g.ldx;
 		s.out += size_t(r) * g.ldo;
+		if (s.out32) s.out32 += size_t(r) * g.ld32;
+		if (s.glu_out) s.glu_out += size_t(r) * g.ld_glu;
+		if (s.route_out) s.route_out += size_t(r) * g.ld_route;
+		if (s.gate) s.gate += size_t(r) * g.ldg;
+		if (s.top) {
+			s.ex_act += size_t(r) * g.top * g.n_ex;
+			s.ex_w += r * g.top;
+			s.ex_id += r * g.top;
+		}
 		if (s.norm_out) s.norm_out += size_t(r) * g.D;
 		TG_TRY(n == 4 ? launch_gemv_r<4>(pro, epi, s, stream) : (n == 2 ? launch_gemv_r<2>(pro, epi, s, stream) : launch_gemv_r<1>(pro, epi, s, stream)));
 		r += n;
@@ -860,6 +627,14 @@ WAttnArgs HybridState::attn_args(const StepDesc &d, int run, const void *p, int 
 	a.scale = L.at.scale;
 	a.window = L.at.window;
 	a.keep = std::min(L.at.keep, c.keep_rows);
+	a.pool = L.at.pool;
+	if (L.at.rot >= 0) {
+		a.rot = L.at.rot_dims;
+		a.cs = cs + size_t(L.at.rot) * max_rows * m->rot_half;
+		a.ld_cs = m->rot_half;
+	}
+	a.vnorm = L.at.vnorm;
+	a.eps = m->eps;
 	a.r1 = L.r1;
 	a.r2 = L.r2;
 	a.p = p;
@@ -867,7 +642,7 @@ WAttnArgs HybridState::attn_args(const StepDesc &d, int run, const void *p, int 
 	a.p_q = L.p_q;
 	a.p_k = L.p_k;
 	a.p_v = L.p_v;
-	a.p_g = L.p_g;
+	a.p_g = L.at.gated ? L.p_g : -1;
 	a.kc = c.kc;
 	a.vc = c.vc;
 	a.ks = c.ks;
@@ -929,6 +704,82 @@ DeltaArgs HybridState::delta_args(const StepDesc &d, int run, const void *p, int
 	return a;
 }
 
+// p: projections of the rows
+LinArgs HybridState::lin_args(const StepDesc &d, int run, const void *p) {
+	const Layer &L = m->layers[m->runs[run].layer];
+	const LinSpec &s = L.li;
+	const RunCache &c = cache[run];
+	LinArgs a = lin;
+	a.d = d;
+	a.kind = s.kind;
+	a.H = s.H;
+	a.G = s.G;
+	a.N = s.N;
+	a.vd = s.vd;
+	a.Np = s.Np;
+	a.vdp = s.vdp;
+	a.p = p;
+	a.ldp = L.ldp;
+	a.p_x = L.p_conv;
+	a.p_q = L.p_q;
+	a.p_k = L.p_k;
+	a.p_v = L.p_v;
+	a.t = T32;
+	a.ldt = L.tail();
+	a.A_log = L.A_log;
+	a.dt_bias = L.dt_bias;
+	a.Dv = L.Dv;
+	a.ib = L.ib;
+	a.fb = L.fb;
+	a.gate_cap = s.gate_cap;
+	a.qscale = s.kind == LIN_MLSTM ? 1.0f / std::sqrt(float(s.N)) : 1.0f;
+	a.cw = L.conv;
+	a.cb = L.conv_b;
+	a.taps = s.taps;
+	a.hist = c.conv;
+	a.xc = xc;
+	a.ldxc = s.xc_cols();
+	if (s.kind == LIN_SSM) {
+		a.rows = xc;
+		a.ldr = a.ldxc;
+		a.o_v = 0;
+		a.o_k = s.H * s.vdp;
+		a.o_q = a.o_k + s.G * s.Np;
+	} else {
+		a.rows = p;
+		a.ldr = L.ldp;
+		a.o_q = L.p_q;
+		a.o_k = L.p_k;
+		a.o_v = L.p_v;
+	}
+	a.S = c.S;
+	a.n = c.n;
+	a.m = c.mx;
+	a.o = o_raw;
+	a.ldo = round_up(s.H * s.vd, 4);
+	a.vsplit = 1;
+	a.err = err_flag;
+	return a;
+}
+
+MoeArgs HybridState::moe_args(const Layer &L) {
+	MoeArgs a = moe;
+	a.z = RL;
+	a.ldz = round_up(L.ff.experts, 8);
+	a.experts = L.ff.experts;
+	a.top = L.ff.top;
+	a.scale = L.ff.route_scale;
+	a.h = h32;
+	a.D = m->D;
+	a.n_glu = L.ff.effp;
+	a.W = L.ex_gu.W;
+	a.ldw = L.ex_gu.ld;
+	a.act = L.ff.act;
+	a.limit = L.ff.limit;
+	a.out = ex32;
+	return a;
+}
+
 namespace {
 template <typename PT, typename CT, typename OT> int launch_token_mix(const WAttnArgs &w, const DeltaArgs &d, int R, cudaStream_t st) {
 	const size_t smem = std::max(wattn_token_smem(w.H / w.G, w.dkp, w.dvp), delta_token_smem(d.dk, d.dv, d.ra, d.rg));
@@ -975,25 +826,99 @@ template <typename PT> int launch_delta(const DeltaArgs &a, int R, int nseg, int
 	count_launch();
 	return check_launch("delta_out");
 }
-template <typename PT> int launch_ln_conv(void *out, int ldo, const float *x, int ldx, float2 *stats, const float *w, const float *cw, float *hist,
-                                          const StepDesc &d, int R, int D, int taps, float eps, cudaStream_t st) {
-	launch_k(ln_stats_kernel, dim3(R), dim3(128), 0, st, stats, x, ldx, D, eps);
+template <typename PT> int launch_stats(float2 *stats, float *x, int ldx, int R, int D, float eps, int rms, const ExpertSum<PT> &add, cudaStream_t st) {
+	launch_k(row_stats_kernel<PT>, dim3(R), dim3(128), 0, st, stats, x, ldx, D, eps, rms, add);
 	count_launch();
-	TG_TRY(check_launch("ln_stats"));
+	return check_launch("row_stats");
+}
+template <typename PT> int launch_norm_conv(void *out, void *plain, int ldo, const float *x, int ldx, const float2 *stats, const float *w, const float *cw, float *hist,
+                                            const StepDesc &d, int R, int D, int taps, cudaStream_t st) {
 	const int cols = (ldo + 511) / 512;
 	int rows = LC_ROWS;
 	while (rows > 1 && (R + rows - 1) / rows * cols < 4 * g_num_sms) rows /= 2;
 	const dim3 grid((R + rows - 1) / rows, cols);
-	if (taps <= 4) launch_k(ln_conv_kernel<PT, 4>, grid, dim3(128), 0, st, static_cast<PT *>(out), ldo, x, ldx, stats, w, cw, hist, d, R, D, taps, rows);
-	else launch_k(ln_conv_kernel<PT, 16>, grid, dim3(128), 0, st, static_cast<PT *>(out), ldo, x, ldx, stats, w, cw, hist, d, R, D, taps, rows);
+	PT *o = static_cast<PT *>(out), *p = static_cast<PT *>(plain);
+	if (taps <= 2) launch_k(norm_conv_kernel<PT, 2>, grid, dim3(128), 0, st, o, p, ldo, x, ldx, stats, w, cw, hist, d, R, D, taps, rows);
+	else if (taps <= 4) launch_k(norm_conv_kernel<PT, 4>, grid, dim3(128), 0, st, o, p, ldo, x, ldx, stats, w, cw, hist, d, R, D, taps, rows);
+	else launch_k(norm_conv_kernel<PT, 16>, grid, dim3(128), 0, st, o, p, ldo, x, ldx, stats, w, cw, hist, d, R, D, taps, rows);
 	count_launch();
-	return check_launch("ln_conv");
+	return check_launch("norm_conv");
 }
-template <typename PT> int launch_ln(void *out, int ldo, const float *x, int ldx, const float *w, const int *rows, int n, int D, float eps, float *out32,
-                                     cudaStream_t st) {
-	launch_k(layer_norm_kernel<PT>, dim3(n), dim3(128), 0, st, static_cast<PT *>(out), ldo, x, ldx, w, rows, n, D, eps, out32);
+template <typename PT> int launch_norm(void *out, int ldo, const float *x, int ldx, const float *w, const int *rows, int n, int D, float eps, int rms, float *out32,
+                                       cudaStream_t st) {
+	launch_k(row_norm_kernel<PT>, dim3(n), dim3(128), 0, st, static_cast<PT *>(out), ldo, x, ldx, w, rows, n, D, eps, rms, out32);
 	count_launch();
-	return check_launch("layer_norm");
+	return check_launch("row_norm");
+}
+// n_exp: CTAs per row of its chosen experts (0: the step's experts are grouped products)
+template <typename PT, typename CT, typename OT> int launch_beside_mix(const WAttnArgs *w, const LinArgs *l, const MoeArgs &e, int n_exp, int R, cudaStream_t st) {
+	const size_t ex = n_exp ? expert_token_smem(e.D) : 0;
+	const int n_mix = w ? w->G * w->nsplit : lin_token_ctas(l->H, l->vd);
+	const size_t smem = std::max(ex, w ? wattn_token_smem(w->H / w->G, w->dkp, w->dvp) : lin_token_smem(l->Np));
+	const dim3 grid(n_mix + n_exp, R);
+	const WAttnArgs wa = w ? *w : WAttnArgs{};
+	const LinArgs la = l ? *l : LinArgs{};
+	if (w) {
+		auto kernel = beside_token_mix_kernel<PT, CT, OT, true>;
+		TG_TRY(allow_smem(kernel, smem));
+		launch_k(kernel, grid, dim3(256), smem, st, wa, la, e, n_mix);
+	} else {
+		auto kernel = beside_token_mix_kernel<PT, CT, OT, false>;
+		TG_TRY(allow_smem(kernel, smem));
+		launch_k(kernel, grid, dim3(256), smem, st, wa, la, e, n_mix);
+	}
+	count_launch();
+	return check_launch("beside_token_mix");
+}
+// portions of a recurrence: raw read-outs of all rows
+template <typename PT> int launch_lin_rows(const LinArgs &a, int R, int nseg, int max_len, cudaStream_t st) {
+	if (a.kind == LIN_SSM) {
+		const dim3 grid((R + LV_ROWS - 1) / LV_ROWS, (a.ldxc + 127) / 128);
+		if (a.taps <= 4) launch_k(lin_conv_kernel<PT, 4>, grid, dim3(128), 0, st, a, R);
+		else launch_k(lin_conv_kernel<PT, 16>, grid, dim3(128), 0, st, a, R);
+		count_launch();
+		TG_TRY(check_launch("lin_conv"));
+	}
+	launch_k(lin_gates_kernel, dim3(a.H, nseg), dim3(256), 0, st, a);
+	count_launch();
+	return check_launch("lin_gates");
+}
+template <typename PT> int launch_lin_scan(const LinArgs &a, int nseg, cudaStream_t st) {
+	const dim3 grid((a.vd + LT_COLS - 1) / LT_COLS, a.H, nseg);
+	if (a.N <= 128) launch_k(lin_scan_kernel<PT, 4>, grid, dim3(256), 0, st, a);
+	else if (a.N <= 256) launch_k(lin_scan_kernel<PT, 8>, grid, dim3(256), 0, st, a);
+	else launch_k(lin_scan_kernel<PT, 16>, grid, dim3(256), 0, st, a);
+	count_launch();
+	return check_launch("lin_scan");
+}
+int launch_lin_chunks(LinArgs a, const CUtensorMap &rows, const CUtensorMap &sh, const CUtensorMap &sl, int nseg, int max_len, cudaStream_t st) {
+	const int chunks = (max_len + LC - 1) / LC, tiles = (a.vdp + 63) / 64;
+	TG_TRY(allow_smem(lin_chunk_state_kernel, lin_state_smem(a.Np)));
+	launch_k(lin_chunk_state_kernel, dim3(chunks, a.H * tiles, nseg), dim3(256), lin_state_smem(a.Np), st, rows, a);
+	count_launch();
+	TG_TRY(check_launch("lin_chunk_state"));
+	const int items = a.H * a.N * (a.vdp / 4) + (a.kind == LIN_MLSTM ? a.H * a.N : 0);
+	launch_k(lin_chunk_scan_kernel, dim3((items + 255) / 256, nseg), dim3(256), 0, st, a);
+	count_launch();
+	TG_TRY(check_launch("lin_chunk_scan"));
+	// (few chunks: more CTAs share a head's columns, each forming the weights again)
+	a.vsplit = std::max(1, std::min(tiles, g_num_sms / std::max(1, chunks * a.H * nseg)));
+	TG_TRY(allow_smem(lin_chunk_out_kernel, lin_out_smem(a.Np)));
+	launch_k(lin_chunk_out_kernel, dim3(chunks, a.H * a.vsplit, nseg), dim3(256), lin_out_smem(a.Np), st, rows, sh, sl, a);
+	count_launch();
+	return check_launch("lin_chunk_out");
+}
+template <typename T> int launch_lin_norm(const LinArgs &a, const Layer &L, void *O, const void *P, int R, float eps, cudaStream_t st) {
+	const int n = a.H * a.vd;
+	launch_k(lin_norm_kernel<T>, dim3((R * L.li.parts + 7) / 8), dim3(256), 0, st, static_cast<T *>(O), L.kcat, a.o, a.ldo, static_cast<const T *>(P) + L.p_z, L.ldp, L.rnorm, R, n,
+	         L.li.parts, a.kind == LIN_SSM ? 1 : 0, eps);
+	count_launch();
+	return check_launch("lin_norm");
+}
+template <typename T> int launch_gather(const MoeArgs &a, const void *h, int ldh, void *xg, int R, cudaStream_t st) {
+	launch_k(expert_gather_kernel<T>, dim3((R + MG_ROWS - 1) / MG_ROWS), dim3(128), 0, st, a, static_cast<const T *>(h), ldh, static_cast<T *>(xg), R);
+	count_launch();
+	return check_launch("expert_gather");
 }
 // portions on CUDA cores
 template <typename PT> int launch_attn_simt(const WAttnArgs &a, int R, cudaStream_t st) {
@@ -1005,117 +930,355 @@ template <typename PT> int launch_attn_simt(const WAttnArgs &a, int R, cudaStrea
 }
 }  // namespace
 
+// attention of a portion, its keys and values being in the cache
+int HybridState::attn_rows(const WAttnArgs &wa, int run, int R, int nseg, int max_len) {
+	const int li = m->runs[run].layer;
+	const RunCache &c = cache[run];
+	static const int use_tc = env_int("TG_WATTN_TC", 1);
+	if (!f32 && use_tc && wa.dkp <= 256 && wa.dvp <= 256) {
+		const WtShape sh = wt_shape(wa.dkp, wa.dvp, wa.window, wa.r1 != nullptr);
+		TG_TRY(allow_smem(window_attn_tc_kernel, sh.total));
+		launch_k(window_attn_tc_kernel, dim3((max_len + 127) / 128, wa.H, nseg), dim3(WT_THREADS), size_t(sh.total), stream, pmap[li], c.kmap, c.vmap,
+		         c.ksmap, c.vsmap, wa);
+		count_launch();
+		TG_TRY(check_launch("window_attn_tc"));
+	} else {
+		if (f32) TG_TRY(launch_attn_simt<float>(wa, R, stream));
+		else TG_TRY(launch_attn_simt<bf16>(wa, R, stream));
+	}
+	return TG_OK;
+}
+
+// how many CTAs share the keys of a (sequence, key/value head) in a step of one token per sequence
+int HybridState::token_splits(const WAttnArgs &wa, int fill) const {
+	const long long second = wa.pool ? max_pos_global / wa.pool : wa.keep, keys = std::min<long long>(wa.window + second, max_pos_global);
+	return int(std::max<long long>(1, std::min<long long>(std::min(nsplit_cap, fill), (keys + WK_KEYS - 1) / WK_KEYS)));
+}
+
+// ---- feed-forward after the mixer
+int HybridState::few_layer(const StepDesc &d, int run, int R) {
+	const Layer &L = m->layers[m->runs[run].layer];
+	const RunCache &c = cache[run];
+	const int D = m->D;
+	GemvArgs g{};
+	g.d = d;
+	g.x = x;
+	g.ldx = ldx;
+	g.D = D;
+	g.embed = m->embed.W;
+	g.lde = m->embed.ld;
+	g.V = m->n_vocab;
+	g.eps = m->eps;
+	g.cw = L.canon;
+	g.hist = c.canon;
+	g.taps = m->taps;
+	g.act = L.ff.act;
+	g.limit = L.ff.limit;
+	const int embed_mode = run == 0 ? 1 : (m->runs[run].add_embed ? 2 : 0);
+	auto product = [&](int pro, int epi, const Lin &w, const float *norm, const float *vec, int ldv, float *out, int ldo, int em) -> int {
+		GemvArgs s = g;
+		s.W = w.W;
+		s.ldw = w.ld;
+		s.N = w.N;
+		s.K = w.K;
+		s.w = norm;
+		s.vec = vec;
+		s.ldv = ldv;
+		s.out = out;
+		s.ldo = ldo;
+		s.embed_mode = em;
+		if (epi == GV_PROJ) {
+			s.p_k = L.p_k;
+			s.n_k = L.at.G * L.at.dkp;
+			s.p_v = L.p_v;
+			s.n_v = L.at.G * L.at.dvp;
+			s.kc = c.kc;
+			s.vc = c.vc;
+			s.ks = c.ks;
+			s.vs = c.vs;
+			s.cap_rows = c.cap;
+			s.keep = std::min(L.at.keep, c.keep_rows);
+			s.keep_rows = c.keep_rows;
+			s.cache_f32 = f32;
+		}
+		return gemv(pro, epi, s, R);
+	};
+	TG_TRY(product(GV_LN_CONV, GV_PROJ, L.proj, L.norm1, nullptr, 0, P32, L.ldp, embed_mode));
+	WAttnArgs wa = attn_args(d, run, P32, L.ldp, O32, L.kc);
+	const DeltaArgs da = delta_args(d, run, P32, L.ldp, O32, L.kc);
+	wa.nsplit = token_splits(wa, nsplit_cap);
+	if (f32) TG_TRY((launch_token_mix<float, float, float>(wa, da, R, stream)));
+	else TG_TRY((launch_token_mix<float, bf16, float>(wa, da, R, stream)));
+	TG_TRY(product(GV_VEC, GV_ADD, L.out, nullptr, O32, L.kc, x, ldx, embed_mode));
+	if (L.ff.ff) {
+		TG_TRY(product(GV_LN, GV_GLU, L.gu, L.norm2, nullptr, 0, act32, L.ff.ffp, 0));
+		TG_TRY(product(GV_VEC, GV_ADD, L.down, nullptr, act32, L.ff.ffp, x, ldx, 0));
+	}
+	return TG_OK;
+}
+
+int HybridState::rows_layer(const StepDesc &d, int run, int R, int nseg, int max_len) {
+	const int li = m->runs[run].layer, D = m->D;
+	const Layer &L = m->layers[li];
+	const bool single = max_len == 1;
+	TG_TRY(norm_in(d, run, R, -1));
+	TG_TRY(gemm(GEMM_STORE, h, m->Dp, &hmap, L.proj, R, P, L.ldp));
+	WAttnArgs wa = attn_args(d, run, P, L.ldp, O, L.kc);
+	const DeltaArgs da = delta_args(d, run, P, L.ldp, O, L.kc);
+	if (f32) launch_k(kv_append_kernel<float, float>, dim3(R), dim3(256), 0, stream, wa);
+	else launch_k(kv_append_kernel<bf16, bf16>, dim3(R), dim3(256), 0, stream, wa);
+	count_launch();
+	TG_TRY(check_launch("kv_append"));
+	if (single) {
+		wa.nsplit = token_splits(wa, std::max(1, 2 * g_num_sms / std::max(1, R * wa.G)));
+		if (f32) TG_TRY((launch_token_mix<float, float, float>(wa, da, R, stream)));
+		else TG_TRY((launch_token_mix<bf16, bf16, bf16>(wa, da, R, stream)));
+	} else {
+		TG_TRY(attn_rows(wa, run, R, nseg, max_len));
+		const size_t esz = f32 ? 4 : 2;
+		const uint8_t *pb = static_cast<const uint8_t *>(P);
+		TG_TRY(gemm(GEMM_STORE32, pb + size_t(L.p_a1) * esz, L.ldp, f32 ? nullptr : &a1map[li], L.a2, R, z, da.ldz));
+		TG_TRY(gemm(GEMM_STORE32, pb + size_t(L.p_g1) * esz, L.ldp, f32 ? nullptr : &g1map[li], L.g2, R, gz, da.ldgz));
+		if (f32) TG_TRY(launch_delta<float>(da, R, nseg, max_len, stream));
+		else TG_TRY(launch_delta<bf16>(da, R, nseg, max_len, stream));
+	}
+	TG_TRY(gemm(GEMM_ADD, O, L.kc, f32 ? nullptr : &omap[li], L.out, R, x, ldx));
+	if (L.ff.ff) {
+		if (f32) TG_TRY(launch_norm<float>(h, m->Dp, x, ldx, L.norm2, nullptr, R, D, m->eps, m->rms, nullptr, stream));
+		else TG_TRY(launch_norm<bf16>(h, m->Dp, x, ldx, L.norm2, nullptr, R, D, m->eps, m->rms, nullptr, stream));
+		GemmOpt glu_opt;
+		glu_opt.act = L.ff.act;
+		glu_opt.limit = L.ff.limit;
+		TG_TRY(gemm(GEMM_GLU, h, m->Dp, &hmap, L.gu, R, act, L.ff.ffp, glu_opt));
+		TG_TRY(gemm(GEMM_ADD, act, L.ff.ffp, f32 ? nullptr : &amap[li], L.down, R, x, ldx));
+	}
+	return TG_OK;
+}
+
+// ---- feed-forward beside the mixer
+int HybridState::beside_few_layer(const StepDesc &d, int run, int R) {
+	const Layer &L = m->layers[m->runs[run].layer];
+	const RunCache &c = cache[run];
+	const FfSpec &F = L.ff;
+	const bool lin_mix = L.li.H > 0;
+	GemvArgs g{};
+	g.d = d;
+	g.x = x;
+	g.ldx = ldx;
+	g.D = m->D;
+	g.embed = m->embed.W;
+	g.lde = m->embed.ld;
+	g.V = m->n_vocab;
+	g.eps = m->eps;
+	g.embed_mode = run == 0 ? 1 : 0;
+	g.act = F.act;
+	g.limit = F.limit;
+	GemvArgs f = g;
+	f.W = L.front.W;
+	f.ldw = L.front.ld;
+	f.N = L.front.N;
+	f.K = L.front.K;
+	f.w = L.norm1;
+	f.cw = L.canon;
+	f.hist = c.canon;
+	f.taps = m->taps;
+	f.out = P32;
+	f.ldo = L.ldp;
+	f.n_proj = L.proj.N;
+	f.n32 = L.n32;
+	f.out32 = T32;
+	f.ld32 = L.tail();
+	f.n_glu = F.ffp;
+	f.glu_out = O32 + L.kc;
+	f.ld_glu = L.kcat;
+	f.n_route = F.experts;
+	f.route_out = RL;
+	f.ld_route = round_up(F.experts, 8);
+	f.norm_out = F.experts ? h32 : nullptr;
+	TG_TRY(gemv(GV_LN_CONV, GV_FRONT, f, R));
+	const MoeArgs ma = moe_args(L);
+	const int n_exp = F.experts ? expert_token_ctas(F.top, F.effp) : 0;
+	if (lin_mix) {
+		LinArgs la = lin_args(d, run, P32);
+		la.o = O32;
+		la.ldo = L.kcat;
+		TG_TRY((launch_beside_mix<float, float, float>(nullptr, &la, ma, n_exp, R, stream)));
+	} else {
+		WAttnArgs wa = attn_args(d, run, P32, L.ldp, O32, L.kcat);
+		wa.append = 1;
+		wa.nsplit = token_splits(wa, nsplit_cap);
+		if (f32) TG_TRY((launch_beside_mix<float, float, float>(&wa, nullptr, ma, n_exp, R, stream)));
+		else TG_TRY((launch_beside_mix<float, bf16, float>(&wa, nullptr, ma, n_exp, R, stream)));
+	}
+	GemvArgs o = g;
+	o.W = L.out.W;
+	o.ldw = L.out.ld;
+	o.N = L.out.N;
+	o.K = L.out.K;
+	o.vec = O32;
+	o.ldv = L.kcat;
+	o.out = x;
+	o.ldo = ldx;
+	o.w = L.rnorm;
+	if (lin_mix) {
+		o.mix_norm = L.li.kind == LIN_SSM ? MIX_GATE_NORM : MIX_NORM_GATE;
+		o.mix_n = L.li.H * L.li.vd;
+		o.parts = L.li.parts;
+		o.gate = P32 + L.p_z;
+		o.ldg = L.ldp;
+	}
+	if (F.experts) {
+		o.top = F.top;
+		o.n_ex = F.effp;
+		o.ex_act = ex32;
+		o.ex_w = moe.w;
+		o.ex_id = moe.id;
+		o.ex_W = L.ex_down.W;
+		o.ld_ex = L.ex_down.ld;
+	}
+	return gemv(GV_MIX, GV_ADD, o, R);
+}
+
+int HybridState::beside_rows_layer(const StepDesc &d, int run, int R, int nseg, int max_len, int pending) {
+	const int li = m->runs[run].layer;
+	const Layer &L = m->layers[li];
+	const FfSpec &F = L.ff;
+	const bool single = max_len == 1;
+	TG_TRY(norm_in(d, run, R, pending));
+	GemmOpt po;
+	po.n32 = L.n32;
+	po.ld32 = L.tail();
+	po.C32 = L.tail() ? T32 : nullptr;
+	TG_TRY(gemm(GEMM_STORE, h, m->Dp, &hmap, L.proj, R, P, L.ldp, po));
+	if (L.at.H) {
+		WAttnArgs wa = attn_args(d, run, P, L.ldp, O, L.kcat);
+		if (single) {
+			wa.append = 1;
+			wa.nsplit = token_splits(wa, std::max(1, 2 * g_num_sms / std::max(1, R * wa.G)));
+			if (f32) TG_TRY((launch_beside_mix<float, float, float>(&wa, nullptr, MoeArgs{}, 0, R, stream)));
+			else TG_TRY((launch_beside_mix<bf16, bf16, bf16>(&wa, nullptr, MoeArgs{}, 0, R, stream)));
+		} else {
+			const int unit = wa.pool ? wa.pool * std::max(1, 16 / wa.pool) : 16;
+			const dim3 grid((max_len + unit - 1) / unit + 1, wa.G, nseg);
+			if (f32) launch_k(kv_transform_kernel<float, float>, grid, dim3(256), 0, stream, wa, unit);
+			else launch_k(kv_transform_kernel<bf16, bf16>, grid, dim3(256), 0, stream, wa, unit);
+			count_launch();
+			TG_TRY(check_launch("kv_transform"));
+			TG_TRY(attn_rows(wa, run, R, nseg, max_len));
+		}
+	} else {
+		const LinArgs la = lin_args(d, run, P);
+		if (single) {
+			if (f32) TG_TRY((launch_beside_mix<float, float, float>(nullptr, &la, MoeArgs{}, 0, R, stream)));
+			else TG_TRY((launch_beside_mix<bf16, bf16, bf16>(nullptr, &la, MoeArgs{}, 0, R, stream)));
+		} else {
+			if (f32) TG_TRY(launch_lin_rows<float>(la, R, nseg, max_len, stream));
+			else TG_TRY(launch_lin_rows<bf16>(la, R, nseg, max_len, stream));
+			if (lin_tc && la.Np <= 256 && max_len > LIN_SCAN_MAX)
+				TG_TRY(launch_lin_chunks(la, la.kind == LIN_SSM ? xcmap[li] : pmap[li], shmap[li], slmap[li], nseg, max_len, stream));
+			else if (f32) TG_TRY(launch_lin_scan<float>(la, nseg, stream));
+			else TG_TRY(launch_lin_scan<bf16>(la, nseg, stream));
+		}
+		if (f32) TG_TRY(launch_lin_norm<float>(la, L, O, P, R, m->eps, stream));
+		else TG_TRY(launch_lin_norm<bf16>(la, L, O, P, R, m->eps, stream));
+	}
+	if (F.any()) {
+		GemmOpt go;
+		go.act = F.act;
+		go.limit = F.limit;
+		go.n32 = 2 * F.ffp;
+		go.C32 = F.experts ? RL : nullptr;
+		go.ld32 = round_up(F.experts, 8);
+		uint8_t *dst = static_cast<uint8_t *>(O) + size_t(L.kc) * (f32 ? 4 : 2);
+		TG_TRY(gemm(GEMM_GLU, hp, m->Dp, &hpmap, L.gu, R, dst, L.kcat, go));
+	}
+	if (F.experts) {
+		const MoeArgs ma = moe_args(L);
+		launch_k(route_kernel, dim3((R + 7) / 8), dim3(256), 0, stream, ma, R);
+		count_launch();
+		TG_TRY(check_launch("route"));
+		if (f32) TG_TRY(launch_gather<float>(ma, hp, m->Dp, xg, R, stream));
+		else TG_TRY(launch_gather<bf16>(ma, hp, m->Dp, xg, R, stream));
+		GemmOpt eo;
+		eo.act = F.act;
+		eo.limit = F.limit;
+		eo.grouped = true;
+		const int most = moe_rows(L, R);
+		eo.est = std::max(1, R * F.top / GB_BM + std::min(F.experts, R * F.top) / 2);
+		TG_TRY(gemm(GEMM_GLU, xg, m->Dp, &xgmap, L.ex_gu, most, xa, F.effp, eo));
+		TG_TRY(gemm(GEMM_STORE, xa, F.effp, f32 ? nullptr : &xamap[li], L.ex_down, most, xy, ldx, eo));
+	}
+	return gemm(GEMM_ADD, O, L.kcat, f32 ? nullptr : &omap[li], L.out, R, x, ldx);
+}
+
+int HybridState::norm_in(const StepDesc &d, int run, int R, int pending) {
+	const Layer &L = m->layers[m->runs[run].layer];
+	float *hist = cache[run].canon;
+	void *plain = L.beside ? hp : nullptr;
+	auto go = [&](auto t) -> int {
+		typedef decltype(t) T;
+		ExpertSum<T> add{};
+		if (pending >= 0) {
+			add.y = static_cast<const T *>(xy);
+			add.ldy = ldx;
+			add.top = m->layers[pending].ff.top;
+			add.slot = moe.place;
+			add.w = moe.w;
+		}
+		if (L.ff.experts) {
+			add.zero = moe.count;
+			add.n_zero = L.ff.experts;
+		}
+		TG_TRY(launch_stats<T>(stats, x, ldx, R, m->D, m->eps, m->rms, add, stream));
+		return launch_norm_conv<T>(h, plain, m->Dp, x, ldx, stats, L.norm1, L.canon, hist, d, R, m->D, m->taps, stream);
+	};
+	return f32 ? go(0.0f) : go(bf16());
+}
+
+// adds the outputs of a layer's experts to the stream (where no norm follows that would do it)
+int HybridState::add_experts(int layer, int R) {
+	auto go = [&](auto t) -> int {
+		typedef decltype(t) T;
+		ExpertSum<T> add{};
+		add.y = static_cast<const T *>(xy);
+		add.ldy = ldx;
+		add.top = m->layers[layer].ff.top;
+		add.slot = moe.place;
+		add.w = moe.w;
+		return launch_stats<T>(stats, x, ldx, R, m->D, m->eps, m->rms, add, stream);
+	};
+	return f32 ? go(0.0f) : go(bf16());
+}
+
 // All layers for R rows in nseg segments (the longest: max_len), leaving the residual stream in x.
 int HybridState::run_layers(const StepDesc &d, int R, int nseg, int max_len) {
-	const bool single = max_len == 1, few = single && R <= FEW_ROWS;
+	const bool few = max_len == 1 && R <= FEW_ROWS;
 	const int D = m->D;
 	auto embed_rows = [&](int add) -> int {
-		launch_k(embed_rows_kernel, dim3(R), dim3(256), 0, stream, x, ldx, m->embed.W, m->embed.ld, d, D, m->n_vocab, add, err_flag);
+		launch_k(embed_rows_kernel, dim3(R), dim3(256), 0, stream, x, ldx, m->embed.W, m->embed.ld, m->embed_scale, d, D, m->n_vocab, add, err_flag);
 		count_launch();
 		return check_launch("embed_rows");
 	};
 	if (!few) TG_TRY(embed_rows(0));
+	if (!m->rots.empty()) {
+		RopeTable t{m->rot_freq, m->rot_factor, cs, max_rows, m->rot_half};
+		launch_k(rope_table_kernel, dim3(R, int(m->rots.size())), dim3(128), 0, stream, t, d);
+		count_launch();
+		TG_TRY(check_launch("rope_table"));
+	}
+	int pending = -1;  // the layer whose experts' outputs are not in x yet
 	for (size_t run = 0; run < m->runs.size(); run++) {
 		const Layer &L = m->layers[m->runs[run].layer];
-		const int li = m->runs[run].layer;
-		const RunCache &c = cache[run];
 		if (few) {
-			GemvArgs g{};
-			g.d = d;
-			g.x = x;
-			g.ldx = ldx;
-			g.D = D;
-			g.embed = m->embed.W;
-			g.lde = m->embed.ld;
-			g.V = m->n_vocab;
-			g.eps = m->eps;
-			g.cw = L.canon;
-			g.hist = c.canon;
-			g.taps = m->taps;
-			const int embed_mode = run == 0 ? 1 : (m->runs[run].add_embed ? 2 : 0);
-			auto product = [&](int pro, int epi, const Lin &w, const float *norm, const float *vec, int ldv, float *out, int ldo, int em) -> int {
-				GemvArgs s = g;
-				s.W = w.W;
-				s.ldw = w.ld;
-				s.N = w.N;
-				s.K = w.K;
-				s.w = norm;
-				s.vec = vec;
-				s.ldv = ldv;
-				s.out = out;
-				s.ldo = ldo;
-				s.embed_mode = em;
-				if (epi == GV_PROJ) {
-					s.p_k = L.p_k;
-					s.n_k = L.at.G * L.at.dkp;
-					s.p_v = L.p_v;
-					s.n_v = L.at.G * L.at.dvp;
-					s.kc = c.kc;
-					s.vc = c.vc;
-					s.ks = c.ks;
-					s.vs = c.vs;
-					s.cap_rows = c.cap;
-					s.keep = std::min(L.at.keep, c.keep_rows);
-					s.keep_rows = c.keep_rows;
-					s.cache_f32 = f32;
-				}
-				return gemv(pro, epi, s, R);
-			};
-			TG_TRY(product(GV_LN_CONV, GV_PROJ, L.proj, L.norm1, nullptr, 0, P32, L.ldp, embed_mode));
-			WAttnArgs wa = attn_args(d, int(run), P32, L.ldp, O32, L.kc);
-			const DeltaArgs da = delta_args(d, int(run), P32, L.ldp, O32, L.kc);
-			const long long keys = std::min<long long>((long long)wa.window + wa.keep, max_pos_global);
-			wa.nsplit = int(std::max<long long>(1, std::min<long long>(nsplit_cap, (keys + WK_KEYS - 1) / WK_KEYS)));
-			if (f32) TG_TRY((launch_token_mix<float, float, float>(wa, da, R, stream)));
-			else TG_TRY((launch_token_mix<float, bf16, float>(wa, da, R, stream)));
-			TG_TRY(product(GV_VEC, GV_ADD, L.out, nullptr, O32, L.kc, x, ldx, embed_mode));
-			if (L.ff) {
-				TG_TRY(product(GV_LN, GV_GEGLU, L.gu, L.norm2, nullptr, 0, act32, L.ffp, 0));
-				TG_TRY(product(GV_VEC, GV_ADD, L.down, nullptr, act32, L.ffp, x, ldx, 0));
-			}
+			TG_TRY(L.beside ? beside_few_layer(d, int(run), R) : few_layer(d, int(run), R));
 		} else {
 			if (m->runs[run].add_embed) TG_TRY(embed_rows(1));
-			if (f32) TG_TRY(launch_ln_conv<float>(h, m->Dp, x, ldx, stats, L.norm1, L.canon, c.canon, d, R, D, m->taps, m->eps, stream));
-			else TG_TRY(launch_ln_conv<bf16>(h, m->Dp, x, ldx, stats, L.norm1, L.canon, c.canon, d, R, D, m->taps, m->eps, stream));
-			TG_TRY(gemm(GEMM_STORE, h, m->Dp, &hmap, L.proj, R, P, L.ldp));
-			WAttnArgs wa = attn_args(d, int(run), P, L.ldp, O, L.kc);
-			const DeltaArgs da = delta_args(d, int(run), P, L.ldp, O, L.kc);
-			if (f32) launch_k(kv_append_kernel<float, float>, dim3(R), dim3(256), 0, stream, wa);
-			else launch_k(kv_append_kernel<bf16, bf16>, dim3(R), dim3(256), 0, stream, wa);
-			count_launch();
-			TG_TRY(check_launch("kv_append"));
-			if (single) {
-				const long long keys = std::min<long long>((long long)wa.window + wa.keep, max_pos_global);
-				const int fill = std::max(1, 2 * g_num_sms / std::max(1, R * wa.G));
-				wa.nsplit = int(std::max<long long>(1, std::min<long long>(std::min(nsplit_cap, fill), (keys + WK_KEYS - 1) / WK_KEYS)));
-				if (f32) TG_TRY((launch_token_mix<float, float, float>(wa, da, R, stream)));
-				else TG_TRY((launch_token_mix<bf16, bf16, bf16>(wa, da, R, stream)));
-			} else {
-				static const int use_tc = env_int("TG_WATTN_TC", 1);
-				if (!f32 && use_tc && wa.dkp <= 256 && wa.dvp <= 256) {
-					const WtShape sh = wt_shape(wa.dkp, wa.dvp, wa.window);
-					TG_TRY(allow_smem(window_attn_tc_kernel, sh.total));
-					launch_k(window_attn_tc_kernel, dim3((max_len + 127) / 128, wa.H, nseg), dim3(WT_THREADS), size_t(sh.total), stream, pmap[li], c.kmap, c.vmap,
-					         c.ksmap, c.vsmap, wa);
-					count_launch();
-					TG_TRY(check_launch("window_attn_tc"));
-				} else {
-					if (f32) TG_TRY(launch_attn_simt<float>(wa, R, stream));
-					else TG_TRY(launch_attn_simt<bf16>(wa, R, stream));
-				}
-				const size_t esz = f32 ? 4 : 2;
-				const uint8_t *pb = static_cast<const uint8_t *>(P);
-				TG_TRY(gemm(GEMM_STORE32, pb + size_t(L.p_a1) * esz, L.ldp, f32 ? nullptr : &a1map[li], L.a2, R, z, da.ldz));
-				TG_TRY(gemm(GEMM_STORE32, pb + size_t(L.p_g1) * esz, L.ldp, f32 ? nullptr : &g1map[li], L.g2, R, gz, da.ldgz));
-				if (f32) TG_TRY(launch_delta<float>(da, R, nseg, max_len, stream));
-				else TG_TRY(launch_delta<bf16>(da, R, nseg, max_len, stream));
-			}
-			TG_TRY(gemm(GEMM_ADD, O, L.kc, f32 ? nullptr : &omap[li], L.out, R, x, ldx));
-			if (L.ff) {
-				if (f32) TG_TRY(launch_ln<float>(h, m->Dp, x, ldx, L.norm2, nullptr, R, D, m->eps, nullptr, stream));
-				else TG_TRY(launch_ln<bf16>(h, m->Dp, x, ldx, L.norm2, nullptr, R, D, m->eps, nullptr, stream));
-				TG_TRY(gemm(GEMM_GEGLU, h, m->Dp, &hmap, L.gu, R, act, L.ffp));
-				TG_TRY(gemm(GEMM_ADD, act, L.ffp, f32 ? nullptr : &amap[li], L.down, R, x, ldx));
+			if (L.beside) TG_TRY(beside_rows_layer(d, int(run), R, nseg, max_len, pending));
+			else TG_TRY(rows_layer(d, int(run), R, nseg, max_len));
+			pending = L.beside && L.ff.experts ? m->runs[run].layer : -1;
+			if (pending >= 0 && (tracing || run + 1 == m->runs.size())) {
+				TG_TRY(add_experts(pending, R));
+				pending = -1;
 			}
 		}
 		if (tracing) {
@@ -1130,9 +1293,11 @@ int HybridState::run_layers(const StepDesc &d, int R, int nseg, int max_len) {
 
 // logits of n rows of x (rows_dev: which; null: 0 .. n-1) -> out [n][ld_logits]
 int HybridState::score_rows(const int *rows_dev, int n, float *out, float *norm_out) {
-	if (f32) TG_TRY(launch_ln<float>(hn, m->Dp, x, ldx, m->final_norm, rows_dev, n, m->D, m->eps, norm_out, stream));
-	else TG_TRY(launch_ln<bf16>(hn, m->Dp, x, ldx, m->final_norm, rows_dev, n, m->D, m->eps, norm_out, stream));
-	return gemm(GEMM_LOGITS, hn, m->Dp, &hnmap, m->embed, n, out, ld_logits, m->softcap);
+	if (f32) TG_TRY(launch_norm<float>(hn, m->Dp, x, ldx, m->final_norm, rows_dev, n, m->D, m->eps, m->rms, norm_out, stream));
+	else TG_TRY(launch_norm<bf16>(hn, m->Dp, x, ldx, m->final_norm, rows_dev, n, m->D, m->eps, m->rms, norm_out, stream));
+	GemmOpt o;
+	o.cap = m->softcap;
+	return gemm(GEMM_LOGITS, hn, m->Dp, &hnmap, m->head, n, out, ld_logits, o);
 }
 
 // ------------------------------------------------------------------ lock-step decoding
@@ -1145,10 +1310,10 @@ int HybridState::enqueue_decode_all() {
 		g.x = x;
 		g.ldx = ldx;
 		g.D = m->D;
-		g.W = m->embed.W;
-		g.ldw = m->embed.ld;
-		g.N = m->embed.N;
-		g.K = m->embed.K;
+		g.W = m->head.W;
+		g.ldw = m->head.ld;
+		g.N = m->head.N;
+		g.K = m->head.K;
 		g.w = m->final_norm;
 		g.eps = m->eps;
 		g.taps = 1;
