@@ -42,6 +42,8 @@ Other modes (one JSON line each, 1 GPU):
     python bench.py --nabelix [--model 270m|1B|3B] [--no-extras]
                                                 prefill and decode throughput of the Nabelix design (bf16, random
                                                 weights) beside int8 Gemma-3 of the same width, depth and vocabulary
+    python bench.py --sominex [--model 270m|1B|3B] [--no-extras]
+                                                the same for the Sominex design, beside Nabelix
 """
 
 from __future__ import annotations
@@ -817,7 +819,7 @@ def run_phase_clocks(args):
     return 0
 
 
-# ------------------------------------------------------------------ Nabelix
+# ------------------------------------------------------------------ layered designs
 def nabelix_work(cfg):
     """per layer-run sums: bf16 weight bytes, matrix-product FLOPs per token, attention FLOPs per (query, key) pair,
     delta-rule FLOPs per token, fp32 state bytes, cache bytes per key"""
@@ -835,11 +837,45 @@ def nabelix_work(cfg):
         w["delta_flops"] += 8.0 * rt["heads"] * rt["dim"] * rt["vdim"]
         w["state_bytes"] += 4.0 * rt["heads"] * rt["dim"] * rt["vdim"]
     w["head_bytes"] = w["head_flops"] = 2.0 * cfg["vocab"] * cfg["width"]
+    win = cfg["layers"][0]["mixer"]["left"]["mask"]["size"] + cfg["layers"][0]["mixer"]["left"]["mask"]["keep_first"]
+    w["keys"] = lambda i: min(i + 1, win)
+    w["expert_bytes"] = lambda rows: 0.0
     return w
 
 
-def run_nabelix(args):
-    """One JSON line. Weights exceed the L2 (0.6 to 4 GB), so nothing is flushed between iterations. Device times from
+def sominex_work(cfg):
+    """the same sums; weight bytes and FLOPs of the experts that one token uses, the bytes of the experts that more rows
+    use taken as the expected number of distinct ones"""
+    w = dict(weight_bytes=0.0, gemm_flops=0.0, attn_flops=0.0, state_bytes=0.0, key_bytes=0.0)
+    synth = importlib.import_module("tiny-gemma_b200.synth")
+    moe = [sp["mlp"] for sp in cfg["layers"] if sp["mlp"] and sp["mlp"]["kind"] == "moe"]
+    for name, shape in synth.sominex_shapes(cfg):
+        if name in ("embed", "head") or len(shape) == 1 or name.endswith("conv") or ".mlp.e" in name:
+            continue
+        w["weight_bytes"] += 2.0 * shape[0] * shape[1]
+        w["gemm_flops"] += 2.0 * shape[0] * shape[1]
+    one = [3 * 2.0 * cfg["width"] * f["expert"]["ff"] for f in moe]  # bytes of an expert, and FLOPs of a token in it
+    w["gemm_flops"] += sum(n * f["router"]["top"] for n, f in zip(one, moe))
+    w["expert_bytes"] = lambda rows: sum(n * f["router"]["experts"] * (1 - (1 - f["router"]["top"] / f["router"]["experts"]) ** rows) for n, f in zip(one, moe))
+    mask = None
+    for sp in cfg["layers"]:
+        c = sp["mixer"]
+        if sp["type"] == "attention":
+            mask = c["mask"]
+            w["attn_flops"] += 2.0 * c["heads"] * (c["dim"] + c["vdim"])
+            w["key_bytes"] += 2.0 * c["kv_heads"] * (c["dim"] + c["vdim"])
+        else:
+            n = c["state"] if sp["type"] == "mamba2" else c["dim"]
+            w["gemm_flops"] += 4.0 * c["heads"] * n * c["vdim"]
+            w["state_bytes"] += 4.0 * c["heads"] * n * c["vdim"]
+    w["keys"] = lambda i: min(i + 1, mask["size"]) + max(0, (int(i) - mask["size"] + 1) // mask["pool"])
+    w["head_bytes"] = w["head_flops"] = 2.0 * cfg["vocab"] * cfg["width"]
+    return w
+
+
+def run_layered(args, design):
+    """One JSON line: a design of the layered family beside the closest other model (Nabelix: int8 Gemma-3; Sominex:
+    Nabelix). Weights exceed the L2 (0.6 to 4 GB), so nothing is flushed between iterations. Device times from
     CUDA events on the state's stream; a prefill's includes the upload of its token ids."""
     import torch
 
@@ -899,10 +935,11 @@ def run_nabelix(args):
     clocks = ClockSampler(0)
     clocks.start()
     rows = []
-    for name in sizes:
-        cfg = synth.nabelix_config(name)
-        w = nabelix_work(cfg)
-        folder = synth.write_random_nabelix(os.path.join(CACHE, "tg_nabelix_%s" % name), cfg)
+
+    def layered(design, name):
+        cfg = synth.LAYERED[design][0](name)
+        w = {"Nabelix": nabelix_work, "Sominex": sominex_work}[design](cfg)
+        folder = synth.write_random_layered(os.path.join(CACHE, "tg_%s_%s" % (design.lower(), name)), cfg)
         t0 = time.perf_counter()
         model = capi.Model.open(folder)
         load_s = time.perf_counter() - t0
@@ -910,17 +947,22 @@ def run_nabelix(args):
         r = measure(model, cfg["vocab"])
         rec = {"size": name, "width": cfg["width"], "ff": cfg["layers"][0]["mlp"]["ff"], "layers": len(cfg["layers"]), "vocab": cfg["vocab"],
                "weight_gb": (w["weight_bytes"] + w["head_bytes"]) / 1e9, "load_s": load_s, "gpu_launches": capi.launch_count(), "prefill": [], "decode": []}
-        win = cfg["layers"][0]["mixer"]["left"]["mask"]["size"] + cfg["layers"][0]["mixer"]["left"]["mask"]["keep_first"]
         for S, ms in r["prefill"]:
-            pairs = sum(min(i + 1, win) for i in range(S))
+            pairs = sum(w["keys"](i) for i in range(S))
             fl = S * w["gemm_flops"] + w["head_flops"] + pairs * w["attn_flops"]
             rec["prefill"].append({"tokens": S, "ms": ms, "tok_s": S / ms * 1e3, "tflops": fl / ms / 1e9, "of_measured_tensor": fl / ms / 1e9 / tf})
         for B, pos, ms in r["decode"]:
-            keys = min(pos + steps / 2, win)
-            by = w["weight_bytes"] + w["head_bytes"] + B * (2 * w["state_bytes"] + keys * w["key_bytes"])
+            keys = w["keys"](pos + steps / 2)
+            by = w["weight_bytes"] + w["expert_bytes"](B) + w["head_bytes"] + B * (2 * w["state_bytes"] + keys * w["key_bytes"])
             rec["decode"].append({"batch": B, "position": pos, "ms_per_step": ms, "tok_s": B / ms * 1e3, "gbs": by / ms / 1e6, "of_measured_hbm": by / ms / 1e6 / hbm})
         model.close()
-        if not args.no_extras and name in synth.CONFIGS:
+        return rec
+
+    for name in sizes:
+        rec = layered(design, name)
+        if design == "Sominex" and not args.no_extras:
+            rec["nabelix"] = layered("Nabelix", name)
+        if design == "Nabelix" and not args.no_extras and name in synth.CONFIGS:
             gm = capi.Model(name).load_file(synth.write_random_model(os.path.join(CACHE, "tg_%s_s%d.bin" % (name, WEIGHT_SEED)), name, WEIGHT_SEED))
             gm.build_tables(1024)
             r = measure(gm, gm.vocab)
@@ -934,7 +976,7 @@ def run_nabelix(args):
                             / ms / 1e6 / hbm} for B, pos, ms in r["decode"]]}
             gm.close()
         rows.append(rec)
-    print(json.dumps({"mode": "nabelix", "dtype": "bf16", "data": "synthetic (random weights and token ids)", "steps": steps,
+    print(json.dumps({"mode": design.lower(), "dtype": "bf16", "data": "synthetic (random weights and token ids)", "steps": steps,
                       "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": src}, "clocks": clocks.stop(), "sizes": rows}), flush=True)
     return 0
 
@@ -948,7 +990,7 @@ def main():
     ap.add_argument("--batch", type=int, default=1, help="total independent sequences (greedy); >1 selects the batched step")
     ap.add_argument("--no-extras", action="store_true", help="skip the matvec sweep and the CPU baseline sample")
     ap.add_argument("--model", default=MODEL, choices=["270m", "1B", "3B"],
-                    help="architecture (3B: only with --nabelix); 1B is the benchmark configuration, 270m is the small case used for profiling")
+                    help="architecture (3B: only with --nabelix or --sominex); 1B is the benchmark configuration, 270m is the small case used for profiling")
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN,
                     help="prompt tokens; 178 is the benchmark configuration, 16384 the long-context one "
                          "(use --no-extras: the CPU baseline sample would prefill the same prompt)")
@@ -959,11 +1001,12 @@ def main():
     ap.add_argument("--greedy", action="store_true", help="with --phase-clocks: argmax instead of the min-p sampler")
     ap.add_argument("--batched-step", action="store_true", help="time the batched step alone (--batch sequences, empty cache)")
     ap.add_argument("--nabelix", action="store_true", help="throughput of the Nabelix design; with --no-extras only --model at --prompt-len and --batch")
+    ap.add_argument("--sominex", action="store_true", help="the same for the Sominex design, beside Nabelix of the same size")
     args = ap.parse_args()
-    if args.model == "3B" and not args.nabelix:
-        ap.error("--model 3B needs --nabelix")
-    if args.nabelix:
-        return run_nabelix(args)
+    if args.model == "3B" and not (args.nabelix or args.sominex):
+        ap.error("--model 3B needs --nabelix or --sominex")
+    if args.nabelix or args.sominex:
+        return run_layered(args, "Nabelix" if args.nabelix else "Sominex")
     globals()["MODEL"] = args.model
     globals()["PROMPT_LEN"] = args.prompt_len
     if args.impl == "reference":

@@ -43,6 +43,7 @@ struct GemmArgs {
 	int ld32;
 	const int *tile_expert;  // GRP: [row tiles] expert of a tile; its weights are rows expert * N ..
 	const int *n_row_tiles;  // GRP: row tiles of this step
+	int splits;              // GEMM_STORE32: CTAs that share a tile's K; split s is stored M * ldc * s further on (0, 1: none)
 };
 
 __device__ __forceinline__ float gelu_tanh(float z) {
@@ -55,6 +56,15 @@ __device__ __forceinline__ float glu(int act, float limit, float g, float u) {
 	g = fminf(g, limit);
 	u = fminf(fmaxf(u, -limit), limit);
 	return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+// the same for results that are rounded to bf16: z sigmoid(y) with the fast exponential (gelu_tanh(z) = z sigmoid(2 u))
+__device__ __forceinline__ float swish_fast(float z, float y) { return __fdividef(z, 1.0f + __expf(-y)); }
+template <int ACT> __device__ __forceinline__ float glu_fast(float limit, float g, float u) {
+	if (ACT == GLU_GELU) return swish_fast(g, 1.5957691216057308f * (g + 0.044715f * g * g * g)) * u;
+	if (ACT == GLU_SILU) return swish_fast(g, g) * u;
+	g = fminf(g, limit);
+	u = fminf(fmaxf(u, -limit), limit);
+	return fmaf(swish_fast(g, 1.702f * g), u, swish_fast(g, 1.702f * g));
 }
 __device__ __forceinline__ float soft_cap(float v, float cap) { return cap > 0.0f ? cap * tanhf(v / cap) : v; }
 __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
@@ -112,9 +122,14 @@ __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 		pdl_wait();
 		a.m_tiles = *a.n_row_tiles;
 	}
-	const int tiles = a.m_tiles * a.n_tiles;
+	constexpr bool SPLIT = EPI == GEMM_STORE32;
+	const int one = a.m_tiles * a.n_tiles, tiles = SPLIT ? one * max(1, a.splits) : one;
+	const int share = SPLIT ? (k_blocks + max(1, a.splits) - 1) / max(1, a.splits) : k_blocks;
+	// K-blocks of tile t: [kb_lo, kb_hi)
+	auto kb_lo = [&](int t) { return SPLIT ? t / one * share : 0; };
+	auto kb_hi = [&](int t) { return SPLIT ? min(k_blocks, (t / one + 1) * share) : k_blocks; };
 	// first weight row of a tile
-	auto w_row = [&](int t) { return (t / a.m_tiles) * BN + (GRP ? a.tile_expert[t % a.m_tiles] * a.N : 0); };
+	auto w_row = [&](int t) { return (SPLIT ? t % one : t) / a.m_tiles * BN + (GRP ? a.tile_expert[t % a.m_tiles] * a.N : 0); };
 	if (tid == 0) {
 		for (int s = 0; s < NS; s++) {
 			mbar_init(&full_bar[s], 1);
@@ -145,17 +160,17 @@ __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 			const int first = int(blockIdx.x);
 			int ahead = 0;
 			if (first < tiles) {
-				ahead = min(NS, k_blocks);
+				ahead = min(NS, kb_hi(first) - kb_lo(first));
 				for (int s = 0; s < ahead; s++) {
 					mbar_expect_tx(&full_bar[s], SH::STAGE);
-					tma_load_2d(smem + s * SH::STAGE + SH::A_BYTES, &wmap, s * GB_BK, w_row(first), &full_bar[s]);
+					tma_load_2d(smem + s * SH::STAGE + SH::A_BYTES, &wmap, (kb_lo(first) + s) * GB_BK, w_row(first), &full_bar[s]);
 				}
 			}
 			pdl_wait();
 			int it = 0;
 			for (int t = first; t < tiles && !*(volatile int *)&s_fail; t += gridDim.x) {
 				const int m0 = (t % a.m_tiles) * GB_BM, n0 = w_row(t);
-				for (int kb = 0; kb < k_blocks; kb++, it++) {
+				for (int kb = kb_lo(t), k1 = kb_hi(t); kb < k1; kb++, it++) {
 					const int s = it % NS, use = it / NS;
 					if (use > 0 && !tc_wait(&free_bar[s], (use - 1) & 1, a.err)) {
 						s_fail = 1;
@@ -184,7 +199,8 @@ __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 				tc_fence_after();
 				const uint32_t d = tmem_base + uint32_t(buf * BN);
 				bool ok = true;
-				for (int kb = 0; kb < k_blocks; kb++, it++) {
+				const int k0 = kb_lo(t);
+				for (int kb = k0, k1 = kb_hi(t); kb < k1; kb++, it++) {
 					const int s = it % NS;
 					if (!tc_wait(&full_bar[s], (it / NS) & 1, a.err)) {
 						s_fail = 1;
@@ -195,7 +211,7 @@ __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 					const uint32_t pa = smem_u32(smem + s * SH::STAGE), pw = pa + SH::A_BYTES;
 #pragma unroll
 					for (int j = 0; j < GB_BK / 16; j++)
-						tc_mma(d, tc_sw128_desc(pa + j * 32, 16, 1024), tc_sw128_desc(pw + j * 32, 16, 1024), idesc, (kb > 0 || j > 0) ? 1u : 0u);
+						tc_mma(d, tc_sw128_desc(pa + j * 32, 16, 1024), tc_sw128_desc(pw + j * 32, 16, 1024), idesc, (kb > k0 || j > 0) ? 1u : 0u);
 					tc_commit(&free_bar[s]);
 				}
 				if (!ok) break;
@@ -227,7 +243,8 @@ __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 				break;
 			}
 			tc_fence_after();
-			const int r0 = (t % a.m_tiles) * GB_BM + quad * 32, n0 = (t / a.m_tiles) * BN;
+			const int r0 = (t % a.m_tiles) * GB_BM + quad * 32, n0 = (SPLIT ? t % one : t) / a.m_tiles * BN;
+			const size_t far = SPLIT ? size_t(t / one) * a.M * a.ldc : 0;
 			const uint32_t taddr = tmem_base + (uint32_t(quad * 32) << 16) + uint32_t(buf * BN);
 			const int ncol = (EPI == GEMM_LOGITS) ? a.ldc : a.N;
 #pragma unroll 1
@@ -242,10 +259,14 @@ __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 					const int row = r0 + lane;
 					if (row < a.M) {
 						uint32_t o[8];
+						auto all = [&](auto f) {
 #pragma unroll
-						for (int i = 0; i < 8; i++)
-							o[i] = pack_bf16(glu(a.act, a.limit, __uint_as_float(r[2 * i]), __uint_as_float(r[16 + 2 * i])),
-							                 glu(a.act, a.limit, __uint_as_float(r[2 * i + 1]), __uint_as_float(r[17 + 2 * i])));
+							for (int i = 0; i < 8; i++)
+								o[i] = pack_bf16(f(__uint_as_float(r[2 * i]), __uint_as_float(r[16 + 2 * i])), f(__uint_as_float(r[2 * i + 1]), __uint_as_float(r[17 + 2 * i])));
+						};
+						if (a.act == GLU_GELU) all([&](float g, float u) { return glu_fast<GLU_GELU>(a.limit, g, u); });
+						else if (a.act == GLU_SILU) all([&](float g, float u) { return glu_fast<GLU_SILU>(a.limit, g, u); });
+						else all([&](float g, float u) { return glu_fast<GLU_CLAMP>(a.limit, g, u); });
 						uint4 *dst = reinterpret_cast<uint4 *>(reinterpret_cast<__nv_bfloat16 *>(a.C) + size_t(row) * a.ldc + col / 2);
 						dst[0] = make_uint4(o[0], o[1], o[2], o[3]);
 						dst[1] = make_uint4(o[4], o[5], o[6], o[7]);
@@ -285,7 +306,7 @@ __global__ void __launch_bounds__(GB_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 							const int rr = 4 * i + (lane >> 3);
 							if (r0 + rr < a.M && col + cc < ncol) {
 								float4 v = *reinterpret_cast<const float4 *>(stg + rr * 36 + cc);
-								float4 *dst = reinterpret_cast<float4 *>(reinterpret_cast<float *>(a.C) + size_t(r0 + rr) * a.ldc + col + cc);
+								float4 *dst = reinterpret_cast<float4 *>(reinterpret_cast<float *>(a.C) + far + size_t(r0 + rr) * a.ldc + col + cc);
 								if (EPI == GEMM_ADD) {
 									v.x += add[i].x; v.y += add[i].y; v.z += add[i].z; v.w += add[i].w;
 								}

@@ -71,18 +71,20 @@ constexpr int GV_THREADS = 256;
 __host__ __device__ inline int gv_k8(int K) { return (K + 7) / 8; }
 template <int R, int NR> __host__ __device__ constexpr int gv_red_floats() { return 2 * 8 * NR * R; }
 template <int R, int NR> size_t gv_smem(int K, int pro, int epi, int parts, int ex) {
-	const size_t rows = epi == GV_FRONT ? 2 * R : R, extra = pro == GV_MIX ? 0 : pro;
+	const size_t rows = epi == GV_FRONT ? 2 * R : R, extra = pro == GV_LN ? 1 : (pro == GV_LN_CONV ? 1 + R : 0);
 	return ((rows + extra) * 8 * gv_k8(K) + gv_red_floats<R, NR>() + 32 + (pro == GV_MIX ? size_t(R) * ((parts + 3) / 4 * 4 + ex) : 0)) * 4;
 }
 
-__device__ __forceinline__ float gv_block_sum(float v, float *red) {
+// sum over the threads of a row (8 / R warps), in every one of them
+template <int R> __device__ __forceinline__ float gv_row_sum(float v, float *red) {
 	v = warp_sum(v);
 	__syncthreads();
 	if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
 	__syncthreads();
+	const float *mine = red + (threadIdx.x >> 5) / (8 / R) * (8 / R);
 	float t = 0.0f;
 #pragma unroll
-	for (int w = 0; w < 8; w++) t += red[w];
+	for (int w = 0; w < 8 / R; w++) t += mine[w];
 	return t;
 }
 
@@ -96,7 +98,7 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 	float *red = gv_sm + size_t(R) * 8 * K8;             // [2][row set][KS][NR][R]
 	float *bred = red + gv_red_floats<R, NR>();
 	float *wn = bred + 32, *hc = wn + 8 * K8;            // norm weight (x its factor in the convolution); history's share
-	float *xp = hc + 8 * K8;                             // GV_FRONT: the plain norms, laid out as xs
+	float *xp = hc + size_t(R) * 8 * K8;                 // GV_FRONT: the plain norms, laid out as xs
 	float *prt = bred + 32, *xe = prt + (PRO == GV_MIX ? R * ((a.parts + 3) / 4 * 4) : 0);  // GV_MIX: 1 / deviation of the parts; experts' activations
 	constexpr int SETS = 8 / KS, GROUP = SETS * NR;      // weight rows per CTA and group
 	const int set = warp / KS, ks = warp % KS;
@@ -147,52 +149,79 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 	pdl_wait();
 
 	// ---------------------------------------------------------------- prologue: activations into shared memory
+	// (the rows side by side, TG threads each; global loads in batches of four, ahead of the stores)
 	auto xi = [&](int k) { return ((k >> 2) & 1) * 4 * K8 + (k >> 3) * 4 + (k & 3); };
-#pragma unroll 1
-	for (int r = 0; r < R; r++) {
-		float *xr = xs + size_t(r) * 8 * K8;
-		if (PRO == GV_VEC) {
-			for (int k = tid; k < 8 * K8; k += GV_THREADS) xr[xi(k)] = k < a.K ? a.vec[size_t(r) * a.ldv + k] : 0.0f;
-			continue;
+	constexpr int TG = GV_THREADS / R;
+	const int r = tid / TG, t = tid % TG;
+	float *xr = xs + size_t(r) * 8 * K8;
+	if constexpr (PRO == GV_VEC || PRO == GV_MIX) {
+		const float *vec = a.vec + size_t(r) * a.ldv, *gate = PRO == GV_MIX ? a.gate + size_t(r) * a.ldg : nullptr;
+		const bool pre = PRO == GV_MIX && a.mix_norm == MIX_GATE_NORM;
+		for (int u0 = t; u0 < 2 * K8; u0 += 4 * TG) {  // (K is a multiple of 8)
+			float4 v[4], z[4];
+#pragma unroll
+			for (int e = 0; e < 4; e++) {
+				const int u = u0 + e * TG;
+				if (u < 2 * K8) v[e] = *reinterpret_cast<const float4 *>(vec + 4 * u);
+				if (pre && 4 * u < a.mix_n) z[e] = *reinterpret_cast<const float4 *>(gate + 4 * u);
+			}
+#pragma unroll
+			for (int e = 0; e < 4; e++) {
+				const int u = u0 + e * TG, k = 4 * u;
+				if (u >= 2 * K8) break;
+				if (pre) {
+					if (k < a.mix_n) v[e].x *= silu_f(z[e].x);
+					if (k + 1 < a.mix_n) v[e].y *= silu_f(z[e].y);
+					if (k + 2 < a.mix_n) v[e].z *= silu_f(z[e].z);
+					if (k + 3 < a.mix_n) v[e].w *= silu_f(z[e].w);
+				}
+				*reinterpret_cast<float4 *>(xr + xi(k)) = v[e];
+			}
 		}
 		if (PRO == GV_MIX) {
-			const float *gate = a.gate + size_t(r) * a.ldg;
-			for (int k = tid; k < 8 * K8; k += GV_THREADS) {
-				float v = k < a.K ? a.vec[size_t(r) * a.ldv + k] : 0.0f;
-				if (a.mix_norm == MIX_GATE_NORM && k < a.mix_n) v *= silu_f(gate[k]);
-				xr[xi(k)] = v;
+			const int n4 = a.n_ex / 4, all4 = a.top * n4;
+			float4 *dst = reinterpret_cast<float4 *>(xe + r * a.top * a.n_ex);
+			const float4 *src = reinterpret_cast<const float4 *>(a.ex_act + size_t(r) * a.top * a.n_ex);
+			const float *ew = a.ex_w + r * a.top;
+#pragma unroll 4
+			for (int u = t; u < all4; u += TG) {
+				const float4 v = src[u];
+				const float w = ew[u / n4];
+				dst[u] = make_float4(v.x * w, v.y * w, v.z * w, v.w * w);
 			}
-			for (int k = tid; k < a.top * a.n_ex; k += GV_THREADS)
-				xe[r * a.top * a.n_ex + k] = a.ex_act[size_t(r) * a.top * a.n_ex + k] * a.ex_w[r * a.top + k / a.n_ex];
-			if (a.mix_norm == MIX_NONE) continue;
-			__syncthreads();
-			const int width = a.mix_n / a.parts;
-			for (int p = warp; p < a.parts; p += 8) {
-				float q = 0.0f;
-				for (int k = p * width + lane; k < (p + 1) * width; k += 32) q = fmaf(xr[xi(k)], xr[xi(k)], q);
-				q = warp_sum(q);
-				if (lane == 0) prt[r * a.parts + p] = 1.0f / sqrtf(q / float(width) + a.eps);
+			if (a.mix_norm != MIX_NONE) {
+				__syncthreads();
+				const int width = a.mix_n / a.parts;
+				for (int p = warp % (8 / R); p < a.parts; p += 8 / R) {
+					float q = 0.0f;
+#pragma unroll 4
+					for (int k = p * width + lane; k < (p + 1) * width; k += 32) q = fmaf(xr[xi(k)], xr[xi(k)], q);
+					q = warp_sum(q);
+					if (lane == 0) prt[r * a.parts + p] = 1.0f / sqrtf(q / float(width) + a.eps);
+				}
+				__syncthreads();
+				const bool post = a.mix_norm == MIX_NORM_GATE;
+#pragma unroll 4
+				for (int k = t; k < a.mix_n; k += TG) {
+					const float w = a.w[k], z = post ? gate[k] : 0.0f;
+					const float v = xr[xi(k)] * prt[r * a.parts + k / width] * w;
+					xr[xi(k)] = post ? v * sigmoid_f(z) : v;
+				}
 			}
-			__syncthreads();
-			for (int k = tid; k < a.mix_n; k += GV_THREADS) {
-				float v = xr[xi(k)] * prt[r * a.parts + k / width] * a.w[k];
-				if (a.mix_norm == MIX_NORM_GATE) v *= sigmoid_f(gate[k]);
-				xr[xi(k)] = v;
-			}
-			continue;
 		}
+	} else {
 		const int seg = a.d.row_seg[r];
 		int tok = 0;
 		if (a.embed_mode) {
 			tok = a.d.tok[r];
 			if (tok < 0 || tok >= a.V) {
-				if (blockIdx.x == 0 && tid == 0) *a.err = 1;
+				if (blockIdx.x == 0 && t == 0) *a.err = 1;
 				tok = 0;
 			}
 		}
 		const int H = PRO == GV_LN_CONV ? a.taps - 1 : 0;
 		const float *hr = nullptr;
-		float *hw = nullptr;
+		float *hw = nullptr, *hcr = hc + size_t(r) * 8 * K8;
 		int pos = 0;
 		if (PRO == GV_LN_CONV) {
 			pos = a.d.seg_pos[seg];
@@ -201,48 +230,69 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 			hw = hb + size_t(a.d.seg_par[seg] ^ 1) * H * a.D;
 		}
 		float s = 0.0f;
-#pragma unroll 2
-		for (int k = tid; k < a.D; k += GV_THREADS) {
-			float v = a.embed_mode == 1 ? 0.0f : a.x[size_t(r) * a.ldx + k];
-			if (a.embed_mode) v += a.embed_scale * __bfloat162float(a.embed[size_t(tok) * a.lde + k]);
-			if (PRO == GV_LN_CONV) {
-				float c = 0.0f;
-#pragma unroll 3
-				for (int j = 0; j < H; j++) {
-					const float u = pos - H + j >= 0 ? hr[size_t(j) * a.D + k] : 0.0f;
-					c = fmaf(a.cw[size_t(j) * a.D + k], u, c);
-					if (blockIdx.x == 0 && j > 0) hw[size_t(j - 1) * a.D + k] = u;
-				}
-				hc[k] = c;
+		for (int k0 = t; k0 < a.D; k0 += 4 * TG) {
+			float v[4], c[4] = {}, em[4];
+#pragma unroll
+			for (int e = 0; e < 4; e++) {
+				const int k = k0 + e * TG;
+				v[e] = k < a.D && a.embed_mode != 1 ? a.x[size_t(r) * a.ldx + k] : 0.0f;
+				em[e] = k < a.D && a.embed_mode ? __bfloat162float(a.embed[size_t(tok) * a.lde + k]) : 0.0f;
 			}
-			xr[xi(k)] = v;
-			s += v;
+			if (PRO == GV_LN_CONV) {
+				for (int j = 0; j < H; j++) {
+					float u[4], w[4];
+#pragma unroll
+					for (int e = 0; e < 4; e++) {
+						const int k = k0 + e * TG;
+						u[e] = k < a.D && pos - H + j >= 0 ? hr[size_t(j) * a.D + k] : 0.0f;
+						w[e] = k < a.D ? a.cw[size_t(j) * a.D + k] : 0.0f;
+					}
+#pragma unroll
+					for (int e = 0; e < 4; e++) {
+						c[e] = fmaf(w[e], u[e], c[e]);
+						if (blockIdx.x == 0 && j > 0 && k0 + e * TG < a.D) hw[size_t(j - 1) * a.D + k0 + e * TG] = u[e];
+					}
+				}
+			}
+#pragma unroll
+			for (int e = 0; e < 4; e++) {
+				const int k = k0 + e * TG;
+				if (k >= a.D) break;
+				v[e] = fmaf(a.embed_scale, em[e], v[e]);
+				if (PRO == GV_LN_CONV) hcr[k] = c[e];
+				xr[xi(k)] = v[e];
+				s += v[e];
+			}
 		}
-		const float mean = a.rms ? 0.0f : gv_block_sum(s, bred) / float(a.D);
+		const float mean = a.rms ? 0.0f : gv_row_sum<R>(s, bred) / float(a.D);
 		float q = 0.0f;
-		for (int k = tid; k < a.D; k += GV_THREADS) {
+		for (int k = t; k < a.D; k += TG) {
 			const float c = xr[xi(k)] - mean;
 			q = fmaf(c, c, q);
 		}
-		const float rstd = 1.0f / sqrtf(gv_block_sum(q, bred) / float(a.D) + a.eps);
-		for (int k = tid; k < 8 * K8; k += GV_THREADS) {
-			float y = 0.0f;
-			if (EPI == GV_FRONT) xp[size_t(r) * 8 * K8 + xi(k)] = 0.0f;
-			if (k < a.D) {
-				const float n = (xr[xi(k)] - mean) * rstd;
-				y = n * wn[k];
-				if (EPI == GV_FRONT) {
-					const float plain = n * a.w[k];
-					xp[size_t(r) * 8 * K8 + xi(k)] = plain;
-					if (a.norm_out && blockIdx.x == 0) a.norm_out[size_t(r) * a.D + k] = plain;
+		const float rstd = 1.0f / sqrtf(gv_row_sum<R>(q, bred) / float(a.D) + a.eps);
+		for (int k0 = t; k0 < 8 * K8; k0 += 4 * TG) {
+			float w[4];
+#pragma unroll
+			for (int e = 0; e < 4; e++) w[e] = PRO == GV_LN_CONV && k0 + e * TG < a.D ? a.w[k0 + e * TG] : 0.0f;
+#pragma unroll
+			for (int e = 0; e < 4; e++) {
+				const int k = k0 + e * TG;
+				if (k >= 8 * K8) break;
+				float y = 0.0f, plain = 0.0f;
+				if (k < a.D) {
+					const float n = (xr[xi(k)] - mean) * rstd;
+					plain = n * w[e];
+					y = n * wn[k];
+					if (PRO == GV_LN_CONV) {
+						y += hcr[k];
+						if (blockIdx.x == 0 && H > 0) hw[size_t(H - 1) * a.D + k] = plain;
+					}
+					if (a.norm_out && blockIdx.x == 0) a.norm_out[size_t(r) * a.D + k] = EPI == GV_FRONT ? plain : y;
 				}
-				if (PRO == GV_LN_CONV) {
-					y += hc[k];
-					if (blockIdx.x == 0 && H > 0) hw[size_t(H - 1) * a.D + k] = n * a.w[k];
-				}
-				if (EPI != GV_FRONT && a.norm_out && blockIdx.x == 0) a.norm_out[size_t(r) * a.D + k] = y;
+				if (EPI == GV_FRONT) xp[size_t(r) * 8 * K8 + xi(k)] = plain;
+				xr[xi(k)] = y;
 			}
-			xr[xi(k)] = y;
 		}
 	}
 	__syncthreads();

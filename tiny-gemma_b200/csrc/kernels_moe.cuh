@@ -81,19 +81,38 @@ __device__ __forceinline__ void moe_choose(const float *z, int E, int top, float
 	}
 }
 
-// grid ceil(R / 8), 256 threads
-static __global__ void __launch_bounds__(256) route_kernel(MoeArgs a, int R) {
+// grid ceil(R / (8 rounds)), 256 threads, rounds <= MR_ROUNDS rows per warp. Places are counted within the CTA first: one
+// addition per CTA and expert to the global counters. (A slot's number does not change what is computed there.)
+constexpr int MR_ROUNDS = 8;
+static __global__ void __launch_bounds__(256) route_kernel(MoeArgs a, int R, int rounds) {
 	pdl_trigger();
 	pdl_wait();
-	const int r = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-	if (r >= R) return;
-	int id;
-	float w;
-	moe_choose(a.z + size_t(r) * a.ldz, a.experts, a.top, a.scale, id, w);
-	if (lane < a.top) {
-		a.id[r * a.top + lane] = id;
-		a.w[r * a.top + lane] = w;
-		a.place[r * a.top + lane] = atomicAdd(a.count + id, 1);  // (a slot's number does not change what is computed there)
+	__shared__ int n[MOE_MAX];
+	const int lane = threadIdx.x & 31, r0 = blockIdx.x * 8 * rounds + (threadIdx.x >> 5);
+	for (int e = threadIdx.x; e < a.experts; e += 256) n[e] = 0;
+	__syncthreads();
+	int id[MR_ROUNDS], at[MR_ROUNDS];
+#pragma unroll
+	for (int i = 0; i < MR_ROUNDS; i++) {
+		const int r = r0 + 8 * i;
+		if (i >= rounds || r >= R) break;
+		float w;
+		moe_choose(a.z + size_t(r) * a.ldz, a.experts, a.top, a.scale, id[i], w);
+		if (lane < a.top) {
+			a.id[r * a.top + lane] = id[i];
+			a.w[r * a.top + lane] = w;
+			at[i] = atomicAdd(n + id[i], 1);
+		}
+	}
+	__syncthreads();
+	for (int e = threadIdx.x; e < a.experts; e += 256)
+		if (n[e]) n[e] = atomicAdd(a.count + e, n[e]);
+	__syncthreads();
+#pragma unroll
+	for (int i = 0; i < MR_ROUNDS; i++) {
+		const int r = r0 + 8 * i;
+		if (i >= rounds || r >= R) break;
+		if (lane < a.top) a.place[r * a.top + lane] = n[id[i]] + at[i];
 	}
 }
 

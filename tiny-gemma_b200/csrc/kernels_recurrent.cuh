@@ -10,8 +10,8 @@
 // The raw o_t go to an fp32 buffer; norm and gate follow in lin_norm_kernel or in the prologue of the output product.
 //
 //   lin_token_cta          one token: a CTA per (sequence, head, 32 columns of S)
-//   lin_conv_kernel        convolution and silu of a portion's x, B, C, padded head by head
-//   lin_gates_kernel       log a, b and exp(-m) of a portion's rows
+//   lin_conv_kernel        LIN_SSM: convolution and silu of a portion's x, B, C, padded head by head; log a and b
+//   lin_gates_kernel       LIN_MLSTM: log a, b and exp(-m) of a portion's rows
 //   lin_scan_kernel        a portion token by token, S in registers: 32-bit states, and portions of a few tokens
 //   lin_chunk_*_kernel     portions in chunks of LC = 128 tokens on the tensor cores. With c_t the sum of log a up to t
 //                          within the chunk (fp64 sums kept as pairs of floats: strong decays before weak ones lose
@@ -60,6 +60,7 @@ struct LinArgs {
 	float *dn, *n0;          // [chunks][H][N]
 	float *tot;              // [chunks][H] c_last
 	int vsplit;              // out: CTAs that share the columns of a head
+	int ready;               // one token: LIN_SSM's convolved rows and log a, b are there already
 	int *err;
 };
 
@@ -99,7 +100,7 @@ template <typename PT> __device__ void lin_token_cta(const LinArgs &a, int r, in
 	const int cl = (tid & 7) * 4, c0 = tile * LT_COLS + cl, rg = tid >> 3;
 	float *S = a.S + (size_t(seq) * a.H + h) * N * a.vdp + c0;
 	const bool on = c0 < a.vdp;
-	constexpr int HOLD = 8;  // rows of the state requested ahead
+	constexpr int HOLD = 4;  // rows of the state requested ahead
 	float4 st[HOLD];
 #pragma unroll
 	for (int e = 0; e < HOLD; e++) {
@@ -107,7 +108,14 @@ template <typename PT> __device__ void lin_token_cta(const LinArgs &a, int r, in
 		st[e] = on && !fresh && i < N ? *reinterpret_cast<const float4 *>(S + size_t(i) * a.vdp) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 	}
 	const PT *row = reinterpret_cast<const PT *>(a.p) + size_t(r) * a.ldp;
-	if (a.kind == LIN_SSM) {
+	if (a.kind == LIN_SSM && a.ready) {
+		const PT *rr = reinterpret_cast<const PT *>(a.rows) + size_t(r) * a.ldr;
+		for (int x = tid; x < N; x += 256) {
+			sq[x] = to_f32(rr[a.o_q + g * a.Np + x]);
+			sk[x] = to_f32(rr[a.o_k + g * a.Np + x]);
+		}
+		if (tid < LT_COLS) sv[tid] = tile * LT_COLS + tid < a.vd ? to_f32(rr[a.o_v + h * a.vdp + tile * LT_COLS + tid]) : 0.0f;
+	} else if (a.kind == LIN_SSM) {
 		const int C = lin_channels(a), H = a.taps - 1;
 		float *hb = a.hist + size_t(seq) * 2 * H * C;
 		const float *hr = hb + size_t(par) * H * C;
@@ -136,7 +144,7 @@ template <typename PT> __device__ void lin_token_cta(const LinArgs &a, int r, in
 		}
 		if (tid < LT_COLS) sv[tid] = tile * LT_COLS + tid < a.vd ? to_f32(row[a.p_v + h * a.vdp + tile * LT_COLS + tid]) : 0.0f;
 	}
-	const float2 gi = lin_gate_in(a, r, h);
+	const float2 gi = a.ready && a.kind == LIN_SSM ? make_float2(a.la[size_t(r) * a.H + h], a.b[size_t(r) * a.H + h]) : lin_gate_in(a, r, h);
 	float da, b, mn = 0.0f;
 	if (a.kind == LIN_SSM) {
 		da = expf(gi.x);
@@ -161,7 +169,14 @@ template <typename PT> __device__ void lin_token_cta(const LinArgs &a, int r, in
 #pragma unroll
 		for (int e = 0; e < HOLD; e++)
 			if (rg + 32 * e < N) update(st[e], rg + 32 * e);
-		for (int i = rg + 32 * HOLD; i < N; i += 32) update(fresh ? make_float4(0.0f, 0.0f, 0.0f, 0.0f) : *reinterpret_cast<const float4 *>(S + size_t(i) * a.vdp), i);
+		for (int i0 = rg + 32 * HOLD; i0 < N; i0 += 32 * HOLD) {
+#pragma unroll
+			for (int e = 0; e < HOLD; e++)
+				st[e] = !fresh && i0 + 32 * e < N ? *reinterpret_cast<const float4 *>(S + size_t(i0 + 32 * e) * a.vdp) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+			for (int e = 0; e < HOLD; e++)
+				if (i0 + 32 * e < N) update(st[e], i0 + 32 * e);
+		}
 	}
 	float den = 0.0f;
 	if (a.kind == LIN_MLSTM) {
@@ -204,14 +219,54 @@ template <typename PT> __device__ void lin_token_cta(const LinArgs &a, int r, in
 }
 
 // ------------------------------------------------------------------ portions: convolution, gates
-// grid (ceil(R / LV_ROWS), ceil(ldxc / 128)), 128 threads: a thread walks LV_ROWS rows of one (padded) column, the window in registers
+// V consecutive elements; fast: where the result is rounded to bf16 anyway
+template <int V> __device__ __forceinline__ void lin_load(float (&o)[V], const float *p) {
+	if constexpr (V == 4) {
+		const float4 v = *reinterpret_cast<const float4 *>(p);
+		o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w;
+	} else {
+		o[0] = p[0];
+	}
+}
+template <int V> __device__ __forceinline__ void lin_load(float (&o)[V], const __nv_bfloat16 *p) {
+	if constexpr (V == 4) {
+		const uint2 u = *reinterpret_cast<const uint2 *>(p);
+		o[0] = bf16_lo(u.x); o[1] = bf16_hi(u.x); o[2] = bf16_lo(u.y); o[3] = bf16_hi(u.y);
+	} else {
+		o[0] = __bfloat162float(p[0]);
+	}
+}
+template <int V, typename T> __device__ __forceinline__ void lin_store(T *p, const float (&o)[V]) {
+	if constexpr (V == 4) store4<T>(p, make_float4(o[0], o[1], o[2], o[3]));
+	else p[0] = from_f32<T>(o[0]);
+}
+template <typename T> __device__ __forceinline__ float lin_sigmoid(float z) {
+	return sizeof(T) == 2 ? __fdividef(1.0f, 1.0f + __expf(-z)) : sigmoid_f(z);
+}
+
+// grid (ceil(R / rows), ceil(ldxc / (128 V)) + 1), 128 threads, rows <= LV_ROWS: a thread walks the rows of V (padded)
+// columns, the window in registers. V = 4 if groups of four columns are channels that follow each other. The last blockIdx.y forms the
+// rows' log a and b.
 constexpr int LV_ROWS = 16;
-template <typename PT, int MT> __global__ void __launch_bounds__(128) lin_conv_kernel(LinArgs a, int R) {
+template <typename PT, int MT, int V> __global__ void __launch_bounds__(128) lin_conv_kernel(LinArgs a, int R, int rows) {
 	pdl_trigger();
 	pdl_wait();
-	const int col = blockIdx.y * 128 + threadIdx.x;
+	__shared__ int seg_s[LV_ROWS];
+	const int tid = threadIdx.x, r0 = blockIdx.x * rows, nr = min(rows, R - r0);
+	if (blockIdx.y + 1 == gridDim.y) {
+		for (int x = tid; x < nr * a.H; x += 128) {
+			const int r = r0 + x / a.H, h = x % a.H;
+			const float2 g = lin_gate_in(a, r, h);
+			a.la[size_t(r) * a.H + h] = g.x;
+			a.b[size_t(r) * a.H + h] = g.y;
+		}
+		return;
+	}
+	if (tid < nr) seg_s[tid] = a.d.row_seg[r0 + tid];
+	__syncthreads();
+	const int col = V * (blockIdx.y * 128 + tid);
 	if (col >= a.ldxc) return;
-	const int r0 = blockIdx.x * LV_ROWS, nr = min(LV_ROWS, R - r0), C = lin_channels(a), H = a.taps - 1;
+	const int C = lin_channels(a), H = a.taps - 1;
 	const int xw = a.H * a.vdp, bw = a.G * a.Np;
 	int ch;  // the raw channel, or -1 for padding
 	if (col < xw) ch = col % a.vdp < a.vd ? col / a.vdp * a.vd + col % a.vdp : -1;
@@ -221,22 +276,42 @@ template <typename PT, int MT> __global__ void __launch_bounds__(128) lin_conv_k
 	}
 	PT *out = reinterpret_cast<PT *>(a.xc) + size_t(r0) * a.ldxc + col;
 	if (ch < 0) {
-		for (int i = 0; i < nr; i++) out[size_t(i) * a.ldxc] = from_f32<PT>(0.0f);
+		const float none[V] = {};
+		for (int i = 0; i < nr; i++) lin_store<V, PT>(out + size_t(i) * a.ldxc, none);
 		return;
 	}
 	const PT *in = reinterpret_cast<const PT *>(a.p) + size_t(r0) * a.ldp + a.p_x + ch;
-	const float bias = a.cb[ch];
-	float cf[MT], win[MT], x[LV_ROWS];
+	float bias[V], cf[MT][V], win[MT][V], x[LV_ROWS][V];
+	lin_load<V>(bias, a.cb + ch);
 #pragma unroll
-	for (int j = 0; j < MT; j++) cf[j] = j >= MT - a.taps ? a.cw[size_t(j - (MT - a.taps)) * C + ch] : 0.0f;
+	for (int i = 0; i < LV_ROWS; i++) {
 #pragma unroll
-	for (int i = 0; i < LV_ROWS; i++) x[i] = i < nr ? to_f32(in[size_t(i) * a.ldp]) : 0.0f;
+		for (int e = 0; e < V; e++) x[i][e] = 0.0f;
+		if (i < nr) lin_load<V>(x[i], in + size_t(i) * a.ldp);
+	}
+#pragma unroll
+	for (int j = 0; j < MT; j++) {
+#pragma unroll
+		for (int e = 0; e < V; e++) cf[j][e] = win[j][e] = 0.0f;
+		if (j >= MT - a.taps) lin_load<V>(cf[j], a.cw + size_t(j - (MT - a.taps)) * C + ch);
+	}
 	int seg = -1, row0 = 0, len = 0;
 	float *hw = nullptr;
+	// the rows before the first one are plain rows of its segment in all but the first few rows of a segment
+	const int before = r0 - a.d.seg_row[seg_s[0]];
+	if (before >= H) {
+		seg = seg_s[0];
+		row0 = a.d.seg_row[seg];
+		len = a.d.seg_len[seg];
+		hw = a.hist + (size_t(a.d.seg_seq[seg]) * 2 + (a.d.seg_par[seg] ^ 1)) * H * C;
+#pragma unroll
+		for (int j = 0; j < MT; j++)
+			if (MT - j <= H) lin_load<V>(win[j], in - ptrdiff_t(MT - j) * a.ldp);
+	}
 #pragma unroll
 	for (int i = 0; i < LV_ROWS; i++) {
 		if (i >= nr) break;
-		const int r = r0 + i, sg = a.d.row_seg[r];
+		const int r = r0 + i, sg = seg_s[i];
 		if (sg != seg) {
 			seg = sg;
 			row0 = a.d.seg_row[seg];
@@ -246,42 +321,43 @@ template <typename PT, int MT> __global__ void __launch_bounds__(128) lin_conv_k
 			const float *hr = hb + size_t(a.d.seg_par[seg]) * H * C;
 			hw = hb + size_t(a.d.seg_par[seg] ^ 1) * H * C;
 #pragma unroll
-			for (int j = 0; j < MT; j++) win[j] = MT - j <= H ? lin_conv_in<PT>(a, row0, pos, hr, C, t - (MT - j), ch) : 0.0f;
+			for (int j = 0; j < MT; j++)
+#pragma unroll
+				for (int e = 0; e < V; e++) win[j][e] = MT - j <= H ? lin_conv_in<PT>(a, row0, pos, hr, C, t - (MT - j), ch + e) : 0.0f;
 			if (t == 0)  // inputs before this segment that stay relevant
 				for (int q = 0; q < H; q++)
-					if (len - H + q < 0) hw[size_t(q) * C + ch] = lin_conv_in<PT>(a, row0, pos, hr, C, len - H + q, ch);
+					if (len - H + q < 0)
+						for (int e = 0; e < V; e++) hw[size_t(q) * C + ch + e] = lin_conv_in<PT>(a, row0, pos, hr, C, len - H + q, ch + e);
 		}
-		float y = bias;
+		float y[V];
 #pragma unroll
-		for (int j = 0; j < MT; j++) {
-			win[j] = j + 1 < MT ? win[j + 1] : x[i];
-			y = fmaf(cf[j], win[j], y);
+		for (int e = 0; e < V; e++) {
+			y[e] = bias[e];
+#pragma unroll
+			for (int j = 0; j < MT; j++) {
+				win[j][e] = j + 1 < MT ? win[j + 1][e] : x[i][e];
+				y[e] = fmaf(cf[j][e], win[j][e], y[e]);
+			}
+			y[e] = sizeof(PT) == 2 ? swish_fast(y[e], y[e]) : silu_f(y[e]);
 		}
-		out[size_t(i) * a.ldxc] = from_f32<PT>(silu_f(y));
+		lin_store<V, PT>(out + size_t(i) * a.ldxc, y);
 		const int q = (r - row0) - (len - H);
-		if (q >= 0) hw[size_t(q) * C + ch] = x[i];
+		if (q >= 0) lin_store<V, float>(hw + size_t(q) * C + ch, x[i]);
 	}
 }
 
-// grid (H, segments), 256 threads; LIN_MLSTM: a scan of (f, i) pairs, (F1, M1)(F2, M2) = (F1 + F2, max(M1 + F2, M2)),
-// four tokens per thread and round
-static __global__ void __launch_bounds__(256) lin_gates_kernel(LinArgs a) {
+// LIN_MLSTM: log a, b and exp(-m). grid (H, segments), LG_THREADS; a scan of (f, i) pairs, (F1, M1)(F2, M2) =
+// (F1 + F2, max(M1 + F2, M2)), four tokens per thread and round
+constexpr int LG_THREADS = 1024;
+static __global__ void __launch_bounds__(LG_THREADS) lin_gates_kernel(LinArgs a) {
 	pdl_trigger();
 	pdl_wait();
-	__shared__ float sF[8], sM[8];
+	__shared__ float sF[LG_THREADS / 32], sM[LG_THREADS / 32];
 	const int h = blockIdx.x, seg = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
 	const int len = a.d.seg_len[seg], row0 = a.d.seg_row[seg];
-	if (a.kind == LIN_SSM) {
-		for (int t = tid; t < len; t += 256) {
-			const float2 g = lin_gate_in(a, row0 + t, h);
-			a.la[size_t(row0 + t) * a.H + h] = g.x;
-			a.b[size_t(row0 + t) * a.H + h] = g.y;
-		}
-		return;
-	}
 	const int seq = a.d.seg_seq[seg], par = a.d.seg_par[seg];
 	float m0 = a.d.seg_pos[seg] == 0 ? 0.0f : a.m[(size_t(seq) * 2 + par) * a.H + h];
-	for (int t0 = 0; t0 < len; t0 += 1024) {
+	for (int t0 = 0; t0 < len; t0 += 4 * LG_THREADS) {
 		float f[4], in[4];
 		float F = 0.0f, M = -INFINITY;
 #pragma unroll
@@ -323,10 +399,10 @@ static __global__ void __launch_bounds__(256) lin_gates_kernel(LinArgs a) {
 				m = mn;
 			}
 		}
-		for (int w = 0; w < 8; w++) m0 = fmaxf(m0 + sF[w], sM[w]);
+		for (int w = 0; w < LG_THREADS / 32; w++) m0 = fmaxf(m0 + sF[w], sM[w]);
 		// (the carried maximum is the one the last token stored)
 		__syncthreads();
-		if (t0 + 1024 >= len) {
+		if (t0 + 4 * LG_THREADS >= len) {
 			if (tid == (len - 1 - t0) / 4) a.m[(size_t(seq) * 2 + (par ^ 1)) * a.H + h] = m;
 		}
 	}
@@ -810,8 +886,10 @@ static __global__ void __launch_bounds__(256, 2) lin_chunk_out_kernel(const __gr
 }
 
 // ------------------------------------------------------------------ norm and gate of the read-outs
-// out = parts of a row normed; gate before (o silu(z)) or after (times sigmoid(z)). A warp per (row, part).
-template <typename OT>
+// out = parts of a row normed; gate before (o silu(z)) or after (times sigmoid(z)). A warp per (row, part), V columns per
+// lane at a time; the first LN_HOLD of them stay in registers between the two uses.
+constexpr int LN_HOLD = 10;
+template <typename OT, int V>
 __global__ void __launch_bounds__(256) lin_norm_kernel(OT *out, int ldo, const float *o, int ldraw, const OT *gate, int ldg, const float *w, int R, int n, int parts,
                                                        int gate_first, float eps) {
 	pdl_trigger();
@@ -821,16 +899,49 @@ __global__ void __launch_bounds__(256) lin_norm_kernel(OT *out, int ldo, const f
 	const int r = i / parts, width = n / parts, c0 = (i % parts) * width;
 	const float *src = o + size_t(r) * ldraw + c0;
 	const OT *z = gate + size_t(r) * ldg + c0;
+	float v[LN_HOLD][V], g[LN_HOLD][V];
 	float q = 0.0f;
-	for (int c = lane; c < width; c += 32) {
-		const float v = gate_first ? src[c] * silu_f(to_f32(z[c])) : src[c];
-		q = fmaf(v, v, q);
+	auto take = [&](int c, float (&x)[V], float (&y)[V]) {  // y: the gate, x: what is normed
+		lin_load<V>(x, src + c);
+		lin_load<V>(y, z + c);
+	};
+	auto finish = [&](float (&x)[V], float (&y)[V]) {
+#pragma unroll
+		for (int e = 0; e < V; e++) {
+			const float s = lin_sigmoid<OT>(y[e]);
+			if (gate_first) x[e] *= y[e] * s;
+			y[e] = gate_first ? 1.0f : s;
+			q = fmaf(x[e], x[e], q);
+		}
+	};
+#pragma unroll
+	for (int j = 0; j < LN_HOLD; j++)
+		if (V * (lane + 32 * j) < width) take(V * (lane + 32 * j), v[j], g[j]);
+#pragma unroll
+	for (int j = 0; j < LN_HOLD; j++)
+		if (V * (lane + 32 * j) < width) finish(v[j], g[j]);
+	for (int c = V * (lane + 32 * LN_HOLD); c < width; c += 32 * V) {
+		float x[V], y[V];
+		take(c, x, y);
+		finish(x, y);
 	}
 	const float f = 1.0f / sqrtf(warp_sum(q) / float(width) + eps);
 	OT *dst = out + size_t(r) * ldo + c0;
-	for (int c = lane; c < width; c += 32) {
-		const float g = to_f32(z[c]), v = src[c] * f * w[c0 + c];
-		dst[c] = from_f32<OT>(v * (gate_first ? silu_f(g) : sigmoid_f(g)));
+	auto put = [&](int c, const float (&x)[V], const float (&y)[V]) {
+		float u[V];
+		lin_load<V>(u, w + c0 + c);
+#pragma unroll
+		for (int e = 0; e < V; e++) u[e] *= x[e] * f * y[e];
+		lin_store<V, OT>(dst + c, u);
+	};
+#pragma unroll
+	for (int j = 0; j < LN_HOLD; j++)
+		if (V * (lane + 32 * j) < width) put(V * (lane + 32 * j), v[j], g[j]);
+	for (int c = V * (lane + 32 * LN_HOLD); c < width; c += 32 * V) {
+		float x[V], y[V];
+		take(c, x, y);
+		finish(x, y);
+		put(c, x, y);
 	}
 }
 

@@ -129,9 +129,11 @@ __global__ void __launch_bounds__(128) row_norm_kernel(OT *out, int ldo, const f
 // first. hist: [B][2][taps-1][D]. Rows before a sequence's start count as zero, whatever hist holds.
 // Two kernels: mean (0 for an RMS norm) and 1/deviation of every row, then a walk down the rows with the window in registers, four
 // channels per thread, LC_ROWS rows per CTA (the rows before them are normed again, not exchanged).
-// The statistics kernel may first add what the chosen experts of the preceding layer put out (`add`): the row is read
-// here anyway.
-template <typename YT> struct ExpertSum {
+// The statistics kernel may first add what the preceding layer left to be added (`add`): the row is read here anyway.
+template <typename YT> struct RowSum {
+	const float *part;  // partial sums of a product whose K was shared, [n_part][rows][ldx]
+	int n_part;
+	size_t part_stride;
 	const YT *y;        // [slots][ldy] outputs of the experts, or null
 	int ldy, top;
 	const int *slot;    // [R][top]
@@ -145,7 +147,7 @@ __device__ __forceinline__ float4 load4(const __nv_bfloat16 *p) {
 	return make_float4(bf16_lo(u.x), bf16_hi(u.x), bf16_lo(u.y), bf16_hi(u.y));
 }
 template <typename YT>
-__global__ void __launch_bounds__(128) row_stats_kernel(float2 *stats, float *x, int ldx, int D, float eps, int rms, ExpertSum<YT> add) {
+__global__ void __launch_bounds__(128) row_stats_kernel(float2 *stats, float *x, int ldx, int D, float eps, int rms, RowSum<YT> add) {
 	pdl_trigger();
 	pdl_wait();
 	__shared__ float red[4];
@@ -163,6 +165,20 @@ __global__ void __launch_bounds__(128) row_stats_kernel(float2 *stats, float *x,
 			const int c = 4 * (tid + 128 * j);
 			v[j] = c < D ? *reinterpret_cast<const float4 *>(xr + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 		}
+		if (add.n_part) {
+			const float *p = add.part + size_t(blockIdx.x) * ldx;
+#pragma unroll
+			for (int j = 0; j < 8; j++) {
+				const int c = 4 * (tid + 128 * j);
+				if (c < D) {
+#pragma unroll 4
+					for (int e = 0; e < add.n_part; e++) {
+						const float4 u = *reinterpret_cast<const float4 *>(p + e * add.part_stride + c);
+						v[j].x += u.x; v[j].y += u.y; v[j].z += u.z; v[j].w += u.w;
+					}
+				}
+			}
+		}
 		if (add.y) {
 			for (int e = 0; e < add.top; e++) {
 				const YT *y = add.y + size_t(slot[e]) * add.ldy;
@@ -176,6 +192,8 @@ __global__ void __launch_bounds__(128) row_stats_kernel(float2 *stats, float *x,
 					}
 				}
 			}
+		}
+		if (add.y || add.n_part) {
 #pragma unroll
 			for (int j = 0; j < 8; j++)
 				if (4 * (tid + 128 * j) < D) *reinterpret_cast<float4 *>(xr + 4 * (tid + 128 * j)) = v[j];
@@ -192,10 +210,10 @@ __global__ void __launch_bounds__(128) row_stats_kernel(float2 *stats, float *x,
 	} else {
 		for (int c = tid; c < D; c += 128) {
 			float v = xr[c];
-			if (add.y) {
+			for (int e = 0; e < add.n_part; e++) v += add.part[e * add.part_stride + size_t(blockIdx.x) * ldx + c];
+			if (add.y)
 				for (int e = 0; e < add.top; e++) v = fmaf(wt[e], to_f32(add.y[size_t(slot[e]) * add.ldy + c]), v);
-				xr[c] = v;
-			}
+			if (add.y || add.n_part) xr[c] = v;
 			s += v;
 		}
 		mean = rms ? 0.0f : cta_sum<4>(s, red) / float(D);

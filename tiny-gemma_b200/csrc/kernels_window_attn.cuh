@@ -105,12 +105,24 @@ static __global__ void __launch_bounds__(256) kv_transform_kernel(WAttnArgs a, i
 		const int r = row0 + i - pos;
 		PT *row = const_cast<PT *>(reinterpret_cast<const PT *>(a.p)) + size_t(r) * a.ldp;
 		const float2 *cs = a.cs + size_t(r) * a.ld_cs;
-		for (int x = lane; x < per * half; x += 32) {
-			const int c = x % half;
-			PT *q = row + a.p_q + (g * per + x / half) * a.dkp + c;
-			const float u = to_f32(q[0]), v = to_f32(q[half]);
-			q[0] = from_f32<PT>(u * cs[c].x - v * cs[c].y);
-			q[half] = from_f32<PT>(v * cs[c].x + u * cs[c].y);
+		for (int c = lane; c < half; c += 32) {
+			const float2 t = cs[c];
+			PT *q = row + a.p_q + g * per * a.dkp + c;
+			for (int h0 = 0; h0 < per; h0 += 8) {  // (loads of eight heads ahead of their stores)
+				float u[8], v[8];
+#pragma unroll
+				for (int h = 0; h < 8; h++)
+					if (h0 + h < per) {
+						u[h] = to_f32(q[(h0 + h) * a.dkp]);
+						v[h] = to_f32(q[(h0 + h) * a.dkp + half]);
+					}
+#pragma unroll
+				for (int h = 0; h < 8; h++)
+					if (h0 + h < per) {
+						q[(h0 + h) * a.dkp] = from_f32<PT>(u[h] * t.x - v[h] * t.y);
+						q[(h0 + h) * a.dkp + half] = from_f32<PT>(v[h] * t.x + u[h] * t.y);
+					}
+			}
 		}
 		const size_t slot = size_t(seq) * a.cap + i % a.cap;
 		CT *kd = reinterpret_cast<CT *>(a.kc) + slot * nk + g * a.dkp, *vd = reinterpret_cast<CT *>(a.vc) + slot * nv + g * a.dvp;

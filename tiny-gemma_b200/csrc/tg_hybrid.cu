@@ -45,12 +45,13 @@ __global__ void __launch_bounds__(256) hybrid_token_mix_kernel(WAttnArgs w, Delt
 
 // One token per sequence, the feed-forward beside the mixer: the mixer's CTAs, then (few rows) those of the row's chosen
 // experts. grid (mixer CTAs + experts' CTAs, rows)
-template <typename PT, typename CT, typename OT, bool ATTN> __global__ void __launch_bounds__(256) beside_token_mix_kernel(WAttnArgs w, LinArgs l, MoeArgs e, int n_mix) {
+template <typename PT, typename CT, typename OT, bool ATTN, bool EXPERTS>
+__global__ void __launch_bounds__(256, ATTN || EXPERTS ? 2 : 4) beside_token_mix_kernel(WAttnArgs w, LinArgs l, MoeArgs e, int n_mix) {
 	pdl_trigger();
 	pdl_wait();
 	extern __shared__ __align__(16) float mix_sm[];
 	const int x = blockIdx.x;
-	if (x >= n_mix) expert_token_cta(e, blockIdx.y, x - n_mix, mix_sm);
+	if (EXPERTS && x >= n_mix) expert_token_cta(e, blockIdx.y, x - n_mix, mix_sm);
 	else if (ATTN) window_attn_token_cta<PT, CT, OT>(w, blockIdx.y, x / w.nsplit, x % w.nsplit, mix_sm);
 	else lin_token_cta<PT>(l, blockIdx.y, x, mix_sm);
 }
@@ -81,6 +82,13 @@ struct HybridState : tg_state {
 	};
 	std::vector<RunCache> cache;
 	std::vector<void *> mem;
+	// what a layer has computed but not yet added to x (the next norm does): its experts' outputs, partial sums
+	struct Left {
+		int experts = -1;  // layer
+		int parts = 0;
+	} left;
+	float *split_part = nullptr;  // [splits][rows][ldx]
+	size_t split_rows = 0;
 	// activations of a pass
 	float *x = nullptr;
 	int ldx = 0;
@@ -142,6 +150,8 @@ struct HybridState : tg_state {
 		float cap = 0.0f, limit = 0.0f;
 		int act = GLU_GELU, n32 = 0, ld32 = 0;
 		float *C32 = nullptr;
+		int splits = 0;         // GEMM_STORE32
+		int bn = 0;             // columns of a tile (0: the launcher chooses)
 		bool grouped = false;   // by expert: M is the most rows there can be, est the likely row tiles
 		int est = 0;
 	};
@@ -156,9 +166,10 @@ struct HybridState : tg_state {
 	int few_layer(const StepDesc &d, int run, int R);
 	int rows_layer(const StepDesc &d, int run, int R, int nseg, int max_len);
 	int beside_few_layer(const StepDesc &d, int run, int R);
-	int beside_rows_layer(const StepDesc &d, int run, int R, int nseg, int max_len, int pending);
-	int norm_in(const StepDesc &d, int run, int R, int pending);  // norm1 and what follows it; first adds layer `pending`'s experts (-1: none)
-	int add_experts(int layer, int R);
+	int beside_rows_layer(const StepDesc &d, int run, int R, int nseg, int max_len);
+	int norm_in(const StepDesc &d, int run, int R);  // what is left is added; norm1 and what follows it
+	int add_left(int R);
+	template <typename T> RowSum<T> row_sum(int R);
 	int attn_rows(const WAttnArgs &wa, int run, int R, int nseg, int max_len);
 	int token_splits(const WAttnArgs &wa, int fill) const;
 
@@ -220,6 +231,26 @@ int pick_bn(int m_tiles, int N) {
 	return best;
 }
 
+// The same for a product whose K several CTAs may share, their partial sums being added later: what a tile costs is its
+// K-blocks and a fixed part, and a partial sum is written and read once more.
+void pick_split(int M, int N, int K, int *bn, int *splits) {
+	static const int most = env_int("TG_SPLIT_K", 8);
+	const int m_tiles = (M + GB_BM - 1) / GB_BM, kb = (K + GB_BK - 1) / GB_BK;
+	double best = 1e30;
+	for (int b : {256, 128, 64})
+		for (int s = 1; s <= std::min(most, std::max(1, kb / 4)); s++) {
+			if ((s - 1) * ((kb + s - 1) / s) >= kb) continue;  // (every share has work)
+			const int tiles = m_tiles * ((N + b - 1) / b) * s;
+			const double c = double((tiles + g_num_sms - 1) / g_num_sms) * ((kb + s - 1) / s + 4) * (b == 256 ? 0.35 : (b == 128 ? 0.275 : 0.21))  // us
+			                 + (s > 1 ? 1.0 + s * double(M) * N * 8.0 / 6e6 : 0.0);
+			if (c < best) {
+				best = c;
+				*bn = b;
+				*splits = s;
+			}
+		}
+}
+
 template <int BN, int EPI, bool GRP> int launch_gemm_tc(const CUtensorMap &am, const CUtensorMap &wm, const GemmArgs &a, cudaStream_t st) {
 	static bool done[TG_MAX_DEVICES] = {};
 	bool &d = done[current_device_slot()];
@@ -228,14 +259,14 @@ template <int BN, int EPI, bool GRP> int launch_gemm_tc(const CUtensorMap &am, c
 		TG_TRY(allow_smem(kernel, GbShape<BN>::SMEM));
 		d = true;
 	}
-	launch_k(kernel, dim3(std::min(g_num_sms, a.m_tiles * a.n_tiles)), dim3(GB_THREADS), size_t(GbShape<BN>::SMEM), st, am, wm, a);
+	launch_k(kernel, dim3(std::min(g_num_sms, a.m_tiles * a.n_tiles * std::max(1, a.splits))), dim3(GB_THREADS), size_t(GbShape<BN>::SMEM), st, am, wm, a);
 	count_launch();
 	return check_launch("gemm_bf16_tc");
 }
 // est: row tiles that a grouped product is likely to have
-template <int EPI, bool GRP = false> int launch_gemm(const CUtensorMap &am, const Lin &w, GemmArgs a, cudaStream_t st, int est = 0) {
+template <int EPI, bool GRP = false> int launch_gemm(const CUtensorMap &am, const Lin &w, GemmArgs a, cudaStream_t st, int est = 0, int want_bn = 0) {
 	a.m_tiles = (a.M + GB_BM - 1) / GB_BM;
-	const int cols = EPI == GEMM_LOGITS ? a.ldc : a.N, bn = pick_bn(est ? est : a.m_tiles, cols);
+	const int cols = EPI == GEMM_LOGITS ? a.ldc : a.N, bn = want_bn ? want_bn : pick_bn(est ? est : a.m_tiles, cols);
 	a.n_tiles = (cols + bn - 1) / bn;
 	if (bn == 256) return launch_gemm_tc<256, EPI, GRP>(am, w.map[2], a, st);
 	if (bn == 128) return launch_gemm_tc<128, EPI, GRP>(am, w.map[1], a, st);
@@ -362,6 +393,10 @@ int HybridState::alloc() {
 		const size_t nb = size_t(R) / DB + B + 1;
 		TG_TRY(take(&blk, nb * blkn));
 		TG_TRY(take(&bV, nb * blkV));
+	}
+	if (beside && !f32) {
+		split_rows = std::min(size_t(8) * R, size_t(4096));
+		TG_TRY(take(&split_part, split_rows * ldx));
 	}
 	if (linH) {
 		if (xcn) TG_TRY(take_act(&xc, size_t(R) * xcn));
@@ -561,6 +596,7 @@ int HybridState::gemm(int epi, const void *A, int lda, const CUtensorMap *am, co
 	a.ld32 = o.ld32;
 	a.tile_expert = moe.tile_expert;
 	a.n_row_tiles = moe.n_tiles;
+	a.splits = o.splits;
 	if (f32) {
 		const float *Af = static_cast<const float *>(A);
 		switch (epi) {
@@ -573,7 +609,7 @@ int HybridState::gemm(int epi, const void *A, int lda, const CUtensorMap *am, co
 	if (o.grouped) return epi == GEMM_GLU ? launch_gemm<GEMM_GLU, true>(*am, w, a, stream, o.est) : launch_gemm<GEMM_STORE, true>(*am, w, a, stream, o.est);
 	switch (epi) {
 		case GEMM_STORE: return launch_gemm<GEMM_STORE>(*am, w, a, stream);
-		case GEMM_STORE32: return launch_gemm<GEMM_STORE32>(*am, w, a, stream);
+		case GEMM_STORE32: return launch_gemm<GEMM_STORE32>(*am, w, a, stream, 0, o.bn);
 		case GEMM_ADD: return launch_gemm<GEMM_ADD>(*am, w, a, stream);
 		case GEMM_GLU: return launch_gemm<GEMM_GLU>(*am, w, a, stream);
 		default: return launch_gemm<GEMM_LOGITS>(*am, w, a, stream);
@@ -586,7 +622,7 @@ int HybridState::gemv(int pro, int epi, GemvArgs g, int R) {
 	g.embed_scale = m->embed_scale;
 	// (rows whose activations do not fit shared memory together go in smaller groups)
 	int most = R >= 4 ? 4 : (R >= 2 ? 2 : 1);
-	const size_t row_floats = size_t(epi == GV_FRONT ? 2 : 1) * 8 * gv_k8(g.K) + (pro == GV_MIX ? g.top * g.n_ex : 0);
+	const size_t row_floats = size_t(epi == GV_FRONT ? 3 : (pro == GV_LN_CONV ? 2 : 1)) * 8 * gv_k8(g.K) + (pro == GV_MIX ? g.top * g.n_ex : 0);
 	while (most > 1 && most * row_floats * 4 > 160 * 1024) most /= 2;
 	for (int r = 0; r < R;) {
 		int n = most;
@@ -826,7 +862,7 @@ template <typename PT> int launch_delta(const DeltaArgs &a, int R, int nseg, int
 	count_launch();
 	return check_launch("delta_out");
 }
-template <typename PT> int launch_stats(float2 *stats, float *x, int ldx, int R, int D, float eps, int rms, const ExpertSum<PT> &add, cudaStream_t st) {
+template <typename PT> int launch_stats(float2 *stats, float *x, int ldx, int R, int D, float eps, int rms, const RowSum<PT> &add, cudaStream_t st) {
 	launch_k(row_stats_kernel<PT>, dim3(R), dim3(128), 0, st, stats, x, ldx, D, eps, rms, add);
 	count_launch();
 	return check_launch("row_stats");
@@ -858,28 +894,30 @@ template <typename PT, typename CT, typename OT> int launch_beside_mix(const WAt
 	const dim3 grid(n_mix + n_exp, R);
 	const WAttnArgs wa = w ? *w : WAttnArgs{};
 	const LinArgs la = l ? *l : LinArgs{};
-	if (w) {
-		auto kernel = beside_token_mix_kernel<PT, CT, OT, true>;
+	auto go = [&](auto kernel) -> int {
 		TG_TRY(allow_smem(kernel, smem));
 		launch_k(kernel, grid, dim3(256), smem, st, wa, la, e, n_mix);
-	} else {
-		auto kernel = beside_token_mix_kernel<PT, CT, OT, false>;
-		TG_TRY(allow_smem(kernel, smem));
-		launch_k(kernel, grid, dim3(256), smem, st, wa, la, e, n_mix);
-	}
+		return TG_OK;
+	};
+	if (w) TG_TRY(n_exp ? go(beside_token_mix_kernel<PT, CT, OT, true, true>) : go(beside_token_mix_kernel<PT, CT, OT, true, false>));
+	else TG_TRY(n_exp ? go(beside_token_mix_kernel<PT, CT, OT, false, true>) : go(beside_token_mix_kernel<PT, CT, OT, false, false>));
 	count_launch();
 	return check_launch("beside_token_mix");
 }
-// portions of a recurrence: raw read-outs of all rows
-template <typename PT> int launch_lin_rows(const LinArgs &a, int R, int nseg, int max_len, cudaStream_t st) {
-	if (a.kind == LIN_SSM) {
-		const dim3 grid((R + LV_ROWS - 1) / LV_ROWS, (a.ldxc + 127) / 128);
-		if (a.taps <= 4) launch_k(lin_conv_kernel<PT, 4>, grid, dim3(128), 0, st, a, R);
-		else launch_k(lin_conv_kernel<PT, 16>, grid, dim3(128), 0, st, a, R);
-		count_launch();
-		TG_TRY(check_launch("lin_conv"));
-	}
-	launch_k(lin_gates_kernel, dim3(a.H, nseg), dim3(256), 0, st, a);
+// portions of a recurrence: its inputs
+template <typename PT, int V> int launch_lin_conv(const LinArgs &a, int R, cudaStream_t st) {
+	const int cols = (a.ldxc + 128 * V - 1) / (128 * V) + 1;
+	int rows = LV_ROWS;
+	while (rows > 1 && (R + rows - 1) / rows * cols < 4 * g_num_sms) rows /= 2;
+	const dim3 grid((R + rows - 1) / rows, cols);
+	if (a.taps <= 4) launch_k(lin_conv_kernel<PT, 4, V>, grid, dim3(128), 0, st, a, R, rows);
+	else launch_k(lin_conv_kernel<PT, 16, V>, grid, dim3(128), 0, st, a, R, rows);
+	count_launch();
+	return check_launch("lin_conv");
+}
+template <typename PT> int launch_lin_inputs(const LinArgs &a, int R, int nseg, cudaStream_t st) {
+	if (a.kind == LIN_SSM) return a.vd % 4 == 0 && a.N % 4 == 0 && a.p_x % 4 == 0 ? launch_lin_conv<PT, 4>(a, R, st) : launch_lin_conv<PT, 1>(a, R, st);
+	launch_k(lin_gates_kernel, dim3(a.H, nseg), dim3(LG_THREADS), 0, st, a);
 	count_launch();
 	return check_launch("lin_gates");
 }
@@ -910,8 +948,12 @@ int launch_lin_chunks(LinArgs a, const CUtensorMap &rows, const CUtensorMap &sh,
 }
 template <typename T> int launch_lin_norm(const LinArgs &a, const Layer &L, void *O, const void *P, int R, float eps, cudaStream_t st) {
 	const int n = a.H * a.vd;
-	launch_k(lin_norm_kernel<T>, dim3((R * L.li.parts + 7) / 8), dim3(256), 0, st, static_cast<T *>(O), L.kcat, a.o, a.ldo, static_cast<const T *>(P) + L.p_z, L.ldp, L.rnorm, R, n,
-	         L.li.parts, a.kind == LIN_SSM ? 1 : 0, eps);
+	auto go = [&](auto kernel) {
+		launch_k(kernel, dim3((R * L.li.parts + 7) / 8), dim3(256), 0, st, static_cast<T *>(O), L.kcat, a.o, a.ldo, static_cast<const T *>(P) + L.p_z, L.ldp, L.rnorm, R, n,
+		         L.li.parts, a.kind == LIN_SSM ? 1 : 0, eps);
+	};
+	if (n / L.li.parts % 4 == 0 && L.p_z % 4 == 0) go(lin_norm_kernel<T, 4>);
+	else go(lin_norm_kernel<T, 1>);
 	count_launch();
 	return check_launch("lin_norm");
 }
@@ -1021,7 +1063,7 @@ int HybridState::rows_layer(const StepDesc &d, int run, int R, int nseg, int max
 	const int li = m->runs[run].layer, D = m->D;
 	const Layer &L = m->layers[li];
 	const bool single = max_len == 1;
-	TG_TRY(norm_in(d, run, R, -1));
+	TG_TRY(norm_in(d, run, R));
 	TG_TRY(gemm(GEMM_STORE, h, m->Dp, &hmap, L.proj, R, P, L.ldp));
 	WAttnArgs wa = attn_args(d, run, P, L.ldp, O, L.kc);
 	const DeltaArgs da = delta_args(d, run, P, L.ldp, O, L.kc);
@@ -1139,12 +1181,12 @@ int HybridState::beside_few_layer(const StepDesc &d, int run, int R) {
 	return gemv(GV_MIX, GV_ADD, o, R);
 }
 
-int HybridState::beside_rows_layer(const StepDesc &d, int run, int R, int nseg, int max_len, int pending) {
+int HybridState::beside_rows_layer(const StepDesc &d, int run, int R, int nseg, int max_len) {
 	const int li = m->runs[run].layer;
 	const Layer &L = m->layers[li];
 	const FfSpec &F = L.ff;
 	const bool single = max_len == 1;
-	TG_TRY(norm_in(d, run, R, pending));
+	TG_TRY(norm_in(d, run, R));
 	GemmOpt po;
 	po.n32 = L.n32;
 	po.ld32 = L.tail();
@@ -1167,13 +1209,17 @@ int HybridState::beside_rows_layer(const StepDesc &d, int run, int R, int nseg, 
 			TG_TRY(attn_rows(wa, run, R, nseg, max_len));
 		}
 	} else {
-		const LinArgs la = lin_args(d, run, P);
+		LinArgs la = lin_args(d, run, P);
 		if (single) {
+			if (la.kind == LIN_SSM) {
+				la.ready = 1;
+				TG_TRY(f32 ? launch_lin_inputs<float>(la, R, nseg, stream) : launch_lin_inputs<bf16>(la, R, nseg, stream));
+			}
 			if (f32) TG_TRY((launch_beside_mix<float, float, float>(nullptr, &la, MoeArgs{}, 0, R, stream)));
 			else TG_TRY((launch_beside_mix<bf16, bf16, bf16>(nullptr, &la, MoeArgs{}, 0, R, stream)));
 		} else {
-			if (f32) TG_TRY(launch_lin_rows<float>(la, R, nseg, max_len, stream));
-			else TG_TRY(launch_lin_rows<bf16>(la, R, nseg, max_len, stream));
+			if (f32) TG_TRY(launch_lin_inputs<float>(la, R, nseg, stream));
+			else TG_TRY(launch_lin_inputs<bf16>(la, R, nseg, stream));
 			if (lin_tc && la.Np <= 256 && max_len > LIN_SCAN_MAX)
 				TG_TRY(launch_lin_chunks(la, la.kind == LIN_SSM ? xcmap[li] : pmap[li], shmap[li], slmap[li], nseg, max_len, stream));
 			else if (f32) TG_TRY(launch_lin_scan<float>(la, nseg, stream));
@@ -1194,7 +1240,8 @@ int HybridState::beside_rows_layer(const StepDesc &d, int run, int R, int nseg, 
 	}
 	if (F.experts) {
 		const MoeArgs ma = moe_args(L);
-		launch_k(route_kernel, dim3((R + 7) / 8), dim3(256), 0, stream, ma, R);
+		const int rounds = std::max(1, std::min(MR_ROUNDS, R / (8 * g_num_sms)));
+		launch_k(route_kernel, dim3((R + 8 * rounds - 1) / (8 * rounds)), dim3(256), 0, stream, ma, R, rounds);
 		count_launch();
 		TG_TRY(check_launch("route"));
 		if (f32) TG_TRY(launch_gather<float>(ma, hp, m->Dp, xg, R, stream));
@@ -1208,23 +1255,41 @@ int HybridState::beside_rows_layer(const StepDesc &d, int run, int R, int nseg, 
 		TG_TRY(gemm(GEMM_GLU, xg, m->Dp, &xgmap, L.ex_gu, most, xa, F.effp, eo));
 		TG_TRY(gemm(GEMM_STORE, xa, F.effp, f32 ? nullptr : &xamap[li], L.ex_down, most, xy, ldx, eo));
 	}
+	int bn = 0, splits = 1;
+	if (!f32) pick_split(R, m->D, L.kcat, &bn, &splits);
+	left.experts = F.experts ? li : -1;
+	if (splits > 1 && size_t(splits) * R <= split_rows) {
+		GemmOpt so;
+		so.splits = left.parts = splits;
+		so.bn = bn;
+		return gemm(GEMM_STORE32, O, L.kcat, &omap[li], L.out, R, split_part, ldx, so);
+	}
 	return gemm(GEMM_ADD, O, L.kcat, f32 ? nullptr : &omap[li], L.out, R, x, ldx);
 }
 
-int HybridState::norm_in(const StepDesc &d, int run, int R, int pending) {
+template <typename T> RowSum<T> HybridState::row_sum(int R) {
+	RowSum<T> add{};
+	if (left.experts >= 0) {
+		add.y = static_cast<const T *>(xy);
+		add.ldy = ldx;
+		add.top = m->layers[left.experts].ff.top;
+		add.slot = moe.place;
+		add.w = moe.w;
+	}
+	add.part = split_part;
+	add.n_part = left.parts;
+	add.part_stride = size_t(R) * ldx;
+	left = Left();
+	return add;
+}
+
+int HybridState::norm_in(const StepDesc &d, int run, int R) {
 	const Layer &L = m->layers[m->runs[run].layer];
 	float *hist = cache[run].canon;
 	void *plain = L.beside ? hp : nullptr;
 	auto go = [&](auto t) -> int {
 		typedef decltype(t) T;
-		ExpertSum<T> add{};
-		if (pending >= 0) {
-			add.y = static_cast<const T *>(xy);
-			add.ldy = ldx;
-			add.top = m->layers[pending].ff.top;
-			add.slot = moe.place;
-			add.w = moe.w;
-		}
+		RowSum<T> add = row_sum<T>(R);
 		if (L.ff.experts) {
 			add.zero = moe.count;
 			add.n_zero = L.ff.experts;
@@ -1235,19 +1300,11 @@ int HybridState::norm_in(const StepDesc &d, int run, int R, int pending) {
 	return f32 ? go(0.0f) : go(bf16());
 }
 
-// adds the outputs of a layer's experts to the stream (where no norm follows that would do it)
-int HybridState::add_experts(int layer, int R) {
-	auto go = [&](auto t) -> int {
-		typedef decltype(t) T;
-		ExpertSum<T> add{};
-		add.y = static_cast<const T *>(xy);
-		add.ldy = ldx;
-		add.top = m->layers[layer].ff.top;
-		add.slot = moe.place;
-		add.w = moe.w;
-		return launch_stats<T>(stats, x, ldx, R, m->D, m->eps, m->rms, add, stream);
-	};
-	return f32 ? go(0.0f) : go(bf16());
+// adds to the stream what is left to be added (where no norm follows that would do it)
+int HybridState::add_left(int R) {
+	if (left.experts < 0 && !left.parts) return TG_OK;
+	if (f32) return launch_stats<float>(stats, x, ldx, R, m->D, m->eps, m->rms, row_sum<float>(R), stream);
+	return launch_stats<bf16>(stats, x, ldx, R, m->D, m->eps, m->rms, row_sum<bf16>(R), stream);
 }
 
 // All layers for R rows in nseg segments (the longest: max_len), leaving the residual stream in x.
@@ -1266,20 +1323,16 @@ int HybridState::run_layers(const StepDesc &d, int R, int nseg, int max_len) {
 		count_launch();
 		TG_TRY(check_launch("rope_table"));
 	}
-	int pending = -1;  // the layer whose experts' outputs are not in x yet
+	left = Left();
 	for (size_t run = 0; run < m->runs.size(); run++) {
 		const Layer &L = m->layers[m->runs[run].layer];
 		if (few) {
 			TG_TRY(L.beside ? beside_few_layer(d, int(run), R) : few_layer(d, int(run), R));
 		} else {
 			if (m->runs[run].add_embed) TG_TRY(embed_rows(1));
-			if (L.beside) TG_TRY(beside_rows_layer(d, int(run), R, nseg, max_len, pending));
+			if (L.beside) TG_TRY(beside_rows_layer(d, int(run), R, nseg, max_len));
 			else TG_TRY(rows_layer(d, int(run), R, nseg, max_len));
-			pending = L.beside && L.ff.experts ? m->runs[run].layer : -1;
-			if (pending >= 0 && (tracing || run + 1 == m->runs.size())) {
-				TG_TRY(add_experts(pending, R));
-				pending = -1;
-			}
+			if (tracing || run + 1 == m->runs.size()) TG_TRY(add_left(R));
 		}
 		if (tracing) {
 			const size_t at = trace.size();

@@ -194,15 +194,19 @@ def mt19937_uniforms(n: int, seed: int) -> np.ndarray:
     return out.astype(np.float32)
 
 
-# ------------------------------------------------------------------ Nabelix model folders
+# ------------------------------------------------------------------ model folders
+#                 width    ff layers  vocab
+LAYERED_SIZES = {"270m": (640, 2048, 18, 262144),
+                 "1B": (1152, 6912, 26, 262144),
+                 "3B": (2560, 9216, 24, 65536)}
+
+
+# ---- Nabelix
 def nabelix_config(name: str) -> dict:
     """config.json of layers that resemble a real model's: the widths, feed-forward sizes, depths and vocabularies of
     the Gemma-3 sizes above (a few more weights per layer than theirs), and a wider one"""
-    #          width    ff layers  vocab  left heads/kv  right heads
-    sizes = {"270m": (640, 2048, 18, 262144, 4, 1, 4),
-             "1B": (1152, 6912, 26, 262144, 8, 2, 4),
-             "3B": (2560, 9216, 24, 65536, 20, 4, 20)}
-    width, ff, n, vocab, h, g, r = sizes[name]
+    width, ff, n, vocab = LAYERED_SIZES[name]
+    h, g, r = {"270m": (4, 1, 4), "1B": (8, 2, 4), "3B": (20, 4, 20)}[name]  # left heads, its key/value heads, right heads
     layer = {"type": "parallel", "mlp": {"kind": "dense", "ff": ff},
              "mixer": {"left_scale": 1.0, "right_scale": 1.0,
                        "left": {"heads": h, "kv_heads": g, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
@@ -252,7 +256,73 @@ def nabelix_shapes(cfg: dict):
     yield "final.norm", (D,)
 
 
-def write_random_nabelix(folder: str, cfg: dict, seed: int = 0) -> str:
+# ---- Sominex
+def sominex_config(name: str) -> dict:
+    """the same widths, feed-forward sizes, depths and vocabularies; layers in turns of attention, Mamba-2, mLSTM and
+    Mamba-2, the Mamba-2 ones with a mixture of experts of which a token uses as many weights as the dense layers have"""
+    width, ff, n, vocab = LAYERED_SIZES[name]
+    h, g, groups, lh = {"270m": (4, 1, 2, 4), "1B": (8, 2, 2, 4), "3B": (20, 4, 4, 10)}[name]
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": ff // 8}, "router": {"experts": 32, "top": 4, "scale": 1.0}, "shared": {"ff": ff // 2}}
+    rot = {"base": 10000.0, "dims": 128, "scaling": {"factor": 4.0, "fast": 32.0, "slow": 1.0, "original": 4096}}
+    attention = {"type": "attention", "mlp": dense,
+                 "mixer": {"heads": h, "kv_heads": g, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "rot": rot,
+                           "mask": {"size": 512, "pool": 16}}}
+    mamba = {"type": "mamba2", "mlp": moe,
+             "mixer": {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": groups, "conv": 4, "norm_groups": groups}}
+    mlstm = {"type": "mlstm", "mlp": dense, "mixer": {"heads": lh, "dim": 128, "vdim": 256, "gate_cap": 15.0}}
+    turn = [attention, mamba, mlstm, mamba]
+    return {"architecture": "Sominex", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "layers": [turn[i % 4] for i in range(n)]}
+
+
+def sominex_shapes(cfg: dict):
+    """(tensor name, shape) of every tensor of a Sominex model"""
+    D = cfg["width"]
+    yield "embed", (cfg["vocab"], D)
+    for i, sp in enumerate(cfg["layers"]):
+        p, m, c, ff = "l%d." % i, "l%d.mix." % i, sp["mixer"], sp["mlp"]
+        yield p + "norm1", (D,)
+        yield p + "shift", (D,)
+        if sp["type"] == "attention":
+            out = c["heads"] * c["vdim"]
+            for n, rows in (("q", c["heads"] * c["dim"]), ("k", c["kv_heads"] * c["dim"]), ("v", c["kv_heads"] * c["vdim"])):
+                yield m + n, (rows, D)
+        elif sp["type"] == "mamba2":
+            out = c["heads"] * c["vdim"]
+            ch = out + 2 * c["groups"] * c["state"]
+            yield m + "in", (out + ch + c["heads"], D)
+            yield m + "conv", (ch, c["conv"])
+            yield m + "conv.b", (ch,)
+            for n in ("dt_bias", "A_log", "D"):
+                yield m + n, (c["heads"],)
+            yield m + "norm", (out,)
+        else:
+            out = c["heads"] * c["vdim"]
+            for n, rows in (("q", c["heads"] * c["dim"]), ("k", c["heads"] * c["dim"]), ("v", out), ("g", out), ("i", c["heads"]), ("f", c["heads"])):
+                yield m + n, (rows, D)
+            yield m + "i.b", (c["heads"],)
+            yield m + "f.b", (c["heads"],)
+            yield m + "norm", (out,)
+        yield m + "o", (D, out)
+        parts = []
+        if ff and ff["kind"] == "dense":
+            parts = [("", ff["ff"])]
+        elif ff:
+            yield p + "mlp.router", (ff["router"]["experts"], D)
+            parts = [("e%d." % e, ff["expert"]["ff"]) for e in range(ff["router"]["experts"])] + [("shared.", ff["shared"]["ff"])]
+        for q, n in parts:
+            yield p + "mlp." + q + "gate", (n, D)
+            yield p + "mlp." + q + "up", (n, D)
+            yield p + "mlp." + q + "down", (D, n)
+    yield "final.norm", (D,)
+    yield "head", (cfg["vocab"], D)
+
+
+LAYERED = {"Nabelix": (nabelix_config, nabelix_shapes), "Sominex": (sominex_config, sominex_shapes)}
+
+
+def write_random_layered(folder: str, cfg: dict, seed: int = 0) -> str:
     """config.json and model.safetensors with seeded random bfloat16 weights. Matrices are N(0, 1/columns), cut from one
     block of random numbers at random offsets (drawing billions of them would take minutes)."""
     import json
@@ -270,7 +340,7 @@ def write_random_nabelix(folder: str, cfg: dict, seed: int = 0) -> str:
         os.unlink(done)
     g = np.random.default_rng(seed)
     block = g.standard_normal(1 << 24, dtype=np.float32)
-    shapes = list(nabelix_shapes(cfg))
+    shapes = list(LAYERED[cfg["architecture"]][1](cfg))
     head, at = {}, 0
     for name, shape in shapes:
         n = 2 * int(np.prod(shape))
@@ -290,8 +360,10 @@ def write_random_nabelix(folder: str, cfg: dict, seed: int = 0) -> str:
         for name, shape in shapes:
             n = int(np.prod(shape))
             if len(shape) == 1:
-                leaf = name.rsplit(".", 1)[-1]
-                x = {"A_log": g.uniform(-3, 0, n), "dt_bias": g.uniform(-4, 0, n), "r1": g.uniform(0.1, 1, n), "r2": g.uniform(0.1, 1, n)}.get(
+                leaf = name.split(".mix.")[-1]
+                leaf = leaf if leaf in ("i.b", "f.b", "conv.b") else leaf.rsplit(".", 1)[-1]
+                x = {"A_log": g.uniform(-3, 0, n), "dt_bias": g.uniform(-4, 0, n), "r1": g.uniform(0.1, 1, n), "r2": g.uniform(0.1, 1, n),
+                     "shift": g.uniform(0, 1, n), "i.b": g.uniform(-3, 0, n), "f.b": g.uniform(2, 6, n), "conv.b": 0.1 * g.standard_normal(n)}.get(
                     leaf, 1.0 + 0.1 * g.standard_normal(n))
                 f.write(bf16(x).tobytes())
                 continue
