@@ -130,7 +130,7 @@ struct HybridModel : tg_model {
 	std::vector<tg::Layer> layers;
 	std::vector<tg::Run> runs;
 	std::vector<tg::Rotation> rots;
-	int rot_half = 0;             // most pairs of a rotation
+	int rot_half = 0;             // most pairs of a rotation, an even number
 	double *rot_freq = nullptr;   // [rotations][rot_half]
 	float *rot_factor = nullptr;  // [rotations]
 	tg::Lin embed, head;          // head: the output matrix (the embedding's, if tied)
@@ -637,7 +637,7 @@ inline int read_sominex(const json::Value &c, HybridModel *m) {
 					A.rot = int(std::find(m->rots.begin(), m->rots.end(), t) - m->rots.begin());
 					if (size_t(A.rot) == m->rots.size()) m->rots.push_back(t);
 					A.rot_dims = t.dims;
-					m->rot_half = std::max(m->rot_half, t.dims / 2);
+					m->rot_half = std::max(m->rot_half, round_up(t.dims / 2, 2));
 				}
 			}
 		} else if (type == "mamba2" || type == "mlstm") {

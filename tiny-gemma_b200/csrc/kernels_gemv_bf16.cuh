@@ -70,9 +70,9 @@ struct GemvArgs {
 constexpr int GV_THREADS = 256;
 __host__ __device__ inline int gv_k8(int K) { return (K + 7) / 8; }
 template <int R, int NR> __host__ __device__ constexpr int gv_red_floats() { return 2 * 8 * NR * R; }
-template <int R, int NR> size_t gv_smem(int K, int pro, int epi, int parts, int ex) {
+template <int R, int NR> size_t gv_smem(int K, int pro, int epi, int parts, int top, int ex) {
 	const size_t rows = epi == GV_FRONT ? 2 * R : R, extra = pro == GV_LN ? 1 : (pro == GV_LN_CONV ? 1 + R : 0);
-	return ((rows + extra) * 8 * gv_k8(K) + gv_red_floats<R, NR>() + 32 + (pro == GV_MIX ? size_t(R) * ((parts + 3) / 4 * 4 + ex) : 0)) * 4;
+	return ((rows + extra) * 8 * gv_k8(K) + gv_red_floats<R, NR>() + 32 + (pro == GV_MIX ? size_t(R) * ((parts + 3) / 4 * 4 + ex + top) : 0)) * 4;
 }
 
 // sum over the threads of a row (8 / R warps), in every one of them
@@ -100,6 +100,7 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 	float *wn = bred + 32, *hc = wn + 8 * K8;            // norm weight (x its factor in the convolution); history's share
 	float *xp = hc + size_t(R) * 8 * K8;                 // GV_FRONT: the plain norms, laid out as xs
 	float *prt = bred + 32, *xe = prt + (PRO == GV_MIX ? R * ((a.parts + 3) / 4 * 4) : 0);  // GV_MIX: 1 / deviation of the parts; experts' activations
+	int *xid = reinterpret_cast<int *>(xe + (PRO == GV_MIX ? R * a.top * a.n_ex : 0));  // the rows' chosen experts
 	constexpr int SETS = 8 / KS, GROUP = SETS * NR;      // weight rows per CTA and group
 	const int set = warp / KS, ks = warp % KS;
 	const int n_out = EPI == GV_GLU ? a.N / 2 : (EPI == GV_LOGITS ? a.ldo : a.N);
@@ -183,6 +184,7 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 			float4 *dst = reinterpret_cast<float4 *>(xe + r * a.top * a.n_ex);
 			const float4 *src = reinterpret_cast<const float4 *>(a.ex_act + size_t(r) * a.top * a.n_ex);
 			const float *ew = a.ex_w + r * a.top;
+			for (int u = t; u < a.top; u += TG) xid[r * a.top + u] = a.ex_id[r * a.top + u];
 #pragma unroll 4
 			for (int u = t; u < all4; u += TG) {
 				const float4 v = src[u];
@@ -328,19 +330,24 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_bf16_kernel(GemvArgs a) {
 #pragma unroll
 			for (int i = 0; i < NR; i++) cur[i] = nxt[i];
 		}
-		if (PRO == GV_MIX && a.top) {  // each row's own experts: 16 bytes of (expert, k) per lane
+		if (PRO == GV_MIX && a.top) {  // each row's own experts: 16 bytes of (expert, k) per lane, the rows' loads together
 			const int e8 = a.n_ex / 8, n0 = grp * GROUP + set * NR;
+			for (int j = ks * 32 + lane; j < a.top * e8; j += 32 * KS) {
+				const int k = j / e8, o = 8 * (j % e8);
+				int4 w[R][NR];
 #pragma unroll
-			for (int r = 0; r < R; r++) {
-				const float *xv = xe + r * a.top * a.n_ex;
-#pragma unroll 2
-				for (int j = ks * 32 + lane; j < a.top * e8; j += 32 * KS) {
-					const __nv_bfloat16 *w = a.ex_W + size_t(a.ex_id[r * a.top + j / e8]) * a.N * a.ld_ex + 8 * (j % e8);
-					const float4 x0 = *reinterpret_cast<const float4 *>(xv + 8 * j), x1 = *reinterpret_cast<const float4 *>(xv + 8 * j + 4);
+				for (int r = 0; r < R; r++) {
+					const __nv_bfloat16 *W = a.ex_W + size_t(xid[r * a.top + k]) * a.N * a.ld_ex + o;
+#pragma unroll
+					for (int i = 0; i < NR; i++) w[r][i] = n0 + i < a.N ? ld_stream_int4(W + size_t(n0 + i) * a.ld_ex) : make_int4(0, 0, 0, 0);
+				}
+#pragma unroll
+				for (int r = 0; r < R; r++) {
+					const float *xv = xe + r * a.top * a.n_ex + 8 * j;
+					const float4 x0 = *reinterpret_cast<const float4 *>(xv), x1 = *reinterpret_cast<const float4 *>(xv + 4);
 #pragma unroll
 					for (int i = 0; i < NR; i++) {
-						if (n0 + i >= a.N) break;
-						const int4 v = ld_stream_int4(w + size_t(n0 + i) * a.ld_ex);
+						const int4 &v = w[r][i];
 						float s = acc[r][i];
 						s = fmaf(bf16_lo(v.x), x0.x, s);
 						s = fmaf(bf16_hi(v.x), x0.y, s);

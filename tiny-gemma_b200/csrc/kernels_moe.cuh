@@ -116,12 +116,12 @@ static __global__ void __launch_bounds__(256) route_kernel(MoeArgs a, int R, int
 	}
 }
 
-// grid ceil(R / MG_ROWS), 128 threads: h rows of ldh (a multiple of 8) -> xg[slot]
+// grid ceil(R / rows), 128 threads, rows <= MG_ROWS: h rows of ldh (a multiple of 8) -> xg[slot]
 constexpr int MG_ROWS = 4;
-template <typename T> __global__ void __launch_bounds__(128) expert_gather_kernel(MoeArgs a, const T *h, int ldh, T *xg, int R) {
+template <typename T> __global__ void __launch_bounds__(128) expert_gather_kernel(MoeArgs a, const T *h, int ldh, T *xg, int R, int rows) {
 	pdl_trigger();
 	pdl_wait();
-	__shared__ int first[MOE_MAX + 1], part[4];
+	__shared__ int first[MOE_MAX], part[4], slot[MG_ROWS * MOE_TOP];
 	const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
 	// first tile of every expert: thread t owns experts 4 t .. 4 t + 3
 	int c[4], sum = 0;
@@ -130,6 +130,8 @@ template <typename T> __global__ void __launch_bounds__(128) expert_gather_kerne
 		c[j] = 4 * tid + j < a.experts ? (a.count[4 * tid + j] + GB_BM - 1) / GB_BM : 0;
 		sum += c[j];
 	}
+	const int r0 = blockIdx.x * rows, nr = min(rows, R - r0), items = nr * a.top;
+	const int id = tid < items ? a.id[r0 * a.top + tid] : 0, place = tid < items ? a.place[r0 * a.top + tid] : 0;
 	int inc = sum;
 #pragma unroll
 	for (int x = 1; x < 32; x *= 2) {
@@ -149,19 +151,16 @@ template <typename T> __global__ void __launch_bounds__(128) expert_gather_kerne
 	}
 	if (blockIdx.x == 0 && tid == 127) *a.n_tiles = at;
 	__syncthreads();
-	constexpr int V = 16 / int(sizeof(T));
-	const int n = ldh / V;
-	for (int i = 0; i < MG_ROWS; i++) {
-		const int r = blockIdx.x * MG_ROWS + i;
-		if (r >= R) break;
-		for (int k = 0; k < a.top; k++) {
-			const int e = a.id[r * a.top + k], slot = first[e] * GB_BM + a.place[r * a.top + k];
-			const uint4 *src = reinterpret_cast<const uint4 *>(h + size_t(r) * ldh);
-			uint4 *dst = reinterpret_cast<uint4 *>(xg + size_t(slot) * ldh);
-			for (int x = tid; x < n; x += 128) dst[x] = src[x];
-			__syncthreads();  // (everybody has read the place)
-			if (tid == 0) a.place[r * a.top + k] = slot;
-		}
+	if (tid < items) {  // (MG_ROWS * MOE_TOP = 128)
+		slot[tid] = first[id] * GB_BM + place;
+		a.place[r0 * a.top + tid] = slot[tid];
+	}
+	__syncthreads();
+	const int n = ldh * int(sizeof(T)) / 16;
+	for (int x = tid; x < nr * n; x += 128) {
+		const int i = x / n, o = x % n;
+		const uint4 v = reinterpret_cast<const uint4 *>(h + size_t(r0 + i) * ldh)[o];
+		for (int k = 0; k < a.top; k++) reinterpret_cast<uint4 *>(xg + size_t(slot[i * a.top + k]) * ldh)[o] = v;
 	}
 }
 
@@ -186,7 +185,7 @@ static __device__ void expert_token_cta(const MoeArgs &a, int r, int item, float
 	__syncthreads();
 	const __nv_bfloat16 *W = a.W + (size_t(s_id) * 2 * a.n_glu + 32 * blk + 2 * warp) * a.ldw;
 	float s[4] = {};
-#pragma unroll 2
+#pragma unroll 4
 	for (int k8 = lane; k8 < K8; k8 += 32) {
 		const float4 x0 = *reinterpret_cast<const float4 *>(sm + 8 * k8), x1 = *reinterpret_cast<const float4 *>(sm + 8 * k8 + 4);
 #pragma unroll

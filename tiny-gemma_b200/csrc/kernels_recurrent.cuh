@@ -281,14 +281,8 @@ template <typename PT, int MT, int V> __global__ void __launch_bounds__(128) lin
 		return;
 	}
 	const PT *in = reinterpret_cast<const PT *>(a.p) + size_t(r0) * a.ldp + a.p_x + ch;
-	float bias[V], cf[MT][V], win[MT][V], x[LV_ROWS][V];
+	float bias[V], cf[MT][V], win[MT][V];
 	lin_load<V>(bias, a.cb + ch);
-#pragma unroll
-	for (int i = 0; i < LV_ROWS; i++) {
-#pragma unroll
-		for (int e = 0; e < V; e++) x[i][e] = 0.0f;
-		if (i < nr) lin_load<V>(x[i], in + size_t(i) * a.ldp);
-	}
 #pragma unroll
 	for (int j = 0; j < MT; j++) {
 #pragma unroll
@@ -308,41 +302,51 @@ template <typename PT, int MT, int V> __global__ void __launch_bounds__(128) lin
 		for (int j = 0; j < MT; j++)
 			if (MT - j <= H) lin_load<V>(win[j], in - ptrdiff_t(MT - j) * a.ldp);
 	}
+#pragma unroll 1
+	for (int i0 = 0; i0 < nr; i0 += 4) {
+		float x[4][V];
 #pragma unroll
-	for (int i = 0; i < LV_ROWS; i++) {
-		if (i >= nr) break;
-		const int r = r0 + i, sg = seg_s[i];
-		if (sg != seg) {
-			seg = sg;
-			row0 = a.d.seg_row[seg];
-			len = a.d.seg_len[seg];
-			const int pos = a.d.seg_pos[seg], t = r - row0;
-			float *hb = a.hist + size_t(a.d.seg_seq[seg]) * 2 * H * C;
-			const float *hr = hb + size_t(a.d.seg_par[seg]) * H * C;
-			hw = hb + size_t(a.d.seg_par[seg] ^ 1) * H * C;
+		for (int u = 0; u < 4; u++) {
 #pragma unroll
-			for (int j = 0; j < MT; j++)
-#pragma unroll
-				for (int e = 0; e < V; e++) win[j][e] = MT - j <= H ? lin_conv_in<PT>(a, row0, pos, hr, C, t - (MT - j), ch + e) : 0.0f;
-			if (t == 0)  // inputs before this segment that stay relevant
-				for (int q = 0; q < H; q++)
-					if (len - H + q < 0)
-						for (int e = 0; e < V; e++) hw[size_t(q) * C + ch + e] = lin_conv_in<PT>(a, row0, pos, hr, C, len - H + q, ch + e);
+			for (int e = 0; e < V; e++) x[u][e] = 0.0f;
+			if (i0 + u < nr) lin_load<V>(x[u], in + size_t(i0 + u) * a.ldp);
 		}
-		float y[V];
 #pragma unroll
-		for (int e = 0; e < V; e++) {
-			y[e] = bias[e];
+		for (int u = 0; u < 4; u++) {
+			const int i = i0 + u, r = r0 + i;
+			if (i >= nr) break;
+			if (seg_s[i] != seg) {
+				seg = seg_s[i];
+				row0 = a.d.seg_row[seg];
+				len = a.d.seg_len[seg];
+				const int pos = a.d.seg_pos[seg], t = r - row0;
+				float *hb = a.hist + size_t(a.d.seg_seq[seg]) * 2 * H * C;
+				const float *hr = hb + size_t(a.d.seg_par[seg]) * H * C;
+				hw = hb + size_t(a.d.seg_par[seg] ^ 1) * H * C;
 #pragma unroll
-			for (int j = 0; j < MT; j++) {
-				win[j][e] = j + 1 < MT ? win[j + 1][e] : x[i][e];
-				y[e] = fmaf(cf[j][e], win[j][e], y[e]);
+				for (int j = 0; j < MT; j++)
+#pragma unroll
+					for (int e = 0; e < V; e++) win[j][e] = MT - j <= H ? lin_conv_in<PT>(a, row0, pos, hr, C, t - (MT - j), ch + e) : 0.0f;
+				if (t == 0)  // inputs before this segment that stay relevant
+					for (int q = 0; q < H; q++)
+						if (len - H + q < 0)
+							for (int e = 0; e < V; e++) hw[size_t(q) * C + ch + e] = lin_conv_in<PT>(a, row0, pos, hr, C, len - H + q, ch + e);
 			}
-			y[e] = sizeof(PT) == 2 ? swish_fast(y[e], y[e]) : silu_f(y[e]);
+			float y[V];
+#pragma unroll
+			for (int e = 0; e < V; e++) {
+				y[e] = bias[e];
+#pragma unroll
+				for (int j = 0; j < MT; j++) {
+					win[j][e] = j + 1 < MT ? win[j + 1][e] : x[u][e];
+					y[e] = fmaf(cf[j][e], win[j][e], y[e]);
+				}
+				y[e] = sizeof(PT) == 2 ? swish_fast(y[e], y[e]) : silu_f(y[e]);
+			}
+			lin_store<V, PT>(out + size_t(i) * a.ldxc, y);
+			const int q = (r - row0) - (len - H);
+			if (q >= 0) lin_store<V, float>(hw + size_t(q) * C + ch, x[u]);
 		}
-		lin_store<V, PT>(out + size_t(i) * a.ldxc, y);
-		const int q = (r - row0) - (len - H);
-		if (q >= 0) lin_store<V, float>(hw + size_t(q) * C + ch, x[i]);
 	}
 }
 
@@ -567,16 +571,23 @@ static __global__ void __launch_bounds__(256) lin_chunk_state_kernel(const __gri
 			for (int c = 0; c < kch; c++) tma_load_2d(smem + c * 16384, &rmap, a.o_k + g * a.Np + 64 * c, row0 + t0, &k_bar);
 		}
 		const float b = tid < n ? a.b[size_t(row0 + t0 + tid) * a.H + h] : 0.0f;
+		const __nv_bfloat16 *vb = reinterpret_cast<const __nv_bfloat16 *>(a.rows) + size_t(row0 + t0) * a.ldr + a.o_v + h * a.vdp + 64 * tile;
+		const int c8n = cols / 8;
+		uint4 vr[4];  // 16 bytes of V per thread and round; at most four rounds
+#pragma unroll
+		for (int e = 0; e < 4; e++) {
+			const int x = tid + 256 * e, s = x / c8n;
+			vr[e] = s < n ? *reinterpret_cast<const uint4 *>(vb + size_t(s) * a.ldr + 8 * (x % c8n)) : make_uint4(0, 0, 0, 0);
+		}
 		lin_cumulate(tid < n ? a.la[size_t(row0 + t0 + tid) * a.H + h] : 0.0f, ch, cl, part);
 		if (tid < LC) sw[tid] = b * exp2f((ch[LC - 1] - ch[tid]) + (cl[LC - 1] - cl[tid]));
 		if (tid == 0 && tile == 0) a.tot[hc] = ch[LC - 1] + cl[LC - 1];
 		__syncthreads();
-		const __nv_bfloat16 *vb = reinterpret_cast<const __nv_bfloat16 *>(a.rows) + size_t(row0 + t0) * a.ldr + a.o_v + h * a.vdp + 64 * tile;
-		const int c8n = cols / 8;
-		for (int x = tid; x < LC * c8n; x += 256) {
-			const int s = x / c8n, c8 = x % c8n;
-			uint4 u = make_uint4(0, 0, 0, 0);
-			if (s < n) u = *reinterpret_cast<const uint4 *>(vb + size_t(s) * a.ldr + 8 * c8);
+#pragma unroll
+		for (int r = 0; r < 4; r++) {
+			const int x = tid + 256 * r, s = x / c8n, c8 = x % c8n;
+			if (s >= LC) break;
+			const uint4 u = vr[r];
 			const float w = sw[s];
 			const uint32_t in[4] = {u.x, u.y, u.z, u.w};
 			uint32_t hi[4], lo[4];
@@ -778,6 +789,11 @@ static __global__ void __launch_bounds__(256, 2) lin_chunk_out_kernel(const __gr
 			const int last = min(row, n - 1) - 64 * half;  // columns of this half up to `last` are visible
 #pragma unroll
 			for (int e = 0; e < 2; e++) {
+				if (64 * half + 32 * e > 32 * quad + 31) {  // (the whole warp: nothing of this block is visible)
+#pragma unroll
+					for (int c = 0; c < 16; c++) w[16 * e + c] = 0;
+					continue;
+				}
 				uint32_t ra[32];
 				tc_ld32(tmem + lane_addr + uint32_t(64 * half + 32 * e), ra);
 				asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");

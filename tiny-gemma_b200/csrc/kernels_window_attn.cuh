@@ -83,11 +83,19 @@ template <typename CT, int NT> __device__ __forceinline__ void wa_pool_block(con
 		const int n = isk ? nk : nv, col = isk ? g * a.dkp + c : g * a.dvp + c - a.dkp;
 		const CT *ring = reinterpret_cast<const CT *>(isk ? a.kc : a.vc) + size_t(seq) * a.cap * n + col;
 		float s = 0.0f;
-#pragma unroll 4
-		for (int j = 0; j < a.pool; j++) s += to_f32(ring[size_t((b * a.pool + j) % a.cap) * n]);
+		const int first = (b * a.pool) % a.cap, wrap = a.cap - first;  // (row j lies at slot first + j, or that minus cap)
+#pragma unroll 8
+		for (int j = 0; j < a.pool; j++) s += to_f32(ring[size_t(first + j - (j >= wrap ? a.cap : 0)) * n]);
 		reinterpret_cast<CT *>(isk ? a.ks : a.vs)[(size_t(seq) * a.keep_rows + b) * n + col] = from_f32<CT>(s / float(a.pool));
 	}
 }
+__device__ __forceinline__ float2 load2(const float *p) { return *reinterpret_cast<const float2 *>(p); }
+__device__ __forceinline__ float2 load2(const __nv_bfloat16 *p) {
+	const uint32_t u = *reinterpret_cast<const uint32_t *>(p);
+	return make_float2(bf16_lo(u), bf16_hi(u));
+}
+__device__ __forceinline__ void store2(float *p, float2 v) { *reinterpret_cast<float2 *>(p) = v; }
+__device__ __forceinline__ void store2(__nv_bfloat16 *p, float2 v) { *reinterpret_cast<uint32_t *>(p) = pack_bf16(v.x, v.y); }
 // Portions: rotates q in place, puts rotated keys and normed values into the ring, and pools the blocks that the step
 // completes. A CTA owns `unit` positions (a multiple of `pool`, counted from the sequence's start) of a key/value head, so
 // that what a block needs is either its own or an earlier step's. grid (units of the longest segment + 1, G, segments)
@@ -105,36 +113,54 @@ static __global__ void __launch_bounds__(256) kv_transform_kernel(WAttnArgs a, i
 		const int r = row0 + i - pos;
 		PT *row = const_cast<PT *>(reinterpret_cast<const PT *>(a.p)) + size_t(r) * a.ldp;
 		const float2 *cs = a.cs + size_t(r) * a.ld_cs;
-		for (int c = lane; c < half; c += 32) {
-			const float2 t = cs[c];
-			PT *q = row + a.p_q + g * per * a.dkp + c;
-			for (int h0 = 0; h0 < per; h0 += 8) {  // (loads of eight heads ahead of their stores)
-				float u[8], v[8];
-#pragma unroll
-				for (int h = 0; h < 8; h++)
-					if (h0 + h < per) {
-						u[h] = to_f32(q[(h0 + h) * a.dkp]);
-						v[h] = to_f32(q[(h0 + h) * a.dkp + half]);
-					}
-#pragma unroll
-				for (int h = 0; h < 8; h++)
-					if (h0 + h < per) {
-						q[(h0 + h) * a.dkp] = from_f32<PT>(u[h] * t.x - v[h] * t.y);
-						q[(h0 + h) * a.dkp + half] = from_f32<PT>(v[h] * t.x + u[h] * t.y);
-					}
+		PT *q0 = row + a.p_q + g * per * a.dkp;
+		if (half % 2 == 0) {
+			for (int c = 2 * lane; c < half; c += 64) {
+				const float4 t = *reinterpret_cast<const float4 *>(cs + c);  // cos, sin, cos, sin
+#pragma unroll 4
+				for (int h = 0; h < per; h++) {
+					PT *q = q0 + h * a.dkp + c;
+					const float2 u = load2(q), v = load2(q + half);
+					store2(q, make_float2(u.x * t.x - v.x * t.y, u.y * t.z - v.y * t.w));
+					store2(q + half, make_float2(v.x * t.x + u.x * t.y, v.y * t.z + u.y * t.w));
+				}
 			}
+		} else {
+			for (int c = lane; c < half; c += 32)
+				for (int h = 0; h < per; h++) {
+					PT *q = q0 + h * a.dkp + c;
+					const float u = to_f32(q[0]), v = to_f32(q[half]);
+					q[0] = from_f32<PT>(u * cs[c].x - v * cs[c].y);
+					q[half] = from_f32<PT>(v * cs[c].x + u * cs[c].y);
+				}
 		}
 		const size_t slot = size_t(seq) * a.cap + i % a.cap;
 		CT *kd = reinterpret_cast<CT *>(a.kc) + slot * nk + g * a.dkp, *vd = reinterpret_cast<CT *>(a.vc) + slot * nv + g * a.dvp;
 		const PT *ks = row + a.p_k + g * a.dkp, *vs = row + a.p_v + g * a.dvp;
-		for (int c = lane; c < a.dkp; c += 32) kd[c] = from_f32<CT>(wa_rotated(a, ks, cs, c));
+		if (half % 2 == 0) {
+			for (int c = 2 * lane; c < half; c += 64) {
+				const float4 t = *reinterpret_cast<const float4 *>(cs + c);
+				const float2 u = load2(ks + c), v = load2(ks + half + c);
+				store2(kd + c, make_float2(u.x * t.x - v.x * t.y, u.y * t.z - v.y * t.w));
+				store2(kd + half + c, make_float2(v.x * t.x + u.x * t.y, v.y * t.z + u.y * t.w));
+			}
+			for (int c = a.rot + 2 * lane; c < a.dkp; c += 64) store2(kd + c, load2(ks + c));
+		} else {
+			for (int c = lane; c < a.dkp; c += 32) kd[c] = from_f32<CT>(wa_rotated(a, ks, cs, c));
+		}
 		float f = 1.0f;
-		if (a.vnorm) {
+		if (a.vnorm) {  // (padding columns are zero)
 			float s = 0.0f;
-			for (int c = lane; c < a.dv; c += 32) s = fmaf(to_f32(vs[c]), to_f32(vs[c]), s);
+			for (int c = 2 * lane; c < a.dvp; c += 64) {
+				const float2 v = load2(vs + c);
+				s = fmaf(v.x, v.x, fmaf(v.y, v.y, s));
+			}
 			f = 1.0f / sqrtf(warp_sum(s) / float(a.dv) + a.eps);
 		}
-		for (int c = lane; c < a.dvp; c += 32) vd[c] = from_f32<CT>(to_f32(vs[c]) * f);
+		for (int c = 2 * lane; c < a.dvp; c += 64) {
+			const float2 v = load2(vs + c);
+			store2(vd + c, make_float2(v.x * f, v.y * f));
+		}
 	}
 	if (!a.pool) return;
 	__syncthreads();

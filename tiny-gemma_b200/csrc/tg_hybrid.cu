@@ -172,6 +172,7 @@ struct HybridState : tg_state {
 	template <typename T> RowSum<T> row_sum(int R);
 	int attn_rows(const WAttnArgs &wa, int run, int R, int nseg, int max_len);
 	int token_splits(const WAttnArgs &wa, int fill) const;
+	int few_rows() const;
 
 	struct Entry {
 		int seq, count, done;
@@ -280,7 +281,7 @@ template <int EPI, bool GRP = false> int launch_gemm_f32(const float *A, int lda
 }
 
 template <int R, int NR, int KS, int PRO, int EPI> int launch_gemv(const GemvArgs &g, cudaStream_t st) {
-	const size_t smem = gv_smem<R, NR>(g.K, PRO, EPI, g.parts, g.top * g.n_ex);
+	const size_t smem = gv_smem<R, NR>(g.K, PRO, EPI, g.parts, g.top, g.top * g.n_ex);
 	auto kernel = gemv_bf16_kernel<R, NR, KS, PRO, EPI>;
 	TG_TRY(allow_smem(kernel, smem));
 	int occ = 1;
@@ -958,7 +959,8 @@ template <typename T> int launch_lin_norm(const LinArgs &a, const Layer &L, void
 	return check_launch("lin_norm");
 }
 template <typename T> int launch_gather(const MoeArgs &a, const void *h, int ldh, void *xg, int R, cudaStream_t st) {
-	launch_k(expert_gather_kernel<T>, dim3((R + MG_ROWS - 1) / MG_ROWS), dim3(128), 0, st, a, static_cast<const T *>(h), ldh, static_cast<T *>(xg), R);
+	const int rows = R >= 4 * MG_ROWS * g_num_sms ? MG_ROWS : 1;
+	launch_k(expert_gather_kernel<T>, dim3((R + rows - 1) / rows), dim3(128), 0, st, a, static_cast<const T *>(h), ldh, static_cast<T *>(xg), R, rows);
 	count_launch();
 	return check_launch("expert_gather");
 }
@@ -995,6 +997,12 @@ int HybridState::attn_rows(const WAttnArgs &wa, int run, int R, int nseg, int ma
 int HybridState::token_splits(const WAttnArgs &wa, int fill) const {
 	const long long second = wa.pool ? max_pos_global / wa.pool : wa.keep, keys = std::min<long long>(wa.window + second, max_pos_global);
 	return int(std::max<long long>(1, std::min<long long>(std::min(nsplit_cap, fill), (keys + WK_KEYS - 1) / WK_KEYS)));
+}
+
+// rows up to which a step of one token per sequence is made of matrix-vector products
+int HybridState::few_rows() const {
+	static const int most = env_int("TG_FEW_ROWS", FEW_ROWS);
+	return std::min(most, FEW_ROWS);
 }
 
 // ---- feed-forward after the mixer
@@ -1309,7 +1317,7 @@ int HybridState::add_left(int R) {
 
 // All layers for R rows in nseg segments (the longest: max_len), leaving the residual stream in x.
 int HybridState::run_layers(const StepDesc &d, int R, int nseg, int max_len) {
-	const bool few = max_len == 1 && R <= FEW_ROWS;
+	const bool few = max_len == 1 && R <= few_rows();
 	const int D = m->D;
 	auto embed_rows = [&](int add) -> int {
 		launch_k(embed_rows_kernel, dim3(R), dim3(256), 0, stream, x, ldx, m->embed.W, m->embed.ld, m->embed_scale, d, D, m->n_vocab, add, err_flag);
@@ -1357,7 +1365,7 @@ int HybridState::score_rows(const int *rows_dev, int n, float *out, float *norm_
 int HybridState::enqueue_decode_all() {
 	const StepDesc d = lockstep_desc();
 	TG_TRY(run_layers(d, B, B, 1));
-	if (B <= FEW_ROWS) {
+	if (B <= few_rows()) {
 		GemvArgs g{};
 		g.d = d;
 		g.x = x;
