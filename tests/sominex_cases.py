@@ -112,7 +112,7 @@ def weights(cfg, seed, gain=1.0):
         if ff and ff["kind"] == "dense":
             glu(W, p + "mlp.", ff["ff"])
         elif ff:
-            W[p + "mlp.router"] = lin(ff["router"]["experts"], D, 1.5)
+            W[p + "mlp.router"] = lin(ff["router"]["experts"], D, 5.0)  # (few close calls)
             for e in range(ff["router"]["experts"]):
                 glu(W, p + "mlp.e%d." % e, ff["expert"]["ff"])
             if ff.get("shared"):
@@ -126,17 +126,35 @@ def tokens(cfg, n, seed):
     return np.random.default_rng(seed).integers(0, cfg["vocab"], n).astype(np.int32)
 
 
-def close_route(cfg, W, trace, scale=1.0):
-    """smallest gap between the last chosen and the first not chosen router score of any token of a traced sequence"""
-    import sominex_plain as P
+# ------------------------------------------------------------------ a model in which one key decides
+# Token KEY's key and token QUERY's query point the same way (strongly enough for the mean of a block to stand out);
+# everybody else's are nearly zero. At a QUERY position the attention either finds the KEY, itself or in a pooled block, or
+# is spread evenly, so whether one certain position is visible decides the output.
+KEY, QUERY = 1, 2
 
-    gap = np.inf
-    for i, sp in enumerate(cfg["layers"]):
-        ff = sp["mlp"]
-        if not ff or ff["kind"] != "moe" or ff["router"]["top"] == ff["router"]["experts"]:
-            continue
-        W64 = {k: np.asarray(v, np.float64) for k, v in W.items()}
-        h = P.unit_rms(trace[i], cfg["norm"]["eps"]) * W64["l%d.norm1" % i]
-        z = np.sort(h @ W64["l%d.mlp.router" % i].T, axis=1)[:, ::-1]
-        gap = min(gap, (z[:, ff["router"]["top"] - 1] - z[:, ff["router"]["top"]]).min())
-    return gap
+
+def beacon(window, pool, seed=5, **kw):
+    cfg = config([attn(None, size=window, pool=pool, heads=2, kv_heads=1, dim=32, vdim=32, scale=0.4, rot=0)], **kw)
+    W = weights(cfg, seed)
+    e, m = np.array(W["embed"]), "l0.mix."
+    e[:, :2] = 0.0
+    e[KEY, 0] = e[QUERY, 1] = 12.0
+    W["embed"] = e
+    W["l0.shift"] = np.zeros_like(W["l0.shift"])
+    W["l0.norm1"] = np.ones_like(W["l0.norm1"])
+    q, k = 0.02 * np.array(W[m + "q"]), 0.02 * np.array(W[m + "k"])
+    q[::32, 1] = k[::32, 0] = 3.0
+    W[m + "q"], W[m + "k"] = q, k
+    v = np.array(W[m + "v"])
+    v[:, 0] = 4.0 * np.random.default_rng(seed).standard_normal(v.shape[0])
+    W[m + "v"] = v
+    W[m + "o"] = 4.0 * np.array(W[m + "o"])
+    return cfg, {k_: to_bf16(x) for k_, x in W.items()}
+
+
+def without_mixers(W, cfg):
+    """the same weights with every mixer's output projection zero: what a layer adds is its feed-forward's"""
+    W = dict(W)
+    for i in range(len(cfg["layers"])):
+        W["l%d.mix.o" % i] = np.zeros_like(W["l%d.mix.o" % i])
+    return W
