@@ -33,19 +33,19 @@ struct MoeArgs {
 	float *out;          // [R][top][n_glu]
 };
 
-// the warp's choice for one row; lane k < top returns the k-th (expert, weight)
-__device__ __forceinline__ void moe_choose(const float *z, int E, int top, float scale, int &id, float &w) {
+// the warp's choice for one row; lane k < top returns the k-th (expert, weight). NL: experts per lane
+template <int NL> __device__ __forceinline__ void moe_choose_n(const float *z, int E, int top, float scale, int &id, float &w) {
 	const int lane = threadIdx.x & 31;
-	float s[MOE_LANE], mx = -INFINITY;
+	float s[NL], mx = -INFINITY;
 #pragma unroll
-	for (int j = 0; j < MOE_LANE; j++) {
+	for (int j = 0; j < NL; j++) {
 		s[j] = lane + 32 * j < E ? z[lane + 32 * j] : -INFINITY;
 		mx = fmaxf(mx, s[j]);
 	}
 	mx = warp_max(mx);
 	float sum = 0.0f;
 #pragma unroll
-	for (int j = 0; j < MOE_LANE; j++) {
+	for (int j = 0; j < NL; j++) {
 		if (32 * j >= E) break;
 		sum += expf(s[j] - mx);
 	}
@@ -56,7 +56,7 @@ __device__ __forceinline__ void moe_choose(const float *z, int E, int top, float
 		float best = -INFINITY;
 		int at = 0x7fffffff;
 #pragma unroll
-		for (int j = 0; j < MOE_LANE; j++)
+		for (int j = 0; j < NL; j++)
 			if (s[j] > best) {
 				best = s[j];
 				at = lane + 32 * j;
@@ -72,13 +72,18 @@ __device__ __forceinline__ void moe_choose(const float *z, int E, int top, float
 		}
 		if (at >= E) at = 0;  // (logits that are not numbers)
 #pragma unroll
-		for (int j = 0; j < MOE_LANE; j++)
+		for (int j = 0; j < NL; j++)
 			if (lane + 32 * j == at) s[j] = -INFINITY;
 		if (lane == k) {
 			id = at;
 			w = expf(best - mx) / sum * scale;
 		}
 	}
+}
+__device__ __forceinline__ void moe_choose(const float *z, int E, int top, float scale, int &id, float &w) {
+	if (E <= 32) moe_choose_n<1>(z, E, top, scale, id, w);
+	else if (E <= 128) moe_choose_n<4>(z, E, top, scale, id, w);
+	else moe_choose_n<MOE_LANE>(z, E, top, scale, id, w);
 }
 
 // grid ceil(R / (8 rounds)), 256 threads, rounds <= MR_ROUNDS rows per warp. Places are counted within the CTA first: one
