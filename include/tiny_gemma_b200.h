@@ -80,7 +80,8 @@ int tg_config_by_name(const char *name, tg_config *out);
  *                  norms, attention scores and recurrent states in 32-bit.
  *   dtype TG_F32:  everything in 32-bit (the weights are the same bfloat16 values).
  * Architectures: "Nabelix" (pre-norm decoder whose mixer runs windowed attention with kept first tokens and a
- * gated delta rule side by side). Entry points of this header that name a Gemma structure (tg_model_load_*,
+ * gated delta rule side by side), "Sominex" (feed-forwards beside the mixers; windowed attention with pooled
+ * blocks, Mamba-2 or mLSTM; dense layers and mixtures of experts). Entry points of this header that name a Gemma structure (tg_model_load_*,
  * tg_model_set_*, tg_kv_read, tg_decode_hidden, the tg_dev_ calls on a handle) return TG_EINVAL on such a model. */
 enum { TG_BF16 = 0, TG_F32 = 1 };
 int tg_model_open(const char *dir, int device, int dtype, tg_model **out);
