@@ -552,6 +552,7 @@ static __global__ void __launch_bounds__(256) lin_chunk_state_kernel(const __gri
 		mbar_init(&d_bar, 1);
 		asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
 	}
+	pdl_wait();  // (before the allocation: a CTA that holds TMEM waits for no earlier kernel)
 	if (warp == 0) {
 		asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_base_s)), "r"(ncols) : "memory");
 		asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
@@ -560,7 +561,6 @@ static __global__ void __launch_bounds__(256) lin_chunk_state_kernel(const __gri
 	__syncthreads();
 	tc_fence_after();
 	const uint32_t tmem = tmem_base_s;
-	pdl_wait();
 	const int vt = (a.vdp + 63) / 64, h = blockIdx.y / vt, tile = blockIdx.y % vt, seg = blockIdx.z, g = h / (a.H / a.G);
 	const int len = a.d.seg_len[seg], row0 = a.d.seg_row[seg], t0 = blockIdx.x * LC;
 	if (t0 < len) {
@@ -733,6 +733,7 @@ static __global__ void __launch_bounds__(256, 2) lin_chunk_out_kernel(const __gr
 		mbar_init(&o_bar, 1);
 		asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
 	}
+	pdl_wait();  // (before the allocation: a CTA that holds TMEM waits for no earlier kernel)
 	if (warp == 0) {
 		asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_base_s)), "r"(256) : "memory");
 		asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
@@ -741,7 +742,6 @@ static __global__ void __launch_bounds__(256, 2) lin_chunk_out_kernel(const __gr
 	__syncthreads();
 	tc_fence_after();
 	const uint32_t tmem = tmem_base_s;
-	pdl_wait();
 	const int h = blockIdx.y / a.vsplit, vs = blockIdx.y % a.vsplit, seg = blockIdx.z, g = h / (a.H / a.G);
 	const int len = a.d.seg_len[seg], row0 = a.d.seg_row[seg], t0 = blockIdx.x * LC;
 	const int tiles = (a.vdp + 63) / 64, share = (tiles + a.vsplit - 1) / a.vsplit, tl0 = vs * share, tl1 = min(tiles, tl0 + share);
